@@ -13,9 +13,11 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libmonofab.so")
-SOURCES = ["api.cu", "moe_aux.cu", "expert_gemm.cu", "pack_static.cu", "fabric_device.cu", "fabric_host.cu", "attention.cu", "host_loop.cu", "ep_exchange.cu", "release.cu", "plan_model.cu", "plan_admission.cu", "plan_api.cu"]
+SOURCES = ["api.cu", "moe_aux.cu", "expert_gemm.cu", "pack_static.cu", "fabric_device.cu", "fabric_layer_rows.cu", "fabric_layer_scan.cu", "fabric_layer_memory.cu", "fabric_layer_latent.cu", "fabric_host.cu", "attention.cu", "host_loop.cu", "ep_exchange.cu", "release.cu", "plan_model.cu", "plan_admission.cu", "plan_api.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr"]
+# The fabric kernel calls the tiles of the fabric_layer_*.cu files across translation units.
+RELOCATABLE = {s for s in SOURCES if s == "fabric_device.cu" or s.startswith("fabric_layer_")}
 
 
 def _nvcc():
@@ -43,7 +45,7 @@ def build(verbose=False, force=False):
         s = os.path.join(CSRC, src)
         o = os.path.join(OBJ, src.replace(".cu", ".o"))
         if force or not os.path.exists(o) or os.path.getmtime(o) < max(os.path.getmtime(s), hdr_t):
-            cmd = [nvcc, *NVCC_FLAGS, "-c", s, "-o", o]
+            cmd = [nvcc, *NVCC_FLAGS, *(["-rdc=true"] if src in RELOCATABLE else []), "-c", s, "-o", o]
             if verbose:
                 cmd.insert(1, "-Xptxas=-v")
             jobs.append(cmd)
@@ -54,7 +56,7 @@ def build(verbose=False, force=False):
             raise RuntimeError("nvcc failed:\n" + " ".join(cmd) + "\n" + r.stdout + r.stderr)
         return r.stderr
 
-    with ThreadPoolExecutor(max_workers=4) as ex:
+    with ThreadPoolExecutor(max_workers=8) as ex:
         logs = list(ex.map(run, jobs))
     if verbose:
         for log in logs:

@@ -287,6 +287,17 @@ const std::string& layouts_json() {
     MF_JSON_STRUCT(AttnPlanArgs, MF_ATTN_PLAN_ARGS)
     MF_JSON_STRUCT(LogitsArgs, MF_LOGITS_ARGS)
     MF_JSON_STRUCT(CombineArgs, MF_COMBINE_ARGS)
+    MF_JSON_STRUCT(StreamArgs, MF_STREAM_ARGS)
+    MF_JSON_STRUCT(ProductArgs, MF_PRODUCT_ARGS)
+    MF_JSON_STRUCT(GatedArgs, MF_GATED_ARGS)
+    MF_JSON_STRUCT(SumArgs, MF_SUM_ARGS)
+    MF_JSON_STRUCT(ConvArgs, MF_CONV_ARGS)
+    MF_JSON_STRUCT(ScanArgs, MF_SCAN_ARGS)
+    MF_JSON_STRUCT(MemGateArgs, MF_MEM_GATE_ARGS)
+    MF_JSON_STRUCT(MemoryArgs, MF_MEMORY_ARGS)
+    MF_JSON_STRUCT(HeadNormArgs, MF_HEAD_NORM_ARGS)
+    MF_JSON_STRUCT(LatentArgs, MF_LATENT_ARGS)
+    MF_JSON_STRUCT(LatentAttnArgs, MF_LATENT_ATTN_ARGS)
     MF_JSON_STRUCT(StagingArgs, MF_STAGING_ARGS)
     s += "}";
     return s;

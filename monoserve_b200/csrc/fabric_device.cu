@@ -31,6 +31,7 @@
 #include <cuda_runtime.h>
 
 #include "attention_core.cuh"
+#include "fabric_layer_tiles.cuh"
 #include "fabric_sched.cuh"
 #include "fabric_types.h"
 #include "gemm_core.cuh"
@@ -41,7 +42,6 @@
 namespace mf {
 namespace fab {
 
-constexpr int kExecThreads = 128;
 constexpr int kSlots = 4;   // work records the scheduler may run ahead of the exec warps
 constexpr int kWorkerThreads = 32 + kExecThreads + 64;   // scheduler, exec/epilogue, TMA producer, MMA
 
@@ -57,7 +57,8 @@ struct WorkSlot {
   AttnWork attn;          // filled by the scheduler for attention work items
   const ProgramDesc* prog;
   uint32_t stage, tile_lane, link, index, cmd, worker_lane, is_gemm, is_attn;
-  uint32_t counts, pad;   // counts: this record completes its tile (0 for all but the last row block of a kind-45 tile)
+  uint32_t counts, is_wide;   // counts: this record completes its tile (0 for all but the last row block of a kind-45 tile);
+                            // is_wide: the exec warps use the operand ring as scratch memory
 };
 
 // A GEMM tile (kind 32) in the reference's operand convention
@@ -84,7 +85,7 @@ __device__ bool make_gemm_work(const TileDesc& t, GemmWork& w, uint32_t block = 
   if (A.bm < 16 || A.bm > kGemmMaxN || (A.bm & (A.bm - 1))) return false;
   const CUtensorMap* wrec = reinterpret_cast<const CUtensorMap*>(t.a[1]);
   const CUtensorMap* xrec = reinterpret_cast<const CUtensorMap*>(t.a[2]);
-  const bool silu = A.epi == kEpiSiluMul;
+  const bool silu = epi_gated(static_cast<int>(A.epi));
   const bool atomic_slabs = A.epi == kEpiAtomicF32 && A.up_offset != 0;
   const bool packed = silu && __ldcg(reinterpret_cast<const unsigned int*>(wrec + 3)) != 0;
   w.a_map = ((silu && !packed) || atomic_slabs) ? wrec + 1 : wrec + 2;
@@ -115,7 +116,7 @@ __device__ bool make_gemm_work(const TileDesc& t, GemmWork& w, uint32_t block = 
   w.block = -1;
   w.w_fp8 = A.w_fp8 != 0;   // e4m3 weights: the exec warps expand every stage to bf16 before its MMAs
   w.fetch = 0;
-  return w.k_tiles > 0 && A.epi <= kEpiRowsF32;
+  return w.k_tiles > 0 && A.epi <= kEpiGeluMul;
 }
 
 // Fetch tile (kind 49): i0 bytes from a[0] (host-resident weights) to a[1] (an HBM staging buffer).
@@ -147,7 +148,6 @@ __device__ bool make_fetch_work(const TileDesc& t, GemmWork& w) {
 }
 
 // ---------------------------------------------------------------- core tiles
-__device__ __forceinline__ void exec_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kExecThreads) : "memory"); }
 // Barrier of the exec threads that also tells each whether `v` held in all of them.
 __device__ __forceinline__ bool exec_all(bool v) {
   int r;
@@ -174,6 +174,7 @@ __device__ void trace_tile(unsigned long long base, uint32_t idx, unsigned long 
 // Scratch of the tile the exec warps are running; tiles run one at a time per worker,
 // so they share one block instead of each holding static shared memory of its own.
 constexpr int kExecScratchInts = 5 * (kMaxExperts + 1) + 16 + 64;
+static_assert(kExecScratchInts >= kLayerScratchInts, "scratch of the layer tiles");
 __shared__ __align__(16) int s_exec_scratch[kExecScratchInts];
 
 }  // namespace fab
@@ -191,8 +192,9 @@ __device__ void tile_asym_reduce(const TileDesc& t, int tid);
 __device__ void tile_norm_logits(const TileDesc& t, int tid);
 __device__ void tile_expand(const TileDesc& t, const ProgramDesc* P, DeviceState& S, int tid);
 
-// tid: index among the exec threads.
-__device__ bool run_core_tile(DeviceState& S, const WorkSlot& w, int tid, uint32_t worker, unsigned long long* sh_t0) {
+// tid: index among the exec threads.  ring: the operand ring, for a wide tile.
+__device__ bool run_core_tile(DeviceState& S, const WorkSlot& w, int tid, uint32_t worker, unsigned long long* sh_t0,
+                              uint8_t* ring) {
   const TileDesc& t = w.tile;
   switch (t.kind) {
     case kTileNop:
@@ -283,7 +285,7 @@ __device__ bool run_core_tile(DeviceState& S, const WorkSlot& w, int tid, uint32
       tile_attn_plan(t, w.prog, S, tid);
       return true;
     default:
-      return false;
+      return run_layer_tile(t, tid, s_exec_scratch, ring);
   }
 }
 
@@ -1094,6 +1096,7 @@ __global__ void __launch_bounds__(kWorkerThreads, 1) fabric_kernel(DeviceState* 
           w.worker_lane = ws.lane;
           w.is_gemm = 0;
           w.is_attn = 0;
+          w.is_wide = tile_is_wide(w.tile.kind);
           if (w.tile.kind == kTileAttnPrefill || w.tile.kind == kTileAttnDecode) {
             if (make_attn_work(w.tile, w.attn)) {
               w.is_attn = 1;
@@ -1156,7 +1159,9 @@ __global__ void __launch_bounds__(kWorkerThreads, 1) fabric_kernel(DeviceState* 
       if (w.is_attn || prev_attn)
         ok = __all_sync(0xffffffffu, (wait_counter(&sh.tiles_done, n, abort_flag) || attn_gave_up(sh.attn, 13)) &&
                                          (wait_counter(&sh.mma_done, n, abort_flag) || attn_gave_up(sh.attn, 14)));
-      prev_attn = w.is_attn != 0;
+      // A wide tile needs no wait of its own: the exec warps reach it when they are through with every earlier record,
+      // whose loads have then arrived and been consumed; only what follows it must stay out of the ring.
+      prev_attn = w.is_attn != 0 || w.is_wide != 0;
       if (ok && w.is_attn) {
         AttnCtx c = attn_ctx(w.attn, sh.attn, abort_flag, ring, tmem_base, aq, ab, &sh.wait_note[0]);
         attn_produce(w.attn, c);
@@ -1240,7 +1245,10 @@ __global__ void __launch_bounds__(kWorkerThreads, 1) fabric_kernel(DeviceState* 
         ok = ok && gemm_epilogue(w.gemm, sh.bar, tmem_base, g & 1, (g >> 1) & 1, abort_flag);
         if (!ok && tid == 0) raise_error(S, kFabErrTileWait);
         ++g;
-      } else if (!run_core_tile(S, w, tid, worker, &sh.t0) && tid == 0) {
+      } else if (w.is_wide) {
+        if (!run_core_tile(S, w, tid, worker, &sh.t0, ring) && tid == 0) raise_error(S, kFabErrBadTile);
+        fence_proxy_async_smem();   // the exec warps' accesses of the ring before the next record's TMA writes
+      } else if (!run_core_tile(S, w, tid, worker, &sh.t0, nullptr) && tid == 0) {
         raise_error(S, kFabErrBadTile);
       }
       exec_sync();

@@ -10,15 +10,6 @@
 namespace mf {
 namespace fab {
 
-template <class T>
-__device__ __forceinline__ void load_block(T& dst, unsigned long long addr) {
-  static_assert(sizeof(T) % 16 == 0, "operand blocks are multiples of 16 bytes");
-  const uint4* src = reinterpret_cast<const uint4*>(addr);
-  uint4* d = reinterpret_cast<uint4*>(&dst);
-#pragma unroll
-  for (int i = 0; i < static_cast<int>(sizeof(T) / 16); ++i) d[i] = __ldcg(src + i);
-}
-
 // An attention work item (kinds 33 prefill / 34 decode, one code path):
 //   a[0] AttnArgs*; i0 first query token (row of q / out); i1 = query tokens | kv head << 16;
 //   i2 first key (a multiple of 128); i3 one past the last key (0: no limit);
@@ -227,18 +218,7 @@ __device__ void tile_embed(const TileDesc& t, int tid) {
   for (uint32_t r = t.i0 + warp; r < t.i0 + t.i1; r += kExecThreads / 32) {
     int token;
     if (A.step) {
-      const int slot = reinterpret_cast<const int*>(St.row_req)[r];
-      token = reinterpret_cast<const int*>(St.last_token)[slot];
-      if (lane == 0) {
-        int* seq_len = reinterpret_cast<int*>(St.seq_len);
-        const int pos = min(seq_len[slot], static_cast<int>(St.bt_stride) * page - 1);
-        seq_len[slot] = pos + 1;
-        reinterpret_cast<int*>(St.tok_pos)[r] = pos;
-        const int pg = reinterpret_cast<const int*>(St.block_table)[static_cast<size_t>(slot) * St.bt_stride + pos / page];
-        reinterpret_cast<int*>(St.tok_slot)[r] = pg * page + pos % page;
-        int4* info = reinterpret_cast<int4*>(St.req_info);
-        info[r] = make_int4(static_cast<int>(r), pos, 1, pos + 1);
-      }
+      token = step_row(St, page, static_cast<int>(r), lane);
     } else {
       token = reinterpret_cast<const int*>(A.tokens)[r];
     }

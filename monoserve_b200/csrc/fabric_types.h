@@ -46,6 +46,19 @@ enum TileKind : uint16_t {
                             // or 41 with slabs) and then the router projection of those rows against experts
                             // [i2, i2 + i3) (a[1] LogitsArgs): the norm stage of a small batch folded into the
                             // projection's tiles (every expert-range tile of a row group writes the same norm)
+  // Layer-list decoders (fabric_layer_tiles.cuh); none of these is in the reference.
+  kTileProduct32 = 51,      // a block of a matrix product in 32-bit arithmetic
+  kTileGatedAct = 52,       // gelu_tanh(gate) * up of fp32 rows
+  kTileStreams = 53,        // hyper-connection update of the residual streams, next sublayer's input and its norm
+  kTileConv = 54,           // causal convolution per channel + silu
+  kTileScan = 55,           // selective scan of a request's rows
+  kTileMemGates = 56,       // log gates of the matrix memory
+  kTileMemory = 57,         // matrix memory over a request's rows
+  kTileHeadNorm = 58,       // per-head norm and output gate
+  kTileLatentKv = 59,       // latent norm, rotation, cache append, query parts
+  kTileLatentAttn = 60,     // attention over the cached latents, one key range
+  kTileLatentMerge = 61,    // merge of the key ranges
+  kTileSumSlabs = 62,       // sum of a K-split product's slabs
 };
 constexpr int kFabChunk = 16;   // rows per router / permute tile = rank chunk of the stable pack
 

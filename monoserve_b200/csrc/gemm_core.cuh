@@ -45,6 +45,9 @@ constexpr int kEpiWeightedAdd = 2;  // out32[pair_token[m]][n] += pair_weight[m]
 constexpr int kEpiStoreF32 = 3;    // out32[m][n] = acc (+ bias[n])
 constexpr int kEpiAtomicF32 = 4;   // out32[m][n] += acc : K-split partial sums
 constexpr int kEpiRowsF32 = 5;     // out32[m][n] = acc : per-pair rows for the deterministic combine (not in the reference)
+constexpr int kEpiGeluMul = 6;     // as kEpiSiluMul with the tanh form of gelu on the gate (not in the reference)
+// A tile of 64 gate and 64 up rows whose epilogue multiplies act(gate) by up.
+__host__ __device__ __forceinline__ bool epi_gated(int epi) { return epi == kEpiSiluMul || epi == kEpiGeluMul; }
 
 // Everything the three roles need to know about one tile; lives in shared memory.
 struct GemmWork {
@@ -184,7 +187,7 @@ __device__ __forceinline__ bool gemm_produce(const GemmWork& w, uint8_t* ring, G
   // SwiGLU tiles of a tensor in the reference row order gather eight 16-row boxes;
   // every other tile is one 128-row box (a packed SwiGLU tensor stores gate/up
   // groups of 16 rows alternately, so its tile starts at row 2 * a_row_lo).
-  const bool slab2 = w.epi == kEpiSiluMul || (w.a_packed & 4);
+  const bool slab2 = epi_gated(w.epi) || (w.a_packed & 4);
   const bool gather = slab2 && !(w.a_packed & 1);
   const int a_row = gather ? ((lane & 1) ? w.a_row_hi : w.a_row_lo) + 16 * ((lane & 7) >> 1)
                            : (slab2 ? 2 * w.a_row_lo : w.a_row_lo);
@@ -382,6 +385,12 @@ __device__ __forceinline__ bool gemm_convert(const GemmWork& w, uint8_t* ring, G
 
 __device__ __forceinline__ float silu_mul(float g, float u) { return __fdividef(g, 1.f + __expf(-g)) * u; }
 
+// gelu in its tanh form, times u: 0.5 g (1 + tanh(t)) = g / (1 + exp(-2 t)), t = sqrt(2 / pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float gelu_mul(float g, float u) {
+  const float t2 = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+  return __fdividef(g, 1.f + __expf(-t2)) * u;
+}
+
 // Epilogue of one tile from accumulator buffer `buf` (the four epilogue warps
 // call): everything except handing the buffer back to the MMA warp.
 template <bool kFetch = true>
@@ -397,7 +406,7 @@ __device__ __forceinline__ bool gemm_epilogue_body(const GemmWork& w, GemmBarrie
     return true;
   }
   const uint32_t tacc = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + buf * kAccCols;
-  const bool silu = w.epi == kEpiSiluMul;
+  const bool silu = epi_gated(w.epi), gelu = w.epi == kEpiGeluMul;
   // output feature of this lane, and the weight row its accumulator row came from
   int f, wrow;
   if (silu || (w.a_packed & 4)) {
@@ -437,7 +446,8 @@ __device__ __forceinline__ bool gemm_epilogue_body(const GemmWork& w, GemmBarrie
         const float mine_keep = __uint_as_float(lo ? r[j] : r[16 + j]) * sc;
         const float send = __uint_as_float(lo ? r[16 + j] : r[j]) * sc;
         const float other = __shfl_xor_sync(0xffffffffu, send, 16);
-        hv[j] = __bfloat16_as_ushort(__float2bfloat16(silu_mul(lo ? mine_keep : other, lo ? other : mine_keep)));
+        const float gate = lo ? mine_keep : other, up = lo ? other : mine_keep;
+        hv[j] = __bfloat16_as_ushort(__float2bfloat16(gelu ? gelu_mul(gate, up) : silu_mul(gate, up)));
       }
       if (f_ok) {
         const int m_hi = w.rows - t0;

@@ -80,6 +80,62 @@ namespace mf {
   U64(y) U64(pair_pos) U64(topk_w) U64(x2) U64(x) U64(w) U64(out) U32(K) U32(H) F32(eps) U32(reserved0) \
   U64(shared)
 
+/* Operand blocks of the layer-list decoders (hyper-connected residual streams, selective scan, matrix memory,
+ * latent attention; fabric_layer_tiles.cuh).  None of them is in the reference.  Activations are bf16, or fp32
+ * where a block's `f32` is set; `ld_*` are row strides in elements.
+ *
+ * StreamArgs: the residual streams xs fp32 [rows][streams][W].  hc_mix [from][to] and hc_out [to] belong to the
+ * sublayer that has just produced y (y_parts fp32 slabs of y_rows rows; 0 parts: no update), hc_in to the one
+ * that follows, w is the norm's multiplier (fp32).  embed set: the streams start as copies of the token's row. */
+#define MF_STREAM_ARGS(U64, U32, F32) \
+  U64(xs) U64(y) U64(hc_out) U64(hc_mix) U64(hc_in) U64(w) U64(h16) U64(h32) U64(gather) U64(out16) U64(out32) \
+  U64(embed) U64(tokens) U64(step) U64(sum_out) U32(W) U32(streams) U32(ld_h16) U32(ld_h32) U32(ld_out) \
+  U32(y_parts) U32(y_rows) F32(eps)
+
+/* out fp32 = x (fp32, or bf16 with f32 = 0) times w^T (bf16 rows), fp32 products and sums. */
+#define MF_PRODUCT_ARGS(U64, U32, F32) \
+  U64(x) U64(w) U64(out) U32(ld_x) U32(ld_w) U32(ld_out) U32(K) U32(N) U32(f32)
+
+#define MF_GATED_ARGS(U64, U32, F32) U64(in) U64(out) U32(ff) U32(ld_in) U32(ld_out)
+
+/* Adds `parts` fp32 slabs of part_rows rows; out32 receives every column, out16 the first c16 rounded to bf16. */
+#define MF_SUM_ARGS(U64, U32, F32) \
+  U64(in) U64(out32) U64(out16) U32(cols) U32(parts) U32(part_rows) U32(ld_in) U32(ld_32) U32(ld_16) U32(c16)
+
+/* Causal convolution per channel over a request's rows, then silu; tail fp32 [slot][taps - 1][channels] holds the
+ * inputs before the portion (read here, advanced by the scan tile). */
+#define MF_CONV_ARGS(U64, U32, F32) \
+  U64(x) U64(tail) U64(w) U64(bias) U64(out) U64(tok_pos) U32(ld_x) U32(ld_out) U32(channels) U32(taps) U32(f32)
+
+#define MF_SCAN_ARGS(U64, U32, F32) \
+  U64(x) U64(z) U64(dt) U64(dt_bias) U64(b) U64(c) U64(A) U64(D) U64(state) U64(tail) U64(x_in) U64(y) \
+  U64(tok_pos) U32(ld_x) U32(ld_z) U32(ld_dt) U32(ld_bc) U32(ld_y) U32(channels) U32(n) U32(taps) U32(f32)
+
+/* Log input and forget gates of the matrix memory: out fp32 [rows][2 heads]. */
+#define MF_MEM_GATE_ARGS(U64, U32, F32) \
+  U64(h) U64(wi) U64(wf) U64(bi) U64(bf) U64(out) U32(K) U32(heads) U32(ld_h) F32(cap)
+
+/* state fp32 [slot][head][e + 1][d] (column e: the normaliser), m fp32 [slot][head]; out fp32 [rows][heads][e + 1],
+ * its last column the denominator. */
+#define MF_MEMORY_ARGS(U64, U32, F32) \
+  U64(q) U64(k) U64(v) U64(gates) U64(state) U64(m) U64(out) U64(tok_pos) U32(ld_qkv) U32(heads) U32(d) U32(e) \
+  U32(f32) F32(q_scale)
+
+#define MF_HEAD_NORM_ARGS(U64, U32, F32) \
+  U64(o) U64(g) U64(w) U64(out) U32(heads) U32(e) U32(ld_g) U32(ld_out) U32(f32) F32(eps)
+
+/* qc fp32 [rows][heads * (d + r) | kv_rank | r]: queries, latent, shared rotated key part.  q_un [head][rows_max][ld_un]
+ * unrotated query parts; q_all [head][rows_max][ld_q] = kv_rank absorbed columns (written by a product) then r rotated
+ * ones; cache [page slots][ld_cache]. */
+#define MF_LATENT_ARGS(U64, U32, F32) \
+  U64(qc) U64(c_norm) U64(q_un) U64(q_all) U64(cache) U64(tok_pos) U64(tok_slot) U64(cos_sin) U32(ld_qc) U32(heads) \
+  U32(d) U32(r) U32(kv_rank) U32(ld_un) U32(ld_q) U32(rows_max) U32(ld_cache) U32(max_pos) U32(f32) F32(eps)
+
+/* ws_o fp32 [(row * heads + head) * parts + part][kv_rank], ws_ml float2 of the same rows. */
+#define MF_LATENT_ATTN_ARGS(U64, U32, F32) \
+  U64(q) U64(cache) U64(block_table) U64(out) U64(ws_o) U64(ws_ml) U64(tok_pos) U32(ld_q) U32(heads) U32(kv_rank) \
+  U32(r) U32(ld_cache) U32(page) U32(bt_stride) U32(rows_max) U32(ld_out) U32(f32) F32(scale)
+
 #define MF_FIELD_U64(name) unsigned long long name;
 #define MF_FIELD_U32(name) uint32_t name;
 #define MF_FIELD_F32(name) float name;
@@ -104,5 +160,16 @@ MF_DECLARE(SampleArgs, MF_SAMPLE_ARGS, 64)
 MF_DECLARE(AttnPlanArgs, MF_ATTN_PLAN_ARGS, 64)
 MF_DECLARE(LogitsArgs, MF_LOGITS_ARGS, 64)
 MF_DECLARE(CombineArgs, MF_COMBINE_ARGS, 128)
+MF_DECLARE(StreamArgs, MF_STREAM_ARGS, 192)
+MF_DECLARE(ProductArgs, MF_PRODUCT_ARGS, 64)
+MF_DECLARE(GatedArgs, MF_GATED_ARGS, 64)
+MF_DECLARE(SumArgs, MF_SUM_ARGS, 64)
+MF_DECLARE(ConvArgs, MF_CONV_ARGS, 128)
+MF_DECLARE(ScanArgs, MF_SCAN_ARGS, 192)
+MF_DECLARE(MemGateArgs, MF_MEM_GATE_ARGS, 64)
+MF_DECLARE(MemoryArgs, MF_MEMORY_ARGS, 128)
+MF_DECLARE(HeadNormArgs, MF_HEAD_NORM_ARGS, 64)
+MF_DECLARE(LatentArgs, MF_LATENT_ARGS, 128)
+MF_DECLARE(LatentAttnArgs, MF_LATENT_ATTN_ARGS, 128)
 
 }  // namespace mf

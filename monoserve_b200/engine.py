@@ -6,7 +6,7 @@ arrive, prompts are batched into a prefill pass under a token budget, a request 
 prompt is done joins the decode batch, the decode lane's program is rebuilt in the buffer
 that is not running and replaces the running one at an iteration boundary, KV pages are
 kept ahead of the sequences, and new tokens are collected from pinned rings.  This module
-is that loop for this library's lanes (`ModelLane`), without the reference's admission
+is that loop for this library's lanes (of every family in monoserve_b200/registry.py), without the reference's admission
 control: requests are admitted first come first served while slots, pages and the token
 budget allow, and the published plan is a fixed SM split (the plan search of
 monoserve_b200.control can supply another one).
@@ -27,6 +27,7 @@ import time
 import numpy as np
 import torch
 
+from monoserve_b200 import registry
 from monoserve_b200.fabric import Program, Tile
 from monoserve_b200.model import ModelLane
 
@@ -165,10 +166,11 @@ class Engine:
         self.max_decode, self.token_budget = max_decode, token_budget
         self.max_len = max_len or table.bt_stride * kv.page
         shared = dict(bt_stride=table.bt_stride, requests=table)
-        self.pre = ModelLane(fab, PREFILL, cfg, weights, kv, max_tokens=token_budget, max_slots=table.slots,
-                             logit_rows=table.slots, **shared)
-        self.dec = [ModelLane(fab, DECODE, cfg, weights, kv, max_tokens=max_decode, max_slots=table.slots,
-                              logit_rows=max_decode, **shared) for _ in range(2)]
+        lane_of = registry.lane_class(cfg, default=ModelLane)
+        self.pre = lane_of(fab, PREFILL, cfg, weights, kv, max_tokens=token_budget, max_slots=table.slots,
+                           logit_rows=table.slots, **shared)
+        self.dec = [lane_of(fab, DECODE, cfg, weights, kv, max_tokens=max_decode, max_slots=table.slots,
+                            logit_rows=max_decode, **shared) for _ in range(2)]
         for lane in [self.pre] + self.dec:
             lane.keep_base = len(lane._keep)   # operand blocks made at construction stay; those of a build go with its program
         n = fab.num_workers

@@ -1,0 +1,643 @@
+"""Layer-list decoders (the Sinotar design) as fabric lane programs: the mixer of every layer is named by the
+configuration (selective scan, latent attention, matrix memory), the residual is a set of hyper-connected streams, and
+a span of layers may run several times in a row.
+
+`LayerListLane` builds the chain of one batch on the fabric's tiles, one run of a layer after the other:
+
+  streams (53: update of the streams by the sublayer before, the next sublayer's input, its norm)
+    selective scan:    in GEMM (32) -> conv + silu (54) -> x GEMM (K ranges) -> slab sum (62) -> dt GEMM -> scan (55) -> o GEMM
+    matrix memory:     q k v g GEMM, gates (56) beside it -> memory (57) -> head norm (58) -> o GEMM
+    latent attention:  q + latent GEMM -> latent norm, rotation, cache append (59) -> per head W_uk^T q GEMM ->
+                       attention over the cached latents (60, 61) -> per head W_uv GEMM -> o GEMM
+  streams -> gate / up GEMM with the gelu epilogue -> down GEMM
+  ... -> final streams (gather) -> head GEMM (fp32) -> sample (43)
+
+Residual streams, norms, positions, gates, scores and recurrent state are 32-bit; GEMM operands are bf16.  With
+cfg.f32 set every activation is fp32 and every product runs in 32-bit arithmetic (tile 51): the exact form of the same
+programs, for checking.
+
+State: `LayerListCache` holds, per layer run, either pages of latents (addressed through the lane's block table) or
+slot-indexed recurrent state.  A request that starts at position 0 finds the state of its slot ignored (the tiles take
+it as zero), so slots and pages are handed on without clearing.
+"""
+import types
+
+import numpy as np
+import torch
+
+from monoserve_b200 import _C
+from monoserve_b200.checkpoint import checkpoint_files, safetensors_tensors
+from monoserve_b200.fabric import Program, Tile, tile_array
+from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_STORE, HEIGHTS, K_GEMM, K_SAMPLE, SPLIT_PARTS, SPLIT_ROWS,
+                                      LaneBase, _block, _bm, _retarget)
+
+K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEM_GATES, K_MEMORY = 51, 52, 53, 54, 55, 56, 57
+K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM = 58, 59, 60, 61, 62
+MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
+SCAN_CHANNELS, MEMORY_COLUMNS = 32, 32   # of one tile
+WIDE_ROWS, WIDE_PARTS = 512, 4           # K ranges of the products that end a sublayer, up to this many rows
+MAX_ATTN_PARTS = 32
+
+
+def up(n, m):
+    return -(-n // m) * m
+
+
+# ---------------------------------------------------------------------------------------------- configuration
+def read_config(c, dtype="bfloat16"):
+    """The model shape from a parsed config.json with a list of layers."""
+    if dtype not in ("bfloat16", "float32"):
+        raise ValueError(f"dtype {dtype}")
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        kind, m, mlp = e["type"], dict(e["mixer"]), e.get("mlp")
+        if kind not in MIXERS:
+            raise NotImplementedError(f"layer {i}: mixer {kind}")
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']}")
+        MIXERS[kind].check(i, m)
+        layers.append(types.SimpleNamespace(kind=kind, m=types.SimpleNamespace(**m), ff=mlp["ff"] if mlp else 0))
+    loop = c.get("loop")
+    order = list(range(len(layers)))
+    if loop:
+        a, b = loop["start"], loop["stop"]
+        order = order[:a] + order[a:b] * loop["times"] + order[b:]
+    streams = c["streams"]
+    if not 1 <= streams <= MAX_STREAMS:
+        raise NotImplementedError(f"{streams} residual streams (1 to {MAX_STREAMS})")
+    return types.SimpleNamespace(model_type="sinotar", hidden=c["width"], vocab=c["vocab"], eps=float(c["norm"]["eps"]),
+                                 streams=streams, layers=layers, order=order, num_layers=len(layers),
+                                 f32=dtype == "float32")
+
+
+def read_tensors(folder):
+    """{name: CPU tensor} of a checkpoint folder."""
+    return {name: t.clone() for path in checkpoint_files(folder) for name, t in safetensors_tensors(path)}
+
+
+class Weights:
+    """Device placement of one decoder's tensors ({name: tensor}, linear weights [out, in]): matrices in bf16 with rows
+    padded to whole 64-element K steps, everything that enters 32-bit arithmetic in fp32.  Products that read the same
+    input are stacked.  Layers that run several times are placed once."""
+
+    def __init__(self, cfg, tensors):
+        self.cfg = cfg
+        t = tensors
+        self.embed = t["embed"].to(torch.bfloat16).contiguous().cuda()
+        self.head = self.mat(t["head"])
+        self.final_norm = self.f32(1 + t["final.norm"].float())
+        self.ones = torch.ones(cfg.streams, device="cuda")
+        self.layers = []
+        for l, layer in enumerate(cfg.layers):
+            g = lambda name: t[f"l{l}.{name}"]  # noqa: B023, E731
+            w = types.SimpleNamespace(norm1=self.f32(1 + g("norm1").float()))
+            w.hc1 = [self.f32(g(f"hc1.{n}").float()) for n in ("in", "out", "mix")]
+            MIXERS[layer.kind].place(self, w, layer.m, lambda name: g("mix." + name))
+            if layer.ff:
+                w.norm2 = self.f32(1 + g("norm2").float())
+                w.hc2 = [self.f32(g(f"hc2.{n}").float()) for n in ("in", "out", "mix")]
+                w.gate_up = self.mat(torch.cat([g("mlp.gate"), g("mlp.up")]))
+                w.down = self.mat(g("mlp.down"))
+            self.layers.append(w)
+
+    @staticmethod
+    def f32(t):
+        return t.float().contiguous().cuda()
+
+    @staticmethod
+    def mat(t):
+        """bf16 [.., out, in padded to 64]."""
+        k = t.shape[-1]
+        return torch.nn.functional.pad(t.to(torch.bfloat16), (0, up(k, 64) - k)).contiguous().cuda()
+
+
+class LayerListCache:
+    """Cache and state of every layer run, shared by the lanes: `page` tokens per page of latents (page 0 is the sink
+    unused block-table entries point at), `slots` requests' recurrent state."""
+
+    def __init__(self, cfg, n_pages, page_size=16, slots=8):
+        self.n_pages, self.page, self.slots = n_pages, page_size, slots
+        self.runs = [MIXERS[cfg.layers[l].kind].state(cfg, cfg.layers[l].m, n_pages * page_size, slots) for l in cfg.order]
+
+
+# ---------------------------------------------------------------------------------------------- mixers
+class SelectiveScan:
+    """x, z = W_in h; x through a causal convolution per channel and silu; dt, B, C from x;
+    S <- exp(dt A) S + dt x B, y = S C + D x, y silu(z), W_o."""
+
+    @staticmethod
+    def check(i, m):
+        if m["state"] > MAX_SCAN_STATE or not 1 <= m["conv"] <= MAX_TAPS:
+            raise NotImplementedError(f"layer {i}: state {m['state']} (to {MAX_SCAN_STATE}), {m['conv']} taps (to {MAX_TAPS})")
+
+    @staticmethod
+    def place(W, w, m, g):
+        w.in_, w.x, w.dt, w.o = W.mat(g("in")), W.mat(g("x")), W.mat(g("dt")), W.mat(g("o"))
+        w.conv, w.conv_b, w.dt_b, w.D = W.f32(g("conv")), W.f32(g("conv.b")), W.f32(g("dt.b")), W.f32(g("D"))
+        w.A = W.f32(-torch.exp(g("A_log").float()))
+
+    @staticmethod
+    def state(cfg, m, rows, slots):
+        return dict(state=torch.zeros(slots, m.inner, m.state, device="cuda"),
+                    tail=torch.zeros(slots, max(1, m.conv - 1), m.inner, device="cuda"))
+
+    @staticmethod
+    def sizes(m):
+        return dict(proj=2 * m.inner, act=m.inner, mix=m.inner, small=m.dt_rank + 2 * m.state, dt=m.inner, dt_in=m.dt_rank)
+
+    @staticmethod
+    def build(lane, p, l, run, b, prev):
+        m, w, st, T = lane.cfg.layers[l].m, lane.w.layers[l], lane.kv.runs[run], b.T
+        f32, R = int(lane.cfg.f32), m.dt_rank + 2 * m.state
+        s = lane.product(p, prev, lane.h, w.in_, lane.proj, T, 2 * m.inner, lane.cfg.hidden, ("scan_in", run), out16=True)
+        conv = lane._dev("ConvArgs", x=lane.proj.addr, tail=st["tail"], w=w.conv, bias=w.conv_b, out=lane.act.addr,
+                         tok_pos=lane.tok_pos, ld_x=lane.proj.ld, ld_out=lane.act.ld, channels=m.inner, taps=m.conv, f32=f32)
+        s_conv = p.stage(_retarget(b.conv_tiles(m.inner), a0=conv.data_ptr()), label=("conv", run))
+        p.after(s, s_conv)
+        if f32:
+            s_x = lane.product(p, s_conv, lane.act, w.x, lane.small, T, R, m.inner, ("scan_x", run))
+            dt_in = lane.small
+        else:
+            parts = lane.split_parts(T, m.inner)
+            s_x = lane.product(p, s_conv, lane.act, w.x, lane.slabs, T, R, m.inner, ("scan_x", run), parts=parts, ld_out=R)
+            sm = lane._dev("SumArgs", out32=lane.small.addr, out16=lane.dt_in.addr, cols=R, parts=parts,
+                           part_rows=lane.slab_rows(T), ld_in=R, ld_32=lane.small.ld, ld_16=lane.dt_in.ld, c16=m.dt_rank,
+                           **{"in": lane.slabs.addr})
+            s_sum = p.stage(lane._rows(K_SUM, sm, T, lane._per(T)), label=("scan_sum", run))
+            p.after(s_x, s_sum)
+            s_x, dt_in = s_sum, lane.dt_in
+        s_dt = lane.product(p, s_x, dt_in, w.dt, lane.dt, T, m.inner, m.dt_rank, ("scan_dt", run))
+        es = lane.proj.es
+        sc = lane._dev("ScanArgs", x=lane.act.addr, z=lane.proj.addr + m.inner * es, dt=lane.dt.addr, dt_bias=w.dt_b,
+                       b=lane.small.addr + 4 * m.dt_rank, c=lane.small.addr + 4 * (m.dt_rank + m.state), A=w.A, D=w.D,
+                       state=st["state"], tail=st["tail"], x_in=lane.proj.addr, y=lane.mix.addr, tok_pos=lane.tok_pos,
+                       ld_x=lane.act.ld, ld_z=lane.proj.ld, ld_dt=lane.dt.ld, ld_bc=lane.small.ld, ld_y=lane.mix.ld,
+                       channels=m.inner, n=m.state, taps=m.conv, f32=f32)
+        s_sc = p.stage(_retarget(b.scan_tiles(m.inner), a0=sc.data_ptr()), label=("scan", run))
+        p.after(s_dt, s_sc)
+        return lane.closing(p, s_sc, lane.mix, w.o, T, m.inner, ("scan_o", run))
+
+
+class MatrixMemory:
+    """q, k, v, g from h; log gates i = cap tanh((W_i h + b) / cap), f = logsigmoid(cap tanh(..)); per head
+    S <- e^(f + m' - m) S + e^(i - m) k v^T with the running maximum m, read by q over max(|n q|, e^-m); head norm, gate."""
+
+    @staticmethod
+    def check(i, m):
+        if m["dim"] > MAX_MEMORY_DIM:
+            raise NotImplementedError(f"layer {i}: memory of {m['dim']} key dimensions (to {MAX_MEMORY_DIM})")
+
+    @staticmethod
+    def place(W, w, m, g):
+        w.qkvg, w.o = W.mat(torch.cat([g(n) for n in "qkvg"])), W.mat(g("o"))
+        w.wi, w.wf = (g(n).to(torch.bfloat16).contiguous().cuda() for n in "if")
+        w.bi, w.bf, w.norm = W.f32(g("i.b")), W.f32(g("f.b")), W.f32(g("norm"))
+
+    @staticmethod
+    def state(cfg, m, rows, slots):
+        return dict(S=torch.zeros(slots, m.heads, m.vdim + 1, up(m.dim, 4), device="cuda"),
+                    m=torch.zeros(slots, m.heads, up(m.vdim + 1, MEMORY_COLUMNS) // MEMORY_COLUMNS, device="cuda"))
+
+    @staticmethod
+    def sizes(m):
+        return dict(proj=2 * m.heads * (m.dim + m.vdim), mix=m.heads * m.vdim, small=2 * m.heads, raw=m.heads * (m.vdim + 1),
+                    h32=1)
+
+    @staticmethod
+    def build(lane, p, l, run, b, prev):
+        m, w, st, T = lane.cfg.layers[l].m, lane.w.layers[l], lane.kv.runs[run], b.T
+        f32, H, d, e, es = int(lane.cfg.f32), m.heads, m.dim, m.vdim, lane.proj.es
+        s = lane.product(p, prev, lane.h, w.qkvg, lane.proj, T, 2 * H * (d + e), lane.cfg.hidden, ("memory_in", run), out16=True)
+        gates = lane._dev("MemGateArgs", h=lane.h32.addr, wi=w.wi, wf=w.wf, bi=w.bi, bf=w.bf, out=lane.small.addr,
+                          K=lane.cfg.hidden, heads=H, ld_h=lane.h32.ld, cap=m.gate_cap)
+        s_g = p.stage(_retarget(b.gate_tiles(2 * H), a0=gates.data_ptr()), label=("memory_gates", run))
+        p.after(prev, s_g)
+        at = lane.proj.addr
+        mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=lane.small.addr, state=st["S"],
+                        m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos, ld_qkv=lane.proj.ld, heads=H, d=d, e=e, f32=f32,
+                        q_scale=d ** -0.5)
+        s_m = p.stage(_retarget(b.memory_tiles(H, e), a0=mem.data_ptr()), label=("memory", run))
+        p.after(s, s_m)
+        p.after(s_g, s_m)
+        nrm = lane._dev("HeadNormArgs", o=lane.raw.addr, g=at + es * H * (2 * d + e), w=w.norm, out=lane.mix.addr, heads=H,
+                        e=e, ld_g=lane.proj.ld, ld_out=lane.mix.ld, f32=f32, eps=lane.cfg.eps)
+        s_n = p.stage(lane._rows(K_HEAD_NORM, nrm, T * H, lane.items_per(T * H)), label=("head_norm", run))
+        p.after(s_m, s_n)
+        return lane.closing(p, s_n, lane.mix, w.o, T, H * e, ("memory_o", run))
+
+
+class LatentAttention:
+    """Causal attention whose keys and values are linear maps of a cached latent (plus one rotated key part shared by
+    the heads), in the absorbed form: W_uk^T q meets the latents themselves, W_uv maps their weighted sum."""
+
+    @staticmethod
+    def check(i, m):
+        if m["kv_rank"] + m["rot_dim"] > MAX_LATENT_DIM:
+            raise NotImplementedError(f"layer {i}: latent of {m['kv_rank']} + {m['rot_dim']} columns (to {MAX_LATENT_DIM})")
+        if m["rot"]["dims"] != m["rot_dim"] or m["rot_dim"] % 2:
+            raise NotImplementedError(f"layer {i}: rotation of {m['rot']['dims']} of {m['rot_dim']} columns")
+
+    @staticmethod
+    def place(W, w, m, g):
+        w.qkv, w.o, w.c_norm = W.mat(torch.cat([g("q"), g("dkv")])), W.mat(g("o")), W.f32(g("dkv.norm"))
+        w.uk = W.mat(g("uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2))    # [head][latent][dim]
+        w.uv = W.mat(g("uv").view(m.heads, m.vdim, m.kv_rank))                   # [head][value][latent]
+
+    @staticmethod
+    def state(cfg, m, rows, slots):
+        return dict(cache=torch.zeros(rows, up(m.kv_rank + m.rot_dim, 8), device="cuda",
+                                      dtype=torch.float32 if cfg.f32 else torch.bfloat16))
+
+    @staticmethod
+    def sizes(m):
+        return dict(qc=m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim, mix=m.heads * m.vdim,
+                    q_un=(m.heads, m.dim), q_all=(m.heads, m.kv_rank + m.rot_dim), o_lat=(m.heads, m.kv_rank),
+                    ws=(m.heads, m.kv_rank))
+
+    @staticmethod
+    def build(lane, p, l, run, b, prev):
+        m, w, st, T = lane.cfg.layers[l].m, lane.w.layers[l], lane.kv.runs[run], b.T
+        f32, H, d, r, c = int(lane.cfg.f32), m.heads, m.dim, m.rot_dim, m.kv_rank
+        s = lane.product(p, prev, lane.h, w.qkv, lane.qc, T, H * (d + r) + c + r, lane.cfg.hidden, ("latent_in", run))
+        ld_q, ld_o = up(c + r, 8), up(c, 64)
+        kv = lane._dev("LatentArgs", qc=lane.qc.addr, c_norm=w.c_norm, q_un=lane.q_un.addr, q_all=lane.q_all.addr,
+                       cache=st["cache"], tok_pos=lane.tok_pos, tok_slot=lane.tok_slot, cos_sin=lane.cos_sin(m.rot["base"], r),
+                       ld_qc=lane.qc.ld, heads=H, d=d, r=r, kv_rank=c, ld_un=up(d, 64), ld_q=ld_q, rows_max=lane.T,
+                       ld_cache=st["cache"].shape[1], max_pos=lane.max_pos, f32=f32, eps=lane.cfg.eps)
+        s_kv = p.stage(lane._rows(K_LATENT_KV, kv, T * (H + 1), lane.items_per(T * (H + 1))), label=("latent_kv", run))
+        p.after(s, s_kv)
+        s_q = lane.head_product(p, s_kv, lane.q_un.addr, up(d, 64), w.uk, lane.q_all.addr, ld_q, lane.T * ld_q, T, c, d,
+                                ("latent_q", run))
+        parts = lane.attn_parts(T, H, c)
+        at = lane._dev("LatentAttnArgs", q=lane.q_all.addr, cache=st["cache"], block_table=lane.bt, out=lane.o_lat.addr,
+                       ws_o=lane.ws.data_ptr(), ws_ml=lane.ws_ml.data_ptr(), tok_pos=lane.tok_pos, ld_q=ld_q, heads=H,
+                       kv_rank=c, r=r, ld_cache=st["cache"].shape[1], page=lane.kv.page, bt_stride=lane.bt_stride,
+                       rows_max=lane.T, ld_out=ld_o, f32=f32, scale=m.scale)
+        s_at = p.stage(_retarget(b.attn_tiles(H, parts), a0=at.data_ptr()), label=("latent_attn", run))
+        p.after(s_q, s_at)
+        if parts > 1:
+            tiles = lane._rows(K_LATENT_MERGE, at, T * H, lane.items_per(T * H))
+            tiles[:, 2] = parts
+            s_mg = p.stage(tiles, label=("latent_merge", run))
+            p.after(s_at, s_mg)
+            s_at = s_mg
+        s_v = lane.head_product(p, s_at, lane.o_lat.addr, ld_o, w.uv, lane.mix.addr, lane.mix.ld, m.vdim, T, m.vdim, c,
+                                ("latent_v", run))
+        return lane.closing(p, s_v, lane.mix, w.o, T, H * m.vdim, ("latent_o", run))
+
+
+MIXERS = {"mamba1": SelectiveScan, "mlstm": MatrixMemory, "latent_attention": LatentAttention}
+
+
+# ---------------------------------------------------------------------------------------------- the lane
+class _Buf:
+    """An activation buffer [rows][ld] and its tensor maps (bf16 operands of a GEMM)."""
+
+    def __init__(self, lane, rows, cols, dtype, maps=False):
+        self.ld = up(cols, 64)
+        self.t = torch.zeros(rows, self.ld, dtype=dtype, device="cuda")
+        self.addr, self.es = self.t.data_ptr(), self.t.element_size()
+        self.lane, self.rows, self._maps = lane, rows, {}
+
+    def data_ptr(self):
+        return self.addr
+
+    def maps(self, k):
+        """Maps of the first k columns (zero beyond them)."""
+        if k not in self._maps:
+            self._maps[k] = [self.lane.fab.tensor_map(self.addr, [k, self.rows], [self.ld * 2], [64, bm]) for bm in HEIGHTS]
+        return self._maps[k]
+
+
+class _Batch:
+    """The rows of one program: requests [(first row, rows, slot)], and the tile lists that depend on them only (made
+    once per program and re-addressed per layer)."""
+
+    def __init__(self, lane, requests):
+        self.lane, self.requests = lane, requests
+        self.T = sum(n for _, n, _ in requests)
+        self._made = {}
+
+    def _once(self, key, make):
+        if key not in self._made:
+            self._made[key] = make()
+        return self._made[key]
+
+    def conv_tiles(self, channels):
+        rows_per, ch_per = 64, 256
+
+        def make():
+            out = []
+            for row0, n, slot in self.requests:
+                r, c = np.meshgrid(np.arange(0, n, rows_per), np.arange(0, channels, ch_per), indexing="ij")
+                out.append(tile_array(K_CONV, i0=row0, i1=row0 + r,
+                                      i2=np.minimum(rows_per, n - r) | (np.minimum(ch_per, channels - c) << 16), i3=slot, a1=c))
+            return np.concatenate(out)
+        return self._once(("conv", channels), make)
+
+    def scan_tiles(self, channels):
+        return self._once(("scan", channels), lambda: np.concatenate(
+            [tile_array(K_SCAN, i0=row0, i1=n, i2=np.arange(0, channels, SCAN_CHANNELS), i3=slot)
+             for row0, n, slot in sorted(self.requests, key=lambda q: -q[1])]))
+
+    def memory_tiles(self, heads, e):
+        def make():
+            blocks = -(-(e + 1) // MEMORY_COLUMNS)
+            h, c = np.meshgrid(np.arange(heads), np.arange(blocks), indexing="ij")
+            return np.concatenate([tile_array(K_MEMORY, i0=row0, i1=n, i2=h | (c << 16), i3=slot)
+                                   for row0, n, slot in sorted(self.requests, key=lambda q: -q[1])])
+        return self._once(("memory", heads, e), make)
+
+    def gate_tiles(self, outputs):
+        per_out, per_row = (4, 8) if self.T <= SPLIT_ROWS else (outputs, 16)
+
+        def make():
+            r, o = np.meshgrid(np.arange(0, self.T, per_row), np.arange(0, outputs, per_out), indexing="ij")
+            return tile_array(K_MEM_GATES, i0=r, i1=np.minimum(per_row, self.T - r), i2=o, i3=np.minimum(per_out, outputs - o))
+        return self._once(("gates", outputs), make)
+
+    def attn_tiles(self, heads, parts):
+        """One tile per row, group of heads and part, the rows that see most keys first."""
+        per = 4 if parts > 1 or self.T * -(-heads // 4) <= 4 * self.lane.fab.num_workers else heads
+
+        def make():
+            rows = np.concatenate([np.arange(row0 + n - 1, row0 - 1, -1) for row0, n, _ in self.requests])
+            slots = np.concatenate([np.full(n, slot) for _, n, slot in self.requests])
+            h = np.arange(0, heads, per)
+            return tile_array(K_LATENT_ATTN, i0=rows[:, None, None], i1=(h | (np.minimum(per, heads - h) << 16))[None, :, None],
+                              i2=np.arange(parts)[None, None, :], i3=parts, a1=slots[:, None, None])
+        return self._once(("attn", heads, parts), make)
+
+
+class LayerListLane(LaneBase):
+    """One lane of the fabric running a layer-list decoder; the interface of ModelLane."""
+
+    def __init__(self, fab, lane_id, cfg, weights, kv, max_tokens, max_slots, bt_stride, logit_rows=None, requests=None,
+                 keep_residual=False):
+        """keep_residual: every program also stores the sum of the streams after each layer run (`residual`)."""
+        self.fab, self.lane_id, self.cfg, self.w, self.kv = fab, lane_id, cfg, weights, kv
+        assert max_slots <= kv.slots, "the cache holds recurrent state for fewer slots"
+        self.T, self.S, self.bt_stride = max_tokens, max_slots, bt_stride
+        self.logit_rows = logit_rows or max(max_tokens, max_slots)
+        T, H = max_tokens, cfg.hidden
+        act, f32 = torch.float32 if cfg.f32 else torch.bfloat16, torch.float32
+        z = lambda *shape, dt=torch.float32: torch.zeros(*shape, dtype=dt, device="cuda")  # noqa: E731
+        sizes = {}
+        for layer in cfg.layers:
+            for name, v in MIXERS[layer.kind].sizes(layer.m).items():
+                if isinstance(v, tuple):   # per head: the largest block of heads x padded columns
+                    sizes[name] = max(sizes.get(name, 0), v[0] * up(v[1], 64))
+                else:
+                    sizes[name] = max(sizes.get(name, 0), v)
+        self.xs = z(T, cfg.streams, H)
+        self.h = _Buf(self, T, H, act)
+        self.h32 = self.h if cfg.f32 else (_Buf(self, T, H, f32) if "h32" in sizes else None)
+        ff = max([layer.ff for layer in cfg.layers] + [0])
+        self.hd = _Buf(self, T, ff, act) if ff else None
+        self.gu = _Buf(self, T, 2 * ff, f32) if ff and cfg.f32 else None
+        for name, dt in (("proj", act), ("act", act), ("mix", act), ("dt_in", act), ("small", f32), ("dt", f32), ("qc", f32),
+                         ("raw", f32)):
+            setattr(self, name, _Buf(self, T, sizes[name], dt) if name in sizes else None)
+        for name in ("q_un", "q_all", "o_lat"):   # [head][T][columns]: addressed by the layer's own strides
+            if name in sizes:
+                buf = types.SimpleNamespace(t=z(T * sizes[name], dt=act))
+                buf.addr = buf.t.data_ptr()
+                setattr(self, name, buf)
+        # fp32 slabs of the K-split products: y of a sublayer, and the scan's x projection
+        self.rows_slab = max(SPLIT_PARTS * SPLIT_ROWS, WIDE_PARTS * min(WIDE_ROWS, up(T, 64)), T)
+        self.y = types.SimpleNamespace(t=z(self.rows_slab, H))
+        self.y.addr = self.y.t.data_ptr()
+        if "small" in sizes:
+            self.slabs = types.SimpleNamespace(t=z(self.rows_slab * sizes["small"]))
+            self.slabs.addr = self.slabs.t.data_ptr()
+        if "ws" in sizes:
+            self.ws_rows = max(min(T, SPLIT_ROWS), 1) * MAX_ATTN_PARTS * max(x.m.heads for x in cfg.layers if x.kind == "latent_attention")
+            self.ws, self.ws_ml = z(self.ws_rows * max(x.m.kv_rank for x in cfg.layers if x.kind == "latent_attention")), z(self.ws_rows, 2)
+        self.xlast, self.logits = _Buf(self, self.logit_rows, H, act), z(self.logit_rows, cfg.vocab)
+        self.residual = z(len(cfg.order), T, H) if keep_residual else None
+        self._request_state(T, self.S, requests)
+        self.max_pos = bt_stride * kv.page
+        self._cos_sin, self._wmaps, self._hmaps = {}, {}, {}
+        for layer in cfg.layers:
+            if layer.kind == "latent_attention":
+                self.cos_sin(layer.m.rot["base"], layer.m.rot_dim)
+        self._build_state((48 << 10) * (len(cfg.order) + 2))
+        self.sample_args, self.step_args = self._sample_block(cfg.vocab), self._step_block()
+        self._prepare()
+
+    def _prepare(self):
+        """Make every tensor map a program can name now: none may be made while the fabric is resident."""
+        if self.cfg.f32:
+            return
+        cfg, w = self.cfg, self.w
+        wm = self.weight_map
+        wm(w.head)
+        self.h.maps(cfg.hidden)
+        self.xlast.maps(cfg.hidden)
+        for layer, lw in zip(cfg.layers, w.layers):
+            m = layer.m
+            if layer.ff:
+                wm(lw.gate_up), wm(lw.down), self.hd.maps(layer.ff)
+            wm(lw.o)
+            if layer.kind == "mamba1":
+                wm(lw.in_), wm(lw.x), wm(lw.dt), self.act.maps(m.inner), self.dt_in.maps(m.dt_rank), self.mix.maps(m.inner)
+            elif layer.kind == "mlstm":
+                wm(lw.qkvg), self.mix.maps(m.heads * m.vdim)
+            else:
+                wm(lw.qkv), wm(lw.uk), wm(lw.uv), self.mix.maps(m.heads * m.vdim)
+                self.head_maps(self.q_un.addr, up(m.dim, 64), m.dim, m.heads)
+                self.head_maps(self.o_lat.addr, up(m.kv_rank, 64), m.kv_rank, m.heads)
+
+    def cos_sin(self, base, r):
+        """fp32 [max_pos][r / 2][cos, sin] of the angles pos * base^(-2 i / r)."""
+        if (base, r) not in self._cos_sin:
+            f = float(base) ** (-2.0 * torch.arange(r // 2, dtype=torch.float64) / r)
+            a = torch.arange(self.max_pos, dtype=torch.float64)[:, None] * f[None]
+            self._cos_sin[base, r] = torch.stack([a.cos(), a.sin()], -1).float().contiguous().cuda()
+        return self._cos_sin[base, r]
+
+    # ------------------------------------------------------------------ products
+    def weight_map(self, t):
+        if t.data_ptr() not in self._wmaps:
+            self._wmaps[t.data_ptr()] = self._wmap(t)
+        return self._wmaps[t.data_ptr()]
+
+    def head_maps(self, addr, ld, k, heads):
+        """Maps of the first k columns of a [head * T][ld] operand (zero beyond them)."""
+        key = addr, ld, k, heads
+        if key not in self._hmaps:
+            self._hmaps[key] = [self.fab.tensor_map(addr, [k, heads * self.T], [ld * 2], [64, bm]) for bm in HEIGHTS]
+        return self._hmaps[key]
+
+    def split_parts(self, rows, k):
+        """K ranges of a product that ends in fp32 slabs."""
+        if rows > min(WIDE_ROWS, up(self.T, 64)):
+            return 1
+        return max(1, min(SPLIT_PARTS if rows <= SPLIT_ROWS else WIDE_PARTS, -(-k // 64) // 8))
+
+    def slab_rows(self, rows):
+        return SPLIT_ROWS if rows <= SPLIT_ROWS else min(WIDE_ROWS, up(self.T, 64)) if rows <= WIDE_ROWS else self.T
+
+    def product(self, p, prev, x, w, out, rows, n, k, label, out16=False, parts=1, ld_out=None, epi=None, up_offset=0):
+        """A stage out[rows][n] = x[rows][k] w[n][k]^T after `prev`.  out16: the output is of the activations' type,
+        else fp32; parts > 1: that many fp32 slabs."""
+        ld = ld_out or out.ld
+        if self.cfg.f32:
+            args = self._dev("ProductArgs", x=x.addr, w=w, out=out.addr, ld_x=x.ld, ld_w=w.shape[-1], ld_out=ld, K=k, N=n, f32=1)
+            s = p.stage(_retarget(self._product_tiles(rows, n), a0=args.data_ptr()), label=label)
+        elif parts > 1:
+            s = self._gemm_split(p, self.weight_map(w), x.maps(k), rows, n, k, out.t, parts, label,
+                                 slab_rows=self.slab_rows(rows))
+        else:
+            s = self._gemm(p, self.weight_map(w), x.maps(k), rows, n, k, out.t, ld,
+                           epi if epi is not None else (EPI_STORE if out16 else EPI_F32), label, up_offset=up_offset)
+        p.after(prev, s)
+        return s
+
+    def _product_tiles(self, rows, n):
+        key = ("product", rows, n)
+        if key not in self._templates:
+            r, c = np.meshgrid(np.arange(0, rows, 32), np.arange(0, n, 32), indexing="ij")
+            self._templates[key] = tile_array(K_PRODUCT, i0=r, i1=np.minimum(32, rows - r), i2=c, i3=np.minimum(32, n - c))
+        return self._templates[key]
+
+    def head_product(self, p, prev, x_addr, ld_x, w, out_addr, ld_out, head_stride, rows, n, k, label):
+        """Per head h: out[.. + h * head_stride][rows][n] = x[h * T ..][k] w[h][n][k]^T, activations' type out."""
+        heads = w.shape[0]
+        if self.cfg.f32:
+            # tile 51 stores fp32, which is the activations' type here
+            args = self._dev("ProductArgs", x=x_addr, w=w, out=out_addr, ld_x=ld_x, ld_w=w.shape[-1], ld_out=ld_out, K=k, N=n, f32=1)
+            base = self._product_tiles(rows, n)
+            tiles = np.tile(base, (heads, 1))
+            h = np.repeat(np.arange(heads, dtype=np.uint64), len(base))
+            tiles[:, 3] = args.data_ptr()
+            tiles[:, 4] = h * np.uint64(4 * self.T * ld_x)
+            tiles[:, 5] = h * np.uint64(2 * w.shape[1] * w.shape[2])
+            tiles[:, 6] = h * np.uint64(4 * head_stride)
+            s = p.stage(tiles, label=label)
+        else:
+            bm = _bm(rows)
+            # the tile's activation rows are h * T + m and its output row is counted from there: the base makes up for it
+            args = [self.arena.put(_C.gemm_args(out=(out_addr + 2 * (h * head_stride - h * self.T * ld_out)) % (1 << 64),
+                                                ld_out=ld_out, k_tiles=-(-k // 64), epi=EPI_STORE, bm=bm, n_limit=n)).data_ptr()
+                    for h in range(heads)]
+            h, m0, n0 = np.meshgrid(np.arange(heads), np.arange(0, rows, bm), np.arange(0, n, 128), indexing="ij")
+            tiles = tile_array(K_GEMM, i0=n0, i1=h * self.T + m0, i2=np.minimum(bm, rows - m0), i3=h,
+                               a0=np.asarray(args, dtype=np.int64)[h], a1=self.weight_map(w),
+                               a2=self.head_maps(x_addr, ld_x, k, heads)[HEIGHTS.index(bm)])
+            s = p.stage(tiles, label=label)
+        p.after(prev, s)
+        return s
+
+    def closing(self, p, prev, x, w, rows, k, label):
+        """The product that ends a sublayer: y as fp32 slabs for the streams tile."""
+        parts = 1 if self.cfg.f32 else self.split_parts(rows, k)
+        s = self.product(p, prev, x, w, self.y, rows, self.cfg.hidden, k, label, parts=parts, ld_out=self.cfg.hidden)
+        return s, parts, self.slab_rows(rows) if parts > 1 else 0
+
+    def items_per(self, items):
+        """Items (one warp each) per tile of an item-wise stage: a multiple of four, about two rounds of tiles."""
+        return max(4, up(-(-items // (2 * self.fab.num_workers)), 4))
+
+    def attn_parts(self, rows, heads, kv_rank):
+        """Key ranges per row: enough tiles to give every worker about two."""
+        tiles = rows * -(-heads // 4)
+        want = min(MAX_ATTN_PARTS, 2 * self.fab.num_workers // tiles)
+        return max(1, min(want, self.ws_rows // (rows * heads)))
+
+    # ------------------------------------------------------------------ programs
+    def _streams(self, p, rows, prev, sub, before, label, h32=False, gather=False, step=False):
+        """The streams stage in front of sublayer `sub` = (hc_in, norm): `before` = ((hc_out, hc_mix), parts, slab rows,
+        run whose residual this completes or None) of the sublayer behind it, or None at the embedding."""
+        cfg = self.cfg
+        hc_in, norm = sub
+        f = dict(xs=self.xs, hc_in=hc_in, w=norm, W=cfg.hidden, streams=cfg.streams, eps=cfg.eps)
+        if before is None:
+            f.update(embed=self.w.embed, **({"step": self.step_args} if step else {"tokens": self.tokens}))
+        else:
+            (hc_out, hc_mix), parts, slab_rows, run = before
+            f.update(y=self.y.addr, hc_out=hc_out, hc_mix=hc_mix, y_parts=parts, y_rows=slab_rows)
+            if run is not None and self.residual is not None:
+                f.update(sum_out=self.residual[run])
+        if gather:
+            f.update(gather=self.gather, ld_out=self.xlast.ld, **{"out32" if cfg.f32 else "out16": self.xlast.addr})
+        else:
+            if cfg.f32:
+                f.update(h32=self.h.addr, ld_h32=self.h.ld)
+            else:
+                f.update(h16=self.h.addr, ld_h16=self.h.ld)
+                if h32:
+                    f.update(h32=self.h32.addr, ld_h32=self.h32.ld)
+        args = self._dev("StreamArgs", **f)
+        s = p.stage(self._rows(K_STREAMS, args, rows, self._per(rows)), label=label)
+        if prev is not None:
+            p.after(prev, s)
+        return s
+
+    def _chain(self, p, b, step):
+        """Every layer run; returns (first stage, final streams stage)."""
+        cfg, T = self.cfg, b.T
+        first = prev = None
+        before = None
+        for run, l in enumerate(cfg.order):
+            layer, w = cfg.layers[l], self.w.layers[l]
+            prev = self._streams(p, T, prev, (w.hc1[0], w.norm1), before, ("streams", run), h32=layer.kind == "mlstm", step=step)
+            first = prev if first is None else first
+            prev, parts, slab = MIXERS[layer.kind].build(self, p, l, run, b, prev)
+            before = (w.hc1[1:], parts, slab, None if layer.ff else run)
+            if layer.ff:
+                prev = self._streams(p, T, prev, (w.hc2[0], w.norm2), before, ("streams_ff", run))
+                if cfg.f32:
+                    s = self.product(p, prev, self.h, w.gate_up, self.gu, T, 2 * layer.ff, cfg.hidden, ("ff_in", run))
+                    g = self._dev("GatedArgs", out=self.hd.addr, ff=layer.ff, ld_in=self.gu.ld, ld_out=self.hd.ld,
+                                  **{"in": self.gu.addr})
+                    s_g = p.stage(self._rows(K_GATED, g, T, self._per(T)), label=("ff_act", run))
+                    p.after(s, s_g)
+                    s = s_g
+                else:
+                    s = self.product(p, prev, self.h, w.gate_up, self.hd, T, layer.ff, cfg.hidden, ("ff_in", run),
+                                     epi=EPI_GELU_MUL, up_offset=layer.ff)
+                prev, parts, slab = self.closing(p, s, self.hd, w.down, T, layer.ff, ("ff_out", run))
+                before = (w.hc2[1:], parts, slab, run)
+        last = self._streams(p, T, prev, (self.w.ones, self.w.final_norm), before, ("final", len(cfg.order)), gather=True)
+        return first, last
+
+    def _finish(self, p, prev, n_rows, sample_rows):
+        if n_rows:
+            s = self.product(p, prev, self.xlast, self.w.head, types.SimpleNamespace(t=self.logits, addr=self.logits.data_ptr(),
+                                                                                     ld=self.cfg.vocab),
+                             n_rows, self.cfg.vocab, self.cfg.hidden, ("head", -1))
+            tiles = [Tile(K_SAMPLE, i=(row, slot), a=(self.sample_args.data_ptr(),)) for row, slot in sample_rows if row >= 0]
+            if tiles:
+                s_s = p.stage(tiles, label=("sample", -1))
+                p.after(s, s_s)
+        self.rows_out = n_rows
+        self.labels = p.labels()
+        self.arena.flush()
+
+    def build_prefill(self, batch, iterations=1, all_logits=False, want=None):
+        """batch: [(slot, tokens, pos0)], a prompt or a portion of one each, pages in place.  Computes the rows, advances
+        the requests' caches and states, and samples one next token per request, as ModelLane.build_prefill does.
+        want: per request, the places among its tokens whose logits are kept instead (row by row in `logits`); then
+        nothing is sampled."""
+        self._reset_build()
+        places = want if want is not None else [[len(toks) - 1] for _, toks, _ in batch]
+        T, req_info, sample_rows = self._batch_rows(batch, places, all_logits)
+        p = Program()
+        b = _Batch(self, [(row0, n, slot) for (row0, _, n, _), (slot, _, _) in zip(req_info, batch)])
+        first, last = self._chain(p, b, step=False)
+        self._finish(p, last, T if all_logits else sum(len(v) for v in places), sample_rows if want is None else [])
+        return p.upload(self.fab, first=first, iterations=iterations)
+
+    def build_decode(self, slots, iterations=1, chunk_keys=0):
+        """One decode step per iteration for the requests in `slots` (row r = slots[r])."""
+        R = len(slots)
+        assert 0 < R <= min(self.T, self.logit_rows)
+        self._reset_build()
+        self._put(self.row_req, slots)
+        self._put(self.gather, np.arange(R))
+        p = Program()
+        b = _Batch(self, [(r, 1, slot) for r, slot in enumerate(slots)])
+        first, last = self._chain(p, b, step=True)
+        self._finish(p, last, R, list(enumerate(slots)))
+        return p.upload(self.fab, first=first, iterations=iterations)

@@ -20,110 +20,21 @@ import torch
 
 from monoserve_b200 import _C
 from monoserve_b200.attention import SCALE_LOG2, fabric_maps, fabric_tiles, plan_items
-from monoserve_b200.fabric import Program, Tile, tile_array
+from monoserve_b200.fabric import Program, Tile
 from monoserve_b200.fabric.args import pack
 from monoserve_b200.lane import SUB, logits_tiles
+from monoserve_b200.lane_base import (EPI_F32, EPI_ROWS_F32, EPI_SILU_MUL, EPI_STORE, HEIGHTS, K_SAMPLE, SPLIT_PARTS,  # noqa: F401
+                                      SPLIT_ROWS, LaneBase, Mat, _Arena, _Blob, _block, _retarget, _u64, rope_table)
 
-K_GEMM, K_ATTN_PREFILL, K_ATTN_DECODE, K_ATTN_MERGE, K_RMSNORM, K_QKROPE = 32, 33, 34, 35, 36, 37
+K_ATTN_PREFILL, K_ATTN_DECODE, K_ATTN_MERGE, K_RMSNORM, K_QKROPE = 33, 34, 35, 36, 37
 K_ADDNORM, K_NORM_LOGITS = 41, 50
 FUSE_ROWS, FUSE_PERMUTE_ROWS = 32, 16   # batches this small fold the norm into the projection's tiles, and the permute into expand
-SPLIT_ROWS, SPLIT_PARTS, QKV_PARTS = 64, 8, 2   # a dense GEMM of at most SPLIT_ROWS rows may run as up to SPLIT_PARTS K ranges
+QKV_PARTS = 2
 O_SPLIT_ROWS, O_WIDE_PARTS = 512, 4   # the o projection (a residual epilogue of 2-byte loads and stores) keeps the form up to here
-K_ROUTER, K_EXPAND, K_PERMUTE, K_EMBED, K_SAMPLE, K_ATTN_PLAN, K_COMBINE, K_LOGITS = 38, 39, 40, 42, 43, 44, 47, 48
-EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_ROWS_F32 = 0, 1, 3, 5
+K_ROUTER, K_EXPAND, K_PERMUTE, K_EMBED, K_ATTN_PLAN, K_COMBINE, K_LOGITS = 38, 39, 40, 42, 44, 47, 48
 REGION_HOST, REGION_HOT = 0, 1
 CHUNK = 16            # rows per router / permute tile = rank chunk of the stable pack
 ROPE_ITEMS = 48       # (row, head) items per qk_rope tile (monoserve/runtime/lane.py:27)
-HEIGHTS = [16, 32, 64, 128, 256]
-
-
-def _block(name, **fields):
-    return torch.frombuffer(bytearray(pack(name, **fields)), dtype=torch.uint8).cuda()
-
-
-def _u64(values):
-    return torch.tensor([int(v) for v in values], dtype=torch.int64).cuda()
-
-
-class _Blob:
-    """A piece of device memory by address (what `pack` and the tile builders need of a tensor)."""
-
-    def __init__(self, addr, nbytes):
-        self.addr, self.nbytes = addr, nbytes
-
-    def data_ptr(self):
-        return self.addr
-
-
-class _Arena:
-    """Device memory for the operand blocks of one program build, carved from one buffer that is
-    allocated with the lane and filled through Fabric.write: a build then neither allocates device
-    memory nor launches a kernel, both of which would wait for a resident fabric kernel."""
-
-    def __init__(self, fab, nbytes):
-        self.fab, self.buf, self.at = fab, torch.zeros(nbytes, dtype=torch.uint8, device="cuda"), 0
-        self.host, self.flushed = bytearray(nbytes), 0   # the blocks of the current build; [flushed, at) not yet written
-
-    def reset(self):
-        self.at = self.flushed = 0
-
-    def put(self, data):
-        """Room for `data` in the arena; the bytes reach the device with the next flush()."""
-        size = (len(data) + 255) & ~255
-        if self.at + size > self.buf.numel():
-            raise RuntimeError("monofab: the lane's operand arena is full")
-        blob = _Blob(self.buf.data_ptr() + self.at, len(data))
-        self.host[self.at:self.at + len(data)] = data
-        self.at += size
-        return blob
-
-    def patch(self, blob, data):
-        """Replace the contents of a block put earlier in this build."""
-        at = blob.addr - self.buf.data_ptr()
-        assert self.flushed <= at and at + len(data) <= self.at, "the block is not of the current build"
-        self.host[at:at + len(data)] = data
-
-    def flush(self):
-        """One write of everything put since the last flush (a build has hundreds of blocks of 64 to 256 bytes)."""
-        if self.at > self.flushed:
-            self.fab.write(self.buf.data_ptr() + self.flushed, bytes(self.host[self.flushed:self.at]))
-            self.flushed = self.at
-
-
-def _bm(rows):
-    """Row-block height of a dense GEMM over `rows` activation rows."""
-    for h in HEIGHTS:
-        if rows <= h:
-            return h
-    return HEIGHTS[-1]
-
-
-def _retarget(template, a0=None, a1=None, a2=None, a4=None):
-    """A copy of a tile array with other operand addresses.  The tiles of a stage depend on the layer only
-    through the addresses they name, so a lane keeps one array per shape and re-addresses a copy per layer."""
-    t = template.copy()
-    for col, v in ((3, a0), (4, a1), (5, a2), (7, a4)):
-        if v is not None:
-            t[:, col] = v
-    return t
-
-
-def rope_table(theta, rot_dim, max_pos):
-    """cos/sin fp32 [max_pos][rot_dim / 2][2], computed as the reference's oracle does
-    (tests/test_fabric_model.py:35-42; the lane's host table: monoserve/runtime/lane.py:36-48)."""
-    half = rot_dim // 2
-    j = torch.arange(half, dtype=torch.float32)
-    inv = 1.0 / torch.pow(torch.tensor(theta, dtype=torch.float32), 2 * j / rot_dim)
-    ang = torch.arange(max_pos, dtype=torch.float32)[:, None] * inv[None]
-    return torch.stack([ang.cos(), ang.sin()], -1).contiguous()
-
-
-class Mat:
-    """A weight matrix on the device: bf16, or e4m3 bytes with an fp32 scale per output row."""
-
-    def __init__(self, data, scale=None):
-        self.data, self.scale = data, scale
-        self.fp8 = data.dtype == torch.uint8
 
 
 class ModelWeights:
@@ -233,7 +144,7 @@ class KVCache:
         self.v = [torch.zeros(shape, dtype=torch.bfloat16, device="cuda") for _ in range(cfg.num_layers)]
 
 
-class ModelLane:
+class ModelLane(LaneBase):
     """One lane of the fabric running the decoder: buffers, operand blocks and tensor maps are
     made once; `build_prefill` / `build_decode` upload programs over them.
 
@@ -294,49 +205,15 @@ class ModelLane:
         wide = max(self.Id, self.Is)
         self.hd = z(T + 256, wide, dt=bf) if wide else None
         self.y_shared = z(T, H, dt=torch.float32) if self.Is else None
-        # token and request state
-        self.tokens, self.tok_pos, self.tok_slot, self.gather = z(T), z(T), z(T), z(T)
-        self.req_info = z(max(T, S), 4)
-        self.row_req = z(max(T, S))
-        if requests is not None:
-            assert requests.slots >= S and requests.bt_stride == bt_stride
-            self.bt, self.seq_len, self.last_token, self.steps = requests.bt, requests.seq_len, requests.last_token, requests.steps
-            self.temperature, self.ring = requests.temperature, requests.ring
-            self.host_tokens, self.host_steps = requests.host_tokens, requests.host_steps
-        else:
-            self.bt = z(S, bt_stride)
-            self.seq_len, self.last_token, self.steps = z(S), z(S), z(S)
-            self.temperature = z(S, dt=torch.float32)
-            self.ring = 64
-            self.host_tokens = torch.zeros(S, self.ring, dtype=torch.int32).pin_memory()
-            self.host_steps = torch.zeros(S, dtype=torch.int64).pin_memory()
+        self._request_state(T, S, requests)
         # attention split workspace: (max, sum) pairs after the fp32 rows
         self.ws_rows = max(max_chunks * S * hq, 4 * T * hq // 8 + 1024)
         self.ws = z(self.ws_rows * 130, dt=torch.float32)
         max_pos = max_pos or bt_stride * kv.page
         self.max_pos = max_pos
         self.cos_sin = rope_table(cfg.rope_theta, cfg.rotary_dim, max_pos).cuda()
-        self._keep = []
-        self.arena = _Arena(fab, (64 << 10) * (L + 2))
-        self._templates = {}   # tile arrays by shape, re-addressed per layer (_retarget)
+        self._build_state((64 << 10) * (L + 2))
         self._maps()
-
-    # ------------------------------------------------------------------ maps and operand blocks
-    def _wmap(self, t, base=None, packed=False):
-        if isinstance(t, Mat):
-            t = t.data
-        if t.dim() == 2:
-            rows, k, zdim = t.shape[0], t.shape[1], 1
-        else:
-            zdim, rows, k = t.shape
-        base = base if base is not None else t.data_ptr()
-        if t.dtype == torch.uint8:   # e4m3 bytes: byte strides, no swizzle (monoserve/runtime/weights.py:38-40)
-            return self.fab.tensor_map(base, [k, rows, zdim], [k, rows * k], [128, 64, 1], dtype=2, swizzle=0, packed=packed)
-        return self.fab.tensor_map(base, [k, rows, zdim], [k * 2, rows * k * 2], [64, 64, 1], packed=packed)
-
-    def _amaps(self, t, rows, k):
-        """Activation maps of a [rows][k] bf16 buffer for every row-block height."""
-        return [self.fab.tensor_map(t.data_ptr(), [k, rows], [k * 2], [64, bm]) for bm in HEIGHTS]
 
     def _maps(self):
         cfg, w, fab = self.cfg, self.w, self.fab
@@ -411,95 +288,10 @@ class ModelLane:
                                    fill=self.fill, pair_token=self.pair_token, pair_weight=self.pair_weight,
                                    src=self.xn, dst=self.xp, K=K, H=H, chunk_prefix=self.chunk_prefix,
                                    pair_pos=self.pair_pos, E=E)
-        self.step_args = _block("StepArgs", row_req=self.row_req, last_token=self.last_token, seq_len=self.seq_len,
-                                block_table=self.bt, tok_pos=self.tok_pos, tok_slot=self.tok_slot,
-                                req_info=self.req_info, bt_stride=self.bt_stride, page_size=self.kv.page)
-        self.sample_args = _block("SampleArgs", logits=self.logits, temperature=self.temperature,
-                                  last_token=self.last_token, steps=self.steps,
-                                  host_tokens=_C.host_device_pointer(self.host_tokens.data_ptr()),
-                                  host_steps=_C.host_device_pointer(self.host_steps.data_ptr()), seed=0x5eed,
-                                  V=cfg.vocab, ring=self.ring)
-
-    # ------------------------------------------------------------------ device memory of a build
-    def _dev(self, name, **fields):
-        """An operand block in the lane's arena."""
-        return self.arena.put(pack(name, **fields))
-
-    def _put(self, tensor, values, dtype=np.int32):
-        """Write the first len(values) elements of a device tensor without launching a kernel."""
-        data = np.ascontiguousarray(values, dtype=dtype)
-        if data.size:
-            self.fab.write(tensor.data_ptr(), data.tobytes())
+        self.step_args = self._step_block()
+        self.sample_args = self._sample_block(cfg.vocab)
 
     # ------------------------------------------------------------------ stage builders
-    def _gemm_split(self, p, wmap, amaps, rows, n_out, k, slabs, parts, label, mark=None, mat=None, bias=None,
-                    slab_rows=SPLIT_ROWS):
-        """The same product for few rows as `parts` K ranges, every range storing its fp32 partial sums in its own
-        slab of `slabs` ([parts][slab_rows][n_out]); the add-norm tile behind it adds the slabs in order.  A 128-row
-        weight slice over all of K is a megabyte that one worker streams alone; the ranges spread it over
-        parts x n_out / 128 workers, and the sum keeps a defined order (no atomics)."""
-        bm = _bm(rows)
-        fp8 = mat is not None and mat.fp8
-        xm = amaps[HEIGHTS.index(bm)]
-        kt = k // 64
-        per = -(-kt // parts)
-        ptrs, ranges = [], []
-        for q in range(parts):
-            k0, kn = q * per, min(per, kt - q * per)
-            args = self.arena.put(_C.gemm_args(out=slabs.data_ptr() + 4 * q * slab_rows * n_out, ld_out=n_out, k_tiles=kt,
-                                               epi=EPI_F32, bm=bm, n_limit=n_out, w_fp8=int(fp8),
-                                               bias=bias.data_ptr() if bias is not None else 0))   # added by the first range
-            ptrs.append(args.data_ptr())
-            ranges.append(k0 | (kn << 16))
-        key = ("split", rows, bm, n_out, parts, kt)
-        tmpl = self._templates.get(key)
-        if tmpl is None:
-            m0, n0 = np.meshgrid(np.arange(0, rows, bm), np.arange(0, n_out, 128), indexing="ij")
-            by_range = np.asarray(ranges, dtype=np.int64)[:, None, None]   # (range, row block, slice)
-            tmpl = self._templates[key] = tile_array(K_GEMM, i0=n0[None], i1=m0[None], i2=np.minimum(bm, rows - m0)[None],
-                                                     a3=by_range)
-        per_range = len(tmpl) // parts
-        tiles = _retarget(tmpl, a0=np.repeat(np.asarray(ptrs, dtype=np.uint64), per_range), a1=wmap, a2=xm,
-                          a4=mat.scale.data_ptr() if fp8 else 0)
-        return p.stage(tiles, mark=mark, label=label)
-
-    def _gemm(self, p, wmap, amaps, rows, n_out, k, out, ld_out, epi, label, residual=None, ld_res=0, mark=None,
-              mat=None, bias=None, up_offset=0):
-        """A dense GEMM stage: out[rows][n_out] = act[rows][k] x weight[n_out (x2 for SiLU-mul)][k]^T.
-        mat: the weight's Mat (e4m3 weights carry their scales into the tiles)."""
-        bm = _bm(rows)
-        fp8 = mat is not None and mat.fp8
-        args = self.arena.put(_C.gemm_args(
-            out=out.data_ptr(), ld_out=ld_out, k_tiles=k // 64, epi=epi, bm=bm, n_limit=n_out,
-            residual=residual.data_ptr() if residual is not None else 0, ld_res=ld_res,
-            bias=bias.data_ptr() if bias is not None else 0, up_offset=up_offset, w_fp8=int(fp8)))
-        xm = amaps[HEIGHTS.index(bm)]
-        step = 64 if epi == EPI_SILU_MUL else 128
-        key = ("gemm", rows, bm, n_out, step)
-        tmpl = self._templates.get(key)
-        if tmpl is None:
-            m0, n0 = np.meshgrid(np.arange(0, rows, bm), np.arange(0, n_out, step), indexing="ij")
-            tmpl = self._templates[key] = tile_array(K_GEMM, i0=n0, i1=m0, i2=np.minimum(bm, rows - m0))
-        tiles = _retarget(tmpl, a0=args.data_ptr(), a1=wmap, a2=xm, a4=mat.scale.data_ptr() if fp8 else 0)
-        return p.stage(tiles, mark=mark, label=label)
-
-    def _rows(self, kind, args, rows, per):
-        key = ("rows", kind, rows, per)
-        tmpl = self._templates.get(key)
-        if tmpl is None:
-            r0 = np.arange(0, rows, per)
-            tmpl = self._templates[key] = tile_array(kind, i0=r0, i1=np.minimum(per, rows - r0))
-        return _retarget(tmpl, a0=args.data_ptr())
-
-    def _per(self, T):
-        """Rows per tile of a stage whose tiles give each exec warp one row at a time: up to four rows per tile
-        while that keeps the stage to one round of tiles over the workers (150 tiles on 148 workers are two
-        rounds), a multiple of four beyond."""
-        nw = self.fab.num_workers
-        if T <= 4 * nw:
-            return max(1, -(-T // nw))
-        return -(-(-(-T // (2 * nw))) // 4) * 4
-
     def _logit_rows(self, T, E):
         """Rows per router-projection tile (of 16 experts): the height in 8 .. 32 that costs the fewest rounds x
         (rows + 4), the 4 standing for what a tile costs before its first row."""
@@ -510,14 +302,6 @@ class ModelLane:
             if best is None or cost < best[0]:
                 best = (cost, rows)
         return best[1]
-
-    def _one(self, kind, args):
-        """The single tile of an expand or plan stage."""
-        key = ("one", kind)
-        tmpl = self._templates.get(key)
-        if tmpl is None:
-            tmpl = self._templates[key] = tile_array(kind)
-        return _retarget(tmpl, a0=args.data_ptr())
 
     def _logits(self, args, T, E):
         key = ("logits", T, E)
@@ -702,38 +486,9 @@ class ModelLane:
         pos0 .. (its pages must already be in the lane's block table row `slot`).  The program
         computes the batch, appends K/V to the caches, and samples one next token per request.
         all_logits: keep the logits of every row (row r of `logits`), not only each request's last."""
-        page = self.kv.page
-        self.arena.reset()   # the operand blocks of this lane's previous program: it must have ended
-        if len(self._templates) > 256:   # shapes of many different batches: start over rather than grow
-            self._templates.clear()
-        tokens, pos, slots, req_info, sample_rows = [], [], [], [], []
-        gather = []
-        stride = self.bt.shape[1]
-        row = 0
-        for r, (slot, toks, pos0) in enumerate(batch):
-            n = len(toks)
-            req_info.append((row, pos0, n, pos0 + n))
-            # the request's row of the block table (read through the fabric: nothing may be launched beside it)
-            pages = np.frombuffer(self.fab.read(self.bt.data_ptr() + 4 * slot * stride, 4 * stride), dtype=np.int32)
-            ppos = pos0 + np.arange(n)
-            tokens.append(np.asarray(toks, dtype=np.int32))
-            pos.append(ppos.astype(np.int32))
-            slots.append((pages[ppos // page].astype(np.int64) * page + ppos % page).astype(np.int32))
-            if all_logits:
-                gather.append(np.arange(row, row + n, dtype=np.int32))
-            else:
-                g = np.full(n, -1, dtype=np.int32)
-                g[n - 1] = r
-                gather.append(g)
-            sample_rows.append((row + n - 1 if all_logits else r, slot))
-            row += n
-        T = row
-        assert 0 < T <= self.T and (T if all_logits else len(batch)) <= self.logit_rows
-        self._put(self.tokens, np.concatenate(tokens))
-        self._put(self.tok_pos, np.concatenate(pos))
-        self._put(self.tok_slot, np.concatenate(slots))
-        self._put(self.gather, np.concatenate(gather))
-        self._put(self.req_info, req_info)
+        self._reset_build()
+        T, req_info, sample_rows = self._batch_rows(batch, None if all_logits else [[len(toks) - 1] for _, toks, _ in batch],
+                                                    all_logits)
         cfg = self.cfg
         hq, hkv = cfg.num_heads, cfg.num_kv_heads
         items, merge, ws_rows = plan_items(req_info, hq, hkv, sms=self.fab.num_workers)
@@ -770,9 +525,7 @@ class ModelLane:
         cfg = self.cfg
         R = len(slots)
         assert 0 < R <= min(self.T, 256, self.logit_rows)
-        self.arena.reset()   # the operand blocks of this lane's previous program: it must have ended
-        if len(self._templates) > 256:   # shapes of many different batches: start over rather than grow
-            self._templates.clear()
+        self._reset_build()
         self._put(self.row_req, slots)
         self._put(self.gather, np.arange(R))
         hq, hkv = cfg.num_heads, cfg.num_kv_heads
@@ -806,16 +559,3 @@ class ModelLane:
         self.labels = p.labels()
         self.arena.flush()
         return p.upload(self.fab, first=s_embed, iterations=iterations)
-
-    # ------------------------------------------------------------------ request state
-    def set_pages(self, slot, pages):
-        row = np.zeros(self.bt_stride, dtype=np.int32)
-        row[:len(pages)] = pages
-        self.fab.write(self.bt.data_ptr() + 4 * slot * self.bt_stride, row.tobytes())
-
-    def set_request(self, slot, seq_len, last_token, temperature=0.0):
-        import struct
-        self.fab.write(self.seq_len.data_ptr() + 4 * slot, struct.pack("<i", seq_len))
-        self.fab.write(self.last_token.data_ptr() + 4 * slot, struct.pack("<i", last_token))
-        self.fab.write(self.steps.data_ptr() + 4 * slot, struct.pack("<i", 0))
-        self.fab.write(self.temperature.data_ptr() + 4 * slot, struct.pack("<f", temperature))
