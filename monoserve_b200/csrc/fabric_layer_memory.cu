@@ -78,7 +78,7 @@ __device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigne
 // the augmented memory, whose column e accumulates k alone: the normaliser); slot i3.  A wide tile: `ring` is the
 // worker's operand ring.  A warp holds eight columns, a lane four-row groups 4 lane + 128 i of each, in registers for
 // the whole portion.  32 tokens at a time: keys and scaled queries as fp32 in shared memory, and each lane prepares
-// one token's gates: with F the running sum of the log forget gates, m_t = F_t + max(m_0, max_{s <= t} (i_s - F_s)).
+// one token's gates, with F the running sum of the log forget gates.
 constexpr int kMemTokens = 32, kMemColumns = 32;
 
 template <int ND>
@@ -135,16 +135,18 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
       const float v = __shfl_up_sync(0xffffffffu, F, o);
       if (lane >= o) F += v;
     }
-    float mx = gi - F;
+    // M_t = max(m_0, max_{s <= t} (i_s - F_s)): m_t = F_t + M_t, so f_t + m_(t-1) - m_t is M_(t-1) - M_t, which is
+    // exactly zero while the maximum decays, and i_t - m_t is (i_t - F_t) - M_t
+    const float rel = gi - F;
+    float M = rel;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float v = __shfl_up_sync(0xffffffffu, mx, o);
-      if (lane >= o) mx = fmaxf(mx, v);
+      const float v = __shfl_up_sync(0xffffffffu, M, o);
+      if (lane >= o) M = fmaxf(M, v);
     }
-    const float m = F + fmaxf(m0, mx);
-    const float m_up = __shfl_up_sync(0xffffffffu, m, 1);
-    const float m_prev = lane == 0 ? m0 : m_up;
-    const float keep = expf(gf + m_prev - m), add = expf(gi - m), floor_ = expf(-m);
+    M = fmaxf(m0, M);
+    const float M_up = __shfl_up_sync(0xffffffffu, M, 1), m = F + M;
+    const float keep = expf((lane == 0 ? m0 : M_up) - M), add = expf(rel - M), floor_ = expf(-m);
     m0 = __shfl_sync(0xffffffffu, m, nt - 1);
     exec_sync();
     for (int tok = 0; tok < nt; ++tok) {

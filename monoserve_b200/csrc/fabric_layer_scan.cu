@@ -91,9 +91,9 @@ __device__ void tile_conv(const TileDesc& t, int tid) {
 // finishes token p of the four (step size, input, output gate), so what a channel needs once per token is computed
 // once; the four state updates of a token run in all lanes.  The loads of the next four tokens are issued before
 // the current four are computed.
-constexpr int kScanChannels = kExecThreads / 4;
-
-template <int NS>
+// F32: the exact form.  It multiplies by e^x as S + S (e^x - 1), so that the rounding of a factor just below one does
+// not add up over a long memory.
+template <int NS, bool F32>
 __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
   ScanArgs A;
   load_block(A, t.a[0]);
@@ -102,7 +102,6 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
   const int p = tid & 3, lane = tid & 31, quad = lane & ~3;
   const int c = min(static_cast<int>(t.i2) + (tid >> 2), C - 1);   // a channel past the end repeats the last one
   const bool c_ok = static_cast<int>(t.i2) + (tid >> 2) < C;
-  const bool f32 = A.f32 != 0;
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
   const int s0 = p * NS;
   float S[NS], a[NS];
@@ -122,8 +121,8 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
   auto fetch = [&](int r, Four& f) {
     const int mine = min(r + p, row0 + rows - 1);   // rows past the end repeat the last one and are not used
     f.dt = f32p(A.dt)[static_cast<size_t>(mine) * A.ld_dt + c];
-    f.x = act_ld(A.x, static_cast<size_t>(mine) * A.ld_x + c, f32);
-    f.z = act_ld(A.z, static_cast<size_t>(mine) * A.ld_z + c, f32);
+    f.x = act_ld(A.x, static_cast<size_t>(mine) * A.ld_x + c, F32);
+    f.z = act_ld(A.z, static_cast<size_t>(mine) * A.ld_z + c, F32);
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       const size_t at = static_cast<size_t>(min(r + k, row0 + rows - 1)) * A.ld_bc + s0;
@@ -155,7 +154,8 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
         float y = 0.f;
 #pragma unroll
         for (int i = 0; i < NS; ++i) {
-          S[i] = fmaf(expf(dk * a[i]), S[i], xk * f.B[k][i]);
+          if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), xk * f.B[k][i]);
+          else S[i] = fmaf(expf(dk * a[i]), S[i], xk * f.B[k][i]);
           y = fmaf(S[i], f.Cc[k][i], y);
         }
         y += __shfl_xor_sync(0xffffffffu, y, 1);
@@ -165,7 +165,7 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
     }
     if (c_ok && r + p < row0 + rows) {
       const float y = fmaf(D, f.x, mine);
-      act_st(A.y, static_cast<size_t>(r + p) * A.ld_y + c, f32, y * (f.z / (1.f + expf(-f.z))));
+      act_st(A.y, static_cast<size_t>(r + p) * A.ld_y + c, F32, y * (f.z / (1.f + expf(-f.z))));
     }
   };
   if constexpr (NS <= 8) {
@@ -195,24 +195,31 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
     for (int j = 0; j < taps - 1; ++j) {
       const int k = rows + j;
       tail[static_cast<size_t>(j) * C] =
-          k >= taps - 1 ? act_ld(A.x_in, static_cast<size_t>(row0 + k - (taps - 1)) * A.ld_z + c, f32)
+          k >= taps - 1 ? act_ld(A.x_in, static_cast<size_t>(row0 + k - (taps - 1)) * A.ld_z + c, F32)
                         : (fresh ? 0.f : tail[static_cast<size_t>(k) * C]);
     }
   }
 }
 
 __device__ bool tile_scan(const TileDesc& t, int tid) {
-  const uint32_t n = __ldcg(&reinterpret_cast<const ScanArgs*>(t.a[0])->n);
-  const uint32_t ns = (n + 3) / 4;
-  if (ns <= 1) scan_rows<1>(t, tid);
-  else if (ns <= 2) scan_rows<2>(t, tid);
-  else if (ns <= 4) scan_rows<4>(t, tid);
-  else if (ns <= 6) scan_rows<6>(t, tid);
-  else if (ns <= 8) scan_rows<8>(t, tid);
-  else if (ns <= 16) scan_rows<16>(t, tid);
-  else if (ns <= 32) scan_rows<32>(t, tid);
-  else return false;
-  return true;
+  const ScanArgs* p = reinterpret_cast<const ScanArgs*>(t.a[0]);
+  const uint32_t ns = (__ldcg(&p->n) + 3) / 4;
+  const bool f32 = __ldcg(&p->f32) != 0;
+#define MF_SCAN(N)                       \
+  if (ns <= N) {                         \
+    if (f32) scan_rows<N, true>(t, tid); \
+    else scan_rows<N, false>(t, tid);    \
+    return true;                         \
+  }
+  MF_SCAN(1)
+  MF_SCAN(2)
+  MF_SCAN(4)
+  MF_SCAN(6)
+  MF_SCAN(8)
+  MF_SCAN(16)
+  MF_SCAN(32)
+#undef MF_SCAN
+  return false;
 }
 
 }  // namespace fab

@@ -103,8 +103,9 @@ class RequestTable:
 
 
 class _Req:
-    def __init__(self, rid, prompt, max_tokens, arrival, eos=()):
+    def __init__(self, rid, prompt, max_tokens, arrival, eos=(), temperature=0.0):
         self.rid, self.prompt, self.max_tokens, self.arrival = rid, list(prompt), max_tokens, arrival
+        self.temperature = temperature
         self.eos, self.reason = frozenset(eos), None   # reason: "stop" (an eos token), "length" (max_tokens, or no KV page left)
         self.slot, self.pages, self.delivered = None, [], 0
         self.tokens, self.token_times, self.first_time, self.finish_time = [], [], None, None
@@ -196,12 +197,12 @@ class Engine:
     def now(self):
         return time.perf_counter() - self.t0
 
-    def submit(self, rid, prompt, max_tokens, arrival=None, eos=()):
+    def submit(self, rid, prompt, max_tokens, arrival=None, eos=(), temperature=0.0):
         if len(prompt) + max_tokens > self.max_len:
             raise ValueError(f"request {rid}: {len(prompt)} + {max_tokens} tokens exceed max_len {self.max_len}")
         if len(prompt) > self.token_budget:
             raise ValueError(f"request {rid}: a prompt of {len(prompt)} tokens exceeds the pass budget {self.token_budget}")
-        r = _Req(rid, prompt, max_tokens, self.now() if arrival is None else arrival, eos)
+        r = _Req(rid, prompt, max_tokens, self.now() if arrival is None else arrival, eos, temperature)
         self.reqs[rid] = r
         self.queue.append(r)
 
@@ -252,7 +253,7 @@ class Engine:
             self.queue.pop(0)
             r.slot, r.pages = self.free_slots.pop(), self.pool.take(need)
             self.table.set_pages(r.slot, r.pages)
-            self.table.open(r.slot, len(r.prompt))
+            self.table.open(r.slot, len(r.prompt), r.temperature)
             batch.append(r)
             tokens += len(r.prompt)
         if not batch:
@@ -367,7 +368,7 @@ class Engine:
         return True
 
     # ------------------------------------------------------------------ a whole run
-    def serve(self, requests, poll_s=2e-4, timeout_s=600.0):
+    def serve(self, requests, poll_s=2e-4, timeout_s=600.0, eos=(), temperature=0.0):
         """requests: [(arrival seconds, rid, prompt tokens, max_tokens)].  Submits each at its arrival
         time on the wall clock and runs the loop until all have finished.  Returns {rid: record}."""
         pending = sorted(requests, key=lambda q: q[0])
@@ -383,7 +384,7 @@ class Engine:
                                    f"decoding {len(self.dec_batch)}, pending switch {self.dec_pending is not None}")
             while pending and pending[0][0] <= now:
                 t, rid, prompt, max_tokens = pending.pop(0)
-                self.submit(rid, prompt, max_tokens, arrival=t)
+                self.submit(rid, prompt, max_tokens, arrival=t, eos=eos, temperature=temperature)
             n_done += len(self.step())
             time.sleep(poll_s)
         while self.busy():   # let the last switch (to the idle program) go through

@@ -137,9 +137,10 @@ def layer_order(config):
 
 
 @torch.no_grad()
-def model_logits(config, weights, tokens, dtype=torch.float64, runs=None, rows=None):
+def model_logits(config, weights, tokens, dtype=torch.float64, runs=None, rows=None, jitter=0.0):
     """Logits [T, vocab] of one sequence.  runs (a list) receives the summed streams after every layer run;
-    rows: only these positions' logits."""
+    rows: only these positions' logits.  jitter: every sublayer's input and output is multiplied by 1 + up to this much at
+    random, which shows how far rounding of that size carries."""
     w = {k: v.to(dtype) for k, v in weights.items()}
     eps = config["norm"]["eps"]
     x = w["embed"][torch.as_tensor(tokens)]
@@ -148,9 +149,14 @@ def model_logits(config, weights, tokens, dtype=torch.float64, runs=None, rows=N
     def sub(prefix):
         return {k[len(prefix):]: v for k, v in w.items() if k.startswith(prefix)}
 
+    gen = torch.Generator().manual_seed(0)
+
+    def shake(x):
+        return x * (1 + jitter * (2 * torch.rand(x.shape, generator=gen, dtype=torch.float64) - 1)) if jitter else x
+
     def mixed(streams, hc, f):
         u = sum(a * x for a, x in zip(hc["in"], streams))
-        y = f(u)
+        y = shake(f(u))
         return [sum(hc["mix"][s, t] * streams[s] for s in range(len(streams))) + hc["out"][t] * y
                 for t in range(len(streams))]
 
@@ -158,10 +164,10 @@ def model_logits(config, weights, tokens, dtype=torch.float64, runs=None, rows=N
         spec, p = config["layers"][l], sub(f"l{l}.")
         mix = sub(f"l{l}.mix.")
         streams = mixed(streams, sub(f"l{l}.hc1."),
-                        lambda u: MIXERS[spec["type"]](norm_around_one(u, p["norm1"], eps), mix, spec["mixer"], eps))
+                        lambda u: MIXERS[spec["type"]](shake(norm_around_one(u, p["norm1"], eps)), mix, spec["mixer"], eps))
         if spec.get("mlp"):
             streams = mixed(streams, sub(f"l{l}.hc2."),
-                            lambda u: gated_ffn(norm_around_one(u, p["norm2"], eps), sub(f"l{l}.mlp.")))
+                            lambda u: gated_ffn(shake(norm_around_one(u, p["norm2"], eps)), sub(f"l{l}.mlp.")))
         if runs is not None:
             runs.append(sum(streams))
     x = sum(streams)
