@@ -194,7 +194,7 @@ __device__ void tile_expand(const TileDesc& t, const ProgramDesc* P, DeviceState
 
 // tid: index among the exec threads.  ring: the operand ring, for a wide tile.
 __device__ bool run_core_tile(DeviceState& S, const WorkSlot& w, int tid, uint32_t worker, unsigned long long* sh_t0,
-                              uint8_t* ring) {
+                              uint8_t* ring, uint32_t tmem_base, volatile int* abort_flag) {
   const TileDesc& t = w.tile;
   switch (t.kind) {
     case kTileNop:
@@ -285,7 +285,7 @@ __device__ bool run_core_tile(DeviceState& S, const WorkSlot& w, int tid, uint32
       tile_attn_plan(t, w.prog, S, tid);
       return true;
     default:
-      return run_layer_tile(t, tid, s_exec_scratch, ring);
+      return run_layer_tile(t, tid, LayerCtx{s_exec_scratch, ring, tmem_base, abort_flag});
   }
 }
 
@@ -1246,9 +1246,9 @@ __global__ void __launch_bounds__(kWorkerThreads, 1) fabric_kernel(DeviceState* 
         if (!ok && tid == 0) raise_error(S, kFabErrTileWait);
         ++g;
       } else if (w.is_wide) {
-        if (!run_core_tile(S, w, tid, worker, &sh.t0, ring) && tid == 0) raise_error(S, kFabErrBadTile);
+        if (!run_core_tile(S, w, tid, worker, &sh.t0, ring, tmem_base, abort_flag) && tid == 0) raise_error(S, kFabErrBadTile);
         fence_proxy_async_smem();   // the exec warps' accesses of the ring before the next record's TMA writes
-      } else if (!run_core_tile(S, w, tid, worker, &sh.t0, nullptr) && tid == 0) {
+      } else if (!run_core_tile(S, w, tid, worker, &sh.t0, nullptr, tmem_base, abort_flag) && tid == 0) {
         raise_error(S, kFabErrBadTile);
       }
       exec_sync();

@@ -1,0 +1,328 @@
+// Latent attention on the tensor cores: the bf16 form of the tile in fabric_layer_latent.cu (fabric_layer_tiles.cuh).
+//
+// Keys are the MMA's M dimension and (head, token) pairs its N dimension, so one cached latent row serves every head
+// of the tile and a decode step with sixteen heads wastes nothing:
+//   S^T [128 keys][N]          = K [128][latent | rotated part] . Q^T      (A K-major)
+//   O^T [latent dims, 128 at a time][N] += V^T [dims][128 keys] . P^T      (A MN-major: the same tile, read as V)
+// A key tile comes through one TMA box per page in groups of eight keys: [group][64-element chunk][8 keys][128 bytes],
+// 128-byte swizzle, which serves both as K (rows = keys) and as V^T (rows = latent columns).
+//
+// The tile is wide: it runs on the exec warps alone, with the operand ring as its shared memory and the worker's TMEM
+// (nothing else of the worker is in flight meanwhile).  Thread = key: a thread turns its key's N scores into P^T; the
+// row maxima move only when a score exceeds the reference by more than kSlack (in the exp2 domain), so the reductions
+// over keys are rare, and the sums stay in registers to the end.  S of the next key tile is issued right behind O of this
+// one.  Every wait is bounded; the threads agree on going on once per key tile.
+#include "fabric_layer_tiles.cuh"
+#include "ptx.cuh"
+
+namespace mf {
+namespace fab {
+
+constexpr unsigned long long kLatentWaitNs = 4000000000ull;
+constexpr float kSlack = 8.f;
+constexpr int kKeyTile = 128;
+
+__device__ __forceinline__ uint64_t sw128_desc(uint32_t addr, uint32_t lead, uint32_t stride) {
+  return static_cast<uint64_t>((addr & 0x3ffffu) >> 4) | (static_cast<uint64_t>(lead >> 4) << 16) |
+         (static_cast<uint64_t>(stride >> 4) << 32) | (static_cast<uint64_t>(1) << 46) | (static_cast<uint64_t>(2) << 61);
+}
+__device__ __forceinline__ void tma_box_3d(void* smem, unsigned long long map, uint64_t* bar, int x, int y, int z) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];" ::"r"(
+          smem_u32(smem)),
+      "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z)
+      : "memory");
+}
+__device__ __forceinline__ void tma_box_4d(void* smem, unsigned long long map, uint64_t* bar, int x, int y, int z, int w) {
+  asm volatile(
+      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];" ::"r"(
+          smem_u32(smem)),
+      "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z), "r"(w)
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
+      "%16};" ::"r"(taddr),
+      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
+      "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+      : "memory");
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// Barrier of the exec threads that also tells each whether `v` held in all / any of them.
+__device__ __forceinline__ bool exec_and(bool v) {
+  int r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.b32 q, %1, 0;\n\tbar.red.and.pred p, 1, %2, q;\n\tselp.b32 %0, 1, 0, p;\n\t}"
+      : "=r"(r) : "r"(static_cast<int>(v)), "n"(kExecThreads) : "memory");
+  return r != 0;
+}
+
+// N columns: (head of the group) * tokens + token.
+template <int N>
+__device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerCtx& ctx) {
+  LatentAttnArgs A;
+  load_block(A, t.a[0]);
+  __builtin_assume(__isShared(ctx.ring));
+  __builtin_assume(__isShared(ctx.scratch));
+  const int warp = tid >> 5, lane = tid & 31, quad = (warp + 1) & 3;   // exec warps are warps 1 .. 4 of the CTA
+  const int row0 = static_cast<int>(t.i0), n_tok = static_cast<int>(t.i1 & 0xffffu), h0 = static_cast<int>(t.i1 >> 16);
+  const int part = static_cast<int>(t.i2), parts = static_cast<int>(t.i3);
+  const int H = static_cast<int>(A.heads), kvr = static_cast<int>(A.kv_rank), page = static_cast<int>(A.page);
+  const int box_tok = static_cast<int>(A.tokens), hg = static_cast<int>(A.group), n_h = min(hg, H - h0);
+  const int chunks = (kvr + static_cast<int>(A.r) + 63) / 64, blocks = (kvr + 127) / 128;
+  const int pos0 = reinterpret_cast<const int*>(A.tok_pos)[row0];
+  const int keys = pos0 + n_tok;
+  const int per = (keys + parts - 1) / parts;
+  const int k_lo = min(part * per, keys), k_hi = min(k_lo + per, keys);
+
+  uint64_t* const bar = reinterpret_cast<uint64_t*>(ctx.scratch);   // q, k[2], s, o
+  uint64_t *const bar_q = bar, *const bar_k = bar + 1, *const bar_s = bar + 3, *const bar_o = bar + 4;
+  float* const s_m = reinterpret_cast<float*>(ctx.scratch) + 16;    // [64] reference of each column
+  float* const s_a = s_m + 64;                                      // [64] factor of the last move, later 1 / sum
+  float* const s_red = s_a + 64;                                    // [4][64]
+  const uint32_t group_bytes = chunks * 1024u, tile_bytes = (kKeyTile / 8) * group_bytes;
+  const uint32_t q_bytes = chunks * N * 128u, p_bytes = N * 256u;
+  uint8_t* const sQ = ctx.ring;
+  uint8_t* const sP = ctx.ring + q_bytes;
+  uint8_t* const sK = sP + ((p_bytes + 1023u) & ~1023u);
+  const int nbuf = A.buffers > 1 ? 2 : 1;
+  const uint32_t tmem_s = ctx.tmem_base, tmem_o = ctx.tmem_base + 64;
+  const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
+
+  if (tid == 0) {
+    for (int i = 0; i < 5; ++i) mbar_init(bar + i, 1);
+    fence_barrier_init();
+  }
+  if (tid < N) s_m[tid] = -1e30f;
+  exec_sync();
+
+  const int* bt = reinterpret_cast<const int*>(A.block_table) + static_cast<size_t>(t.a[1] & 0xffffffffull) * A.bt_stride;
+  const int last_page = (max(k_hi, 1) - 1) / page, per_tile = kKeyTile / page;
+  const int first_key = k_lo / page * page;   // key tiles start at a page
+  const int tiles = k_hi > k_lo ? (k_hi - first_key + kKeyTile - 1) / kKeyTile : 0;
+  auto load_keys = [&](int j) {   // warp 0
+    const int s = j % nbuf;
+    if (lane == 0) {
+      fence_proxy_async_all();
+      mbar_arrive_expect_tx(bar_k + s, tile_bytes);
+    }
+    __syncwarp();
+    if (lane < per_tile) {
+      // pages past the visible range repeat the last visible page; their keys are masked
+      const int pg = bt[min(first_key / page + j * per_tile + lane, last_page)];
+      tma_box_4d(sK + s * tile_bytes + lane * (page / 8) * group_bytes, A.kv_map, bar_k + s, 0, 0, 0, pg * (page / 8));
+    }
+  };
+  auto issue_s = [&](int j) {   // one thread: S^T of key tile j
+    const uint32_t k_addr = smem_u32(sK + (j % nbuf) * tile_bytes), q_addr = smem_u32(sQ);
+    const uint32_t idesc = umma_idesc_bf16(128, N);
+    for (int c = 0; c < chunks; ++c)
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        umma_bf16(tmem_s, sw128_desc(k_addr + c * 1024u + i * 32u, 0, group_bytes),
+                  sw128_desc(q_addr + c * (N * 128u) + i * 32u, 0, 1024), idesc, (c | i) != 0);
+    umma_commit(bar_s);
+  };
+
+  bool ok = true;
+  if (warp == 0 && tiles > 0) {
+    if (lane == 0) {
+      fence_proxy_async_all();
+      mbar_arrive_expect_tx(bar_q, static_cast<uint32_t>(chunks) * 128u * box_tok * hg);
+      for (int c = 0; c < chunks; ++c) tma_box_3d(sQ + c * (N * 128u), A.q_map, bar_q, c * 64, row0, h0);
+    }
+    __syncwarp();
+    load_keys(0);
+    if (nbuf > 1 && tiles > 1) load_keys(1);
+  }
+  if (tid == 0 && tiles > 0) {
+    ok = mbar_wait_bounded(bar_q, 0, ctx.abort_flag, kLatentWaitNs) && mbar_wait_bounded(bar_k, 0, ctx.abort_flag, kLatentWaitNs);
+    if (ok) {
+      tc_fence_after_sync();
+      issue_s(0);
+    }
+  }
+  const float scale = A.scale * 1.4426950408889634f;
+  float l[N];
+#pragma unroll
+  for (int c = 0; c < N; ++c) l[c] = 0.f;
+  const int n_col = box_tok * hg;
+  const int my_key = quad * 32 + lane;
+  for (int j = 0; j < tiles; ++j) {
+    ok = ok && mbar_wait_bounded(bar_s, j & 1, ctx.abort_flag, kLatentWaitNs) &&
+         (j == 0 || mbar_wait_bounded(bar_o, (j - 1) & 1, ctx.abort_flag, kLatentWaitNs));
+    if (!exec_and(ok)) {
+      ok = false;
+      break;
+    }
+    tc_fence_after_sync();
+    float v[N];
+#pragma unroll
+    for (int c0 = 0; c0 < N; c0 += 16) {
+      __syncwarp();
+      tmem_ld_32x16(tmem_s + lane_off + c0, *reinterpret_cast<uint32_t(*)[16]>(&v[c0]));
+    }
+    tmem_ld_wait();
+    const int key = first_key + j * kKeyTile + my_key;
+    // token t of a column sees the key when pos0 + t >= key; keys outside [k_lo, k_hi) belong to another part
+    const int t_min = (key < k_lo || key >= k_hi) ? 0x7fffffff : key - pos0;
+    bool move = false;
+    {
+      int tok = 0;
+#pragma unroll
+      for (int c = 0; c < N; ++c) {
+        const bool see = c < n_col && tok >= t_min;
+        v[c] = see ? v[c] * scale : -INFINITY;
+        move |= v[c] > s_m[c] + kSlack;
+        if (++tok == box_tok) tok = 0;
+      }
+    }
+    if (!exec_and(!move)) {   // some column's reference moves: reduce over the tile's keys, rescale O
+#pragma unroll
+      for (int c = 0; c < N; ++c) {
+        float m = v[c];
+#pragma unroll
+        for (int o = 16; o; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        if (lane == 0) s_red[warp * 64 + c] = m;
+      }
+      exec_sync();
+      if (tid < N) {
+        const float old = s_m[tid];
+        const float m = fmaxf(fmaxf(s_red[tid], s_red[64 + tid]), fmaxf(s_red[128 + tid], s_red[192 + tid]));
+        const float now = m > old + kSlack ? m : old;
+        s_m[tid] = now;
+        s_a[tid] = ex2(old - now);
+      }
+      exec_sync();
+#pragma unroll
+      for (int c = 0; c < N; ++c) l[c] *= s_a[c];
+      if (j > 0)   // O of the tiles before is complete: S of this tile was issued behind it
+        for (int b = 0; b < blocks; ++b)
+#pragma unroll
+          for (int c0 = 0; c0 < N; c0 += 16) {
+            uint32_t o[16];
+            __syncwarp();
+            tmem_ld_32x16(tmem_o + lane_off + b * N + c0, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_a[c0 + i]);
+            tmem_st_32x16(tmem_o + lane_off + b * N + c0, o);
+          }
+      asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+    }
+    // P^T as bf16: row = column of S^T, 64 keys per 128-byte row, 128-byte swizzle
+    uint8_t* const p_half = sP + (my_key >> 6) * (N * 128);
+    const int k6 = my_key & 63;
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+      const __nv_bfloat16 p = __float2bfloat16(ex2(v[c] - s_m[c]));
+      l[c] += __bfloat162float(p);
+      *reinterpret_cast<__nv_bfloat16*>(p_half + c * 128 + ((((k6 >> 3) ^ (c & 7)) << 4) | ((k6 & 7) << 1))) = p;
+    }
+    tc_fence_before_sync();
+    fence_proxy_async_smem();
+    exec_sync();
+    if (tid == 0) {
+      tc_fence_after_sync();
+      const uint32_t k_addr = smem_u32(sK + (j % nbuf) * tile_bytes), p_addr = smem_u32(sP);
+      const uint32_t idesc = umma_idesc_bf16(128, N) | (1u << 15);   // A is MN-major
+      for (int b = 0; b < blocks; ++b)
+#pragma unroll
+        for (int i = 0; i < kKeyTile / 16; ++i)
+          umma_bf16(tmem_o + b * N, sw128_desc(k_addr + b * 2048u + i * 2u * group_bytes, 1024, group_bytes),
+                    sw128_desc(p_addr + (i >> 2) * (N * 128u) + (i & 3) * 32u, 0, 1024), idesc, (j | i) != 0);
+      umma_commit(bar_o);
+      if (nbuf > 1 && j + 1 < tiles) {
+        ok = mbar_wait_bounded(bar_k + ((j + 1) & 1), ((j + 1) >> 1) & 1, ctx.abort_flag, kLatentWaitNs);
+        if (ok) {
+          tc_fence_after_sync();
+          issue_s(j + 1);
+        }
+      }
+    }
+    // the key tile's buffer goes to the loads of tile j + nbuf when O has read it
+    if (warp == 0 && j + nbuf < tiles) {
+      const bool free_ = mbar_wait_bounded(bar_o, j & 1, ctx.abort_flag, kLatentWaitNs);
+      if (__all_sync(0xffffffffu, free_)) load_keys(j + nbuf);
+      else ok = false;
+      if (nbuf == 1 && tid == 0 && ok) {
+        ok = mbar_wait_bounded(bar_k, (j + 1) & 1, ctx.abort_flag, kLatentWaitNs);
+        if (ok) {
+          tc_fence_after_sync();
+          issue_s(j + 1);
+        }
+      }
+    }
+  }
+  if (ok && tiles > 0) ok = mbar_wait_bounded(bar_o, (tiles - 1) & 1, ctx.abort_flag, kLatentWaitNs);
+  ok = exec_and(ok);
+  tc_fence_after_sync();
+  if (ok) {
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+      const float s = warp_sum(l[c]);
+      if (lane == 0) s_red[warp * 64 + c] = s;
+    }
+    exec_sync();
+    if (tid < N) {
+      const float s = s_red[tid] + s_red[64 + tid] + s_red[128 + tid] + s_red[192 + tid];
+      s_a[tid] = parts == 1 ? 1.f / s : s;
+    }
+    exec_sync();
+    if (parts > 1 && tid < n_tok * n_h) {
+      const int h = tid / n_tok, tok = tid - h * n_tok, c = h * box_tok + tok;
+      const size_t w = (static_cast<size_t>(row0 + tok) * H + h0 + h) * parts + part;
+      reinterpret_cast<float2*>(A.ws_ml)[w] = tiles ? make_float2(s_m[c] * 0.6931471805599453f, s_a[c]) : make_float2(-INFINITY, 0.f);
+    }
+    for (int b = 0; b < blocks; ++b) {
+      const int dim = b * 128 + quad * 32 + lane;
+#pragma unroll
+      for (int c0 = 0; c0 < N; c0 += 16) {
+        uint32_t o[16];
+        __syncwarp();
+        if (tiles > 0) {
+          tmem_ld_32x16(tmem_o + lane_off + b * N + c0, o);
+          tmem_ld_wait();
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) o[i] = 0u;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const int c = c0 + i, h = c / box_tok, tok = c - h * box_tok;
+          if (h >= n_h || tok >= n_tok || dim >= kvr) continue;
+          const float x = __uint_as_float(o[i]);
+          if (parts == 1) {
+            reinterpret_cast<__nv_bfloat16*>(A.out)[(static_cast<size_t>(h0 + h) * A.rows_max + row0 + tok) * A.ld_out + dim] =
+                __float2bfloat16(x * s_a[c]);
+          } else {
+            reinterpret_cast<float*>(A.ws_o)[((static_cast<size_t>(row0 + tok) * H + h0 + h) * parts + part) * kvr + dim] = x;
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before_sync();
+  exec_sync();
+  if (tid == 0)
+    for (int i = 0; i < 5; ++i) asm volatile("mbarrier.inval.shared::cta.b64 [%0];" ::"r"(smem_u32(bar + i)) : "memory");
+  return ok;
+}
+
+__device__ bool tile_latent_mma(const TileDesc& t, int tid, const LayerCtx& ctx) {
+  const LatentAttnArgs* p = reinterpret_cast<const LatentAttnArgs*>(t.a[0]);
+  const uint32_t n = __ldcg(&p->tokens) * __ldcg(&p->group);
+  if (n <= 16) return latent_mma<16>(t, tid, ctx);
+  if (n <= 32) return latent_mma<32>(t, tid, ctx);
+  if (n <= 64) return latent_mma<64>(t, tid, ctx);
+  return false;
+}
+
+}  // namespace fab
+}  // namespace mf

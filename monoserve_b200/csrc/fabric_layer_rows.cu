@@ -253,7 +253,8 @@ __device__ void tile_streams(const TileDesc& t, int tid, int* scratch) {
   else streams_rows<1, kMaxStreams>(t, tid, scratch);
 }
 
-__device__ bool run_layer_tile(const TileDesc& t, int tid, int* scratch, uint8_t* ring) {
+__device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx) {
+  int* const scratch = ctx.scratch;
   switch (t.kind) {
     case kTileProduct32: tile_product32(t, tid, scratch); return true;
     case kTileGatedAct: tile_gated_act(t, tid); return true;
@@ -261,10 +262,11 @@ __device__ bool run_layer_tile(const TileDesc& t, int tid, int* scratch, uint8_t
     case kTileConv: tile_conv(t, tid); return true;
     case kTileScan: return tile_scan(t, tid);
     case kTileMemGates: tile_mem_gates(t, tid); return true;
-    case kTileMemory: return tile_memory(t, tid, ring);
+    case kTileMemory: return tile_memory(t, tid, ctx.ring);
     case kTileHeadNorm: tile_head_norm(t, tid); return true;
     case kTileLatentKv: tile_latent_kv(t, tid); return true;
     case kTileLatentAttn: return tile_latent_attn(t, tid);
+    case kTileLatentMma: return tile_latent_mma(t, tid, ctx);
     case kTileLatentMerge: tile_latent_merge(t, tid); return true;
     case kTileSumSlabs: tile_sum_slabs(t, tid); return true;
     default: return false;

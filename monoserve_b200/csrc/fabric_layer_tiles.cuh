@@ -25,11 +25,21 @@ constexpr int kLayerScratchInts = 1120;
 constexpr int kMaxStreams = 8;
 constexpr int kMaxTaps = 8;
 
-// Runs tile kinds kTileProduct32 .. kTileSumSlabs: false for a kind or size these tiles do not take.  All exec threads
-// call it with the same tile.  ring: the operand ring, for wide tiles (tile_is_wide).
-__device__ bool run_layer_tile(const TileDesc& t, int tid, int* scratch, uint8_t* ring);
-// Tiles whose exec warps use the operand ring as scratch memory.
-__device__ __forceinline__ bool tile_is_wide(uint32_t kind) { return kind == kTileMemory; }
+// What the worker lends a tile.
+struct LayerCtx {
+  int* scratch;              // kLayerScratchInts ints of shared memory
+  uint8_t* ring;             // the operand ring (shared memory, 1024-byte aligned), for wide tiles only
+  uint32_t tmem_base;        // all of the worker's TMEM, for wide tiles only
+  volatile int* abort_flag;
+};
+
+// Runs tile kinds kTileProduct32 .. kTileLatentMma: false for a kind or size these tiles do not take, or when a bounded
+// wait gave up.  All exec threads call it with the same tile.
+__device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx);
+// Wide tiles: their exec warps use the operand ring as scratch memory, and TMEM.
+__device__ __forceinline__ bool tile_is_wide(uint32_t kind) {
+  return kind == kTileMemory || kind == kTileLatentMma;
+}
 
 __device__ void tile_streams(const TileDesc& t, int tid, int* scratch);
 __device__ void tile_product32(const TileDesc& t, int tid, int* scratch);
@@ -42,6 +52,7 @@ __device__ bool tile_memory(const TileDesc& t, int tid, uint8_t* ring);
 __device__ void tile_head_norm(const TileDesc& t, int tid);
 __device__ void tile_latent_kv(const TileDesc& t, int tid);
 __device__ bool tile_latent_attn(const TileDesc& t, int tid);
+__device__ bool tile_latent_mma(const TileDesc& t, int tid, const LayerCtx& ctx);
 __device__ void tile_latent_merge(const TileDesc& t, int tid);
 
 __device__ __forceinline__ void exec_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kExecThreads) : "memory"); }

@@ -59,6 +59,7 @@ enum TileKind : uint16_t {
   kTileLatentAttn = 60,     // attention over the cached latents, one key range
   kTileLatentMerge = 61,    // merge of the key ranges
   kTileSumSlabs = 62,       // sum of a K-split product's slabs
+  kTileLatentMma = 63,      // attention over the cached latents on the tensor cores: heads x tokens, one key range
 };
 constexpr int kFabChunk = 16;   // rows per router / permute tile = rank chunk of the stable pack
 

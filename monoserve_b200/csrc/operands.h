@@ -131,10 +131,13 @@ namespace mf {
   U64(qc) U64(c_norm) U64(q_un) U64(q_all) U64(cache) U64(tok_pos) U64(tok_slot) U64(cos_sin) U32(ld_qc) U32(heads) \
   U32(d) U32(r) U32(kv_rank) U32(ld_un) U32(ld_q) U32(rows_max) U32(ld_cache) U32(max_pos) U32(f32) F32(eps)
 
-/* ws_o fp32 [(row * heads + head) * parts + part][kv_rank], ws_ml float2 of the same rows. */
+/* ws_o fp32 [(row * heads + head) * parts + part][kv_rank], ws_ml float2 of the same rows.  For the tensor-core tile:
+ * q_map dims (kv_rank + r, rows_max, heads), box (64, tokens, group); kv_map dims (64, 8, chunks, page slots / 8), box
+ * (64, 8, chunks, page / 8); buffers: key tiles of 128 in shared memory. */
 #define MF_LATENT_ATTN_ARGS(U64, U32, F32) \
-  U64(q) U64(cache) U64(block_table) U64(out) U64(ws_o) U64(ws_ml) U64(tok_pos) U32(ld_q) U32(heads) U32(kv_rank) \
-  U32(r) U32(ld_cache) U32(page) U32(bt_stride) U32(rows_max) U32(ld_out) U32(f32) F32(scale)
+  U64(q) U64(cache) U64(block_table) U64(out) U64(ws_o) U64(ws_ml) U64(tok_pos) U64(q_map) U64(kv_map) U32(ld_q) \
+  U32(heads) U32(kv_rank) U32(r) U32(ld_cache) U32(page) U32(bt_stride) U32(rows_max) U32(ld_out) U32(f32) F32(scale) \
+  U32(tokens) U32(group) U32(buffers)
 
 #define MF_FIELD_U64(name) unsigned long long name;
 #define MF_FIELD_U32(name) uint32_t name;

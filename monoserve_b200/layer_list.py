@@ -32,11 +32,12 @@ from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_STORE, HEIGHTS,
                                       LaneBase, _block, _bm, _retarget)
 
 K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEM_GATES, K_MEMORY = 51, 52, 53, 54, 55, 56, 57
-K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM = 58, 59, 60, 61, 62
+K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA = 58, 59, 60, 61, 62, 63
 MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
 SCAN_CHANNELS, MEMORY_COLUMNS = 32, 32   # of one tile
 WIDE_ROWS, WIDE_PARTS = 512, 4           # K ranges of the products that end a sublayer, up to this many rows
 MAX_ATTN_PARTS = 32
+RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys per step of the tensor-core attention tile
 
 
 def up(n, m):
@@ -118,6 +119,25 @@ class LayerListCache:
     def __init__(self, cfg, n_pages, page_size=16, slots=8):
         self.n_pages, self.page, self.slots = n_pages, page_size, slots
         self.runs = [MIXERS[cfg.layers[l].kind].state(cfg, cfg.layers[l].m, n_pages * page_size, slots) for l in cfg.order]
+
+
+def latent_tile(m, page, tokens_per_request):
+    """(tokens, heads, key-tile buffers) of a tensor-core attention tile (kind 63), or None where its operands do not fit
+    the worker's shared memory or TMEM, or the page size does not divide a key tile (kind 60 then)."""
+    chunks, blocks = -(-(m.kv_rank + m.rot_dim) // 64), -(-m.kv_rank // 128)
+    if page % 8 or KEY_TILE % page:
+        return None
+
+    def room(cols, buffers):
+        return cols * (chunks * 128 + 256) + buffers * chunks * KEY_TILE * 128 <= RING_BYTES and blocks * cols <= 448
+
+    most = next((n for n in (64, 32, 16) if room(n, 1)), None)
+    if most is None:
+        return None
+    heads = -(-m.heads // -(-m.heads // most))
+    tokens = max(1, min(most // heads, tokens_per_request))
+    cols = next(n for n in (16, 32, 64) if n >= tokens * heads)
+    return tokens, heads, 2 if room(cols, 2) else 1
 
 
 # ---------------------------------------------------------------------------------------------- mixers
@@ -245,7 +265,7 @@ class LatentAttention:
 
     @staticmethod
     def state(cfg, m, rows, slots):
-        return dict(cache=torch.zeros(rows, up(m.kv_rank + m.rot_dim, 8), device="cuda",
+        return dict(cache=torch.zeros(rows, up(m.kv_rank + m.rot_dim, 64), device="cuda",
                                       dtype=torch.float32 if cfg.f32 else torch.bfloat16))
 
     @staticmethod
@@ -268,12 +288,23 @@ class LatentAttention:
         p.after(s, s_kv)
         s_q = lane.head_product(p, s_kv, lane.q_un.addr, up(d, 64), w.uk, lane.q_all.addr, ld_q, lane.T * ld_q, T, c, d,
                                 ("latent_q", run))
-        parts = lane.attn_parts(T, H, c)
-        at = lane._dev("LatentAttnArgs", q=lane.q_all.addr, cache=st["cache"], block_table=lane.bt, out=lane.o_lat.addr,
-                       ws_o=lane.ws.data_ptr(), ws_ml=lane.ws_ml.data_ptr(), tok_pos=lane.tok_pos, ld_q=ld_q, heads=H,
-                       kv_rank=c, r=r, ld_cache=st["cache"].shape[1], page=lane.kv.page, bt_stride=lane.bt_stride,
-                       rows_max=lane.T, ld_out=ld_o, f32=f32, scale=m.scale)
-        s_at = p.stage(_retarget(b.attn_tiles(H, parts), a0=at.data_ptr()), label=("latent_attn", run))
+        shape = None if f32 else latent_tile(m, lane.kv.page, max(n for _, n, _ in b.requests))
+        fields = dict(q=lane.q_all.addr, cache=st["cache"], block_table=lane.bt, out=lane.o_lat.addr, ws_o=lane.ws.data_ptr(),
+                      ws_ml=lane.ws_ml.data_ptr(), tok_pos=lane.tok_pos, ld_q=ld_q, heads=H, kv_rank=c, r=r,
+                      ld_cache=st["cache"].shape[1], page=lane.kv.page, bt_stride=lane.bt_stride, rows_max=lane.T, ld_out=ld_o,
+                      f32=f32, scale=m.scale)
+        if shape:
+            tokens, heads, buffers = shape
+            blocks = sum(-(-n // tokens) for _, n, _ in b.requests) * -(-H // heads)
+            parts = lane.attn_parts(T, H, blocks)
+            fields.update(q_map=lane.q_map(m, tokens, heads), kv_map=lane.kv_map(m, st["cache"]), tokens=tokens, group=heads,
+                          buffers=buffers)
+            tiles = b.latent_tiles(H, tokens, heads, parts)
+        else:
+            parts = lane.attn_parts(T, H, T * -(-H // 4))
+            tiles = b.attn_tiles(H, parts)
+        at = lane._dev("LatentAttnArgs", **fields)
+        s_at = p.stage(_retarget(tiles, a0=at.data_ptr()), label=("latent_attn", run))
         p.after(s_q, s_at)
         if parts > 1:
             tiles = lane._rows(K_LATENT_MERGE, at, T * H, lane.items_per(T * H))
@@ -368,6 +399,20 @@ class _Batch:
                               i2=np.arange(parts)[None, None, :], i3=parts, a1=slots[:, None, None])
         return self._once(("attn", heads, parts), make)
 
+    def latent_tiles(self, heads, tokens, group, parts):
+        """One tile per block of `tokens` rows of a request, group of heads and part, the blocks that see most keys first
+        (as far as the rows' order in their requests tells)."""
+        def make():
+            first = np.concatenate([row0 + np.arange(0, n, tokens) for row0, n, _ in self.requests])
+            count = np.concatenate([np.minimum(tokens, n - np.arange(0, n, tokens)) for _, n, _ in self.requests])
+            place = np.concatenate([np.arange(0, n, tokens) for _, n, _ in self.requests])
+            slots = np.concatenate([np.full(-(-n // tokens), slot) for _, n, slot in self.requests])
+            order = np.argsort(-place, kind="stable")
+            r, n, s = (v[order][:, None, None] for v in (first, count, slots))
+            h = np.arange(0, heads, group)[None, :, None]
+            return tile_array(K_LATENT_MMA, i0=r, i1=n | (h << 16), i2=np.arange(parts)[None, None, :], i3=parts, a1=s)
+        return self._once(("latent", heads, tokens, group, parts), make)
+
 
 class LayerListLane(LaneBase):
     """One lane of the fabric running a layer-list decoder; the interface of ModelLane."""
@@ -424,6 +469,9 @@ class LayerListLane(LaneBase):
         self._build_state((48 << 10) * (len(cfg.order) + 2))
         self.sample_args, self.step_args = self._sample_block(cfg.vocab), self._step_block()
         self._prepare()
+        for l, state in zip(cfg.order, kv.runs):
+            if cfg.layers[l].kind == "latent_attention" and not cfg.f32 and latent_tile(cfg.layers[l].m, kv.page, 1):
+                self.kv_map(cfg.layers[l].m, state["cache"])
 
     def _prepare(self):
         """Make every tensor map a program can name now: none may be made while the fabric is resident."""
@@ -447,6 +495,10 @@ class LayerListLane(LaneBase):
                 wm(lw.qkv), wm(lw.uk), wm(lw.uv), self.mix.maps(m.heads * m.vdim)
                 self.head_maps(self.q_un.addr, up(m.dim, 64), m.dim, m.heads)
                 self.head_maps(self.o_lat.addr, up(m.kv_rank, 64), m.kv_rank, m.heads)
+                for n in range(1, 65):   # a program's tile shape follows its longest request
+                    shape = latent_tile(m, self.kv.page, n)
+                    if shape:
+                        self.q_map(m, *shape[:2])
 
     def cos_sin(self, base, r):
         """fp32 [max_pos][r / 2][cos, sin] of the angles pos * base^(-2 i / r)."""
@@ -539,9 +591,27 @@ class LayerListLane(LaneBase):
         """Items (one warp each) per tile of an item-wise stage: a multiple of four, about two rounds of tiles."""
         return max(4, up(-(-items // (2 * self.fab.num_workers)), 4))
 
-    def attn_parts(self, rows, heads, kv_rank):
-        """Key ranges per row: enough tiles to give every worker about two."""
-        tiles = rows * -(-heads // 4)
+    def q_map(self, m, tokens, heads):
+        """The absorbed queries [head][T][columns], boxes of 64 columns x tokens x heads."""
+        key = "q", m.kv_rank, m.rot_dim, m.heads, tokens, heads
+        if key not in self._hmaps:
+            ld = up(m.kv_rank + m.rot_dim, 8)
+            self._hmaps[key] = self.fab.tensor_map(self.q_all.addr, [m.kv_rank + m.rot_dim, self.T, m.heads],
+                                                   [ld * 2, self.T * ld * 2], [64, tokens, heads])
+        return self._hmaps[key]
+
+    def kv_map(self, m, cache):
+        """A cache of latents, one box per page: groups of eight rows, their 64-column chunks side by side."""
+        key = cache.data_ptr()
+        if key not in self._hmaps:
+            rows, ld = cache.shape
+            chunks = -(-(m.kv_rank + m.rot_dim) // 64)
+            self._hmaps[key] = self.fab.tensor_map(cache.data_ptr(), [64, 8, chunks, rows // 8], [ld * 2, 128, 16 * ld],
+                                                   [64, 8, chunks, self.kv.page // 8])
+        return self._hmaps[key]
+
+    def attn_parts(self, rows, heads, tiles):
+        """Key ranges per row: enough of them to give every worker about two tiles."""
         want = min(MAX_ATTN_PARTS, 2 * self.fab.num_workers // tiles)
         return max(1, min(want, self.ws_rows // (rows * heads)))
 
