@@ -298,6 +298,7 @@ const std::string& layouts_json() {
     MF_JSON_STRUCT(HeadNormArgs, MF_HEAD_NORM_ARGS)
     MF_JSON_STRUCT(LatentArgs, MF_LATENT_ARGS)
     MF_JSON_STRUCT(LatentAttnArgs, MF_LATENT_ATTN_ARGS)
+    MF_JSON_STRUCT(LatentDirectArgs, MF_LATENT_DIRECT_ARGS)
     MF_JSON_STRUCT(StagingArgs, MF_STAGING_ARGS)
     s += "}";
     return s;

@@ -14,53 +14,12 @@
 // one.  Every wait is bounded; the threads agree on going on once per key tile.
 #include "fabric_layer_tiles.cuh"
 #include "ptx.cuh"
+#include "wide_tile.cuh"
 
 namespace mf {
 namespace fab {
 
-constexpr unsigned long long kLatentWaitNs = 4000000000ull;
-constexpr float kSlack = 8.f;
 constexpr int kKeyTile = 128;
-
-__device__ __forceinline__ uint64_t sw128_desc(uint32_t addr, uint32_t lead, uint32_t stride) {
-  return static_cast<uint64_t>((addr & 0x3ffffu) >> 4) | (static_cast<uint64_t>(lead >> 4) << 16) |
-         (static_cast<uint64_t>(stride >> 4) << 32) | (static_cast<uint64_t>(1) << 46) | (static_cast<uint64_t>(2) << 61);
-}
-__device__ __forceinline__ void tma_box_3d(void* smem, unsigned long long map, uint64_t* bar, int x, int y, int z) {
-  asm volatile(
-      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];" ::"r"(
-          smem_u32(smem)),
-      "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z)
-      : "memory");
-}
-__device__ __forceinline__ void tma_box_4d(void* smem, unsigned long long map, uint64_t* bar, int x, int y, int z, int w) {
-  asm volatile(
-      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];" ::"r"(
-          smem_u32(smem)),
-      "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z), "r"(w)
-      : "memory");
-}
-__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-      "%16};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
-      "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
-}
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Barrier of the exec threads that also tells each whether `v` held in all / any of them.
-__device__ __forceinline__ bool exec_and(bool v) {
-  int r;
-  asm volatile(
-      "{\n\t.reg .pred p, q;\n\tsetp.ne.b32 q, %1, 0;\n\tbar.red.and.pred p, 1, %2, q;\n\tselp.b32 %0, 1, 0, p;\n\t}"
-      : "=r"(r) : "r"(static_cast<int>(v)), "n"(kExecThreads) : "memory");
-  return r != 0;
-}
 
 // N columns: (head of the group) * tokens + token.
 template <int N>
@@ -141,7 +100,7 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
     if (nbuf > 1 && tiles > 1) load_keys(1);
   }
   if (tid == 0 && tiles > 0) {
-    ok = mbar_wait_bounded(bar_q, 0, ctx.abort_flag, kLatentWaitNs) && mbar_wait_bounded(bar_k, 0, ctx.abort_flag, kLatentWaitNs);
+    ok = mbar_wait_bounded(bar_q, 0, ctx.abort_flag, kWideWaitNs) && mbar_wait_bounded(bar_k, 0, ctx.abort_flag, kWideWaitNs);
     if (ok) {
       tc_fence_after_sync();
       issue_s(0);
@@ -154,8 +113,8 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
   const int n_col = box_tok * hg;
   const int my_key = quad * 32 + lane;
   for (int j = 0; j < tiles; ++j) {
-    ok = ok && mbar_wait_bounded(bar_s, j & 1, ctx.abort_flag, kLatentWaitNs) &&
-         (j == 0 || mbar_wait_bounded(bar_o, (j - 1) & 1, ctx.abort_flag, kLatentWaitNs));
+    ok = ok && mbar_wait_bounded(bar_s, j & 1, ctx.abort_flag, kWideWaitNs) &&
+         (j == 0 || mbar_wait_bounded(bar_o, (j - 1) & 1, ctx.abort_flag, kWideWaitNs));
     if (!exec_and(ok)) {
       ok = false;
       break;
@@ -213,7 +172,7 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
             for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_a[c0 + i]);
             tmem_st_32x16(tmem_o + lane_off + b * N + c0, o);
           }
-      asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+      tmem_st_done();
     }
     // P^T as bf16: row = column of S^T, 64 keys per 128-byte row, 128-byte swizzle
     uint8_t* const p_half = sP + (my_key >> 6) * (N * 128);
@@ -238,7 +197,7 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
                     sw128_desc(p_addr + (i >> 2) * (N * 128u) + (i & 3) * 32u, 0, 1024), idesc, (j | i) != 0);
       umma_commit(bar_o);
       if (nbuf > 1 && j + 1 < tiles) {
-        ok = mbar_wait_bounded(bar_k + ((j + 1) & 1), ((j + 1) >> 1) & 1, ctx.abort_flag, kLatentWaitNs);
+        ok = mbar_wait_bounded(bar_k + ((j + 1) & 1), ((j + 1) >> 1) & 1, ctx.abort_flag, kWideWaitNs);
         if (ok) {
           tc_fence_after_sync();
           issue_s(j + 1);
@@ -247,11 +206,11 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
     }
     // the key tile's buffer goes to the loads of tile j + nbuf when O has read it
     if (warp == 0 && j + nbuf < tiles) {
-      const bool free_ = mbar_wait_bounded(bar_o, j & 1, ctx.abort_flag, kLatentWaitNs);
+      const bool free_ = mbar_wait_bounded(bar_o, j & 1, ctx.abort_flag, kWideWaitNs);
       if (__all_sync(0xffffffffu, free_)) load_keys(j + nbuf);
       else ok = false;
       if (nbuf == 1 && tid == 0 && ok) {
-        ok = mbar_wait_bounded(bar_k, (j + 1) & 1, ctx.abort_flag, kLatentWaitNs);
+        ok = mbar_wait_bounded(bar_k, (j + 1) & 1, ctx.abort_flag, kWideWaitNs);
         if (ok) {
           tc_fence_after_sync();
           issue_s(j + 1);
@@ -259,7 +218,7 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
       }
     }
   }
-  if (ok && tiles > 0) ok = mbar_wait_bounded(bar_o, (tiles - 1) & 1, ctx.abort_flag, kLatentWaitNs);
+  if (ok && tiles > 0) ok = mbar_wait_bounded(bar_o, (tiles - 1) & 1, ctx.abort_flag, kWideWaitNs);
   ok = exec_and(ok);
   tc_fence_after_sync();
   if (ok) {
@@ -311,7 +270,7 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
   tc_fence_before_sync();
   exec_sync();
   if (tid == 0)
-    for (int i = 0; i < 5; ++i) asm volatile("mbarrier.inval.shared::cta.b64 [%0];" ::"r"(smem_u32(bar + i)) : "memory");
+    for (int i = 0; i < 5; ++i) mbar_inval(bar + i);
   return ok;
 }
 

@@ -1,52 +1,65 @@
 // The matrix memory of the layer-list decoders (fabric_layer_tiles.cuh).
 #include "fabric_layer_tiles.cuh"
+#include "wide_tile.cuh"
 
 namespace mf {
 namespace fab {
 
 // ------------------------------------------------------------------ matrix memory
 // Kind 56, MemGateArgs: rows [i0, i0 + i1), outputs [i2, i2 + i3) of the 2 heads (input gates, then forget gates).
-// A warp takes one output and four rows at a time.
+// A warp takes one row and eight outputs at a time, 2048 columns of the row in registers.
 __device__ void tile_mem_gates(const TileDesc& t, int tid) {
+  constexpr int NV = 16;
   MemGateArgs A;
   load_block(A, t.a[0]);
   const int warp = tid >> 5, lane = tid & 31, K = static_cast<int>(A.K), H = static_cast<int>(A.heads);
-  for (int o = static_cast<int>(t.i2) + warp; o < static_cast<int>(t.i2 + t.i3); o += kExecThreads / 32) {
-    const bool forget = o >= H;
-    const int h = forget ? o - H : o;
-    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(forget ? A.wf : A.wi) + static_cast<size_t>(h) * K;
-    const float bias = f32p(forget ? A.bf : A.bi)[h];
-    for (uint32_t r = t.i0; r < t.i0 + t.i1; r += 4) {
-      const float* x[4];
+  const int o_lo = static_cast<int>(t.i2), o_hi = static_cast<int>(t.i2 + t.i3);
+  auto weights = [&](int o) {
+    return reinterpret_cast<const __nv_bfloat16*>(o >= H ? A.wf : A.wi) + static_cast<size_t>(o >= H ? o - H : o) * K;
+  };
+  for (uint32_t r = t.i0 + warp; r < t.i0 + t.i1; r += kExecThreads / 32) {
+    const float* x = f32p(A.h) + static_cast<size_t>(r) * A.ld_h;
+    for (int o0 = o_lo; o0 < o_hi; o0 += 8) {
+      float acc[8] = {};
+      if ((K & 3) == 0) {
+        for (int k0 = 0; k0 < K; k0 += 128 * NV) {
+          float4 v[NV];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) x[i] = f32p(A.h) + static_cast<size_t>(min(r + i, t.i0 + t.i1 - 1)) * A.ld_h;
-      float acc[4] = {};
-      if ((K & 3) == 0 && (A.ld_h & 3) == 0) {
-#pragma unroll 4
-        for (int k = 4 * lane; k < K; k += 128) {
-          const uint2 raw = __ldg(reinterpret_cast<const uint2*>(w + k));
-          const float2 wa = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-          const float2 wb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+          for (int i = 0; i < NV; ++i) {
+            const int k = k0 + i * 128 + lane * 4;
+            v[i] = k < K ? *reinterpret_cast<const float4*>(x + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
 #pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            const float4 v = *reinterpret_cast<const float4*>(x[i] + k);
-            acc[i] = fmaf(v.x, wa.x, fmaf(v.y, wa.y, fmaf(v.z, wb.x, fmaf(v.w, wb.y, acc[i]))));
+          for (int o = 0; o < 8; ++o) {
+            const __nv_bfloat16* w = weights(min(o0 + o, o_hi - 1));
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+              const int k = k0 + i * 128 + lane * 4;
+              const uint2 raw = k < K ? __ldg(reinterpret_cast<const uint2*>(w + k)) : make_uint2(0u, 0u);
+              const float2 wa = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+              const float2 wb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+              acc[o] = fmaf(v[i].x, wa.x, fmaf(v[i].y, wa.y, fmaf(v[i].z, wb.x, fmaf(v[i].w, wb.y, acc[o]))));
+            }
           }
         }
       } else {
-        for (int k = lane; k < K; k += 32) {
-          const float wv = __bfloat162float(w[k]);
 #pragma unroll
-          for (int i = 0; i < 4; ++i) acc[i] = fmaf(x[i][k], wv, acc[i]);
+        for (int o = 0; o < 8; ++o) {
+          const __nv_bfloat16* w = weights(min(o0 + o, o_hi - 1));
+          for (int k = lane; k < K; k += 32) acc[o] = fmaf(x[k], __bfloat162float(w[k]), acc[o]);
         }
       }
+      float mine = 0.f;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[i] = warp_sum(acc[i]);
-      if (lane < 4 && r + lane < t.i0 + t.i1) {
-        const float z = (lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3]) + bias;
-        const float g = A.cap * tanhf(z / A.cap);
-        reinterpret_cast<float*>(A.out)[static_cast<size_t>(r + lane) * 2 * H + o] =
-            forget ? fminf(g, 0.f) - log1pf(expf(-fabsf(g))) : g;
+      for (int o = 0; o < 8; ++o) {
+        const float s = warp_sum(acc[o]);
+        if (lane == o) mine = s;
+      }
+      if (lane < 8 && o0 + lane < o_hi) {
+        const int o = o0 + lane;
+        const bool forget = o >= H;
+        const float g = A.cap * tanhf((mine + f32p(forget ? A.bf : A.bi)[forget ? o - H : o]) / A.cap);
+        reinterpret_cast<float*>(A.out)[static_cast<size_t>(r) * 2 * H + o] = forget ? fminf(g, 0.f) - log1pf(expf(-fabsf(g))) : g;
       }
     }
   }
@@ -75,27 +88,37 @@ __device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigne
 }
 
 // Kind 57, MemoryArgs: rows [i0, i0 + i1) of one request; i2 = head | column block << 16 (32 of the e + 1 columns of
-// the augmented memory, whose column e accumulates k alone: the normaliser); slot i3.  A wide tile: `ring` is the
-// worker's operand ring.  A warp holds eight columns, a lane four-row groups 4 lane + 128 i of each, in registers for
-// the whole portion.  32 tokens at a time: keys and scaled queries as fp32 in shared memory, and each lane prepares
+// the augmented memory, whose column e accumulates k alone: the normaliser); slot i3.  A wide tile: keys, queries and
+// values come `tokens` rows at a time through double-buffered asynchronous copies into the operand ring.  A warp holds
+// eight columns, a lane four-row groups 4 lane + 128 i of each, in registers for the whole portion.  Each lane prepares
 // one token's gates, with F the running sum of the log forget gates.
-constexpr int kMemTokens = 32, kMemColumns = 32;
+constexpr int kMemColumns = 32;
 
-template <int ND>
+template <bool F32>
+__device__ __forceinline__ float4 ld_four(const void* p) {
+  if constexpr (F32) return *reinterpret_cast<const float4*>(p);
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                     __uint_as_float(u.y & 0xffff0000u));
+}
+
+template <int ND, bool F32>
 __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ring) {
+  using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
+  constexpr int kPer16 = 16 / static_cast<int>(sizeof(T));
+  constexpr int kTokens = (ND == 4 && F32) ? 16 : 32;
   MemoryArgs A;
   load_block(A, t.a[0]);
+  __builtin_assume(__isShared(ring));
   const int row0 = static_cast<int>(t.i0), rows = static_cast<int>(t.i1), slot = static_cast<int>(t.i3);
   const int head = static_cast<int>(t.i2 & 0xffffu), col0 = static_cast<int>(t.i2 >> 16) * kMemColumns;
   const int H = static_cast<int>(A.heads), d = static_cast<int>(A.d), e = static_cast<int>(A.e);
-  const int dp = (d + 3) & ~3, warp = tid >> 5, lane = tid & 31;
-  const bool f32 = A.f32 != 0;
+  const int dp = (d + 3) & ~3, ds = (d + 7) & ~7, oe = (e + 4) & ~3, warp = tid >> 5, lane = tid & 31;
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
-  __builtin_assume(__isShared(ring));
-  float* const sk = reinterpret_cast<float*>(ring);      // [32][dp]
-  float* const sq = sk + kMemTokens * dp;                // [32][dp]
-  float* const sv = sq + kMemTokens * dp;                // [32][32]
-  const int c_lo = col0 + warp * 8;                      // this warp's first column
+  T* const buf = reinterpret_cast<T*>(ring);
+  const int buf_elems = kTokens * (2 * ds + kMemColumns);   // k, q, v
+  const int c_lo = col0 + warp * 8;                          // this warp's first column
+  const int n_v = min(kMemColumns, e - col0);                // columns of v in this block (at most 0: only the normaliser)
   float* const state = reinterpret_cast<float*>(A.state) + (static_cast<size_t>(slot) * H + head) * (e + 1) * dp;
   unsigned long long S[8][ND][2];
 #pragma unroll
@@ -113,22 +136,57 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
                          (static_cast<size_t>(slot) * H + head) * ((e + kMemColumns) / kMemColumns) + (t.i2 >> 16);
   float m0 = fresh ? 0.f : *m_state;
   const float* gates = f32p(A.gates);
-  for (int base = 0; base < rows; base += kMemTokens) {
-    const int nt = min(kMemTokens, rows - base);
+  const T *gk = reinterpret_cast<const T*>(A.k) + head * d, *gq = reinterpret_cast<const T*>(A.q) + head * d;
+  const T* gv = reinterpret_cast<const T*>(A.v) + head * e + col0;
+  const bool kq16 = d % kPer16 == 0 && ((A.k | A.q) & 15) == 0;
+  const bool v16 = e % kPer16 == 0 && n_v > 0 && n_v % kPer16 == 0 && (A.v & 15) == 0;
+  if (d & 3) {   // the padding of keys and queries stays zero
+    for (int i = tid; i < 2 * buf_elems; i += kExecThreads) buf[i] = static_cast<T>(0.f);
     exec_sync();
-    for (int i = tid; i < nt * dp; i += kExecThreads) {
-      const int tok = i / dp, k = i - tok * dp;
-      const size_t at = static_cast<size_t>(row0 + base + tok) * A.ld_qkv + head * d + k;
-      sk[i] = k < d ? act_ld(A.k, at, f32) : 0.f;
-      sq[i] = k < d ? act_ld(A.q, at, f32) * A.q_scale : 0.f;
+  }
+  auto stage = [&](int base, T* b) {
+    const int nt = min(kTokens, rows - base);
+    for (int tok = warp; tok < nt; tok += kExecThreads / 32) {
+      const size_t at = static_cast<size_t>(row0 + base + tok) * A.ld_qkv;
+      T *k = b + tok * ds, *q = b + (kTokens + tok) * ds, *v = b + 2 * kTokens * ds + tok * kMemColumns;
+      if (kq16) {
+        for (int p = lane; p < d / kPer16; p += 32) {
+          cp16(k + p * kPer16, gk + at + p * kPer16);
+          cp16(q + p * kPer16, gq + at + p * kPer16);
+        }
+      } else {
+        for (int p = lane; p < d; p += 32) {
+          k[p] = gk[at + p];
+          q[p] = gq[at + p];
+        }
+      }
+      if (v16) {
+        if (lane < n_v / kPer16) cp16(v + lane * kPer16, gv + at + lane * kPer16);
+      } else if (lane < n_v) {
+        v[lane] = gv[at + lane];
+      }
     }
-    for (int i = tid; i < nt * kMemColumns; i += kExecThreads) {
-      const int tok = i / kMemColumns, c = col0 + (i & (kMemColumns - 1));
-      sv[i] = c < e ? act_ld(A.v, static_cast<size_t>(row0 + base + tok) * A.ld_qkv + head * e + c, f32) : (c == e ? 1.f : 0.f);
+    cp_commit();
+  };
+  auto load_gates = [&](int base, float& gi, float& gf) {   // one token per lane
+    const int nt = min(kTokens, rows - base);
+    const size_t at = static_cast<size_t>(row0 + base + min(lane, nt - 1)) * 2 * H + head;
+    gi = lane < nt ? gates[at] : -INFINITY;
+    gf = lane < nt ? gates[at + H] : 0.f;
+  };
+  stage(0, buf);
+  float gi, gf;
+  load_gates(0, gi, gf);
+  for (int base = 0, s = 0; base < rows; base += kTokens, s ^= 1) {
+    const int nt = min(kTokens, rows - base);
+    float gi_next = 0.f, gf_next = 0.f;
+    if (base + kTokens < rows) {
+      stage(base + kTokens, buf + (s ^ 1) * buf_elems);
+      load_gates(base + kTokens, gi_next, gf_next);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
     }
-    // gates of this chunk, one token per lane
-    const size_t gat = static_cast<size_t>(row0 + base + min(lane, nt - 1)) * 2 * H + head;
-    const float gi = lane < nt ? gates[gat] : -INFINITY, gf = lane < nt ? gates[gat + H] : 0.f;
     float F = gf;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -149,67 +207,74 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
     const float keep = expf((lane == 0 ? m0 : M_up) - M), add = expf(rel - M), floor_ = expf(-m);
     m0 = __shfl_sync(0xffffffffu, m, nt - 1);
     exec_sync();
+    const T* const sk = buf + s * buf_elems;
+    const T* const sq = sk + kTokens * ds;
+    const T* const sv = sq + kTokens * ds + warp * 8;
     for (int tok = 0; tok < nt; ++tok) {
       const float kp = __shfl_sync(0xffffffffu, keep, tok), ad = __shfl_sync(0xffffffffu, add, tok);
       const unsigned long long kp2 = pk2(kp, kp);
-      unsigned long long acc[8];
-#pragma unroll
-      for (int c = 0; c < 8; ++c) acc[c] = 0ull;
-      const float4 va = *reinterpret_cast<const float4*>(sv + tok * kMemColumns + warp * 8);
-      const float4 vb = *reinterpret_cast<const float4*>(sv + tok * kMemColumns + warp * 8 + 4);
+      unsigned long long acc[8], av2[8];
+      const float4 va = ld_four<F32>(sv + tok * kMemColumns), vb = ld_four<F32>(sv + tok * kMemColumns + 4);
       const float v[8] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        const float av = c_lo + c < e ? ad * v[c] : (c_lo + c == e ? ad : 0.f);
+        av2[c] = pk2(av, av);
+        acc[c] = 0ull;
+      }
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
         const int at = i * 128 + lane * 4;
-        if (ND == 1 && at >= dp) continue;
         float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
         if (at < dp) {
-          k4 = *reinterpret_cast<const float4*>(sk + tok * dp + at);
-          q4 = *reinterpret_cast<const float4*>(sq + tok * dp + at);
+          k4 = ld_four<F32>(sk + tok * ds + at);
+          q4 = ld_four<F32>(sq + tok * ds + at);
         }
         const unsigned long long k0 = pk2(k4.x, k4.y), k1 = pk2(k4.z, k4.w), q0 = pk2(q4.x, q4.y), q1 = pk2(q4.z, q4.w);
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
-          const float av = ad * v[c];
-          const unsigned long long av2 = pk2(av, av);
-          S[c][i][0] = fma2(av2, k0, mul2(kp2, S[c][i][0]));
-          S[c][i][1] = fma2(av2, k1, mul2(kp2, S[c][i][1]));
+          S[c][i][0] = fma2(av2[c], k0, mul2(kp2, S[c][i][0]));
+          S[c][i][1] = fma2(av2[c], k1, mul2(kp2, S[c][i][1]));
           acc[c] = fma2(S[c][i][0], q0, acc[c]);
           acc[c] = fma2(S[c][i][1], q1, acc[c]);
         }
       }
-      float s[8];
+      float r[8];
 #pragma unroll
       for (int c = 0; c < 8; ++c) {
         const float2 f = unpk2(acc[c]);
-        s[c] = f.x + f.y;
+        r[c] = f.x + f.y;
       }
-      // the eight columns' sums over the warp; lane ends with column (lane >> 2) & 7 bit-reversed through the halves
+      // the eight columns' sums over the warp: each step halves the columns a lane carries, then plain sums
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const bool hi = lane & 16;
-        const float give = hi ? s[c] : s[c + 4], have = hi ? s[c + 4] : s[c];
-        s[c] = have + __shfl_xor_sync(0xffffffffu, give, 16);
+        const float give = hi ? r[c] : r[c + 4], have = hi ? r[c + 4] : r[c];
+        r[c] = have + __shfl_xor_sync(0xffffffffu, give, 16);
       }
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         const bool hi = lane & 8;
-        const float give = hi ? s[c] : s[c + 2], have = hi ? s[c + 2] : s[c];
-        s[c] = have + __shfl_xor_sync(0xffffffffu, give, 8);
+        const float give = hi ? r[c] : r[c + 2], have = hi ? r[c + 2] : r[c];
+        r[c] = have + __shfl_xor_sync(0xffffffffu, give, 8);
       }
       {
         const bool hi = lane & 4;
-        const float give = hi ? s[0] : s[1], have = hi ? s[1] : s[0];
-        s[0] = have + __shfl_xor_sync(0xffffffffu, give, 4);
+        const float give = hi ? r[0] : r[1], have = hi ? r[1] : r[0];
+        r[0] = have + __shfl_xor_sync(0xffffffffu, give, 4);
       }
-      s[0] += __shfl_xor_sync(0xffffffffu, s[0], 2);
-      s[0] += __shfl_xor_sync(0xffffffffu, s[0], 1);
+      r[0] += __shfl_xor_sync(0xffffffffu, r[0], 2);
+      r[0] += __shfl_xor_sync(0xffffffffu, r[0], 1);
       const float fl = __shfl_sync(0xffffffffu, floor_, tok);
       const int c = c_lo + ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);
+      const float read = r[0] * A.q_scale;
       if ((lane & 3) == 0 && c <= e)
-        reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row0 + base + tok) * H + head) * (e + 1) + c] =
-            c < e ? s[0] : fmaxf(fabsf(s[0]), fl) + 1e-6f;
+        reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row0 + base + tok) * H + head) * oe + c] =
+            c < e ? read : fmaxf(fabsf(read), fl) + 1e-6f;
     }
+    gi = gi_next;
+    gf = gf_next;
+    exec_sync();
   }
 #pragma unroll
   for (int c = 0; c < 8; ++c)
@@ -225,36 +290,111 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
 }
 
 __device__ bool tile_memory(const TileDesc& t, int tid, uint8_t* ring) {
-  const uint32_t d = __ldcg(&reinterpret_cast<const MemoryArgs*>(t.a[0])->d);
-  if (d <= 128) memory_rows<1>(t, tid, ring);
-  else if (d <= 256) memory_rows<2>(t, tid, ring);
-  else if (d <= 512) memory_rows<4>(t, tid, ring);
-  else return false;
-  return true;
+  const MemoryArgs* p = reinterpret_cast<const MemoryArgs*>(t.a[0]);
+  const uint32_t d = __ldcg(&p->d);
+  const bool f32 = __ldcg(&p->f32) != 0;
+#define MF_MEMORY(N)                             \
+  if (d <= 128 * N) {                            \
+    if (f32) memory_rows<N, true>(t, tid, ring); \
+    else memory_rows<N, false>(t, tid, ring);    \
+    return true;                                 \
+  }
+  MF_MEMORY(1)
+  MF_MEMORY(2)
+  MF_MEMORY(4)
+#undef MF_MEMORY
+  return false;
 }
 
-// Kind 58, HeadNormArgs: items [i0, i0 + i1), item = row * heads + head, one warp each: the head's output over its
-// denominator, over its root mean square, times the norm weight and sigmoid(g).
-__device__ void tile_head_norm(const TileDesc& t, int tid) {
+// Kind 58, HeadNormArgs: items [i0, i0 + i1), item = row * heads + head, one warp each: the head's read-out over its
+// denominator, over its root mean square, times the norm weight and sigmoid(g).  An item of `o` is e values, the
+// denominator, and padding to a multiple of four.
+template <int V>
+__device__ __noinline__ void head_norm_items(const TileDesc& t, int tid) {
+  constexpr int NV = 8;   // V-element pieces per lane kept in registers
   HeadNormArgs A;
   load_block(A, t.a[0]);
-  const int warp = tid >> 5, lane = tid & 31, e = static_cast<int>(A.e);
+  const int warp = tid >> 5, lane = tid & 31, e = static_cast<int>(A.e), oe = (e + 4) & ~3;
+  const bool f32 = A.f32 != 0;
   for (uint32_t it = t.i0 + warp; it < t.i0 + t.i1; it += kExecThreads / 32) {
     const uint32_t row = it / A.heads, head = it % A.heads;
-    const float* o = f32p(A.o) + static_cast<size_t>(it) * (e + 1);
-    const float inv_den = 1.f / o[e];
-    float ss = 0.f;
-    for (int c = lane; c < e; c += 32) {
-      const float v = o[c] * inv_den;
-      ss = fmaf(v, v, ss);
-    }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(e) + A.eps);
+    const float* o = f32p(A.o) + static_cast<size_t>(it) * oe;
     const size_t g0 = static_cast<size_t>(row) * A.ld_g + head * e, o0 = static_cast<size_t>(row) * A.ld_out + head * e;
-    for (int c = lane; c < e; c += 32) {
-      const float g = act_ld(A.g, g0 + c, A.f32);
-      act_st(A.out, o0 + c, A.f32, o[c] * inv_den * inv * f32p(A.w)[head * e + c] * sigmoid32(g));
+    const float* w = f32p(A.w) + head * e;
+    const float inv_den = 1.f / o[e];
+    auto gate = [&](int c, float (&g)[V]) {
+      if constexpr (V == 4) {
+        if (!f32) {
+          const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(A.g) + g0 + c);
+          const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+          const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+          g[0] = a.x; g[1] = a.y; g[2] = b.x; g[3] = b.y;
+          return;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) g[j] = act_ld(A.g, g0 + c + j, f32);
+    };
+    auto put = [&](int c, const float (&v)[V], const float (&g)[V], const float (&ww)[V], float inv) {
+      float x[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] = v[j] * inv_den * inv * ww[j] * (f32 ? sigmoid32(g[j]) : __fdividef(1.f, 1.f + __expf(-g[j])));
+      if constexpr (V == 4) {
+        if (!f32) {
+          const __nv_bfloat162 q[2] = {__floats2bfloat162_rn(x[0], x[1]), __floats2bfloat162_rn(x[2], x[3])};
+          *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(A.out) + o0 + c) = *reinterpret_cast<const uint2*>(q);
+          return;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) act_st(A.out, o0 + c + j, f32, x[j]);
+    };
+    float ss = 0.f;
+    if (e <= 32 * V * NV) {
+      float v[NV][V], g[NV][V], ww[NV][V];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * 32 + lane) * V;
+        if (c < e) {
+          ld_vec<V>(o + c, v[i]);
+          gate(c, g[i]);
+          ld_vec<V>(w + c, ww[i]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if ((i * 32 + lane) * V < e)
+#pragma unroll
+          for (int j = 0; j < V; ++j) ss = fmaf(v[i][j] * inv_den, v[i][j] * inv_den, ss);
+      const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(e) + A.eps);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * 32 + lane) * V;
+        if (c < e) put(c, v[i], g[i], ww[i], inv);
+      }
+    } else {
+      for (int c = lane * V; c < e; c += 32 * V) {
+        float v[V];
+        ld_vec<V>(o + c, v);
+#pragma unroll
+        for (int j = 0; j < V; ++j) ss = fmaf(v[j] * inv_den, v[j] * inv_den, ss);
+      }
+      const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(e) + A.eps);
+      for (int c = lane * V; c < e; c += 32 * V) {
+        float v[V], g[V], ww[V];
+        ld_vec<V>(o + c, v);
+        gate(c, g);
+        ld_vec<V>(w + c, ww);
+        put(c, v, g, ww, inv);
+      }
     }
   }
+}
+
+__device__ void tile_head_norm(const TileDesc& t, int tid) {
+  const HeadNormArgs* p = reinterpret_cast<const HeadNormArgs*>(t.a[0]);
+  if ((__ldcg(&p->e) & 3) == 0 && (__ldcg(&p->g) & 7) == 0) head_norm_items<4>(t, tid);
+  else head_norm_items<1>(t, tid);
 }
 
 }  // namespace fab

@@ -28,15 +28,21 @@ __device__ void tile_product32(const TileDesc& t, int tid, int* scratch) {
       sw[lr * LD + lk + i] = (lr < cols && k < K) ? act_ld(w, static_cast<size_t>(t.i2 + lr) * A.ld_w + k, false) : 0.f;
     }
     exec_sync();
+    float part[2][4] = {};   // sums of KC products are added up, not single products: the rounding of a long sum stays small
 #pragma unroll
     for (int k = 0; k < KC; ++k) {
       const float x0 = sx[r * LD + k], x1 = sx[(r + 1) * LD + k];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float wv = sw[(c + j) * LD + k];
-        acc[0][j] = fmaf(x0, wv, acc[0][j]);
-        acc[1][j] = fmaf(x1, wv, acc[1][j]);
+        part[0][j] = fmaf(x0, wv, part[0][j]);
+        part[1][j] = fmaf(x1, wv, part[1][j]);
       }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      acc[0][j] += part[0][j];
+      acc[1][j] += part[1][j];
     }
     exec_sync();
   }
@@ -61,20 +67,40 @@ __device__ void tile_gated_act(const TileDesc& t, int tid) {
   }
 }
 
-// Kind 62, SumArgs: rows [i0, i0 + i1).
-__device__ void tile_sum_slabs(const TileDesc& t, int tid) {
+// Kind 62, SumArgs: rows [i0, i0 + i1), V columns at a time.
+template <int V>
+__device__ __noinline__ void sum_rows(const TileDesc& t, int tid) {
   SumArgs A;
   load_block(A, t.a[0]);
   const size_t slab = static_cast<size_t>(A.part_rows) * A.ld_in;
-  const uint32_t n = t.i1 * A.cols;
+  const uint32_t per = A.cols / V, n = t.i1 * per;
   for (uint32_t i = tid; i < n; i += kExecThreads) {
-    const uint32_t r = t.i0 + i / A.cols, c = i % A.cols;
+    const uint32_t r = t.i0 + i / per, c = (i % per) * V;
     const float* in = f32p(A.in) + static_cast<size_t>(r) * A.ld_in + c;
-    float v = __ldcg(in);
-    for (uint32_t q = 1; q < A.parts; ++q) v += __ldcg(in + q * slab);
-    if (A.out32) reinterpret_cast<float*>(A.out32)[static_cast<size_t>(r) * A.ld_32 + c] = v;
-    if (c < A.c16) reinterpret_cast<__nv_bfloat16*>(A.out16)[static_cast<size_t>(r) * A.ld_16 + c] = __float2bfloat16(v);
+    float v[V];
+    ld_vec<V>(in, v);
+    for (uint32_t q0 = 1; q0 < A.parts; q0 += 4) {
+      float b[4][V];
+#pragma unroll
+      for (uint32_t q = 0; q < 4; ++q) ld_vec<V>(in + min(q0 + q, A.parts - 1) * slab, b[q]);
+#pragma unroll
+      for (uint32_t q = 0; q < 4; ++q)
+        if (q0 + q < A.parts)
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] += b[q][j];
+    }
+    if (A.out32) st_vec<V>(reinterpret_cast<float*>(A.out32) + static_cast<size_t>(r) * A.ld_32 + c, v);
+    __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(A.out16) + static_cast<size_t>(r) * A.ld_16 + c;
+#pragma unroll
+    for (int j = 0; j < V; ++j)
+      if (c + j < A.c16) o[j] = __float2bfloat16(v[j]);
   }
+}
+
+__device__ void tile_sum_slabs(const TileDesc& t, int tid) {
+  const SumArgs* p = reinterpret_cast<const SumArgs*>(t.a[0]);
+  if (((__ldcg(&p->cols) | __ldcg(&p->ld_in)) & 3) == 0) sum_rows<4>(t, tid);
+  else sum_rows<1>(t, tid);
 }
 
 // ------------------------------------------------------------------ residual streams
@@ -260,13 +286,14 @@ __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx) 
     case kTileGatedAct: tile_gated_act(t, tid); return true;
     case kTileStreams: tile_streams(t, tid, scratch); return true;
     case kTileConv: tile_conv(t, tid); return true;
-    case kTileScan: return tile_scan(t, tid);
+    case kTileScan: return tile_scan(t, tid, ctx.ring);
     case kTileMemGates: tile_mem_gates(t, tid); return true;
     case kTileMemory: return tile_memory(t, tid, ctx.ring);
     case kTileHeadNorm: tile_head_norm(t, tid); return true;
     case kTileLatentKv: tile_latent_kv(t, tid); return true;
     case kTileLatentAttn: return tile_latent_attn(t, tid);
     case kTileLatentMma: return tile_latent_mma(t, tid, ctx);
+    case kTileLatentDirect: return tile_latent_direct(t, tid, ctx);
     case kTileLatentMerge: tile_latent_merge(t, tid); return true;
     case kTileSumSlabs: tile_sum_slabs(t, tid); return true;
     default: return false;

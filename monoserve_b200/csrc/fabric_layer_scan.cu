@@ -1,77 +1,90 @@
 // Short convolution and selective scan of the layer-list decoders (fabric_layer_tiles.cuh).
 #include "fabric_layer_tiles.cuh"
+#include "wide_tile.cuh"
 
 namespace mf {
 namespace fab {
 
 // ------------------------------------------------------------------ short convolution
 // Kind 54, ConvArgs: i0 the request's first row, i1 first row of this tile, i2 rows | channels << 16, i3 slot,
-// a[1] first channel.  A thread walks down one channel (two in bf16) with the last `taps` inputs in registers.
-template <bool F32, int V>
+// a[1] first channel.  A thread walks down V channels with the last TAPS - 1 inputs in registers, eight rows' loads in
+// flight.  V = 8: bf16 rows in 16-byte pieces.
+template <bool F32, int V, int TAPS>
 __device__ __noinline__ void conv_rows(const TileDesc& t, int tid) {
   ConvArgs A;
   load_block(A, t.a[0]);
-  const int row0 = static_cast<int>(t.i0), r_lo = static_cast<int>(t.i1), rows = static_cast<int>(t.i2 & 0xffffu);
+  const int row0 = static_cast<int>(t.i0), r_lo = static_cast<int>(t.i1), r_hi = r_lo + static_cast<int>(t.i2 & 0xffffu);
   const int n_ch = static_cast<int>(t.i2 >> 16), ch0 = static_cast<int>(t.a[1]), taps = static_cast<int>(A.taps);
   const int C = static_cast<int>(A.channels);
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
   const float* tail = f32p(A.tail) + static_cast<size_t>(t.i3) * (taps - 1) * C;
-  auto load = [&](int r, int c, float (&v)[V]) {   // the input at row r of the portion, r < row0: before it
-    if (r < row0) {
-      const int k = r - row0 + taps - 1;   // place in the tail
+  using Raw = typename std::conditional<V == 8, uint4, float>::type;
+  auto load = [&](int r, int c) -> Raw {   // row r >= row0
+    const size_t at = static_cast<size_t>(r) * A.ld_x + c;
+    if constexpr (V == 8) return *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(A.x) + at);
+    else return act_ld(A.x, at, F32);
+  };
+  auto unpack = [&](const Raw& raw, float (&v)[V]) {
+    if constexpr (V == 8) {
+      const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
-      for (int j = 0; j < V; ++j) v[j] = (fresh || k < 0) ? 0.f : tail[static_cast<size_t>(k) * C + c + j];
-    } else if constexpr (!F32 && V == 2) {
-      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(
-          reinterpret_cast<const __nv_bfloat16*>(A.x) + static_cast<size_t>(r) * A.ld_x + c));
-      v[0] = f.x; v[1] = f.y;
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        v[2 * i] = f.x;
+        v[2 * i + 1] = f.y;
+      }
     } else {
-#pragma unroll
-      for (int j = 0; j < V; ++j) v[j] = act_ld(A.x, static_cast<size_t>(r) * A.ld_x + c + j, F32);
+      v[0] = raw;
     }
   };
   for (int c = ch0 + tid * V; c < ch0 + n_ch; c += kExecThreads * V) {
-    float w[kMaxTaps][V], bias[V], win[kMaxTaps][V];   // win: the inputs at rows r - 7 .. r, newest last
+    float w[TAPS][V], bias[V], win[TAPS][V];   // win: the inputs at rows r - TAPS + 1 .. r, newest last
 #pragma unroll
-    for (int k = 0; k < kMaxTaps; ++k) {
-      const int tap = k - (kMaxTaps - taps);
+    for (int k = 0; k < TAPS; ++k) {
+      const int tap = k - (TAPS - taps);
 #pragma unroll
       for (int j = 0; j < V; ++j) w[k][j] = tap >= 0 ? f32p(A.w)[static_cast<size_t>(c + j) * taps + tap] : 0.f;
     }
 #pragma unroll
     for (int j = 0; j < V; ++j) bias[j] = f32p(A.bias)[c + j];
 #pragma unroll
-    for (int k = 0; k < kMaxTaps - 1; ++k) {
-      if (k >= kMaxTaps - taps) load(r_lo - (kMaxTaps - 1) + k, c, win[k + 1]);
-      else
+    for (int k = 1; k < TAPS; ++k) {
+      const int r = r_lo - TAPS + k, place = r - row0 + taps - 1;   // place in the tail, for rows before the portion
+      if (r >= row0) {
+        unpack(load(r, c), win[k]);
+      } else {
 #pragma unroll
-        for (int j = 0; j < V; ++j) win[k + 1][j] = 0.f;
+        for (int j = 0; j < V; ++j) win[k][j] = (fresh || place < 0) ? 0.f : tail[static_cast<size_t>(place) * C + c + j];
+      }
     }
-    for (int r = r_lo; r < r_lo + rows; r += 8) {
-      float in[8][V];
+    for (int r = r_lo; r < r_hi; r += 8) {
+      Raw in[8];
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
-        if (r + i < r_lo + rows) load(r + i, c, in[i]);
+      for (int i = 0; i < 8; ++i) in[i] = load(min(r + i, r_hi - 1), c);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        if (r + i >= r_lo + rows) break;
-        float o[V];
+        if (r + i >= r_hi) break;
+        float x[V], o[V];
+        unpack(in[i], x);
 #pragma unroll
         for (int j = 0; j < V; ++j) {
 #pragma unroll
-          for (int k = 0; k < kMaxTaps - 1; ++k) win[k][j] = win[k + 1][j];
-          win[kMaxTaps - 1][j] = in[i][j];
+          for (int k = 0; k < TAPS - 1; ++k) win[k][j] = win[k + 1][j];
+          win[TAPS - 1][j] = x[j];
           float acc = bias[j];
 #pragma unroll
-          for (int k = 0; k < kMaxTaps; ++k) acc = fmaf(w[k][j], win[k][j], acc);
-          o[j] = acc / (1.f + expf(-acc));
+          for (int k = 0; k < TAPS; ++k) acc = fmaf(w[k][j], win[k][j], acc);
+          o[j] = F32 ? acc / (1.f + expf(-acc)) : __fdividef(acc, 1.f + __expf(-acc));
         }
         const size_t at = static_cast<size_t>(r + i) * A.ld_out + c;
-        if constexpr (!F32 && V == 2)
-          *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(A.out) + at) = __floats2bfloat162_rn(o[0], o[1]);
-        else
+        if constexpr (V == 8) {
+          __nv_bfloat162 h[4];
 #pragma unroll
-          for (int j = 0; j < V; ++j) act_st(A.out, at + j, F32, o[j]);
+          for (int j = 0; j < 4; ++j) h[j] = __floats2bfloat162_rn(o[2 * j], o[2 * j + 1]);
+          *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(A.out) + at) = *reinterpret_cast<const uint4*>(h);
+        } else {
+          act_st(A.out, at, F32, o[0]);
+        }
       }
     }
   }
@@ -79,29 +92,48 @@ __device__ __noinline__ void conv_rows(const TileDesc& t, int tid) {
 
 __device__ void tile_conv(const TileDesc& t, int tid) {
   const ConvArgs* p = reinterpret_cast<const ConvArgs*>(t.a[0]);
-  const uint32_t f32 = __ldcg(&p->f32), C = __ldcg(&p->channels);
-  if (f32) conv_rows<true, 1>(t, tid);
-  else if ((C & 1) == 0) conv_rows<false, 2>(t, tid);
-  else conv_rows<false, 1>(t, tid);
+  const uint32_t taps = __ldcg(&p->taps);
+  if (__ldcg(&p->f32)) conv_rows<true, 1, kMaxTaps>(t, tid);
+  else if ((__ldcg(&p->channels) & 7) != 0) conv_rows<false, 1, kMaxTaps>(t, tid);
+  else if (taps <= 4) conv_rows<false, 8, 4>(t, tid);
+  else conv_rows<false, 8, kMaxTaps>(t, tid);
 }
 
 // ------------------------------------------------------------------ selective scan
-// Kind 55, ScanArgs: rows [i0, i0 + i1) of one request, channels [i2, i2 + 32) (as many as there are), slot i3.
-// Four lanes share a channel, each with NS of its states.  Four tokens at a time: lane p loads, prepares and
-// finishes token p of the four (step size, input, output gate), so what a channel needs once per token is computed
-// once; the four state updates of a token run in all lanes.  The loads of the next four tokens are issued before
-// the current four are computed.
-// F32: the exact form.  It multiplies by e^x as S + S (e^x - 1), so that the rounding of a factor just below one does
-// not add up over a long memory.
+// Kind 55, ScanArgs: rows [i0, i0 + i1) of one request, channels [i2, i2 + 32) (as many as there are), slot i3.  A wide
+// tile: the inputs come 32 tokens at a time through double-buffered asynchronous copies into the operand ring.  Four
+// lanes share a channel, each with NS of its states in registers.  Four tokens at a time: lane p prepares and finishes
+// token p of the four (step size, output gate), so what a channel needs once per token is computed once; the four state
+// updates of a token run in all lanes.  F32: the exact form.  It multiplies by e^x as S + S (e^x - 1), so that the
+// rounding of a factor just below one does not add up over a long memory.
+constexpr int kScanTokens = 32, kScanChannels = kExecThreads / 4;
+
 template <int NS, bool F32>
-__device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
+__device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring) {
+  using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
+  constexpr int NP = 4 * NS;                              // states, padded
+  constexpr int kPer16 = 16 / static_cast<int>(sizeof(T));
+  struct Chunk {
+    float dt[kScanTokens][kScanChannels];
+    float bc[kScanTokens][2 * NP];                        // B, then C
+    T x[kScanTokens][kScanChannels];
+    T z[kScanTokens][kScanChannels];
+  };
+  struct Shared {
+    Chunk in[2];
+    T y[kScanTokens][kScanChannels];
+  };
+  static_assert(sizeof(Shared) <= 216 * 1024, "the operand ring");
+  __builtin_assume(__isShared(ring));
+  Shared& sh = *reinterpret_cast<Shared*>(ring);
   ScanArgs A;
   load_block(A, t.a[0]);
   const int row0 = static_cast<int>(t.i0), rows = static_cast<int>(t.i1), slot = static_cast<int>(t.i3);
+  const int ch0 = static_cast<int>(t.i2);
   const int n = static_cast<int>(A.n), C = static_cast<int>(A.channels), taps = static_cast<int>(A.taps);
-  const int p = tid & 3, lane = tid & 31, quad = lane & ~3;
-  const int c = min(static_cast<int>(t.i2) + (tid >> 2), C - 1);   // a channel past the end repeats the last one
-  const bool c_ok = static_cast<int>(t.i2) + (tid >> 2) < C;
+  const int warp = tid >> 5, lane = tid & 31, p = tid & 3, quad = lane & ~3, my = tid >> 2;
+  const int c = min(ch0 + my, C - 1);                     // a channel past the end repeats the last one
+  const bool c_ok = ch0 + my < C;
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
   const int s0 = p * NS;
   float S[NS], a[NS];
@@ -110,81 +142,121 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
   for (int i = 0; i < NS; ++i) {
     const bool ok = s0 + i < n;
     S[i] = (ok && !fresh) ? state[s0 + i] : 0.f;
-    a[i] = ok ? f32p(A.A)[static_cast<size_t>(c) * n + s0 + i] : 0.f;
+    a[i] = ok ? f32p(A.A)[static_cast<size_t>(c) * n + s0 + i] * (F32 ? 1.f : 1.4426950408889634f) : 0.f;
   }
   const float D = f32p(A.D)[c], dt_bias = f32p(A.dt_bias)[c];
-  struct Four {
-    float dt, x, z;
-    float B[4][NS], Cc[4][NS];
+  const bool z16 = (A.z & 15) == 0, bc16 = ((A.b | A.c) & 15) == 0 && (n & 3) == 0;
+  if (n < NP) {   // the padding of B and C stays zero
+    for (int i = tid; i < 2 * kScanTokens * 2 * NP; i += kExecThreads)
+      (&sh.in[i / (kScanTokens * 2 * NP)].bc[0][0])[i % (kScanTokens * 2 * NP)] = 0.f;
+    exec_sync();
+  }
+  auto stage = [&](int base, Chunk& k) {
+    const int nt = min(kScanTokens, rows - base);
+    const T* x = reinterpret_cast<const T*>(A.x);
+    const T* z = reinterpret_cast<const T*>(A.z);
+    // rows of 32 channels: 8 pieces of dt, 32 / kPer16 of x and of z; rows are padded, so whole pieces may be read
+    constexpr int kPieces = 8 + kScanChannels / kPer16;
+    for (int i = tid; i < nt * kPieces; i += kExecThreads) {
+      const int tok = i / kPieces, q = i - tok * kPieces;
+      const size_t r = static_cast<size_t>(row0 + base + tok);
+      if (q < 8) cp16(&k.dt[tok][4 * q], f32p(A.dt) + r * A.ld_dt + ch0 + 4 * q);
+      else cp16(&k.x[tok][(q - 8) * kPer16], x + r * A.ld_x + ch0 + (q - 8) * kPer16);
+    }
+    if (z16) {
+      constexpr int kZ = kScanChannels / kPer16;
+      for (int i = tid; i < nt * kZ; i += kExecThreads)
+        cp16(&k.z[i / kZ][(i % kZ) * kPer16], z + static_cast<size_t>(row0 + base + i / kZ) * A.ld_z + ch0 + (i % kZ) * kPer16);
+    } else {
+      for (int tok = warp; tok < nt; tok += kExecThreads / 32)
+        k.z[tok][lane] = z[static_cast<size_t>(row0 + base + tok) * A.ld_z + min(ch0 + lane, C - 1)];
+    }
+    if (bc16) {
+      const int np = n >> 2;
+      for (int tok = warp; tok < nt; tok += kExecThreads / 32) {
+        const size_t at = static_cast<size_t>(row0 + base + tok) * A.ld_bc;
+        for (int q = lane; q < 2 * np; q += 32) {
+          const bool second = q >= np;
+          const int k4 = 4 * (second ? q - np : q);
+          cp16(&k.bc[tok][(second ? NP : 0) + k4], f32p(second ? A.c : A.b) + at + k4);
+        }
+      }
+    } else {
+      for (int tok = warp; tok < nt; tok += kExecThreads / 32) {
+        const size_t at = static_cast<size_t>(row0 + base + tok) * A.ld_bc;
+        for (int q = lane; q < n; q += 32) {
+          k.bc[tok][q] = f32p(A.b)[at + q];
+          k.bc[tok][NP + q] = f32p(A.c)[at + q];
+        }
+      }
+    }
+    cp_commit();
   };
-  const bool vec = (NS & 3) == 0 && n == 4 * NS && (A.ld_bc & 3) == 0 && ((A.b | A.c) & 15) == 0;
-  auto fetch = [&](int r, Four& f) {
-    const int mine = min(r + p, row0 + rows - 1);   // rows past the end repeat the last one and are not used
-    f.dt = f32p(A.dt)[static_cast<size_t>(mine) * A.ld_dt + c];
-    f.x = act_ld(A.x, static_cast<size_t>(mine) * A.ld_x + c, F32);
-    f.z = act_ld(A.z, static_cast<size_t>(mine) * A.ld_z + c, F32);
+  auto value = [](const T& v) -> float {
+    if constexpr (F32) return v;
+    else return __bfloat162float(v);
+  };
+  stage(0, sh.in[0]);
+  for (int base = 0, s = 0; base < rows; base += kScanTokens, s ^= 1) {
+    const int nt = min(kScanTokens, rows - base);
+    if (base + kScanTokens < rows) {
+      stage(base + kScanTokens, sh.in[s ^ 1]);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    exec_sync();
+    const Chunk& k = sh.in[s];
+    for (int t0 = 0; t0 < nt; t0 += 4) {
+      const int mine = min(t0 + p, nt - 1);
+      const float x = value(k.x[mine][my]), z = value(k.z[mine][my]);
+      const float u = k.dt[mine][my] + dt_bias;
+      const float dt = F32 ? softplus32(u) : fmaxf(u, 0.f) + __logf(1.f + __expf(-fabsf(u)));
+      const float dtx = dt * x;
+      float out = 0.f;
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const size_t at = static_cast<size_t>(min(r + k, row0 + rows - 1)) * A.ld_bc + s0;
-      const float *b = f32p(A.b) + at, *cc = f32p(A.c) + at;
-      if (vec) {
-        if constexpr ((NS & 3) == 0) {
+      for (int i4 = 0; i4 < 4; ++i4) {
+        if (t0 + i4 < nt) {   // the same in all threads
+          const float dk = __shfl_sync(0xffffffffu, dt, quad + i4), xk = __shfl_sync(0xffffffffu, dtx, quad + i4);
+          float B[NS], Cv[NS];
+          const float *b = &k.bc[t0 + i4][s0], *cc = &k.bc[t0 + i4][NP + s0];
+          if constexpr ((NS & 3) == 0) {
 #pragma unroll
-          for (int i = 0; i < NS; i += 4) {
-            ld_vec<4>(b + i, *reinterpret_cast<float(*)[4]>(&f.B[k][i]));
-            ld_vec<4>(cc + i, *reinterpret_cast<float(*)[4]>(&f.Cc[k][i]));
+            for (int i = 0; i < NS; i += 4) {
+              ld_vec<4>(b + i, *reinterpret_cast<float(*)[4]>(&B[i]));
+              ld_vec<4>(cc + i, *reinterpret_cast<float(*)[4]>(&Cv[i]));
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < NS; ++i) {
+              B[i] = b[i];
+              Cv[i] = cc[i];
+            }
           }
-        }
-      } else {
+          float y = 0.f;
 #pragma unroll
-        for (int i = 0; i < NS; ++i) {
-          f.B[k][i] = s0 + i < n ? b[i] : 0.f;
-          f.Cc[k][i] = s0 + i < n ? cc[i] : 0.f;
+          for (int i = 0; i < NS; ++i) {
+            if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), xk * B[i]);
+            else S[i] = fmaf(ex2(dk * a[i]), S[i], xk * B[i]);
+            y = fmaf(S[i], Cv[i], y);
+          }
+          y += __shfl_xor_sync(0xffffffffu, y, 1);
+          y += __shfl_xor_sync(0xffffffffu, y, 2);
+          if (i4 == p) out = y;
         }
       }
-    }
-  };
-  auto run = [&](int r, const Four& f) {
-    const float dt = softplus32(f.dt + dt_bias), dtx = dt * f.x;
-    float mine = 0.f;
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      if (r + k < row0 + rows) {
-        const float dk = __shfl_sync(0xffffffffu, dt, quad + k), xk = __shfl_sync(0xffffffffu, dtx, quad + k);
-        float y = 0.f;
-#pragma unroll
-        for (int i = 0; i < NS; ++i) {
-          if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), xk * f.B[k][i]);
-          else S[i] = fmaf(expf(dk * a[i]), S[i], xk * f.B[k][i]);
-          y = fmaf(S[i], f.Cc[k][i], y);
-        }
-        y += __shfl_xor_sync(0xffffffffu, y, 1);
-        y += __shfl_xor_sync(0xffffffffu, y, 2);
-        if (k == p) mine = y;
+      if (t0 + p < nt) {
+        const float y = fmaf(D, x, out) * (F32 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)));
+        if constexpr (F32) sh.y[t0 + p][my] = y;
+        else sh.y[t0 + p][my] = __float2bfloat16(y);
       }
     }
-    if (c_ok && r + p < row0 + rows) {
-      const float y = fmaf(D, f.x, mine);
-      act_st(A.y, static_cast<size_t>(r + p) * A.ld_y + c, F32, y * (f.z / (1.f + expf(-f.z))));
-    }
-  };
-  if constexpr (NS <= 8) {
-    Four f0, f1;
-    fetch(row0, f0);
-    for (int r = row0; r < row0 + rows; r += 8) {
-      if (r + 4 < row0 + rows) fetch(r + 4, f1);
-      run(r, f0);
-      if (r + 4 < row0 + rows) {
-        if (r + 8 < row0 + rows) fetch(r + 8, f0);
-        run(r + 4, f1);
-      }
-    }
-  } else {
-    Four f0;
-    for (int r = row0; r < row0 + rows; r += 4) {
-      fetch(r, f0);
-      run(r, f0);
-    }
+    exec_sync();
+    // rows of y are padded to whole pieces
+    constexpr int kY = kScanChannels / kPer16;
+    for (int i = tid; i < nt * kY; i += kExecThreads)
+      *reinterpret_cast<uint4*>(reinterpret_cast<T*>(A.y) + static_cast<size_t>(row0 + base + i / kY) * A.ld_y + ch0 + (i % kY) * kPer16) =
+          *reinterpret_cast<const uint4*>(&sh.y[i / kY][(i % kY) * kPer16]);
   }
 #pragma unroll
   for (int i = 0; i < NS; ++i)
@@ -201,15 +273,15 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid) {
   }
 }
 
-__device__ bool tile_scan(const TileDesc& t, int tid) {
+__device__ bool tile_scan(const TileDesc& t, int tid, uint8_t* ring) {
   const ScanArgs* p = reinterpret_cast<const ScanArgs*>(t.a[0]);
   const uint32_t ns = (__ldcg(&p->n) + 3) / 4;
   const bool f32 = __ldcg(&p->f32) != 0;
-#define MF_SCAN(N)                       \
-  if (ns <= N) {                         \
-    if (f32) scan_rows<N, true>(t, tid); \
-    else scan_rows<N, false>(t, tid);    \
-    return true;                         \
+#define MF_SCAN(N)                             \
+  if (ns <= N) {                               \
+    if (f32) scan_rows<N, true>(t, tid, ring); \
+    else scan_rows<N, false>(t, tid, ring);    \
+    return true;                               \
   }
   MF_SCAN(1)
   MF_SCAN(2)

@@ -13,6 +13,8 @@
 #pragma once
 #include <cuda_bf16.h>
 
+#include <type_traits>
+
 #include "fabric_types.h"
 #include "operands.h"
 
@@ -33,12 +35,12 @@ struct LayerCtx {
   volatile int* abort_flag;
 };
 
-// Runs tile kinds kTileProduct32 .. kTileLatentMma: false for a kind or size these tiles do not take, or when a bounded
+// Runs tile kinds kTileProduct32 .. kTileLatentDirect: false for a kind or size these tiles do not take, or when a bounded
 // wait gave up.  All exec threads call it with the same tile.
 __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx);
 // Wide tiles: their exec warps use the operand ring as scratch memory, and TMEM.
 __device__ __forceinline__ bool tile_is_wide(uint32_t kind) {
-  return kind == kTileMemory || kind == kTileLatentMma;
+  return kind == kTileMemory || kind == kTileScan || kind == kTileLatentMma || kind == kTileLatentDirect;
 }
 
 __device__ void tile_streams(const TileDesc& t, int tid, int* scratch);
@@ -46,13 +48,14 @@ __device__ void tile_product32(const TileDesc& t, int tid, int* scratch);
 __device__ void tile_gated_act(const TileDesc& t, int tid);
 __device__ void tile_sum_slabs(const TileDesc& t, int tid);
 __device__ void tile_conv(const TileDesc& t, int tid);
-__device__ bool tile_scan(const TileDesc& t, int tid);
+__device__ bool tile_scan(const TileDesc& t, int tid, uint8_t* ring);
 __device__ void tile_mem_gates(const TileDesc& t, int tid);
 __device__ bool tile_memory(const TileDesc& t, int tid, uint8_t* ring);
 __device__ void tile_head_norm(const TileDesc& t, int tid);
 __device__ void tile_latent_kv(const TileDesc& t, int tid);
 __device__ bool tile_latent_attn(const TileDesc& t, int tid);
 __device__ bool tile_latent_mma(const TileDesc& t, int tid, const LayerCtx& ctx);
+__device__ bool tile_latent_direct(const TileDesc& t, int tid, const LayerCtx& ctx);
 __device__ void tile_latent_merge(const TileDesc& t, int tid);
 
 __device__ __forceinline__ void exec_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kExecThreads) : "memory"); }

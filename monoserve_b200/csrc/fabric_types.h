@@ -60,6 +60,7 @@ enum TileKind : uint16_t {
   kTileLatentMerge = 61,    // merge of the key ranges
   kTileSumSlabs = 62,       // sum of a K-split product's slabs
   kTileLatentMma = 63,      // attention over the cached latents on the tensor cores: heads x tokens, one key range
+  kTileLatentDirect = 64,   // the same for a whole prompt, with keys and values mapped out of the latents
 };
 constexpr int kFabChunk = 16;   // rows per router / permute tile = rank chunk of the stable pack
 

@@ -115,8 +115,8 @@ namespace mf {
 #define MF_MEM_GATE_ARGS(U64, U32, F32) \
   U64(h) U64(wi) U64(wf) U64(bi) U64(bf) U64(out) U32(K) U32(heads) U32(ld_h) F32(cap)
 
-/* state fp32 [slot][head][e + 1][d] (column e: the normaliser), m fp32 [slot][head]; out fp32 [rows][heads][e + 1],
- * its last column the denominator. */
+/* state fp32 [slot][head][e + 1][d] (column e: the normaliser), m fp32 [slot][head][column
+ * block]; out fp32 [rows][heads][e, the denominator, padding to a multiple of four]. */
 #define MF_MEMORY_ARGS(U64, U32, F32) \
   U64(q) U64(k) U64(v) U64(gates) U64(state) U64(m) U64(out) U64(tok_pos) U32(ld_qkv) U32(heads) U32(d) U32(e) \
   U32(f32) F32(q_scale)
@@ -126,10 +126,10 @@ namespace mf {
 
 /* qc fp32 [rows][heads * (d + r) | kv_rank | r]: queries, latent, shared rotated key part.  q_un [head][rows_max][ld_un]
  * unrotated query parts; q_all [head][rows_max][ld_q] = kv_rank absorbed columns (written by a product) then r rotated
- * ones; cache [page slots][ld_cache]. */
+ * ones; cache [page slots][ld_cache]; rows (optional) [rows][ld_rows]: a copy of the cached rows in token order. */
 #define MF_LATENT_ARGS(U64, U32, F32) \
-  U64(qc) U64(c_norm) U64(q_un) U64(q_all) U64(cache) U64(tok_pos) U64(tok_slot) U64(cos_sin) U32(ld_qc) U32(heads) \
-  U32(d) U32(r) U32(kv_rank) U32(ld_un) U32(ld_q) U32(rows_max) U32(ld_cache) U32(max_pos) U32(f32) F32(eps)
+  U64(qc) U64(c_norm) U64(q_un) U64(q_all) U64(cache) U64(rows) U64(tok_pos) U64(tok_slot) U64(cos_sin) U32(ld_qc) U32(heads) \
+  U32(d) U32(r) U32(kv_rank) U32(ld_un) U32(ld_q) U32(rows_max) U32(ld_cache) U32(ld_rows) U32(max_pos) U32(f32) F32(eps)
 
 /* ws_o fp32 [(row * heads + head) * parts + part][kv_rank], ws_ml float2 of the same rows.  For the tensor-core tile:
  * q_map dims (kv_rank + r, rows_max, heads), box (64, tokens, group); kv_map dims (64, 8, chunks, page slots / 8), box
@@ -138,6 +138,12 @@ namespace mf {
   U64(q) U64(cache) U64(block_table) U64(out) U64(ws_o) U64(ws_ml) U64(tok_pos) U64(q_map) U64(kv_map) U32(ld_q) \
   U32(heads) U32(kv_rank) U32(r) U32(ld_cache) U32(page) U32(bt_stride) U32(rows_max) U32(ld_out) U32(f32) F32(scale) \
   U32(tokens) U32(group) U32(buffers)
+
+/* Whole prompts: q_map dims (d, heads * rows_max) and qr_map (r, heads * rows_max), kv_map (heads * (d + e), rows): keys
+ * then values of every head, kr_map (r, rows); boxes (64, 128).  out bf16 [rows][ld_out], head h at column h e. */
+#define MF_LATENT_DIRECT_ARGS(U64, U32, F32) \
+  U64(q_map) U64(qr_map) U64(kv_map) U64(kr_map) U64(out) U32(d) U32(r) U32(e) U32(heads) U32(rows_max) U32(ld_out) \
+  U32(buffers) F32(scale)
 
 #define MF_FIELD_U64(name) unsigned long long name;
 #define MF_FIELD_U32(name) uint32_t name;
@@ -174,5 +180,6 @@ MF_DECLARE(MemoryArgs, MF_MEMORY_ARGS, 128)
 MF_DECLARE(HeadNormArgs, MF_HEAD_NORM_ARGS, 64)
 MF_DECLARE(LatentArgs, MF_LATENT_ARGS, 128)
 MF_DECLARE(LatentAttnArgs, MF_LATENT_ATTN_ARGS, 128)
+MF_DECLARE(LatentDirectArgs, MF_LATENT_DIRECT_ARGS, 128)
 
 }  // namespace mf

@@ -8,7 +8,8 @@ a span of layers may run several times in a row.
     selective scan:    in GEMM (32) -> conv + silu (54) -> x GEMM (K ranges) -> slab sum (62) -> dt GEMM -> scan (55) -> o GEMM
     matrix memory:     q k v g GEMM, gates (56) beside it -> memory (57) -> head norm (58) -> o GEMM
     latent attention:  q + latent GEMM -> latent norm, rotation, cache append (59) -> per head W_uk^T q GEMM ->
-                       attention over the cached latents (60, 61) -> per head W_uv GEMM -> o GEMM
+                       attention over the cached latents (63 on the tensor cores, 60 in 32-bit; 61) -> per head W_uv
+                       GEMM -> o GEMM; for a whole prompt: keys and values GEMM -> attention (64) -> o GEMM
   streams -> gate / up GEMM with the gelu epilogue -> down GEMM
   ... -> final streams (gather) -> head GEMM (fp32) -> sample (43)
 
@@ -32,12 +33,13 @@ from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_STORE, HEIGHTS,
                                       LaneBase, _block, _bm, _retarget)
 
 K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEM_GATES, K_MEMORY = 51, 52, 53, 54, 55, 56, 57
-K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA = 58, 59, 60, 61, 62, 63
+K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA, K_LATENT_DIRECT = 58, 59, 60, 61, 62, 63, 64
 MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
 SCAN_CHANNELS, MEMORY_COLUMNS = 32, 32   # of one tile
 WIDE_ROWS, WIDE_PARTS = 512, 4           # K ranges of the products that end a sublayer, up to this many rows
 MAX_ATTN_PARTS = 32
-RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys per step of the tensor-core attention tile
+RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys per step of the tensor-core attention tiles
+DIRECT_ROWS = 32                         # a prompt of at least this many tokens maps its keys and values out of the latents
 
 
 def up(n, m):
@@ -140,6 +142,14 @@ def latent_tile(m, page, tokens_per_request):
     return tokens, heads, 2 if room(cols, 2) else 1
 
 
+def direct_buffers(m):
+    """Key-tile buffers of the whole-prompt attention tile (kind 64), or 0 where its operands do not fit."""
+    if any(v % 8 for v in (m.dim, m.rot_dim, m.vdim, m.kv_rank)) or m.vdim > 256:
+        return 0
+    nq, ne, room = -(-m.dim // 64) + -(-m.rot_dim // 64), -(-m.vdim // 64), RING_BYTES // (KEY_TILE * 128)
+    return next((b for b in (2, 1) if nq * (1 + b) + ne + 2 <= room), 0)
+
+
 # ---------------------------------------------------------------------------------------------- mixers
 class SelectiveScan:
     """x, z = W_in h; x through a causal convolution per channel and silu; dt, B, C from x;
@@ -220,7 +230,7 @@ class MatrixMemory:
 
     @staticmethod
     def sizes(m):
-        return dict(proj=2 * m.heads * (m.dim + m.vdim), mix=m.heads * m.vdim, small=2 * m.heads, raw=m.heads * (m.vdim + 1),
+        return dict(proj=2 * m.heads * (m.dim + m.vdim), mix=m.heads * m.vdim, small=2 * m.heads, raw=m.heads * up(m.vdim + 1, 4),
                     h32=1)
 
     @staticmethod
@@ -260,6 +270,7 @@ class LatentAttention:
     @staticmethod
     def place(W, w, m, g):
         w.qkv, w.o, w.c_norm = W.mat(torch.cat([g("q"), g("dkv")])), W.mat(g("o")), W.f32(g("dkv.norm"))
+        w.ukv = W.mat(torch.cat([g("uk"), g("uv")]))
         w.uk = W.mat(g("uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2))    # [head][latent][dim]
         w.uv = W.mat(g("uv").view(m.heads, m.vdim, m.kv_rank))                   # [head][value][latent]
 
@@ -271,50 +282,77 @@ class LatentAttention:
     @staticmethod
     def sizes(m):
         return dict(qc=m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim, mix=m.heads * m.vdim,
-                    q_un=(m.heads, m.dim), q_all=(m.heads, m.kv_rank + m.rot_dim), o_lat=(m.heads, m.kv_rank),
+                    kvb=m.heads * (m.dim + m.vdim), c_rows=m.kv_rank + m.rot_dim, q_un=(m.heads, m.dim), q_all=(m.heads, m.kv_rank + m.rot_dim), o_lat=(m.heads, m.kv_rank),
                     ws=(m.heads, m.kv_rank))
 
     @staticmethod
     def build(lane, p, l, run, b, prev):
         m, w, st, T = lane.cfg.layers[l].m, lane.w.layers[l], lane.kv.runs[run], b.T
         f32, H, d, r, c = int(lane.cfg.f32), m.heads, m.dim, m.rot_dim, m.kv_rank
+        buffers = 0 if f32 else direct_buffers(m)
+        whole, rest = b.split() if buffers else ([], b)
         s = lane.product(p, prev, lane.h, w.qkv, lane.qc, T, H * (d + r) + c + r, lane.cfg.hidden, ("latent_in", run))
-        ld_q, ld_o = up(c + r, 8), up(c, 64)
+        ld_q = up(c + r, 8)
+        copy = dict(rows=lane.c_rows.addr, ld_rows=lane.c_rows.ld) if whole else {}
         kv = lane._dev("LatentArgs", qc=lane.qc.addr, c_norm=w.c_norm, q_un=lane.q_un.addr, q_all=lane.q_all.addr,
                        cache=st["cache"], tok_pos=lane.tok_pos, tok_slot=lane.tok_slot, cos_sin=lane.cos_sin(m.rot["base"], r),
                        ld_qc=lane.qc.ld, heads=H, d=d, r=r, kv_rank=c, ld_un=up(d, 64), ld_q=ld_q, rows_max=lane.T,
-                       ld_cache=st["cache"].shape[1], max_pos=lane.max_pos, f32=f32, eps=lane.cfg.eps)
-        s_kv = p.stage(lane._rows(K_LATENT_KV, kv, T * (H + 1), lane.items_per(T * (H + 1))), label=("latent_kv", run))
+                       ld_cache=st["cache"].shape[1], max_pos=lane.max_pos, f32=f32, eps=lane.cfg.eps, **copy)
+        s_kv = p.stage(lane._rows(K_LATENT_KV, kv, T, lane._per(T)), label=("latent_kv", run))
         p.after(s, s_kv)
-        s_q = lane.head_product(p, s_kv, lane.q_un.addr, up(d, 64), w.uk, lane.q_all.addr, ld_q, lane.T * ld_q, T, c, d,
-                                ("latent_q", run))
+        ends = []
+        if whole:
+            ends.append(LatentAttention.direct(lane, p, m, w, whole, buffers, T, run, s_kv))
+        if rest.requests:
+            ends.append(LatentAttention.absorbed(lane, p, m, w, st["cache"], rest, run, s_kv))
+        return lane.closing(p, ends, lane.mix, w.o, T, H * m.vdim, ("latent_o", run))
+
+    @staticmethod
+    def direct(lane, p, m, w, requests, buffers, T, run, prev):
+        """Whole prompts: keys and values of the prompt's own rows, then attention straight into `mix`."""
+        H, d, r, e, c = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
+        s = lane.product(p, prev, lane.c_rows, w.ukv, lane.kvb, T, H * (d + e), c, ("latent_expand", run), out16=True)
+        q_map, qr_map, kv_map, kr_map = lane.direct_maps(m)
+        at = lane._dev("LatentDirectArgs", q_map=q_map, qr_map=qr_map, kv_map=kv_map, kr_map=kr_map, out=lane.mix.addr, d=d, r=r,
+                       e=e, heads=H, rows_max=lane.T, ld_out=lane.mix.ld, buffers=buffers, scale=m.scale)
+        blocks = sorted(((q0, row0, n) for row0, n, _ in requests for q0 in range(0, n, 128)), reverse=True)   # longest first
+        q0, row0, n = (np.array(v)[:, None] for v in zip(*blocks))
+        s_at = p.stage(tile_array(K_LATENT_DIRECT, i0=row0, i1=n, i2=q0, i3=np.arange(H)[None], a0=at.data_ptr()),
+                       label=("latent_attn", run))
+        p.after(s, s_at)
+        return s_at
+
+    @staticmethod
+    def absorbed(lane, p, m, w, cache, b, run, prev):
+        """Rows that attend to cached latents: W_uk^T q, attention over the latents themselves, W_uv."""
+        f32, H, d, r, c = int(lane.cfg.f32), m.heads, m.dim, m.rot_dim, m.kv_rank
+        ld_q, ld_o, spans = up(c + r, 8), up(c, 64), [(row0, n) for row0, n, _ in b.requests]
+        s = lane.head_product(p, prev, lane.q_un.addr, up(d, 64), w.uk, lane.q_all.addr, ld_q, lane.T * ld_q, spans, c, d,
+                              ("latent_q", run))
         shape = None if f32 else latent_tile(m, lane.kv.page, max(n for _, n, _ in b.requests))
-        fields = dict(q=lane.q_all.addr, cache=st["cache"], block_table=lane.bt, out=lane.o_lat.addr, ws_o=lane.ws.data_ptr(),
+        fields = dict(q=lane.q_all.addr, cache=cache, block_table=lane.bt, out=lane.o_lat.addr, ws_o=lane.ws.data_ptr(),
                       ws_ml=lane.ws_ml.data_ptr(), tok_pos=lane.tok_pos, ld_q=ld_q, heads=H, kv_rank=c, r=r,
-                      ld_cache=st["cache"].shape[1], page=lane.kv.page, bt_stride=lane.bt_stride, rows_max=lane.T, ld_out=ld_o,
+                      ld_cache=cache.shape[1], page=lane.kv.page, bt_stride=lane.bt_stride, rows_max=lane.T, ld_out=ld_o,
                       f32=f32, scale=m.scale)
         if shape:
             tokens, heads, buffers = shape
-            blocks = sum(-(-n // tokens) for _, n, _ in b.requests) * -(-H // heads)
-            parts = lane.attn_parts(T, H, blocks)
-            fields.update(q_map=lane.q_map(m, tokens, heads), kv_map=lane.kv_map(m, st["cache"]), tokens=tokens, group=heads,
+            blocks = sum(-(-n // tokens) for _, n in spans) * -(-H // heads)
+            parts = lane.attn_parts(H, blocks)
+            fields.update(q_map=lane.q_map(m, tokens, heads), kv_map=lane.kv_map(m, cache), tokens=tokens, group=heads,
                           buffers=buffers)
             tiles = b.latent_tiles(H, tokens, heads, parts)
         else:
-            parts = lane.attn_parts(T, H, T * -(-H // 4))
+            parts = lane.attn_parts(H, b.T * -(-H // 4))
             tiles = b.attn_tiles(H, parts)
         at = lane._dev("LatentAttnArgs", **fields)
         s_at = p.stage(_retarget(tiles, a0=at.data_ptr()), label=("latent_attn", run))
-        p.after(s_q, s_at)
+        p.after(s, s_at)
         if parts > 1:
-            tiles = lane._rows(K_LATENT_MERGE, at, T * H, lane.items_per(T * H))
-            tiles[:, 2] = parts
-            s_mg = p.stage(tiles, label=("latent_merge", run))
+            s_mg = p.stage(_retarget(b.item_tiles(K_LATENT_MERGE, H, i2=parts), a0=at.data_ptr()), label=("latent_merge", run))
             p.after(s_at, s_mg)
             s_at = s_mg
-        s_v = lane.head_product(p, s_at, lane.o_lat.addr, ld_o, w.uv, lane.mix.addr, lane.mix.ld, m.vdim, T, m.vdim, c,
-                                ("latent_v", run))
-        return lane.closing(p, s_v, lane.mix, w.o, T, H * m.vdim, ("latent_o", run))
+        return lane.head_product(p, s_at, lane.o_lat.addr, ld_o, w.uv, lane.mix.addr, lane.mix.ld, m.vdim, spans, m.vdim, c,
+                                 ("latent_v", run))
 
 
 MIXERS = {"mamba1": SelectiveScan, "mlstm": MatrixMemory, "latent_attention": LatentAttention}
@@ -342,12 +380,28 @@ class _Buf:
 
 class _Batch:
     """The rows of one program: requests [(first row, rows, slot)], and the tile lists that depend on them only (made
-    once per program and re-addressed per layer)."""
+    once per program and re-addressed per layer).  pos0: the requests' first positions, None for a decode step."""
 
-    def __init__(self, lane, requests):
-        self.lane, self.requests = lane, requests
+    def __init__(self, lane, requests, pos0=None):
+        self.lane, self.requests, self.pos0 = lane, requests, pos0
         self.T = sum(n for _, n, _ in requests)
         self._made = {}
+
+    def split(self):
+        """(requests that bring a whole prompt from its start, a _Batch of the others)."""
+        def make():
+            whole = [i for i, (_, n, _) in enumerate(self.requests) if self.pos0 and self.pos0[i] == 0 and n >= DIRECT_ROWS]
+            return [self.requests[i] for i in whole], _Batch(self.lane, [q for i, q in enumerate(self.requests) if i not in whole])
+        return self._once("split", make)
+
+    def item_tiles(self, kind, per_row, **ops):
+        """Item-wise tiles over the batch's rows, items row * per_row + j."""
+        def make():
+            per = self.lane.items_per(self.T * per_row)
+            spans = [(row0 * per_row + i, min(per, n * per_row - i)) for row0, n, _ in self.requests for i in range(0, n * per_row, per)]
+            first, count = (np.array(v) for v in zip(*spans))
+            return tile_array(kind, i0=first, i1=count, **ops)
+        return self._once((kind, per_row, tuple(ops.items())), make)
 
     def _once(self, key, make):
         if key not in self._made:
@@ -355,7 +409,7 @@ class _Batch:
         return self._made[key]
 
     def conv_tiles(self, channels):
-        rows_per, ch_per = 64, 256
+        rows_per, ch_per = 32, 1024
 
         def make():
             out = []
@@ -380,7 +434,7 @@ class _Batch:
         return self._once(("memory", heads, e), make)
 
     def gate_tiles(self, outputs):
-        per_out, per_row = (4, 8) if self.T <= SPLIT_ROWS else (outputs, 16)
+        per_out, per_row = (8, 4) if self.T <= SPLIT_ROWS else (outputs, 16)
 
         def make():
             r, o = np.meshgrid(np.arange(0, self.T, per_row), np.arange(0, outputs, per_out), indexing="ij")
@@ -441,7 +495,7 @@ class LayerListLane(LaneBase):
         self.hd = _Buf(self, T, ff, act) if ff else None
         self.gu = _Buf(self, T, 2 * ff, f32) if ff and cfg.f32 else None
         for name, dt in (("proj", act), ("act", act), ("mix", act), ("dt_in", act), ("small", f32), ("dt", f32), ("qc", f32),
-                         ("raw", f32)):
+                         ("raw", f32)) + (() if cfg.f32 else (("kvb", act), ("c_rows", act))):
             setattr(self, name, _Buf(self, T, sizes[name], dt) if name in sizes else None)
         for name in ("q_un", "q_all", "o_lat"):   # [head][T][columns]: addressed by the layer's own strides
             if name in sizes:
@@ -495,6 +549,9 @@ class LayerListLane(LaneBase):
                 wm(lw.qkv), wm(lw.uk), wm(lw.uv), self.mix.maps(m.heads * m.vdim)
                 self.head_maps(self.q_un.addr, up(m.dim, 64), m.dim, m.heads)
                 self.head_maps(self.o_lat.addr, up(m.kv_rank, 64), m.kv_rank, m.heads)
+                wm(lw.ukv), self.c_rows.maps(m.kv_rank)
+                if direct_buffers(m):
+                    self.direct_maps(m)
                 for n in range(1, 65):   # a program's tile shape follows its longest request
                     shape = latent_tile(m, self.kv.page, n)
                     if shape:
@@ -543,23 +600,25 @@ class LayerListLane(LaneBase):
         else:
             s = self._gemm(p, self.weight_map(w), x.maps(k), rows, n, k, out.t, ld,
                            epi if epi is not None else (EPI_STORE if out16 else EPI_F32), label, up_offset=up_offset)
-        p.after(prev, s)
+        for stage in prev if isinstance(prev, list) else [prev]:
+            p.after(stage, s)
         return s
 
-    def _product_tiles(self, rows, n):
-        key = ("product", rows, n)
+    def _product_tiles(self, rows, n, row0=0):
+        key = ("product", rows, n, row0)
         if key not in self._templates:
             r, c = np.meshgrid(np.arange(0, rows, 32), np.arange(0, n, 32), indexing="ij")
-            self._templates[key] = tile_array(K_PRODUCT, i0=r, i1=np.minimum(32, rows - r), i2=c, i3=np.minimum(32, n - c))
+            self._templates[key] = tile_array(K_PRODUCT, i0=row0 + r, i1=np.minimum(32, rows - r), i2=c, i3=np.minimum(32, n - c))
         return self._templates[key]
 
-    def head_product(self, p, prev, x_addr, ld_x, w, out_addr, ld_out, head_stride, rows, n, k, label):
-        """Per head h: out[.. + h * head_stride][rows][n] = x[h * T ..][k] w[h][n][k]^T, activations' type out."""
+    def head_product(self, p, prev, x_addr, ld_x, w, out_addr, ld_out, head_stride, spans, n, k, label):
+        """Per head h and row span (first, rows): out[h * head_stride + row * ld_out ..n] = x[h * T + row][k] w[h][n][k]^T,
+        activations' type out."""
         heads = w.shape[0]
         if self.cfg.f32:
             # tile 51 stores fp32, which is the activations' type here
             args = self._dev("ProductArgs", x=x_addr, w=w, out=out_addr, ld_x=ld_x, ld_w=w.shape[-1], ld_out=ld_out, K=k, N=n, f32=1)
-            base = self._product_tiles(rows, n)
+            base = np.concatenate([self._product_tiles(rows, n, row0) for row0, rows in spans])
             tiles = np.tile(base, (heads, 1))
             h = np.repeat(np.arange(heads, dtype=np.uint64), len(base))
             tiles[:, 3] = args.data_ptr()
@@ -568,15 +627,19 @@ class LayerListLane(LaneBase):
             tiles[:, 6] = h * np.uint64(4 * head_stride)
             s = p.stage(tiles, label=label)
         else:
-            bm = _bm(rows)
-            # the tile's activation rows are h * T + m and its output row is counted from there: the base makes up for it
-            args = [self.arena.put(_C.gemm_args(out=(out_addr + 2 * (h * head_stride - h * self.T * ld_out)) % (1 << 64),
-                                                ld_out=ld_out, k_tiles=-(-k // 64), epi=EPI_STORE, bm=bm, n_limit=n)).data_ptr()
-                    for h in range(heads)]
-            h, m0, n0 = np.meshgrid(np.arange(heads), np.arange(0, rows, bm), np.arange(0, n, 128), indexing="ij")
-            tiles = tile_array(K_GEMM, i0=n0, i1=h * self.T + m0, i2=np.minimum(bm, rows - m0), i3=h,
-                               a0=np.asarray(args, dtype=np.int64)[h], a1=self.weight_map(w),
-                               a2=self.head_maps(x_addr, ld_x, k, heads)[HEIGHTS.index(bm)])
+            tiles = []
+            for bm in sorted({_bm(rows) for _, rows in spans}):
+                # the tile's activation rows are h * T + m and its output row is counted from there: the base makes up for it
+                args = [self.arena.put(_C.gemm_args(out=(out_addr + 2 * (h * head_stride - h * self.T * ld_out)) % (1 << 64),
+                                                    ld_out=ld_out, k_tiles=-(-k // 64), epi=EPI_STORE, bm=bm, n_limit=n)).data_ptr()
+                        for h in range(heads)]
+                m0, count = (np.array(v) for v in zip(*[(row0 + i, min(bm, rows - i)) for row0, rows in spans if _bm(rows) == bm
+                                                        for i in range(0, rows, bm)]))
+                h, m, n0 = np.meshgrid(np.arange(heads), np.arange(len(m0)), np.arange(0, n, 128), indexing="ij")
+                tiles.append(tile_array(K_GEMM, i0=n0, i1=h * self.T + m0[m], i2=count[m], i3=h,
+                                        a0=np.asarray(args, dtype=np.int64)[h], a1=self.weight_map(w),
+                                        a2=self.head_maps(x_addr, ld_x, k, heads)[HEIGHTS.index(bm)]))
+            tiles = np.concatenate(tiles)
             s = p.stage(tiles, label=label)
         p.after(prev, s)
         return s
@@ -610,10 +673,23 @@ class LayerListLane(LaneBase):
                                                    [64, 8, chunks, self.kv.page // 8])
         return self._hmaps[key]
 
-    def attn_parts(self, rows, heads, tiles):
-        """Key ranges per row: enough of them to give every worker about two tiles."""
+    def attn_parts(self, heads, tiles):
+        """Key ranges per row: enough of them to give every worker about two tiles (the split workspace is addressed by
+        row, so it covers the rows of a small program only)."""
         want = min(MAX_ATTN_PARTS, 2 * self.fab.num_workers // tiles)
-        return max(1, min(want, self.ws_rows // (rows * heads)))
+        return max(1, want) if self.rows_now <= SPLIT_ROWS else 1
+
+    def direct_maps(self, m):
+        """Operands of the whole-prompt attention tile: (q unrotated, q rotated, keys and values, rotated keys)."""
+        key = "direct", m.dim, m.rot_dim, m.vdim, m.kv_rank, m.heads
+        if key not in self._hmaps:
+            box, H, T, ld_q = [64, KEY_TILE], m.heads, self.T, up(m.kv_rank + m.rot_dim, 8)
+            tm = self.fab.tensor_map
+            self._hmaps[key] = (tm(self.q_un.addr, [m.dim, H * T], [2 * up(m.dim, 64)], box),
+                                tm(self.q_all.addr + 2 * m.kv_rank, [m.rot_dim, H * T], [2 * ld_q], box),
+                                tm(self.kvb.addr, [H * (m.dim + m.vdim), T], [2 * self.kvb.ld], box),
+                                tm(self.c_rows.addr + 2 * m.kv_rank, [m.rot_dim, T], [2 * self.c_rows.ld], box))
+        return self._hmaps[key]
 
     # ------------------------------------------------------------------ programs
     def _streams(self, p, rows, prev, sub, before, label, h32=False, gather=False, step=False):
@@ -647,6 +723,7 @@ class LayerListLane(LaneBase):
     def _chain(self, p, b, step):
         """Every layer run; returns (first stage, final streams stage)."""
         cfg, T = self.cfg, b.T
+        self.rows_now = T
         first = prev = None
         before = None
         for run, l in enumerate(cfg.order):
@@ -694,7 +771,7 @@ class LayerListLane(LaneBase):
         places = want if want is not None else [[len(toks) - 1] for _, toks, _ in batch]
         T, req_info, sample_rows = self._batch_rows(batch, places, all_logits)
         p = Program()
-        b = _Batch(self, [(row0, n, slot) for (row0, _, n, _), (slot, _, _) in zip(req_info, batch)])
+        b = _Batch(self, [(row0, n, slot) for (row0, _, n, _), (slot, _, _) in zip(req_info, batch)], [q[2] for q in batch])
         first, last = self._chain(p, b, step=False)
         self._finish(p, last, T if all_logits else sum(len(v) for v in places), sample_rows if want is None else [])
         return p.upload(self.fab, first=first, iterations=iterations)
