@@ -293,7 +293,6 @@ const std::string& layouts_json() {
     MF_JSON_STRUCT(SumArgs, MF_SUM_ARGS)
     MF_JSON_STRUCT(ConvArgs, MF_CONV_ARGS)
     MF_JSON_STRUCT(ScanArgs, MF_SCAN_ARGS)
-    MF_JSON_STRUCT(MemGateArgs, MF_MEM_GATE_ARGS)
     MF_JSON_STRUCT(MemoryArgs, MF_MEMORY_ARGS)
     MF_JSON_STRUCT(HeadNormArgs, MF_HEAD_NORM_ARGS)
     MF_JSON_STRUCT(LatentArgs, MF_LATENT_ARGS)

@@ -64,17 +64,21 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
   const int last_page = (max(k_hi, 1) - 1) / page, per_tile = kKeyTile / page;
   const int first_key = k_lo / page * page;   // key tiles start at a page
   const int tiles = k_hi > k_lo ? (k_hi - first_key + kKeyTile - 1) / kKeyTile : 0;
-  auto load_keys = [&](int j) {   // warp 0
-    const int s = j % nbuf;
+  auto page_of = [&](int j) {   // this lane's page of key tile j; pages past the visible range repeat the last visible one
+    return lane < per_tile ? bt[min(first_key / page + j * per_tile + lane, last_page)] : 0;
+  };
+  int pg_next = 0;
+  auto load_keys = [&](int j) {   // warp 0, in the order of the tiles; the tile behind it is brought to L2
+    const int s = j % nbuf, pg = j == 0 ? page_of(0) : pg_next;
     if (lane == 0) {
-      fence_proxy_async_all();
+      if (j == 0) fence_proxy_async_all();
       mbar_arrive_expect_tx(bar_k + s, tile_bytes);
     }
     __syncwarp();
-    if (lane < per_tile) {
-      // pages past the visible range repeat the last visible page; their keys are masked
-      const int pg = bt[min(first_key / page + j * per_tile + lane, last_page)];
-      tma_box_4d(sK + s * tile_bytes + lane * (page / 8) * group_bytes, A.kv_map, bar_k + s, 0, 0, 0, pg * (page / 8));
+    if (lane < per_tile) tma_box_4d(sK + s * tile_bytes + lane * (page / 8) * group_bytes, A.kv_map, bar_k + s, 0, 0, 0, pg * (page / 8));
+    if (j + 1 < tiles) {
+      pg_next = page_of(j + 1);
+      if (lane < per_tile) tma_prefetch_4d(A.kv_map, 0, 0, 0, pg_next * (page / 8));
     }
   };
   auto issue_s = [&](int j) {   // one thread: S^T of key tile j
@@ -254,7 +258,7 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
         __syncwarp();
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const int c = c0 + i, h = c / box_tok, tok = c - h * box_tok;
+          const int c = c0 + i, h = box_tok == 1 ? c : c / box_tok, tok = c - h * box_tok;
           if (h >= n_h || tok >= n_tok || dim >= kvr) continue;
           const float x = __uint_as_float(o[i]);
           if (parts == 1) {

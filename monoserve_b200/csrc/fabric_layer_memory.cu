@@ -6,65 +6,6 @@ namespace mf {
 namespace fab {
 
 // ------------------------------------------------------------------ matrix memory
-// Kind 56, MemGateArgs: rows [i0, i0 + i1), outputs [i2, i2 + i3) of the 2 heads (input gates, then forget gates).
-// A warp takes one row and eight outputs at a time, 2048 columns of the row in registers.
-__device__ void tile_mem_gates(const TileDesc& t, int tid) {
-  constexpr int NV = 16;
-  MemGateArgs A;
-  load_block(A, t.a[0]);
-  const int warp = tid >> 5, lane = tid & 31, K = static_cast<int>(A.K), H = static_cast<int>(A.heads);
-  const int o_lo = static_cast<int>(t.i2), o_hi = static_cast<int>(t.i2 + t.i3);
-  auto weights = [&](int o) {
-    return reinterpret_cast<const __nv_bfloat16*>(o >= H ? A.wf : A.wi) + static_cast<size_t>(o >= H ? o - H : o) * K;
-  };
-  for (uint32_t r = t.i0 + warp; r < t.i0 + t.i1; r += kExecThreads / 32) {
-    const float* x = f32p(A.h) + static_cast<size_t>(r) * A.ld_h;
-    for (int o0 = o_lo; o0 < o_hi; o0 += 8) {
-      float acc[8] = {};
-      if ((K & 3) == 0) {
-        for (int k0 = 0; k0 < K; k0 += 128 * NV) {
-          float4 v[NV];
-#pragma unroll
-          for (int i = 0; i < NV; ++i) {
-            const int k = k0 + i * 128 + lane * 4;
-            v[i] = k < K ? *reinterpret_cast<const float4*>(x + k) : make_float4(0.f, 0.f, 0.f, 0.f);
-          }
-#pragma unroll
-          for (int o = 0; o < 8; ++o) {
-            const __nv_bfloat16* w = weights(min(o0 + o, o_hi - 1));
-#pragma unroll
-            for (int i = 0; i < NV; ++i) {
-              const int k = k0 + i * 128 + lane * 4;
-              const uint2 raw = k < K ? __ldg(reinterpret_cast<const uint2*>(w + k)) : make_uint2(0u, 0u);
-              const float2 wa = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-              const float2 wb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-              acc[o] = fmaf(v[i].x, wa.x, fmaf(v[i].y, wa.y, fmaf(v[i].z, wb.x, fmaf(v[i].w, wb.y, acc[o]))));
-            }
-          }
-        }
-      } else {
-#pragma unroll
-        for (int o = 0; o < 8; ++o) {
-          const __nv_bfloat16* w = weights(min(o0 + o, o_hi - 1));
-          for (int k = lane; k < K; k += 32) acc[o] = fmaf(x[k], __bfloat162float(w[k]), acc[o]);
-        }
-      }
-      float mine = 0.f;
-#pragma unroll
-      for (int o = 0; o < 8; ++o) {
-        const float s = warp_sum(acc[o]);
-        if (lane == o) mine = s;
-      }
-      if (lane < 8 && o0 + lane < o_hi) {
-        const int o = o0 + lane;
-        const bool forget = o >= H;
-        const float g = A.cap * tanhf((mine + f32p(forget ? A.bf : A.bi)[forget ? o - H : o]) / A.cap);
-        reinterpret_cast<float*>(A.out)[static_cast<size_t>(r) * 2 * H + o] = forget ? fminf(g, 0.f) - log1pf(expf(-fabsf(g))) : g;
-      }
-    }
-  }
-}
-
 // Packed fp32 pairs (each half rounded like the scalar instruction).
 __device__ __forceinline__ unsigned long long pk2(float a, float b) {
   unsigned long long r;
@@ -102,6 +43,27 @@ __device__ __forceinline__ float4 ld_four(const void* p) {
                      __uint_as_float(u.y & 0xffff0000u));
 }
 
+// Log gate of a head from its raw projection: cap tanh(z / cap), the forget gate through log sigmoid.
+__device__ __forceinline__ float capped(float z, float cap) { return cap * tanhf(z / cap); }
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+// R values per lane (R <= 32, a power of two) summed over the warp: lane l ends with the sum of value l / (32 / R).
+template <int R>
+__device__ __forceinline__ float warp_sum_each(float (&r)[R], int lane) {
+#pragma unroll
+  for (int half = R / 2, bit = 16; half >= 1; half >>= 1, bit >>= 1) {
+    const bool hi = lane & bit;
+#pragma unroll
+    for (int c = 0; c < half; ++c) {
+      const float give = hi ? r[c] : r[c + half], have = hi ? r[c + half] : r[c];
+      r[c] = have + __shfl_xor_sync(0xffffffffu, give, bit);
+    }
+  }
+#pragma unroll
+  for (int bit = 16 / R; bit >= 1; bit >>= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], bit);
+  return r[0];
+}
+
 template <int ND, bool F32>
 __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ring) {
   using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
@@ -135,7 +97,7 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
   float* const m_state = reinterpret_cast<float*>(A.m) +
                          (static_cast<size_t>(slot) * H + head) * ((e + kMemColumns) / kMemColumns) + (t.i2 >> 16);
   float m0 = fresh ? 0.f : *m_state;
-  const float* gates = f32p(A.gates);
+  const float *gates = f32p(A.gates), bi = f32p(A.gate_bias)[head], bf = f32p(A.gate_bias)[H + head];
   const T *gk = reinterpret_cast<const T*>(A.k) + head * d, *gq = reinterpret_cast<const T*>(A.q) + head * d;
   const T* gv = reinterpret_cast<const T*>(A.v) + head * e + col0;
   const bool kq16 = d % kPer16 == 0 && ((A.k | A.q) & 15) == 0;
@@ -170,9 +132,9 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
   };
   auto load_gates = [&](int base, float& gi, float& gf) {   // one token per lane
     const int nt = min(kTokens, rows - base);
-    const size_t at = static_cast<size_t>(row0 + base + min(lane, nt - 1)) * 2 * H + head;
-    gi = lane < nt ? gates[at] : -INFINITY;
-    gf = lane < nt ? gates[at + H] : 0.f;
+    const size_t at = static_cast<size_t>(row0 + base + min(lane, nt - 1)) * A.ld_gates + head;
+    gi = lane < nt ? capped(gates[at] + bi, A.cap) : -INFINITY;
+    gf = lane < nt ? log_sigmoid(capped(gates[at + H] + bf, A.cap)) : 0.f;
   };
   stage(0, buf);
   float gi, gf;
@@ -210,65 +172,51 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
     const T* const sk = buf + s * buf_elems;
     const T* const sq = sk + kTokens * ds;
     const T* const sv = sq + kTokens * ds + warp * 8;
-    for (int tok = 0; tok < nt; ++tok) {
-      const float kp = __shfl_sync(0xffffffffu, keep, tok), ad = __shfl_sync(0xffffffffu, add, tok);
-      const unsigned long long kp2 = pk2(kp, kp);
-      unsigned long long acc[8], av2[8];
-      const float4 va = ld_four<F32>(sv + tok * kMemColumns), vb = ld_four<F32>(sv + tok * kMemColumns + 4);
-      const float v[8] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
+    for (int t0 = 0; t0 < nt; t0 += 4) {   // four tokens' read-outs are summed over the warp together
+      float r[32];                        // [token][column]
 #pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        const float av = c_lo + c < e ? ad * v[c] : (c_lo + c == e ? ad : 0.f);
-        av2[c] = pk2(av, av);
-        acc[c] = 0ull;
-      }
-#pragma unroll
-      for (int i = 0; i < ND; ++i) {
-        const int at = i * 128 + lane * 4;
-        float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
-        if (at < dp) {
-          k4 = ld_four<F32>(sk + tok * ds + at);
-          q4 = ld_four<F32>(sq + tok * ds + at);
-        }
-        const unsigned long long k0 = pk2(k4.x, k4.y), k1 = pk2(k4.z, k4.w), q0 = pk2(q4.x, q4.y), q1 = pk2(q4.z, q4.w);
+      for (int u = 0; u < 4; ++u) {
+        const int tok = min(t0 + u, nt - 1);
+        const bool live = t0 + u < nt;      // a token past the end keeps the state and adds nothing
+        const float kp_ = __shfl_sync(0xffffffffu, keep, tok), ad_ = __shfl_sync(0xffffffffu, add, tok);
+        const float kp = live ? kp_ : 1.f, ad = live ? ad_ : 0.f;
+        const unsigned long long kp2 = pk2(kp, kp);
+        unsigned long long acc[8], av2[8];
+        const float4 va = ld_four<F32>(sv + tok * kMemColumns), vb = ld_four<F32>(sv + tok * kMemColumns + 4);
+        const float v[8] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
-          S[c][i][0] = fma2(av2[c], k0, mul2(kp2, S[c][i][0]));
-          S[c][i][1] = fma2(av2[c], k1, mul2(kp2, S[c][i][1]));
-          acc[c] = fma2(S[c][i][0], q0, acc[c]);
-          acc[c] = fma2(S[c][i][1], q1, acc[c]);
+          const float av = c_lo + c < e ? ad * v[c] : (c_lo + c == e ? ad : 0.f);
+          av2[c] = pk2(av, av);
+          acc[c] = 0ull;
+        }
+#pragma unroll
+        for (int i = 0; i < ND; ++i) {
+          const int at = i * 128 + lane * 4;
+          float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
+          if (at < dp) {
+            k4 = ld_four<F32>(sk + tok * ds + at);
+            q4 = ld_four<F32>(sq + tok * ds + at);
+          }
+          const unsigned long long k0 = pk2(k4.x, k4.y), k1 = pk2(k4.z, k4.w), q0 = pk2(q4.x, q4.y), q1 = pk2(q4.z, q4.w);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) {
+            S[c][i][0] = fma2(av2[c], k0, mul2(kp2, S[c][i][0]));
+            S[c][i][1] = fma2(av2[c], k1, mul2(kp2, S[c][i][1]));
+            acc[c] = fma2(S[c][i][0], q0, acc[c]);
+            acc[c] = fma2(S[c][i][1], q1, acc[c]);
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          const float2 f = unpk2(acc[c]);
+          r[u * 8 + c] = f.x + f.y;
         }
       }
-      float r[8];
-#pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        const float2 f = unpk2(acc[c]);
-        r[c] = f.x + f.y;
-      }
-      // the eight columns' sums over the warp: each step halves the columns a lane carries, then plain sums
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const bool hi = lane & 16;
-        const float give = hi ? r[c] : r[c + 4], have = hi ? r[c + 4] : r[c];
-        r[c] = have + __shfl_xor_sync(0xffffffffu, give, 16);
-      }
-#pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        const bool hi = lane & 8;
-        const float give = hi ? r[c] : r[c + 2], have = hi ? r[c + 2] : r[c];
-        r[c] = have + __shfl_xor_sync(0xffffffffu, give, 8);
-      }
-      {
-        const bool hi = lane & 4;
-        const float give = hi ? r[0] : r[1], have = hi ? r[1] : r[0];
-        r[0] = have + __shfl_xor_sync(0xffffffffu, give, 4);
-      }
-      r[0] += __shfl_xor_sync(0xffffffffu, r[0], 2);
-      r[0] += __shfl_xor_sync(0xffffffffu, r[0], 1);
-      const float fl = __shfl_sync(0xffffffffu, floor_, tok);
-      const int c = c_lo + ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);
-      const float read = r[0] * A.q_scale;
-      if ((lane & 3) == 0 && c <= e)
+      const float read = warp_sum_each<32>(r, lane) * A.q_scale;
+      const int tok = t0 + (lane >> 3), c = c_lo + (lane & 7);
+      const float fl = __shfl_sync(0xffffffffu, floor_, tok & 31);
+      if (tok < nt && c <= e)
         reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row0 + base + tok) * H + head) * oe + c] =
             c < e ? read : fmaxf(fabsf(read), fl) + 1e-6f;
     }
@@ -287,6 +235,113 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
       }
     }
   if (tid == 0) *m_state = m0;
+}
+
+// Kind 56, MemoryArgs: one token.  Row i0, i2 = head | first column block << 16, i1 column blocks, slot i3.  The state
+// streams through registers, the next block's loads issued before this one's arithmetic.
+template <int ND, bool F32>
+__device__ __noinline__ void memory_step(const TileDesc& t, int tid) {
+  using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
+  MemoryArgs A;
+  load_block(A, t.a[0]);
+  const int row = static_cast<int>(t.i0), slot = static_cast<int>(t.i3), n_blocks = static_cast<int>(t.i1);
+  const int head = static_cast<int>(t.i2 & 0xffffu), block0 = static_cast<int>(t.i2 >> 16);
+  const int H = static_cast<int>(A.heads), d = static_cast<int>(A.d), e = static_cast<int>(A.e);
+  const int dp = (d + 3) & ~3, oe = (e + 4) & ~3, warp = tid >> 5, lane = tid & 31;
+  const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row] == 0;
+  const size_t at_row = static_cast<size_t>(row) * A.ld_qkv;
+  const T *gk = reinterpret_cast<const T*>(A.k) + at_row + head * d, *gq = reinterpret_cast<const T*>(A.q) + at_row + head * d;
+  const T* gv = reinterpret_cast<const T*>(A.v) + at_row + head * e;
+  float* const m_state = reinterpret_cast<float*>(A.m) + (static_cast<size_t>(slot) * H + head) * ((e + kMemColumns) / kMemColumns);
+  float* const state = reinterpret_cast<float*>(A.state) + (static_cast<size_t>(slot) * H + head) * (e + 1) * dp;
+  const float* gates = f32p(A.gates) + static_cast<size_t>(row) * A.ld_gates;
+  auto value = [](const T& v) -> float {
+    if constexpr (F32) return v;
+    else return __bfloat162float(v);
+  };
+  float4 st[2][8][ND];
+  float v8[2][8];
+  auto fetch = [&](int b, float4 (&S)[8][ND], float (&v)[8]) {
+    const int c_lo = b * kMemColumns + warp * 8;
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+#pragma unroll
+      for (int i = 0; i < ND; ++i) {
+        const int at = i * 128 + lane * 4;
+        S[c][i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (!fresh && at < dp && c_lo + c <= e) S[c][i] = __ldcs(reinterpret_cast<const float4*>(state + static_cast<size_t>(c_lo + c) * dp + at));
+      }
+      v[c] = c_lo + c < e ? value(gv[c_lo + c]) : (c_lo + c == e ? 1.f : 0.f);
+    }
+  };
+  fetch(block0, st[0], v8[0]);
+  const float m_old = fresh ? 0.f : m_state[block0];
+  float k[ND][4], q[ND][4];
+#pragma unroll
+  for (int i = 0; i < ND; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int at = i * 128 + lane * 4 + j;
+      k[i][j] = at < d ? value(gk[at]) : 0.f;
+      q[i][j] = at < d ? value(gq[at]) * A.q_scale : 0.f;
+    }
+  const float gi = capped(gates[head] + f32p(A.gate_bias)[head], A.cap);
+  const float gf = log_sigmoid(capped(gates[H + head] + f32p(A.gate_bias)[H + head], A.cap));
+  const float m = fmaxf(gf + m_old, gi);
+  const float keep = expf(gf + m_old - m), add = expf(gi - m), floor_ = expf(-m);
+  exec_sync();   // every thread has read the old maximum
+  auto run = [&](int b, float4 (&S)[8][ND], const float (&v)[8]) {
+    const int c_lo = b * kMemColumns + warp * 8;
+    float r[8];
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      const float av = add * v[c];
+      r[c] = 0.f;
+#pragma unroll
+      for (int i = 0; i < ND; ++i) {
+        float4 s = S[c][i];
+        s.x = fmaf(av, k[i][0], keep * s.x);
+        s.y = fmaf(av, k[i][1], keep * s.y);
+        s.z = fmaf(av, k[i][2], keep * s.z);
+        s.w = fmaf(av, k[i][3], keep * s.w);
+        r[c] = fmaf(s.x, q[i][0], fmaf(s.y, q[i][1], fmaf(s.z, q[i][2], fmaf(s.w, q[i][3], r[c]))));
+        const int at = i * 128 + lane * 4;
+        if (at < dp && c_lo + c <= e) __stcs(reinterpret_cast<float4*>(state + static_cast<size_t>(c_lo + c) * dp + at), s);
+      }
+    }
+    const float read = warp_sum_each<8>(r, lane);
+    const int c = c_lo + (lane >> 2);
+    if ((lane & 3) == 0 && c <= e)
+      reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row) * H + head) * oe + c] =
+          c < e ? read : fmaxf(fabsf(read), floor_) + 1e-6f;
+  };
+  for (int b = block0; b < block0 + n_blocks; b += 2) {
+    if (b + 1 < block0 + n_blocks) fetch(b + 1, st[1], v8[1]);
+    run(b, st[0], v8[0]);
+    if (b + 1 < block0 + n_blocks) {
+      if (b + 2 < block0 + n_blocks) fetch(b + 2, st[0], v8[0]);
+      run(b + 1, st[1], v8[1]);
+    }
+  }
+  if (tid < n_blocks) m_state[block0 + tid] = m;
+}
+
+__device__ bool tile_memory_step(const TileDesc& t, int tid) {
+  const MemoryArgs* p = reinterpret_cast<const MemoryArgs*>(t.a[0]);
+  const uint32_t d = __ldcg(&p->d);
+  const bool f32 = __ldcg(&p->f32) != 0;
+  if (t.i1 > static_cast<uint32_t>(kExecThreads)) return false;
+#define MF_STEP(N)                         \
+  if (d <= 128 * N) {                      \
+    if (f32) memory_step<N, true>(t, tid); \
+    else memory_step<N, false>(t, tid);    \
+    return true;                           \
+  }
+  MF_STEP(1)
+  MF_STEP(2)
+  MF_STEP(4)
+#undef MF_STEP
+  return false;
 }
 
 __device__ bool tile_memory(const TileDesc& t, int tid, uint8_t* ring) {

@@ -219,8 +219,16 @@ __device__ __forceinline__ void streams_row(const StreamArgs& A, uint32_t r, int
         o[0] = __float2bfloat16(h[0]);
       }
     };
-    if (A.h16) st16(A.h16, static_cast<size_t>(r) * A.ld_h16 + c * V);
     if (g >= 0 && A.out16) st16(A.out16, static_cast<size_t>(g) * A.ld_out + c * V);
+    if (A.h16) {
+      const size_t at = static_cast<size_t>(r) * A.ld_h16 + c * V;
+      st16(A.h16, at);
+      for (uint32_t part = 1; part <= 2 && A.split; ++part) {   // what rounding has left, rounded again
+#pragma unroll
+        for (int j = 0; j < V; ++j) h[j] -= __bfloat162float(__float2bfloat16(h[j]));
+        st16(A.h16, at + part * A.split);
+      }
+    }
   };
   if constexpr (kReg) {
 #pragma unroll
@@ -287,7 +295,8 @@ __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx) 
     case kTileStreams: tile_streams(t, tid, scratch); return true;
     case kTileConv: tile_conv(t, tid); return true;
     case kTileScan: return tile_scan(t, tid, ctx.ring);
-    case kTileMemGates: tile_mem_gates(t, tid); return true;
+    case kTileMemoryStep: return tile_memory_step(t, tid);
+    case kTileScanStep: tile_scan_step(t, tid); return true;
     case kTileMemory: return tile_memory(t, tid, ctx.ring);
     case kTileHeadNorm: tile_head_norm(t, tid); return true;
     case kTileLatentKv: tile_latent_kv(t, tid); return true;

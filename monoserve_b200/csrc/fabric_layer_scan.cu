@@ -207,48 +207,62 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
     }
     exec_sync();
     const Chunk& k = sh.in[s];
-    for (int t0 = 0; t0 < nt; t0 += 4) {
-      const int mine = min(t0 + p, nt - 1);
-      const float x = value(k.x[mine][my]), z = value(k.z[mine][my]);
+    // Step sizes of the chunk, lane p those of tokens p, p + 4, ...; a token past the end gets step 0 and input 0, which
+    // leaves the state as it is.
+    float dts[kScanTokens / 4], xs[kScanTokens / 4];
+#pragma unroll
+    for (int g = 0; g < kScanTokens / 4; ++g) {
+      const int mine = 4 * g + p;
       const float u = k.dt[mine][my] + dt_bias;
       const float dt = F32 ? softplus32(u) : fmaxf(u, 0.f) + __logf(1.f + __expf(-fabsf(u)));
-      const float dtx = dt * x;
-      float out = 0.f;
+      dts[g] = mine < nt ? dt : 0.f;
+      xs[g] = mine < nt ? value(k.x[mine][my]) : 0.f;
+    }
+#pragma unroll
+    for (int g = 0; g < kScanTokens / 4; ++g) {
+      if (4 * g >= nt) break;   // the same in all threads
+      const float dt = dts[g], dtx = dts[g] * xs[g];
+      float part[4];
 #pragma unroll
       for (int i4 = 0; i4 < 4; ++i4) {
-        if (t0 + i4 < nt) {   // the same in all threads
-          const float dk = __shfl_sync(0xffffffffu, dt, quad + i4), xk = __shfl_sync(0xffffffffu, dtx, quad + i4);
-          float B[NS], Cv[NS];
-          const float *b = &k.bc[t0 + i4][s0], *cc = &k.bc[t0 + i4][NP + s0];
-          if constexpr ((NS & 3) == 0) {
+        const float dk = __shfl_sync(0xffffffffu, dt, quad + i4), xk = __shfl_sync(0xffffffffu, dtx, quad + i4);
+        float B[NS], Cv[NS];
+        const float *b = &k.bc[4 * g + i4][s0], *cc = &k.bc[4 * g + i4][NP + s0];
+        if constexpr ((NS & 3) == 0) {
 #pragma unroll
-            for (int i = 0; i < NS; i += 4) {
-              ld_vec<4>(b + i, *reinterpret_cast<float(*)[4]>(&B[i]));
-              ld_vec<4>(cc + i, *reinterpret_cast<float(*)[4]>(&Cv[i]));
-            }
-          } else {
-#pragma unroll
-            for (int i = 0; i < NS; ++i) {
-              B[i] = b[i];
-              Cv[i] = cc[i];
-            }
+          for (int i = 0; i < NS; i += 4) {
+            ld_vec<4>(b + i, *reinterpret_cast<float(*)[4]>(&B[i]));
+            ld_vec<4>(cc + i, *reinterpret_cast<float(*)[4]>(&Cv[i]));
           }
-          float y = 0.f;
+        } else {
 #pragma unroll
           for (int i = 0; i < NS; ++i) {
-            if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), xk * B[i]);
-            else S[i] = fmaf(ex2(dk * a[i]), S[i], xk * B[i]);
-            y = fmaf(S[i], Cv[i], y);
+            B[i] = b[i];
+            Cv[i] = cc[i];
           }
-          y += __shfl_xor_sync(0xffffffffu, y, 1);
-          y += __shfl_xor_sync(0xffffffffu, y, 2);
-          if (i4 == p) out = y;
         }
+        float y = 0.f;
+#pragma unroll
+        for (int i = 0; i < NS; ++i) {
+          // past the end B may be anything (its factor is 0), so it must not be let into the sum
+          const float in = 4 * g + i4 < nt ? xk * B[i] : 0.f;
+          if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), in);
+          else S[i] = fmaf(ex2(dk * a[i]), S[i], in);
+          y = fmaf(S[i], Cv[i], y);
+        }
+        part[i4] = y;
       }
-      if (t0 + p < nt) {
-        const float y = fmaf(D, x, out) * (F32 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)));
-        if constexpr (F32) sh.y[t0 + p][my] = y;
-        else sh.y[t0 + p][my] = __float2bfloat16(y);
+      // the four lanes' sums, lane p ending with token p's
+      const bool odd = p & 1, hi = p & 2;
+      const float t0 = (odd ? part[1] : part[0]) + __shfl_xor_sync(0xffffffffu, odd ? part[0] : part[1], 1);
+      const float t1 = (odd ? part[3] : part[2]) + __shfl_xor_sync(0xffffffffu, odd ? part[2] : part[3], 1);
+      const float out = (hi ? t1 : t0) + __shfl_xor_sync(0xffffffffu, hi ? t0 : t1, 2);
+      const int mine = 4 * g + p;
+      if (mine < nt) {
+        const float z = value(k.z[mine][my]);
+        const float y = fmaf(D, xs[g], out) * (F32 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)));
+        if constexpr (F32) sh.y[mine][my] = y;
+        else sh.y[mine][my] = __float2bfloat16(y);
       }
     }
     exec_sync();
@@ -271,6 +285,87 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
                         : (fresh ? 0.f : tail[static_cast<size_t>(k) * C]);
     }
   }
+}
+
+// Kind 65, ScanArgs: one token.  Row i0, channels [i2, i2 + i1), slot i3; a thread per channel, NS of its states at a
+// time with their loads in flight together.
+template <bool F32>
+__device__ __noinline__ void scan_step(const TileDesc& t, int tid) {
+  constexpr int NS = 16;
+  ScanArgs A;
+  load_block(A, t.a[0]);
+  const int row = static_cast<int>(t.i0), slot = static_cast<int>(t.i3);
+  const int n = static_cast<int>(A.n), C = static_cast<int>(A.channels), taps = static_cast<int>(A.taps);
+  const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row] == 0;
+  const float *gb = f32p(A.b) + static_cast<size_t>(row) * A.ld_bc, *gc = f32p(A.c) + static_cast<size_t>(row) * A.ld_bc;
+  const bool vec = (n & 3) == 0 && ((A.b | A.c) & 15) == 0;
+  auto ld4 = [&](const float* p, int i, float (&v)[4]) {
+    if (vec) {
+      ld_vec<4>(p + i, v);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] = i + j < n ? p[i + j] : 0.f;
+    }
+  };
+  for (int c = static_cast<int>(t.i2) + tid; c < static_cast<int>(t.i2 + t.i1); c += kExecThreads) {
+    const size_t sc = (static_cast<size_t>(slot) * C + c) * n;
+    float* state = reinterpret_cast<float*>(A.state) + sc;
+    const float* a = f32p(A.A) + static_cast<size_t>(c) * n;
+    const float u = f32p(A.dt)[static_cast<size_t>(row) * A.ld_dt + c] + f32p(A.dt_bias)[c];
+    const float x = act_ld(A.x, static_cast<size_t>(row) * A.ld_x + c, F32), z = act_ld(A.z, static_cast<size_t>(row) * A.ld_z + c, F32);
+    const float D = f32p(A.D)[c];
+    float* tail = reinterpret_cast<float*>(A.tail) + static_cast<size_t>(slot) * (taps - 1) * C + c;
+    float old[kMaxTaps];
+#pragma unroll
+    for (int j = 1; j < kMaxTaps; ++j)
+      if (j < taps - 1) old[j] = fresh ? 0.f : tail[static_cast<size_t>(j) * C];
+    const float newest = taps > 1 ? act_ld(A.x_in, static_cast<size_t>(row) * A.ld_z + c, F32) : 0.f;
+    float dt = 0.f, y = 0.f;
+    for (int s0 = 0; s0 < n; s0 += NS) {
+      float S[NS / 4][4], av[NS / 4][4], B[NS / 4][4], Cv[NS / 4][4];
+#pragma unroll
+      for (int i = 0; i < NS / 4; ++i) {
+        const int k = s0 + 4 * i;
+        if (k >= n) break;
+        if (!fresh) ld4(state, k, S[i]);
+        else S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
+        ld4(a, k, av[i]);
+        ld4(gb, k, B[i]);
+        ld4(gc, k, Cv[i]);
+      }
+      if (s0 == 0) dt = F32 ? softplus32(u) : fmaxf(u, 0.f) + __logf(1.f + __expf(-fabsf(u)));
+#pragma unroll
+      for (int i = 0; i < NS / 4; ++i) {
+        const int k = s0 + 4 * i;
+        if (k >= n) break;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          if constexpr (F32) S[i][j] += fmaf(S[i][j], expm1f(dt * av[i][j]), dt * x * B[i][j]);
+          else S[i][j] = fmaf(__expf(dt * av[i][j]), S[i][j], dt * x * B[i][j]);
+          y = fmaf(S[i][j], Cv[i][j], y);
+        }
+        if (vec) {
+          st_vec<4>(state + k, S[i]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (k + j < n) state[k + j] = S[i][j];
+        }
+      }
+    }
+    y = fmaf(D, x, y);
+    act_st(A.y, static_cast<size_t>(row) * A.ld_y + c, F32, y * (F32 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z))));
+#pragma unroll
+    for (int j = 0; j < kMaxTaps - 1; ++j) {
+      if (j < taps - 2) tail[static_cast<size_t>(j) * C] = old[j + 1];
+      else if (j == taps - 2) tail[static_cast<size_t>(j) * C] = newest;
+    }
+  }
+}
+
+__device__ void tile_scan_step(const TileDesc& t, int tid) {
+  if (__ldcg(&reinterpret_cast<const ScanArgs*>(t.a[0])->f32)) scan_step<true>(t, tid);
+  else scan_step<false>(t, tid);
 }
 
 __device__ bool tile_scan(const TileDesc& t, int tid, uint8_t* ring) {

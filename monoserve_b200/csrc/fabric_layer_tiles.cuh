@@ -35,7 +35,7 @@ struct LayerCtx {
   volatile int* abort_flag;
 };
 
-// Runs tile kinds kTileProduct32 .. kTileLatentDirect: false for a kind or size these tiles do not take, or when a bounded
+// Runs tile kinds kTileProduct32 .. kTileScanStep: false for a kind or size these tiles do not take, or when a bounded
 // wait gave up.  All exec threads call it with the same tile.
 __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx);
 // Wide tiles: their exec warps use the operand ring as scratch memory, and TMEM.
@@ -49,7 +49,8 @@ __device__ void tile_gated_act(const TileDesc& t, int tid);
 __device__ void tile_sum_slabs(const TileDesc& t, int tid);
 __device__ void tile_conv(const TileDesc& t, int tid);
 __device__ bool tile_scan(const TileDesc& t, int tid, uint8_t* ring);
-__device__ void tile_mem_gates(const TileDesc& t, int tid);
+__device__ bool tile_memory_step(const TileDesc& t, int tid);
+__device__ void tile_scan_step(const TileDesc& t, int tid);
 __device__ bool tile_memory(const TileDesc& t, int tid, uint8_t* ring);
 __device__ void tile_head_norm(const TileDesc& t, int tid);
 __device__ void tile_latent_kv(const TileDesc& t, int tid);

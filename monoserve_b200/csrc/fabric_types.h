@@ -52,7 +52,7 @@ enum TileKind : uint16_t {
   kTileStreams = 53,        // hyper-connection update of the residual streams, next sublayer's input and its norm
   kTileConv = 54,           // causal convolution per channel + silu
   kTileScan = 55,           // selective scan of a request's rows
-  kTileMemGates = 56,       // log gates of the matrix memory
+  kTileMemoryStep = 56,     // matrix memory, one token
   kTileMemory = 57,         // matrix memory over a request's rows
   kTileHeadNorm = 58,       // per-head norm and output gate
   kTileLatentKv = 59,       // latent norm, rotation, cache append, query parts
@@ -61,6 +61,7 @@ enum TileKind : uint16_t {
   kTileSumSlabs = 62,       // sum of a K-split product's slabs
   kTileLatentMma = 63,      // attention over the cached latents on the tensor cores: heads x tokens, one key range
   kTileLatentDirect = 64,   // the same for a whole prompt, with keys and values mapped out of the latents
+  kTileScanStep = 65,       // selective scan, one token
 };
 constexpr int kFabChunk = 16;   // rows per router / permute tile = rank chunk of the stable pack
 

@@ -86,11 +86,13 @@ namespace mf {
  *
  * StreamArgs: the residual streams xs fp32 [rows][streams][W].  hc_mix [from][to] and hc_out [to] belong to the
  * sublayer that has just produced y (y_parts fp32 slabs of y_rows rows; 0 parts: no update), hc_in to the one
- * that follows, w is the norm's multiplier (fp32).  embed set: the streams start as copies of the token's row. */
+ * that follows, w is the norm's multiplier (fp32).  embed set: the streams start as copies of the token's row.
+ * split > 0: h16's row also receives what bf16 rounding leaves of the row, in two further bf16 parts `split` and
+ * 2 split columns on (the three add up to the fp32 row). */
 #define MF_STREAM_ARGS(U64, U32, F32) \
   U64(xs) U64(y) U64(hc_out) U64(hc_mix) U64(hc_in) U64(w) U64(h16) U64(h32) U64(gather) U64(out16) U64(out32) \
   U64(embed) U64(tokens) U64(step) U64(sum_out) U32(W) U32(streams) U32(ld_h16) U32(ld_h32) U32(ld_out) \
-  U32(y_parts) U32(y_rows) F32(eps)
+  U32(y_parts) U32(y_rows) F32(eps) U32(split)
 
 /* out fp32 = x (fp32, or bf16 with f32 = 0) times w^T (bf16 rows), fp32 products and sums. */
 #define MF_PRODUCT_ARGS(U64, U32, F32) \
@@ -111,15 +113,12 @@ namespace mf {
   U64(x) U64(z) U64(dt) U64(dt_bias) U64(b) U64(c) U64(A) U64(D) U64(state) U64(tail) U64(x_in) U64(y) \
   U64(tok_pos) U32(ld_x) U32(ld_z) U32(ld_dt) U32(ld_bc) U32(ld_y) U32(channels) U32(n) U32(taps) U32(f32)
 
-/* Log input and forget gates of the matrix memory: out fp32 [rows][2 heads]. */
-#define MF_MEM_GATE_ARGS(U64, U32, F32) \
-  U64(h) U64(wi) U64(wf) U64(bi) U64(bf) U64(out) U32(K) U32(heads) U32(ld_h) F32(cap)
-
-/* state fp32 [slot][head][e + 1][d] (column e: the normaliser), m fp32 [slot][head][column
+/* gates fp32 [rows][ld_gates]: raw input gates of the heads, then forget gates; gate_bias fp32 [2 heads].
+ * state fp32 [slot][head][e + 1][d] (column e: the normaliser), m fp32 [slot][head][column
  * block]; out fp32 [rows][heads][e, the denominator, padding to a multiple of four]. */
 #define MF_MEMORY_ARGS(U64, U32, F32) \
-  U64(q) U64(k) U64(v) U64(gates) U64(state) U64(m) U64(out) U64(tok_pos) U32(ld_qkv) U32(heads) U32(d) U32(e) \
-  U32(f32) F32(q_scale)
+  U64(q) U64(k) U64(v) U64(gates) U64(gate_bias) U64(state) U64(m) U64(out) U64(tok_pos) U32(ld_qkv) U32(ld_gates) \
+  U32(heads) U32(d) U32(e) U32(f32) F32(q_scale) F32(cap)
 
 #define MF_HEAD_NORM_ARGS(U64, U32, F32) \
   U64(o) U64(g) U64(w) U64(out) U32(heads) U32(e) U32(ld_g) U32(ld_out) U32(f32) F32(eps)
@@ -175,7 +174,6 @@ MF_DECLARE(GatedArgs, MF_GATED_ARGS, 64)
 MF_DECLARE(SumArgs, MF_SUM_ARGS, 64)
 MF_DECLARE(ConvArgs, MF_CONV_ARGS, 128)
 MF_DECLARE(ScanArgs, MF_SCAN_ARGS, 192)
-MF_DECLARE(MemGateArgs, MF_MEM_GATE_ARGS, 64)
 MF_DECLARE(MemoryArgs, MF_MEMORY_ARGS, 128)
 MF_DECLARE(HeadNormArgs, MF_HEAD_NORM_ARGS, 64)
 MF_DECLARE(LatentArgs, MF_LATENT_ARGS, 128)

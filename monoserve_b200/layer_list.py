@@ -5,8 +5,9 @@ a span of layers may run several times in a row.
 `LayerListLane` builds the chain of one batch on the fabric's tiles, one run of a layer after the other:
 
   streams (53: update of the streams by the sublayer before, the next sublayer's input, its norm)
-    selective scan:    in GEMM (32) -> conv + silu (54) -> x GEMM (K ranges) -> slab sum (62) -> dt GEMM -> scan (55) -> o GEMM
-    matrix memory:     q k v g GEMM, gates (56) beside it -> memory (57) -> head norm (58) -> o GEMM
+    selective scan:    in GEMM (32) -> conv + silu (54) -> x GEMM (K ranges) -> slab sum (62) -> dt GEMM -> scan (55; one
+                       token: 65) -> o GEMM
+    matrix memory:     q k v g GEMM, gates GEMM beside it -> memory (57; one token: 56) -> head norm (58) -> o GEMM
     latent attention:  q + latent GEMM -> latent norm, rotation, cache append (59) -> per head W_uk^T q GEMM ->
                        attention over the cached latents (63 on the tensor cores, 60 in 32-bit; 61) -> per head W_uv
                        GEMM -> o GEMM; for a whole prompt: keys and values GEMM -> attention (64) -> o GEMM
@@ -32,10 +33,10 @@ from monoserve_b200.fabric import Program, Tile, tile_array
 from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_STORE, HEIGHTS, K_GEMM, K_SAMPLE, SPLIT_PARTS, SPLIT_ROWS,
                                       LaneBase, _block, _bm, _retarget)
 
-K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEM_GATES, K_MEMORY = 51, 52, 53, 54, 55, 56, 57
+K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEMORY_STEP, K_MEMORY, K_SCAN_STEP = 51, 52, 53, 54, 55, 56, 57, 65
 K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA, K_LATENT_DIRECT = 58, 59, 60, 61, 62, 63, 64
 MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
-SCAN_CHANNELS, MEMORY_COLUMNS = 32, 32   # of one tile
+SCAN_CHANNELS, MEMORY_COLUMNS, STEP_CHANNELS = 32, 32, 512   # of one tile
 WIDE_ROWS, WIDE_PARTS = 512, 4           # K ranges of the products that end a sublayer, up to this many rows
 MAX_ATTN_PARTS = 32
 RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys per step of the tensor-core attention tiles
@@ -220,8 +221,9 @@ class MatrixMemory:
     @staticmethod
     def place(W, w, m, g):
         w.qkvg, w.o = W.mat(torch.cat([g(n) for n in "qkvg"])), W.mat(g("o"))
-        w.wi, w.wf = (g(n).to(torch.bfloat16).contiguous().cuda() for n in "if")
-        w.bi, w.bf, w.norm = W.f32(g("i.b")), W.f32(g("f.b")), W.f32(g("norm"))
+        gates = W.mat(torch.cat([g("i"), g("f")]))
+        w.gates = gates if W.cfg.f32 else torch.cat([gates] * 3, -1).contiguous()   # one copy per part of a split row
+        w.gate_b, w.norm = W.f32(torch.cat([g("i.b"), g("f.b")])), W.f32(g("norm"))
 
     @staticmethod
     def state(cfg, m, rows, slots):
@@ -231,21 +233,20 @@ class MatrixMemory:
     @staticmethod
     def sizes(m):
         return dict(proj=2 * m.heads * (m.dim + m.vdim), mix=m.heads * m.vdim, small=2 * m.heads, raw=m.heads * up(m.vdim + 1, 4),
-                    h32=1)
+                    split=1)
 
     @staticmethod
     def build(lane, p, l, run, b, prev):
         m, w, st, T = lane.cfg.layers[l].m, lane.w.layers[l], lane.kv.runs[run], b.T
         f32, H, d, e, es = int(lane.cfg.f32), m.heads, m.dim, m.vdim, lane.proj.es
         s = lane.product(p, prev, lane.h, w.qkvg, lane.proj, T, 2 * H * (d + e), lane.cfg.hidden, ("memory_in", run), out16=True)
-        gates = lane._dev("MemGateArgs", h=lane.h32.addr, wi=w.wi, wf=w.wf, bi=w.bi, bf=w.bf, out=lane.small.addr,
-                          K=lane.cfg.hidden, heads=H, ld_h=lane.h32.ld, cap=m.gate_cap)
-        s_g = p.stage(_retarget(b.gate_tiles(2 * H), a0=gates.data_ptr()), label=("memory_gates", run))
-        p.after(prev, s_g)
+        # the gates enter the recurrence: their projection takes the whole 32-bit row, as three bf16 parts on the tensor cores
+        k = lane.cfg.hidden if f32 else 3 * up(lane.cfg.hidden, 64)
+        s_g = lane.product(p, prev, lane.h, w.gates, lane.small, T, 2 * H, k, ("memory_gates", run))
         at = lane.proj.addr
-        mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=lane.small.addr, state=st["S"],
-                        m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos, ld_qkv=lane.proj.ld, heads=H, d=d, e=e, f32=f32,
-                        q_scale=d ** -0.5)
+        mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=lane.small.addr,
+                        gate_bias=w.gate_b, state=st["S"], m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos,
+                        ld_qkv=lane.proj.ld, ld_gates=lane.small.ld, heads=H, d=d, e=e, f32=f32, q_scale=d ** -0.5, cap=m.gate_cap)
         s_m = p.stage(_retarget(b.memory_tiles(H, e), a0=mem.data_ptr()), label=("memory", run))
         p.after(s, s_m)
         p.after(s_g, s_m)
@@ -326,7 +327,7 @@ class LatentAttention:
     def absorbed(lane, p, m, w, cache, b, run, prev):
         """Rows that attend to cached latents: W_uk^T q, attention over the latents themselves, W_uv."""
         f32, H, d, r, c = int(lane.cfg.f32), m.heads, m.dim, m.rot_dim, m.kv_rank
-        ld_q, ld_o, spans = up(c + r, 8), up(c, 64), [(row0, n) for row0, n, _ in b.requests]
+        ld_q, ld_o, spans = up(c + r, 8), up(c, 64), b.spans()
         s = lane.head_product(p, prev, lane.q_un.addr, up(d, 64), w.uk, lane.q_all.addr, ld_q, lane.T * ld_q, spans, c, d,
                               ("latent_q", run))
         shape = None if f32 else latent_tile(m, lane.kv.page, max(n for _, n, _ in b.requests))
@@ -336,7 +337,7 @@ class LatentAttention:
                       f32=f32, scale=m.scale)
         if shape:
             tokens, heads, buffers = shape
-            blocks = sum(-(-n // tokens) for _, n in spans) * -(-H // heads)
+            blocks = sum(-(-n // tokens) for _, n, _ in b.requests) * -(-H // heads)
             parts = lane.attn_parts(H, blocks)
             fields.update(q_map=lane.q_map(m, tokens, heads), kv_map=lane.kv_map(m, cache), tokens=tokens, group=heads,
                           buffers=buffers)
@@ -394,11 +395,21 @@ class _Batch:
             return [self.requests[i] for i in whole], _Batch(self.lane, [q for i, q in enumerate(self.requests) if i not in whole])
         return self._once("split", make)
 
+    def spans(self):
+        """The batch's rows as (first, rows), requests that lie side by side together."""
+        out = []
+        for row0, n, _ in self.requests:
+            if out and sum(out[-1]) == row0:
+                out[-1] = (out[-1][0], out[-1][1] + n)
+            else:
+                out.append((row0, n))
+        return out
+
     def item_tiles(self, kind, per_row, **ops):
         """Item-wise tiles over the batch's rows, items row * per_row + j."""
         def make():
             per = self.lane.items_per(self.T * per_row)
-            spans = [(row0 * per_row + i, min(per, n * per_row - i)) for row0, n, _ in self.requests for i in range(0, n * per_row, per)]
+            spans = [(row0 * per_row + i, min(per, n * per_row - i)) for row0, n in self.spans() for i in range(0, n * per_row, per)]
             first, count = (np.array(v) for v in zip(*spans))
             return tile_array(kind, i0=first, i1=count, **ops)
         return self._once((kind, per_row, tuple(ops.items())), make)
@@ -421,25 +432,34 @@ class _Batch:
         return self._once(("conv", channels), make)
 
     def scan_tiles(self, channels):
-        return self._once(("scan", channels), lambda: np.concatenate(
-            [tile_array(K_SCAN, i0=row0, i1=n, i2=np.arange(0, channels, SCAN_CHANNELS), i3=slot)
-             for row0, n, slot in sorted(self.requests, key=lambda q: -q[1])]))
+        """Portions: a tile per block of channels, the longest first; single tokens: wider blocks of one row each."""
+        def make():
+            out = [tile_array(K_SCAN, i0=row0, i1=n, i2=np.arange(0, channels, SCAN_CHANNELS), i3=slot)
+                   for row0, n, slot in sorted(self.requests, key=lambda q: -q[1]) if n > 1]
+            ones = [(row0, slot) for row0, n, slot in self.requests if n == 1]
+            if ones:
+                row, slot = (np.array(v)[:, None] for v in zip(*ones))
+                c = np.arange(0, channels, STEP_CHANNELS)[None]
+                out.append(tile_array(K_SCAN_STEP, i0=row, i1=np.minimum(STEP_CHANNELS, channels - c), i2=c, i3=slot))
+            return np.concatenate(out)
+        return self._once(("scan", channels), make)
 
     def memory_tiles(self, heads, e):
+        """Portions: a tile per head and block of columns; single tokens: as many column blocks in a tile as leave every
+        worker one."""
         def make():
             blocks = -(-(e + 1) // MEMORY_COLUMNS)
             h, c = np.meshgrid(np.arange(heads), np.arange(blocks), indexing="ij")
-            return np.concatenate([tile_array(K_MEMORY, i0=row0, i1=n, i2=h | (c << 16), i3=slot)
-                                   for row0, n, slot in sorted(self.requests, key=lambda q: -q[1])])
+            out = [tile_array(K_MEMORY, i0=row0, i1=n, i2=h | (c << 16), i3=slot)
+                   for row0, n, slot in sorted(self.requests, key=lambda q: -q[1]) if n > 1]
+            ones = [(row0, slot) for row0, n, slot in self.requests if n == 1]
+            if ones:
+                row, slot = (np.array(v)[:, None, None] for v in zip(*ones))
+                per = min(128, -(-blocks // min(blocks, max(1, self.lane.fab.num_workers // (len(ones) * heads)))))
+                h, c = np.arange(heads)[None, :, None], np.arange(0, blocks, per)[None, None, :]
+                out.append(tile_array(K_MEMORY_STEP, i0=row, i1=np.minimum(per, blocks - c), i2=h | (c << 16), i3=slot))
+            return np.concatenate(out)
         return self._once(("memory", heads, e), make)
-
-    def gate_tiles(self, outputs):
-        per_out, per_row = (8, 4) if self.T <= SPLIT_ROWS else (outputs, 16)
-
-        def make():
-            r, o = np.meshgrid(np.arange(0, self.T, per_row), np.arange(0, outputs, per_out), indexing="ij")
-            return tile_array(K_MEM_GATES, i0=r, i1=np.minimum(per_row, self.T - r), i2=o, i3=np.minimum(per_out, outputs - o))
-        return self._once(("gates", outputs), make)
 
     def attn_tiles(self, heads, parts):
         """One tile per row, group of heads and part, the rows that see most keys first."""
@@ -489,8 +509,9 @@ class LayerListLane(LaneBase):
                 else:
                     sizes[name] = max(sizes.get(name, 0), v)
         self.xs = z(T, cfg.streams, H)
-        self.h = _Buf(self, T, H, act)
-        self.h32 = self.h if cfg.f32 else (_Buf(self, T, H, f32) if "h32" in sizes else None)
+        # a row of h, and behind it what its bf16 rounding has left, for products that take the whole 32-bit row
+        self.split = up(H, 64) if "split" in sizes and not cfg.f32 else 0
+        self.h = _Buf(self, T, 3 * self.split or H, act)
         ff = max([layer.ff for layer in cfg.layers] + [0])
         self.hd = _Buf(self, T, ff, act) if ff else None
         self.gu = _Buf(self, T, 2 * ff, f32) if ff and cfg.f32 else None
@@ -544,7 +565,7 @@ class LayerListLane(LaneBase):
             if layer.kind == "mamba1":
                 wm(lw.in_), wm(lw.x), wm(lw.dt), self.act.maps(m.inner), self.dt_in.maps(m.dt_rank), self.mix.maps(m.inner)
             elif layer.kind == "mlstm":
-                wm(lw.qkvg), self.mix.maps(m.heads * m.vdim)
+                wm(lw.qkvg), wm(lw.gates), self.h.maps(3 * self.split), self.mix.maps(m.heads * m.vdim)
             else:
                 wm(lw.qkv), wm(lw.uk), wm(lw.uv), self.mix.maps(m.heads * m.vdim)
                 self.head_maps(self.q_un.addr, up(m.dim, 64), m.dim, m.heads)
@@ -692,7 +713,7 @@ class LayerListLane(LaneBase):
         return self._hmaps[key]
 
     # ------------------------------------------------------------------ programs
-    def _streams(self, p, rows, prev, sub, before, label, h32=False, gather=False, step=False):
+    def _streams(self, p, rows, prev, sub, before, label, split=False, gather=False, step=False):
         """The streams stage in front of sublayer `sub` = (hc_in, norm): `before` = ((hc_out, hc_mix), parts, slab rows,
         run whose residual this completes or None) of the sublayer behind it, or None at the embedding."""
         cfg = self.cfg
@@ -711,9 +732,7 @@ class LayerListLane(LaneBase):
             if cfg.f32:
                 f.update(h32=self.h.addr, ld_h32=self.h.ld)
             else:
-                f.update(h16=self.h.addr, ld_h16=self.h.ld)
-                if h32:
-                    f.update(h32=self.h32.addr, ld_h32=self.h32.ld)
+                f.update(h16=self.h.addr, ld_h16=self.h.ld, split=self.split if split else 0)
         args = self._dev("StreamArgs", **f)
         s = p.stage(self._rows(K_STREAMS, args, rows, self._per(rows)), label=label)
         if prev is not None:
@@ -728,7 +747,7 @@ class LayerListLane(LaneBase):
         before = None
         for run, l in enumerate(cfg.order):
             layer, w = cfg.layers[l], self.w.layers[l]
-            prev = self._streams(p, T, prev, (w.hc1[0], w.norm1), before, ("streams", run), h32=layer.kind == "mlstm", step=step)
+            prev = self._streams(p, T, prev, (w.hc1[0], w.norm1), before, ("streams", run), split=layer.kind == "mlstm", step=step)
             first = prev if first is None else first
             prev, parts, slab = MIXERS[layer.kind].build(self, p, l, run, b, prev)
             before = (w.hc1[1:], parts, slab, None if layer.ff else run)

@@ -114,6 +114,7 @@ MIXED = config([MEMORY, LATENT, SCAN, LATENT], width=112, vocab=160, streams=2, 
 WIDE = config([(scan(inner=520, state=64, dt_rank=40, conv=5), None), latent(heads=17, dim=64, rot=32, vdim=96, rank=320, base=1e4, scale=0.1),
                memory(heads=1, dim=300, vdim=65, cap=15.0), (memory(heads=4, dim=130, vdim=31, cap=15.0), None)],
               width=1100, vocab=333, streams=4, ff=700)
+SERVED = config([LATENT, SCAN, MEMORY], width=112, vocab=160, streams=2, ff=64)   # magnifies rounding little
 ONES = config([scan(inner=1, state=1, dt_rank=1, conv=2), latent(heads=1, dim=1, rot=2, vdim=1, rank=1, base=10.0, scale=1.0),
                memory(heads=1, dim=1, vdim=2, cap=1.0)], width=16, vocab=16, streams=1, ff=1)
 ALONE = {"scan": config([SCAN], 96, 128, 3), "memory": config([MEMORY], 96, 128, 3), "latent": config([LATENT], 96, 128, 3),

@@ -192,7 +192,7 @@ def test_greedy_generation_through_the_serving_loop(dtype, slack):
     """More requests than decode rows, of unequal lengths, through monoserve_b200.generate: continuous batching, slots and
     pages handed on, one long generation."""
     from monoserve_b200.generate import generate
-    c = lm.MIXED
+    c = lm.SERVED
     t = lm.tensors(c, 9)
     prompts = [lm.tokens(c, n, 60 + n) for n in (33, 1, 12, 50, 7, 21, 2)]
     results = generate(model_of(c, t, dtype), prompts, max_tokens=40, max_decode=3, token_budget=64)
