@@ -47,6 +47,13 @@ __device__ __forceinline__ float4 ld_four(const void* p) {
 __device__ __forceinline__ float capped(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
+// The raw gate at `p`: the sum of a K-split product's slabs.
+__device__ __forceinline__ float raw_gate(const MemoryArgs& A, const float* p) {
+  float v = *p;
+  for (uint32_t q = 1; q < A.gate_parts; ++q) v += p[static_cast<size_t>(q) * A.gate_rows * A.ld_gates];
+  return v;
+}
+
 // R values per lane (R <= 32, a power of two) summed over the warp: lane l ends with the sum of value l / (32 / R).
 template <int R>
 __device__ __forceinline__ float warp_sum_each(float (&r)[R], int lane) {
@@ -68,7 +75,7 @@ template <int ND, bool F32>
 __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ring) {
   using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
   constexpr int kPer16 = 16 / static_cast<int>(sizeof(T));
-  constexpr int kTokens = (ND == 4 && F32) ? 16 : 32;
+  constexpr int kTokens = (ND == 4 && F32) ? 16 : 32, kGroup = ND == 4 ? 2 : 4;
   MemoryArgs A;
   load_block(A, t.a[0]);
   __builtin_assume(__isShared(ring));
@@ -80,6 +87,7 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
   T* const buf = reinterpret_cast<T*>(ring);
   const int buf_elems = kTokens * (2 * ds + kMemColumns);   // k, q, v
   const int c_lo = col0 + warp * 8;                          // this warp's first column
+  const bool edge = c_lo + 8 > e;
   const int n_v = min(kMemColumns, e - col0);                // columns of v in this block (at most 0: only the normaliser)
   float* const state = reinterpret_cast<float*>(A.state) + (static_cast<size_t>(slot) * H + head) * (e + 1) * dp;
   unsigned long long S[8][ND][2];
@@ -133,8 +141,8 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
   auto load_gates = [&](int base, float& gi, float& gf) {   // one token per lane
     const int nt = min(kTokens, rows - base);
     const size_t at = static_cast<size_t>(row0 + base + min(lane, nt - 1)) * A.ld_gates + head;
-    gi = lane < nt ? capped(gates[at] + bi, A.cap) : -INFINITY;
-    gf = lane < nt ? log_sigmoid(capped(gates[at + H] + bf, A.cap)) : 0.f;
+    gi = lane < nt ? capped(raw_gate(A, gates + at) + bi, A.cap) : -INFINITY;
+    gf = lane < nt ? log_sigmoid(capped(raw_gate(A, gates + at + H) + bf, A.cap)) : 0.f;
   };
   stage(0, buf);
   float gi, gf;
@@ -172,24 +180,25 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
     const T* const sk = buf + s * buf_elems;
     const T* const sq = sk + kTokens * ds;
     const T* const sv = sq + kTokens * ds + warp * 8;
-    for (int t0 = 0; t0 < nt; t0 += 4) {   // four tokens' read-outs are summed over the warp together
-      float r[32];                        // [token][column]
+#pragma unroll 1
+    for (int t0 = 0; t0 < nt; t0 += kGroup) {   // the read-outs of kGroup tokens are summed over the warp together
+      float r[8 * kGroup];                       // [token][column]
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
+      for (int u = 0; u < kGroup; ++u) {
         const int tok = min(t0 + u, nt - 1);
-        const bool live = t0 + u < nt;      // a token past the end keeps the state and adds nothing
-        const float kp_ = __shfl_sync(0xffffffffu, keep, tok), ad_ = __shfl_sync(0xffffffffu, add, tok);
-        const float kp = live ? kp_ : 1.f, ad = live ? ad_ : 0.f;
-        const unsigned long long kp2 = pk2(kp, kp);
-        unsigned long long acc[8], av2[8];
-        const float4 va = ld_four<F32>(sv + tok * kMemColumns), vb = ld_four<F32>(sv + tok * kMemColumns + 4);
-        const float v[8] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
-#pragma unroll
-        for (int c = 0; c < 8; ++c) {
-          const float av = c_lo + c < e ? ad * v[c] : (c_lo + c == e ? ad : 0.f);
-          av2[c] = pk2(av, av);
-          acc[c] = 0ull;
+        float kp = __shfl_sync(0xffffffffu, keep, tok), ad = __shfl_sync(0xffffffffu, add, tok);
+        if (t0 + u >= nt) {                      // a token past the end keeps the state and adds nothing
+          kp = 1.f;
+          ad = 0.f;
         }
+        const unsigned long long kp2 = pk2(kp, kp);
+        const float4 va = ld_four<F32>(sv + tok * kMemColumns), vb = ld_four<F32>(sv + tok * kMemColumns + 4);
+        float v[8] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
+        if (edge) {                              // this warp's columns reach past the values: the normaliser's v is 1
+#pragma unroll
+          for (int c = 0; c < 8; ++c) v[c] = c_lo + c < e ? v[c] : (c_lo + c == e ? 1.f : 0.f);
+        }
+        unsigned long long kk[ND][2], qq[ND][2];
 #pragma unroll
         for (int i = 0; i < ND; ++i) {
           const int at = i * 128 + lane * 4;
@@ -198,25 +207,31 @@ __device__ __noinline__ void memory_rows(const TileDesc& t, int tid, uint8_t* ri
             k4 = ld_four<F32>(sk + tok * ds + at);
             q4 = ld_four<F32>(sq + tok * ds + at);
           }
-          const unsigned long long k0 = pk2(k4.x, k4.y), k1 = pk2(k4.z, k4.w), q0 = pk2(q4.x, q4.y), q1 = pk2(q4.z, q4.w);
-#pragma unroll
-          for (int c = 0; c < 8; ++c) {
-            S[c][i][0] = fma2(av2[c], k0, mul2(kp2, S[c][i][0]));
-            S[c][i][1] = fma2(av2[c], k1, mul2(kp2, S[c][i][1]));
-            acc[c] = fma2(S[c][i][0], q0, acc[c]);
-            acc[c] = fma2(S[c][i][1], q1, acc[c]);
-          }
+          kk[i][0] = mul2(pk2(ad, ad), pk2(k4.x, k4.y));
+          kk[i][1] = mul2(pk2(ad, ad), pk2(k4.z, k4.w));
+          qq[i][0] = pk2(q4.x, q4.y);
+          qq[i][1] = pk2(q4.z, q4.w);
         }
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
-          const float2 f = unpk2(acc[c]);
+          unsigned long long acc = 0ull;
+          const unsigned long long v2 = pk2(v[c], v[c]);
+#pragma unroll
+          for (int i = 0; i < ND; ++i)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+              S[c][i][j] = fma2(v2, kk[i][j], mul2(kp2, S[c][i][j]));
+              acc = fma2(S[c][i][j], qq[i][j], acc);
+            }
+          const float2 f = unpk2(acc);
           r[u * 8 + c] = f.x + f.y;
         }
       }
-      const float read = warp_sum_each<32>(r, lane) * A.q_scale;
-      const int tok = t0 + (lane >> 3), c = c_lo + (lane & 7);
+      const float read = warp_sum_each<8 * kGroup>(r, lane) * A.q_scale;
+      constexpr int kStep = 4 / kGroup;          // lanes per sum
+      const int tok = t0 + lane / (8 * kStep), c = c_lo + (lane / kStep) % 8;
       const float fl = __shfl_sync(0xffffffffu, floor_, tok & 31);
-      if (tok < nt && c <= e)
+      if (lane % kStep == 0 && tok < nt && c <= e)
         reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row0 + base + tok) * H + head) * oe + c] =
             c < e ? read : fmaxf(fabsf(read), fl) + 1e-6f;
     }
@@ -285,8 +300,8 @@ __device__ __noinline__ void memory_step(const TileDesc& t, int tid) {
       k[i][j] = at < d ? value(gk[at]) : 0.f;
       q[i][j] = at < d ? value(gq[at]) * A.q_scale : 0.f;
     }
-  const float gi = capped(gates[head] + f32p(A.gate_bias)[head], A.cap);
-  const float gf = log_sigmoid(capped(gates[H + head] + f32p(A.gate_bias)[H + head], A.cap));
+  const float gi = capped(raw_gate(A, gates + head) + f32p(A.gate_bias)[head], A.cap);
+  const float gf = log_sigmoid(capped(raw_gate(A, gates + H + head) + f32p(A.gate_bias)[H + head], A.cap));
   const float m = fmaxf(gf + m_old, gi);
   const float keep = expf(gf + m_old - m), add = expf(gi - m), floor_ = expf(-m);
   exec_sync();   // every thread has read the old maximum

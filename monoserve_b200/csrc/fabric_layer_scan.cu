@@ -131,7 +131,7 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
   const int row0 = static_cast<int>(t.i0), rows = static_cast<int>(t.i1), slot = static_cast<int>(t.i3);
   const int ch0 = static_cast<int>(t.i2);
   const int n = static_cast<int>(A.n), C = static_cast<int>(A.channels), taps = static_cast<int>(A.taps);
-  const int warp = tid >> 5, lane = tid & 31, p = tid & 3, quad = lane & ~3, my = tid >> 2;
+  const int warp = tid >> 5, lane = tid & 31, p = tid & 3, my = tid >> 2;
   const int c = min(ch0 + my, C - 1);                     // a channel past the end repeats the last one
   const bool c_ok = ch0 + my < C;
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
@@ -146,11 +146,10 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
   }
   const float D = f32p(A.D)[c], dt_bias = f32p(A.dt_bias)[c];
   const bool z16 = (A.z & 15) == 0, bc16 = ((A.b | A.c) & 15) == 0 && (n & 3) == 0;
-  if (n < NP) {   // the padding of B and C stays zero
-    for (int i = tid; i < 2 * kScanTokens * 2 * NP; i += kExecThreads)
-      (&sh.in[i / (kScanTokens * 2 * NP)].bc[0][0])[i % (kScanTokens * 2 * NP)] = 0.f;
-    exec_sync();
-  }
+  // the padding of B and C, and their rows past the end of a short chunk, must be finite
+  for (int i = tid; i < 2 * kScanTokens * 2 * NP; i += kExecThreads)
+    (&sh.in[i / (kScanTokens * 2 * NP)].bc[0][0])[i % (kScanTokens * 2 * NP)] = 0.f;
+  exec_sync();
   auto stage = [&](int base, Chunk& k) {
     const int nt = min(kScanTokens, rows - base);
     const T* x = reinterpret_cast<const T*>(A.x);
@@ -206,28 +205,28 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
       cp_wait<0>();
     }
     exec_sync();
-    const Chunk& k = sh.in[s];
+    Chunk& k = sh.in[s];
     // Step sizes of the chunk, lane p those of tokens p, p + 4, ...; a token past the end gets step 0 and input 0, which
-    // leaves the state as it is.
-    float dts[kScanTokens / 4], xs[kScanTokens / 4];
-#pragma unroll
-    for (int g = 0; g < kScanTokens / 4; ++g) {
-      const int mine = 4 * g + p;
+    // leaves the state as it is.  (Loops stay rolled: one warp per scheduler runs this, and a body beyond the instruction
+    // cache costs more than it hides.)
+#pragma unroll 2
+    for (int mine = p; mine < kScanTokens; mine += 4) {
       const float u = k.dt[mine][my] + dt_bias;
       const float dt = F32 ? softplus32(u) : fmaxf(u, 0.f) + __logf(1.f + __expf(-fabsf(u)));
-      dts[g] = mine < nt ? dt : 0.f;
-      xs[g] = mine < nt ? value(k.x[mine][my]) : 0.f;
+      k.dt[mine][my] = mine < nt ? dt : 0.f;
     }
-#pragma unroll
-    for (int g = 0; g < kScanTokens / 4; ++g) {
-      if (4 * g >= nt) break;   // the same in all threads
-      const float dt = dts[g], dtx = dts[g] * xs[g];
+    __syncwarp();
+#pragma unroll 1
+    for (int g = 0; g < nt; g += 4) {
+      const int mine = g + p;
+      const float x = value(k.x[mine][my]), z = value(k.z[mine][my]);
       float part[4];
 #pragma unroll
       for (int i4 = 0; i4 < 4; ++i4) {
-        const float dk = __shfl_sync(0xffffffffu, dt, quad + i4), xk = __shfl_sync(0xffffffffu, dtx, quad + i4);
+        const float dk = k.dt[g + i4][my];
+        const float xk = g + i4 < nt ? dk * value(k.x[g + i4][my]) : 0.f;
         float B[NS], Cv[NS];
-        const float *b = &k.bc[4 * g + i4][s0], *cc = &k.bc[4 * g + i4][NP + s0];
+        const float *b = &k.bc[g + i4][s0], *cc = &k.bc[g + i4][NP + s0];
         if constexpr ((NS & 3) == 0) {
 #pragma unroll
           for (int i = 0; i < NS; i += 4) {
@@ -244,10 +243,8 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
         float y = 0.f;
 #pragma unroll
         for (int i = 0; i < NS; ++i) {
-          // past the end B may be anything (its factor is 0), so it must not be let into the sum
-          const float in = 4 * g + i4 < nt ? xk * B[i] : 0.f;
-          if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), in);
-          else S[i] = fmaf(ex2(dk * a[i]), S[i], in);
+          if constexpr (F32) S[i] += fmaf(S[i], expm1f(dk * a[i]), xk * B[i]);
+          else S[i] = fmaf(ex2(dk * a[i]), S[i], xk * B[i]);
           y = fmaf(S[i], Cv[i], y);
         }
         part[i4] = y;
@@ -257,10 +254,8 @@ __device__ __noinline__ void scan_rows(const TileDesc& t, int tid, uint8_t* ring
       const float t0 = (odd ? part[1] : part[0]) + __shfl_xor_sync(0xffffffffu, odd ? part[0] : part[1], 1);
       const float t1 = (odd ? part[3] : part[2]) + __shfl_xor_sync(0xffffffffu, odd ? part[2] : part[3], 1);
       const float out = (hi ? t1 : t0) + __shfl_xor_sync(0xffffffffu, hi ? t0 : t1, 2);
-      const int mine = 4 * g + p;
       if (mine < nt) {
-        const float z = value(k.z[mine][my]);
-        const float y = fmaf(D, xs[g], out) * (F32 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)));
+        const float y = fmaf(D, x, out) * (F32 ? z / (1.f + expf(-z)) : __fdividef(z, 1.f + __expf(-z)));
         if constexpr (F32) sh.y[mine][my] = y;
         else sh.y[mine][my] = __float2bfloat16(y);
       }

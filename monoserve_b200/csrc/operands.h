@@ -113,12 +113,13 @@ namespace mf {
   U64(x) U64(z) U64(dt) U64(dt_bias) U64(b) U64(c) U64(A) U64(D) U64(state) U64(tail) U64(x_in) U64(y) \
   U64(tok_pos) U32(ld_x) U32(ld_z) U32(ld_dt) U32(ld_bc) U32(ld_y) U32(channels) U32(n) U32(taps) U32(f32)
 
-/* gates fp32 [rows][ld_gates]: raw input gates of the heads, then forget gates; gate_bias fp32 [2 heads].
+/* gates fp32 [rows][ld_gates]: raw input gates of the heads, then forget gates, as gate_parts slabs of
+ * gate_rows rows to be added; gate_bias fp32 [2 heads].
  * state fp32 [slot][head][e + 1][d] (column e: the normaliser), m fp32 [slot][head][column
  * block]; out fp32 [rows][heads][e, the denominator, padding to a multiple of four]. */
 #define MF_MEMORY_ARGS(U64, U32, F32) \
   U64(q) U64(k) U64(v) U64(gates) U64(gate_bias) U64(state) U64(m) U64(out) U64(tok_pos) U32(ld_qkv) U32(ld_gates) \
-  U32(heads) U32(d) U32(e) U32(f32) F32(q_scale) F32(cap)
+  U32(gate_parts) U32(gate_rows) U32(heads) U32(d) U32(e) U32(f32) F32(q_scale) F32(cap)
 
 #define MF_HEAD_NORM_ARGS(U64, U32, F32) \
   U64(o) U64(g) U64(w) U64(out) U32(heads) U32(e) U32(ld_g) U32(ld_out) U32(f32) F32(eps)

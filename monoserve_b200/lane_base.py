@@ -243,10 +243,11 @@ class LaneBase:
         return p.stage(tiles, mark=mark, label=label)
 
     def _gemm(self, p, wmap, amaps, rows, n_out, k, out, ld_out, epi, label, residual=None, ld_res=0, mark=None,
-              mat=None, bias=None, up_offset=0):
+              mat=None, bias=None, up_offset=0, bm=None):
         """A dense GEMM stage: out[rows][n_out] = act[rows][k] x weight[n_out (x2 for SiLU-mul)][k]^T.
-        mat: the weight's Mat (e4m3 weights carry their scales into the tiles)."""
-        bm = _bm(rows)
+        mat: the weight's Mat (e4m3 weights carry their scales into the tiles); bm: the row-block height, when not the
+        largest."""
+        bm = bm or _bm(rows)
         fp8 = mat is not None and mat.fp8
         args = self.arena.put(_C.gemm_args(
             out=out.data_ptr(), ld_out=ld_out, k_tiles=-(-k // 64), epi=epi, bm=bm, n_limit=n_out,

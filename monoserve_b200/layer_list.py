@@ -38,7 +38,7 @@ K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA, K_
 MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
 SCAN_CHANNELS, MEMORY_COLUMNS, STEP_CHANNELS = 32, 32, 512   # of one tile
 WIDE_ROWS, WIDE_PARTS = 512, 4           # K ranges of the products that end a sublayer, up to this many rows
-MAX_ATTN_PARTS = 32
+MAX_ATTN_PARTS, ATTN_ROUNDS = 32, 2
 RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys per step of the tensor-core attention tiles
 DIRECT_ROWS = 32                         # a prompt of at least this many tokens maps its keys and values out of the latents
 
@@ -242,11 +242,13 @@ class MatrixMemory:
         s = lane.product(p, prev, lane.h, w.qkvg, lane.proj, T, 2 * H * (d + e), lane.cfg.hidden, ("memory_in", run), out16=True)
         # the gates enter the recurrence: their projection takes the whole 32-bit row, as three bf16 parts on the tensor cores
         k = lane.cfg.hidden if f32 else 3 * up(lane.cfg.hidden, 64)
-        s_g = lane.product(p, prev, lane.h, w.gates, lane.small, T, 2 * H, k, ("memory_gates", run))
+        parts = 1 if f32 else lane.split_parts(T, k)
+        raw, ld = (lane.slabs, 2 * H) if parts > 1 else (lane.small, lane.small.ld)
+        s_g = lane.product(p, prev, lane.h, w.gates, raw, T, 2 * H, k, ("memory_gates", run), parts=parts, ld_out=ld)
         at = lane.proj.addr
-        mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=lane.small.addr,
-                        gate_bias=w.gate_b, state=st["S"], m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos,
-                        ld_qkv=lane.proj.ld, ld_gates=lane.small.ld, heads=H, d=d, e=e, f32=f32, q_scale=d ** -0.5, cap=m.gate_cap)
+        mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=raw.addr,
+                        gate_parts=parts, gate_rows=lane.slab_rows(T), gate_bias=w.gate_b, state=st["S"], m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos,
+                        ld_qkv=lane.proj.ld, ld_gates=ld, heads=H, d=d, e=e, f32=f32, q_scale=d ** -0.5, cap=m.gate_cap)
         s_m = p.stage(_retarget(b.memory_tiles(H, e), a0=mem.data_ptr()), label=("memory", run))
         p.after(s, s_m)
         p.after(s_g, s_m)
@@ -620,10 +622,19 @@ class LayerListLane(LaneBase):
                                  slab_rows=self.slab_rows(rows))
         else:
             s = self._gemm(p, self.weight_map(w), x.maps(k), rows, n, k, out.t, ld,
-                           epi if epi is not None else (EPI_STORE if out16 else EPI_F32), label, up_offset=up_offset)
+                           epi if epi is not None else (EPI_STORE if out16 else EPI_F32), label, up_offset=up_offset,
+                           bm=self.row_block(rows, n))
         for stage in prev if isinstance(prev, list) else [prev]:
             p.after(stage, s)
         return s
+
+    def row_block(self, rows, n):
+        """Row-block height of a GEMM: the largest that still gives most workers a tile (a narrow product over many rows
+        takes lower blocks), at least 32 rows."""
+        for bm in reversed(HEIGHTS):
+            if bm <= _bm(rows) and -(-rows // bm) * -(-n // 128) * 4 >= 3 * self.fab.num_workers:
+                return bm
+        return min(32, _bm(rows))
 
     def _product_tiles(self, rows, n, row0=0):
         key = ("product", rows, n, row0)
@@ -697,7 +708,7 @@ class LayerListLane(LaneBase):
     def attn_parts(self, heads, tiles):
         """Key ranges per row: enough of them to give every worker about two tiles (the split workspace is addressed by
         row, so it covers the rows of a small program only)."""
-        want = min(MAX_ATTN_PARTS, 2 * self.fab.num_workers // tiles)
+        want = min(MAX_ATTN_PARTS, ATTN_ROUNDS * self.fab.num_workers // tiles)
         return max(1, want) if self.rows_now <= SPLIT_ROWS else 1
 
     def direct_maps(self, m):
