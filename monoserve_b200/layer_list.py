@@ -38,7 +38,7 @@ K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA, K_
 MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
 SCAN_CHANNELS, MEMORY_COLUMNS, STEP_CHANNELS = 32, 32, 512   # of one tile
 WIDE_ROWS, WIDE_PARTS = 512, 4           # K ranges of the products that end a sublayer, up to this many rows
-MAX_ATTN_PARTS, ATTN_ROUNDS = 32, 2
+MAX_ATTN_PARTS, ATTN_ROUNDS = 32, 1
 RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys per step of the tensor-core attention tiles
 DIRECT_ROWS = 32                         # a prompt of at least this many tokens maps its keys and values out of the latents
 
@@ -706,7 +706,7 @@ class LayerListLane(LaneBase):
         return self._hmaps[key]
 
     def attn_parts(self, heads, tiles):
-        """Key ranges per row: enough of them to give every worker about two tiles (the split workspace is addressed by
+        """Key ranges per row: as many as give every worker one tile (the split workspace is addressed by
         row, so it covers the rows of a small program only)."""
         want = min(MAX_ATTN_PARTS, ATTN_ROUNDS * self.fab.num_workers // tiles)
         return max(1, want) if self.rows_now <= SPLIT_ROWS else 1
