@@ -81,16 +81,41 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
       if (lane < per_tile) tma_prefetch_4d(A.kv_map, 0, 0, 0, pg_next * (page / 8));
     }
   };
-  auto issue_s = [&](int j) {   // one thread: S^T of key tile j
-    const uint32_t k_addr = smem_u32(sK + (j % nbuf) * tile_bytes), q_addr = smem_u32(sQ);
+  // The MMAs are issued by warp 0 in step, one elected lane issuing: descriptors are then warp-uniform values that only
+  // their start addresses tell apart (all of them below 2^18, so plain additions of address / 16).
+  const bool leader = warp == 0 && elect_one();
+  const uint64_t desc_q = sw128_desc(smem_u32(sQ), 0, 1024), desc_p = sw128_desc(smem_u32(sP), 0, 1024);
+  auto issue_s = [&](int j) {   // S^T of key tile j
+    uint64_t k = sw128_desc(smem_u32(sK + (j % nbuf) * tile_bytes), 0, group_bytes), q = desc_q;
     const uint32_t idesc = umma_idesc_bf16(128, N);
-    for (int c = 0; c < chunks; ++c)
+    tc_fence_after_sync();
+#pragma unroll 1
+    for (int c = 0; c < chunks; ++c, k += 1024 >> 4, q += (N * 128) >> 4) {
+      if (leader) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        umma_bf16(tmem_s, sw128_desc(k_addr + c * 1024u + i * 32u, 0, group_bytes),
-                  sw128_desc(q_addr + c * (N * 128u) + i * 32u, 0, 1024), idesc, (c | i) != 0);
-    umma_commit(bar_s);
+        for (int i = 0; i < 4; ++i) umma_bf16(tmem_s, k + 2 * i, q + 2 * i, idesc, (c | i) != 0);
+      }
+    }
+    if (leader) umma_commit(bar_s);
+    __syncwarp();
   };
+  auto issue_o = [&](int j) {   // O^T += V^T P^T of key tile j
+    uint64_t v = sw128_desc(smem_u32(sK + (j % nbuf) * tile_bytes), 1024, group_bytes);
+    const uint32_t idesc = umma_idesc_bf16(128, N) | (1u << 15), step = group_bytes >> 3;   // A is MN-major; 16 keys on
+    tc_fence_after_sync();
+#pragma unroll 1
+    for (int b = 0; b < blocks; ++b, v += 2048 >> 4) {
+      if (leader) {
+        uint64_t vi = v;
+#pragma unroll
+        for (int i = 0; i < kKeyTile / 16; ++i, vi += step)
+          umma_bf16(tmem_o + b * N, vi, desc_p + (i >> 2) * ((N * 128) >> 4) + (i & 3) * 2, idesc, (j | i) != 0);
+      }
+    }
+    if (leader) umma_commit(bar_o);
+    __syncwarp();
+  };
+  auto wait = [&](uint64_t* b, int phase) { return mbar_wait_bounded(b, phase & 1, ctx.abort_flag, kWideWaitNs); };
 
   bool ok = true;
   if (warp == 0 && tiles > 0) {
@@ -103,12 +128,9 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
     load_keys(0);
     if (nbuf > 1 && tiles > 1) load_keys(1);
   }
-  if (tid == 0 && tiles > 0) {
-    ok = mbar_wait_bounded(bar_q, 0, ctx.abort_flag, kWideWaitNs) && mbar_wait_bounded(bar_k, 0, ctx.abort_flag, kWideWaitNs);
-    if (ok) {
-      tc_fence_after_sync();
-      issue_s(0);
-    }
+  if (warp == 0 && tiles > 0) {
+    ok = __all_sync(0xffffffffu, wait(bar_q, 0) && wait(bar_k, 0));
+    if (ok) issue_s(0);
   }
   const float scale = A.scale * 1.4426950408889634f;
   float l[N];
@@ -190,34 +212,18 @@ __device__ __noinline__ bool latent_mma(const TileDesc& t, int tid, const LayerC
     tc_fence_before_sync();
     fence_proxy_async_smem();
     exec_sync();
-    if (tid == 0) {
-      tc_fence_after_sync();
-      const uint32_t k_addr = smem_u32(sK + (j % nbuf) * tile_bytes), p_addr = smem_u32(sP);
-      const uint32_t idesc = umma_idesc_bf16(128, N) | (1u << 15);   // A is MN-major
-      for (int b = 0; b < blocks; ++b)
-#pragma unroll
-        for (int i = 0; i < kKeyTile / 16; ++i)
-          umma_bf16(tmem_o + b * N, sw128_desc(k_addr + b * 2048u + i * 2u * group_bytes, 1024, group_bytes),
-                    sw128_desc(p_addr + (i >> 2) * (N * 128u) + (i & 3) * 32u, 0, 1024), idesc, (j | i) != 0);
-      umma_commit(bar_o);
+    if (warp == 0) {
+      issue_o(j);
       if (nbuf > 1 && j + 1 < tiles) {
-        ok = mbar_wait_bounded(bar_k + ((j + 1) & 1), ((j + 1) >> 1) & 1, ctx.abort_flag, kWideWaitNs);
-        if (ok) {
-          tc_fence_after_sync();
-          issue_s(j + 1);
-        }
+        ok = __all_sync(0xffffffffu, wait(bar_k + ((j + 1) & 1), (j + 1) >> 1));
+        if (ok) issue_s(j + 1);
       }
-    }
-    // the key tile's buffer goes to the loads of tile j + nbuf when O has read it
-    if (warp == 0 && j + nbuf < tiles) {
-      const bool free_ = mbar_wait_bounded(bar_o, j & 1, ctx.abort_flag, kWideWaitNs);
-      if (__all_sync(0xffffffffu, free_)) load_keys(j + nbuf);
-      else ok = false;
-      if (nbuf == 1 && tid == 0 && ok) {
-        ok = mbar_wait_bounded(bar_k, (j + 1) & 1, ctx.abort_flag, kWideWaitNs);
-        if (ok) {
-          tc_fence_after_sync();
-          issue_s(j + 1);
+      if (j + nbuf < tiles) {   // the key tile's buffer goes to the loads of tile j + nbuf when O has read it
+        ok = __all_sync(0xffffffffu, ok && wait(bar_o, j));
+        if (ok) load_keys(j + nbuf);
+        if (nbuf == 1 && ok) {
+          ok = __all_sync(0xffffffffu, wait(bar_k, j + 1));
+          if (ok) issue_s(j + 1);
         }
       }
     }
