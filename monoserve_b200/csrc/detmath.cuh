@@ -10,8 +10,8 @@
 
 namespace mf {
 
-// exp(x) for any finite x: Cody-Waite reduction by ln2 (two constants), a
-// degree-5 polynomial in Horner form on |r| <= ln2/2, exp(r) = 1 + r + r^2 P(r),
+// exp(x) for any finite x: Cody-Waite reduction by ln2 (two constants), the
+// degree-5 polynomial of expf in the Cephes library (S. L. Moshier) in Horner form on |r| <= ln2/2, exp(r) = 1 + r + r^2 P(r),
 // and an exact two-step power-of-two scaling (so that results in the denormal
 // range round exactly once).
 __device__ __forceinline__ float det_expf(float x) {

@@ -112,6 +112,21 @@ def test_far_key_through_prompt_and_decoding(dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_portions_run_as_several_passes(dtype):
+    """A portion longer than the session's pass: several programs, whole-prompt attention for the first and the cached
+    latents for the rest, several key tiles; then decode steps whose keys are split over tiles."""
+    from monoserve_b200.session import Session
+    c = lm.SERVED
+    t = lm.tensors(c, 15)
+    toks = lm.tokens(c, 420, 8)
+    ref = oracle.model_logits(c, t, toks)
+    limit = limit_of(c, t, toks, ref, dtype)
+    with Session(model_of(c, t, dtype), max_tokens=512, page=16, pass_tokens=160) as s:
+        assert error(s.step("a", toks[:400], want=range(400)), ref[:400]) < limit
+        assert error(run_portions(s, "a", toks[400:], [1]), ref[400:]) < limit
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_slots_and_pages_are_used_again(dtype):
     """Requests that come and go over few slots and pages: nothing of an earlier request shows, whatever it left."""
     from monoserve_b200.session import Session
