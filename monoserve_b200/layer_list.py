@@ -31,7 +31,7 @@ from monoserve_b200 import _C
 from monoserve_b200.checkpoint import checkpoint_files, safetensors_tensors
 from monoserve_b200.fabric import Program, Tile, tile_array
 from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_STORE, HEIGHTS, K_GEMM, K_SAMPLE, SPLIT_PARTS, SPLIT_ROWS,
-                                      LaneBase, _block, _bm, _retarget)
+                                      LaneBase, _bm, _retarget)
 
 K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEMORY_STEP, K_MEMORY, K_SCAN_STEP = 51, 52, 53, 54, 55, 56, 57, 65
 K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA, K_LATENT_DIRECT = 58, 59, 60, 61, 62, 63, 64
@@ -365,7 +365,7 @@ MIXERS = {"mamba1": SelectiveScan, "mlstm": MatrixMemory, "latent_attention": La
 class _Buf:
     """An activation buffer [rows][ld] and its tensor maps (bf16 operands of a GEMM)."""
 
-    def __init__(self, lane, rows, cols, dtype, maps=False):
+    def __init__(self, lane, rows, cols, dtype):
         self.ld = up(cols, 64)
         self.t = torch.zeros(rows, self.ld, dtype=dtype, device="cuda")
         self.addr, self.es = self.t.data_ptr(), self.t.element_size()
