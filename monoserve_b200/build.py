@@ -13,7 +13,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libmonofab.so")
-SOURCES = ["api.cu", "moe_aux.cu", "expert_gemm.cu", "pack_static.cu", "fabric_device.cu", "fabric_layer_rows.cu", "fabric_layer_scan.cu", "fabric_layer_memory.cu", "fabric_layer_latent.cu", "fabric_layer_latent_mma.cu", "fabric_layer_latent_direct.cu", "fabric_host.cu", "attention.cu", "host_loop.cu", "ep_exchange.cu", "release.cu", "plan_model.cu", "plan_admission.cu", "plan_api.cu"]
+SOURCES = ["api.cu", "moe_aux.cu", "expert_gemm.cu", "pack_static.cu", "fabric_device.cu", "fabric_layer_rows.cu", "fabric_layer_scan.cu", "fabric_layer_memory.cu", "fabric_layer_gated.cu", "fabric_layer_residual.cu", "fabric_layer_attention.cu", "fabric_layer_latent.cu", "fabric_layer_latent_mma.cu", "fabric_layer_latent_direct.cu", "fabric_host.cu", "attention.cu", "host_loop.cu", "ep_exchange.cu", "release.cu", "plan_model.cu", "plan_admission.cu", "plan_api.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr"]
 # The fabric kernel calls the tiles of the fabric_layer_*.cu files across translation units.

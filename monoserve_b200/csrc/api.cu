@@ -298,6 +298,12 @@ const std::string& layouts_json() {
     MF_JSON_STRUCT(LatentArgs, MF_LATENT_ARGS)
     MF_JSON_STRUCT(LatentAttnArgs, MF_LATENT_ATTN_ARGS)
     MF_JSON_STRUCT(LatentDirectArgs, MF_LATENT_DIRECT_ARGS)
+    MF_JSON_STRUCT(ResidualArgs, MF_RESIDUAL_ARGS)
+    MF_JSON_STRUCT(DecayArgs, MF_DECAY_ARGS)
+    MF_JSON_STRUCT(GatedMemoryArgs, MF_GATED_MEMORY_ARGS)
+    MF_JSON_STRUCT(QkvArgs, MF_QKV_ARGS)
+    MF_JSON_STRUCT(GroupedAttnArgs, MF_GROUPED_ATTN_ARGS)
+    MF_JSON_STRUCT(HeadGateArgs, MF_HEAD_GATE_ARGS)
     MF_JSON_STRUCT(StagingArgs, MF_STAGING_ARGS)
     s += "}";
     return s;

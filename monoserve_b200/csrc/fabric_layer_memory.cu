@@ -377,21 +377,20 @@ __device__ bool tile_memory(const TileDesc& t, int tid, uint8_t* ring) {
 }
 
 // Kind 58, HeadNormArgs: items [i0, i0 + i1), item = row * heads + head, one warp each: the head's read-out over its
-// denominator, over its root mean square, times the norm weight and sigmoid(g).  An item of `o` is e values, the
-// denominator, and padding to a multiple of four.
+// denominator (if it has one), over its root mean square, times the norm weight and sigmoid(g) or silu(g).
 template <int V>
 __device__ __noinline__ void head_norm_items(const TileDesc& t, int tid) {
   constexpr int NV = 8;   // V-element pieces per lane kept in registers
   HeadNormArgs A;
   load_block(A, t.a[0]);
-  const int warp = tid >> 5, lane = tid & 31, e = static_cast<int>(A.e), oe = (e + 4) & ~3;
-  const bool f32 = A.f32 != 0;
+  const int warp = tid >> 5, lane = tid & 31, e = static_cast<int>(A.e), oe = (e + (A.divide ? 4 : 3)) & ~3;
+  const bool f32 = A.f32 != 0, silu = A.silu != 0;
   for (uint32_t it = t.i0 + warp; it < t.i0 + t.i1; it += kExecThreads / 32) {
     const uint32_t row = it / A.heads, head = it % A.heads;
     const float* o = f32p(A.o) + static_cast<size_t>(it) * oe;
     const size_t g0 = static_cast<size_t>(row) * A.ld_g + head * e, o0 = static_cast<size_t>(row) * A.ld_out + head * e;
-    const float* w = f32p(A.w) + head * e;
-    const float inv_den = 1.f / o[e];
+    const float* w = f32p(A.w) + head * A.w_head;
+    const float inv_den = A.divide ? 1.f / o[e] : 1.f;
     auto gate = [&](int c, float (&g)[V]) {
       if constexpr (V == 4) {
         if (!f32) {
@@ -408,7 +407,8 @@ __device__ __noinline__ void head_norm_items(const TileDesc& t, int tid) {
     auto put = [&](int c, const float (&v)[V], const float (&g)[V], const float (&ww)[V], float inv) {
       float x[V];
 #pragma unroll
-      for (int j = 0; j < V; ++j) x[j] = v[j] * inv_den * inv * ww[j] * (f32 ? sigmoid32(g[j]) : __fdividef(1.f, 1.f + __expf(-g[j])));
+      for (int j = 0; j < V; ++j)
+        x[j] = v[j] * inv_den * inv * ww[j] * (f32 ? sigmoid32(g[j]) : __fdividef(1.f, 1.f + __expf(-g[j]))) * (silu ? g[j] : 1.f);
       if constexpr (V == 4) {
         if (!f32) {
           const __nv_bfloat162 q[2] = {__floats2bfloat162_rn(x[0], x[1]), __floats2bfloat162_rn(x[2], x[3])};

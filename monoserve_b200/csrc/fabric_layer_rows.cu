@@ -53,7 +53,7 @@ __device__ void tile_product32(const TileDesc& t, int tid, int* scratch) {
       if (r + i < rows && c + j < cols) out[static_cast<size_t>(t.i0 + r + i) * A.ld_out + t.i2 + c + j] = acc[i][j];
 }
 
-// Kind 52, GatedArgs: rows [i0, i0 + i1) of fp32 [gate | up] -> gelu_tanh(gate) * up, fp32.
+// Kind 52, GatedArgs: rows [i0, i0 + i1) of fp32 [gate | up] -> gelu_tanh(gate) * up or silu(gate) * up, fp32.
 __device__ void tile_gated_act(const TileDesc& t, int tid) {
   GatedArgs A;
   load_block(A, t.a[0]);
@@ -62,7 +62,8 @@ __device__ void tile_gated_act(const TileDesc& t, int tid) {
     float* out = reinterpret_cast<float*>(A.out) + static_cast<size_t>(r) * A.ld_out;
     for (uint32_t f = tid; f < A.ff; f += kExecThreads) {
       const float g = in[f];
-      out[f] = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * in[A.ff + f];
+      const float a = A.silu ? g * sigmoid32(g) : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+      out[f] = a * in[A.ff + f];
     }
   }
 }
@@ -305,6 +306,13 @@ __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx) 
     case kTileLatentDirect: return tile_latent_direct(t, tid, ctx);
     case kTileLatentMerge: tile_latent_merge(t, tid); return true;
     case kTileSumSlabs: tile_sum_slabs(t, tid); return true;
+    case kTileResidual: tile_residual(t, tid, scratch); return true;
+    case kTileDecay: tile_decay(t, tid, scratch); return true;
+    case kTileGatedMemory: return tile_gated_memory(t, tid, ctx.ring);
+    case kTileGatedStep: return tile_gated_step(t, tid);
+    case kTileQkv: tile_qkv(t, tid); return true;
+    case kTileGroupedAttn: return tile_grouped_attn(t, tid);
+    case kTileHeadGate: tile_head_gate(t, tid); return true;
     default: return false;
   }
 }

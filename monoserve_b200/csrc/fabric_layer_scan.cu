@@ -7,7 +7,7 @@ namespace fab {
 
 // ------------------------------------------------------------------ short convolution
 // Kind 54, ConvArgs: i0 the request's first row, i1 first row of this tile, i2 rows | channels << 16, i3 slot,
-// a[1] first channel.  A thread walks down V channels with the last TAPS - 1 inputs in registers, eight rows' loads in
+// a[1] first channel, a[2] the request's rows (read with `advance`).  A thread walks down V channels with the last TAPS - 1 inputs in registers, eight rows' loads in
 // flight.  V = 8: bf16 rows in 16-byte pieces.
 template <bool F32, int V, int TAPS>
 __device__ __noinline__ void conv_rows(const TileDesc& t, int tid) {
@@ -17,7 +17,7 @@ __device__ __noinline__ void conv_rows(const TileDesc& t, int tid) {
   const int n_ch = static_cast<int>(t.i2 >> 16), ch0 = static_cast<int>(t.a[1]), taps = static_cast<int>(A.taps);
   const int C = static_cast<int>(A.channels);
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
-  const float* tail = f32p(A.tail) + static_cast<size_t>(t.i3) * (taps - 1) * C;
+  float* tail = reinterpret_cast<float*>(A.tail) + static_cast<size_t>(t.i3) * (taps - 1) * C;
   using Raw = typename std::conditional<V == 8, uint4, float>::type;
   auto load = [&](int r, int c) -> Raw {   // row r >= row0
     const size_t at = static_cast<size_t>(r) * A.ld_x + c;
@@ -46,7 +46,7 @@ __device__ __noinline__ void conv_rows(const TileDesc& t, int tid) {
       for (int j = 0; j < V; ++j) w[k][j] = tap >= 0 ? f32p(A.w)[static_cast<size_t>(c + j) * taps + tap] : 0.f;
     }
 #pragma unroll
-    for (int j = 0; j < V; ++j) bias[j] = f32p(A.bias)[c + j];
+    for (int j = 0; j < V; ++j) bias[j] = A.bias ? f32p(A.bias)[c + j] : 0.f;
 #pragma unroll
     for (int k = 1; k < TAPS; ++k) {
       const int r = r_lo - TAPS + k, place = r - row0 + taps - 1;   // place in the tail, for rows before the portion
@@ -85,6 +85,21 @@ __device__ __noinline__ void conv_rows(const TileDesc& t, int tid) {
         } else {
           act_st(A.out, at, F32, o[0]);
         }
+      }
+    }
+    if (A.advance && r_lo == row0) {   // the last taps - 1 inputs of [old tail, this portion]
+      const int n = static_cast<int>(t.a[2]);
+      for (int place = 0; place < taps - 1; ++place) {
+        const int k = n + place;
+        float in[V];
+        if (k >= taps - 1) {
+          unpack(load(row0 + k - (taps - 1), c), in);
+        } else {
+#pragma unroll
+          for (int j = 0; j < V; ++j) in[j] = fresh ? 0.f : tail[static_cast<size_t>(k) * C + c + j];
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) tail[static_cast<size_t>(place) * C + c + j] = in[j];
       }
     }
   }

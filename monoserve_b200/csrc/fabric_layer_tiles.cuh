@@ -1,6 +1,7 @@
-// Tiles of the layer-list decoders inside the persistent fabric kernel: hyper-connected residual streams with
-// their norms, short causal convolution, selective scan, matrix memory, latent attention over a paged cache of
-// latents, and 32-bit matrix products.  Kinds in fabric_types.h, operand blocks in operands.h.  What the recurrences,
+// Tiles of the layer-list decoders inside the persistent fabric kernel: hyper-connected residual streams or a plain
+// residual with their norms, short causal convolution, selective scan, matrix memory, gated memories (linear attention
+// and delta rule), latent attention over a paged cache of latents, what surrounds grouped-query attention, and 32-bit
+// matrix products.  Kinds in fabric_types.h, operand blocks in operands.h.  What the recurrences,
 // norms, scores and residual sums compute is 32-bit throughout; activations between tiles are bf16, or fp32 when a
 // block's f32 is set.
 //
@@ -35,12 +36,12 @@ struct LayerCtx {
   volatile int* abort_flag;
 };
 
-// Runs tile kinds kTileProduct32 .. kTileScanStep: false for a kind or size these tiles do not take, or when a bounded
+// Runs tile kinds kTileProduct32 .. kTileHeadGate: false for a kind or size these tiles do not take, or when a bounded
 // wait gave up.  All exec threads call it with the same tile.
 __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx);
 // Wide tiles: their exec warps use the operand ring as scratch memory, and TMEM.
 __device__ __forceinline__ bool tile_is_wide(uint32_t kind) {
-  return kind == kTileMemory || kind == kTileScan || kind == kTileLatentMma || kind == kTileLatentDirect;
+  return kind == kTileMemory || kind == kTileScan || kind == kTileGatedMemory || kind == kTileLatentMma || kind == kTileLatentDirect;
 }
 
 __device__ void tile_streams(const TileDesc& t, int tid, int* scratch);
@@ -58,6 +59,13 @@ __device__ bool tile_latent_attn(const TileDesc& t, int tid);
 __device__ bool tile_latent_mma(const TileDesc& t, int tid, const LayerCtx& ctx);
 __device__ bool tile_latent_direct(const TileDesc& t, int tid, const LayerCtx& ctx);
 __device__ void tile_latent_merge(const TileDesc& t, int tid);
+__device__ void tile_residual(const TileDesc& t, int tid, int* scratch);
+__device__ void tile_decay(const TileDesc& t, int tid, int* scratch);
+__device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring);
+__device__ bool tile_gated_step(const TileDesc& t, int tid);
+__device__ void tile_qkv(const TileDesc& t, int tid);
+__device__ bool tile_grouped_attn(const TileDesc& t, int tid);
+__device__ void tile_head_gate(const TileDesc& t, int tid);
 
 __device__ __forceinline__ void exec_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kExecThreads) : "memory"); }
 

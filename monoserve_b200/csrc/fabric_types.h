@@ -48,7 +48,7 @@ enum TileKind : uint16_t {
                             // projection's tiles (every expert-range tile of a row group writes the same norm)
   // Layer-list decoders (fabric_layer_tiles.cuh); none of these is in the reference.
   kTileProduct32 = 51,      // a block of a matrix product in 32-bit arithmetic
-  kTileGatedAct = 52,       // gelu_tanh(gate) * up of fp32 rows
+  kTileGatedAct = 52,       // gelu_tanh(gate) * up, or silu(gate) * up, of fp32 rows
   kTileStreams = 53,        // hyper-connection update of the residual streams, next sublayer's input and its norm
   kTileConv = 54,           // causal convolution per channel + silu
   kTileScan = 55,           // selective scan of a request's rows
@@ -62,6 +62,13 @@ enum TileKind : uint16_t {
   kTileLatentMma = 63,      // attention over the cached latents on the tensor cores: heads x tokens, one key range
   kTileLatentDirect = 64,   // the same for a whole prompt, with keys and values mapped out of the latents
   kTileScanStep = 65,       // selective scan, one token
+  kTileResidual = 66,       // normed sublayer output into the plain residual, next sublayer's input and its norm
+  kTileDecay = 67,          // decays of a gated memory from their low-rank projection
+  kTileGatedMemory = 68,    // gated linear attention / gated delta rule over a request's rows
+  kTileGatedStep = 69,      // the same, one token
+  kTileQkv = 70,            // query / key norms and K / V append of grouped-query attention
+  kTileGroupedAttn = 71,    // grouped-query attention over the paged cache, simple form
+  kTileHeadGate = 72,       // attention output times one gate per head
 };
 constexpr int kFabChunk = 16;   // rows per router / permute tile = rank chunk of the stable pack
 

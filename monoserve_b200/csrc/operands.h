@@ -98,16 +98,18 @@ namespace mf {
 #define MF_PRODUCT_ARGS(U64, U32, F32) \
   U64(x) U64(w) U64(out) U32(ld_x) U32(ld_w) U32(ld_out) U32(K) U32(N) U32(f32)
 
-#define MF_GATED_ARGS(U64, U32, F32) U64(in) U64(out) U32(ff) U32(ld_in) U32(ld_out)
+/* silu: the activation of the gate is silu, else gelu (tanh form). */
+#define MF_GATED_ARGS(U64, U32, F32) U64(in) U64(out) U32(ff) U32(ld_in) U32(ld_out) U32(silu)
 
 /* Adds `parts` fp32 slabs of part_rows rows; out32 receives every column, out16 the first c16 rounded to bf16. */
 #define MF_SUM_ARGS(U64, U32, F32) \
   U64(in) U64(out32) U64(out16) U32(cols) U32(parts) U32(part_rows) U32(ld_in) U32(ld_32) U32(ld_16) U32(c16)
 
 /* Causal convolution per channel over a request's rows, then silu; tail fp32 [slot][taps - 1][channels] holds the
- * inputs before the portion (read here, advanced by the scan tile). */
+ * inputs before the portion (read here; advanced by the scan tile, or with `advance` set by the tile of the request's
+ * first rows, the only one that reads it).  bias may be 0. */
 #define MF_CONV_ARGS(U64, U32, F32) \
-  U64(x) U64(tail) U64(w) U64(bias) U64(out) U64(tok_pos) U32(ld_x) U32(ld_out) U32(channels) U32(taps) U32(f32)
+  U64(x) U64(tail) U64(w) U64(bias) U64(out) U64(tok_pos) U32(ld_x) U32(ld_out) U32(channels) U32(taps) U32(f32) U32(advance)
 
 #define MF_SCAN_ARGS(U64, U32, F32) \
   U64(x) U64(z) U64(dt) U64(dt_bias) U64(b) U64(c) U64(A) U64(D) U64(state) U64(tail) U64(x_in) U64(y) \
@@ -121,8 +123,10 @@ namespace mf {
   U64(q) U64(k) U64(v) U64(gates) U64(gate_bias) U64(state) U64(m) U64(out) U64(tok_pos) U32(ld_qkv) U32(ld_gates) \
   U32(gate_parts) U32(gate_rows) U32(heads) U32(d) U32(e) U32(f32) F32(q_scale) F32(cap)
 
+/* An item of o is e values, with `divide` set their denominator, and padding to a multiple of four.  w: head h's
+ * multipliers at h * w_head; the gate g enters through silu, or else through sigmoid. */
 #define MF_HEAD_NORM_ARGS(U64, U32, F32) \
-  U64(o) U64(g) U64(w) U64(out) U32(heads) U32(e) U32(ld_g) U32(ld_out) U32(f32) F32(eps)
+  U64(o) U64(g) U64(w) U64(out) U32(heads) U32(e) U32(ld_g) U32(ld_out) U32(f32) F32(eps) U32(divide) U32(w_head) U32(silu)
 
 /* qc fp32 [rows][heads * (d + r) | kv_rank | r]: queries, latent, shared rotated key part.  q_un [head][rows_max][ld_un]
  * unrotated query parts; q_all [head][rows_max][ld_q] = kv_rank absorbed columns (written by a product) then r rotated
@@ -144,6 +148,45 @@ namespace mf {
 #define MF_LATENT_DIRECT_ARGS(U64, U32, F32) \
   U64(q_map) U64(qr_map) U64(kv_map) U64(kr_map) U64(out) U32(d) U32(r) U32(e) U32(heads) U32(rows_max) U32(ld_out) \
   U32(buffers) F32(scale)
+
+/* The plain residual x fp32 [rows][W] with a norm on both sides of a sublayer: x += post_w norm(y), then the next
+ * sublayer's input w norm(x) in h16 / h32 (and, for rows with gather >= 0, in out16 / out32).  y is the sum of y0_parts
+ * fp32 slabs of y_rows rows at y0; with y1_parts > 0 it is branch_scale * (w0 norm(y0) + w1 norm(y1)).  embed set: x starts
+ * as embed[token] * embed_scale + pos[position] instead (pos optional, max_pos rows). */
+#define MF_RESIDUAL_ARGS(U64, U32, F32) \
+  U64(x) U64(y0) U64(y1) U64(w0) U64(w1) U64(post_w) U64(w) U64(h16) U64(h32) U64(gather) U64(out16) U64(out32) U64(embed) \
+  U64(pos) U64(tokens) U64(tok_pos) U64(step) U64(sum_out) U32(W) U32(ld_h16) U32(ld_h32) U32(ld_out) U32(y0_parts) \
+  U32(y1_parts) U32(y_rows) U32(max_pos) F32(eps) F32(embed_scale) F32(branch_scale)
+
+/* out fp32 [rows][ld_out] = expm1(-coef[channel / d] * softplus(sign * (x w^T + bias))) for n channels: one minus the
+ * decay of a gated memory, negated.  x: r activations per row, w bf16 [n][ld_w]. */
+#define MF_DECAY_ARGS(U64, U32, F32) \
+  U64(x) U64(w) U64(bias) U64(coef) U64(out) U32(ld_x) U32(ld_w) U32(ld_out) U32(r) U32(n) U32(d) U32(f32) F32(sign)
+
+/* Gated memory: per head S <- diag(1 + decay) S + k u^T, o = S^T q, state fp32 [slot][head][e][d padded to 4].
+ * beta = 0: u = v; else the delta rule u = sigmoid(beta) (v - S^T k) on the decayed S.  unit: keys and queries are
+ * divided by sqrt(sum of squares + 1e-6).  q is multiplied by q_scale; value head h reads key head h / group.  q, k, v,
+ * beta: activations; decay fp32 [rows][heads * d]; out fp32 [rows][heads][e padded to 4]. */
+#define MF_GATED_MEMORY_ARGS(U64, U32, F32) \
+  U64(q) U64(k) U64(v) U64(beta) U64(decay) U64(state) U64(out) U64(tok_pos) U32(ld_qkv) U32(ld_beta) U32(ld_decay) \
+  U32(heads) U32(group) U32(d) U32(e) U32(f32) U32(unit) F32(q_scale)
+
+/* Grouped-query attention around the paged cache.  q, k, v: activations of a row; q_out [rows][heads][ld_q], caches
+ * [page slots][kv_heads][ld_k or ld_v], columns past d (e) are written as zero.  Queries and keys are divided by their
+ * root mean square and multiplied by q_norm / k_norm (fp32 [d]; 0: left as they are). */
+#define MF_QKV_ARGS(U64, U32, F32) \
+  U64(q) U64(k) U64(v) U64(q_norm) U64(k_norm) U64(q_out) U64(k_cache) U64(v_cache) U64(tok_slot) U32(ld_x) U32(heads) \
+  U32(kv_heads) U32(d) U32(e) U32(ld_q) U32(ld_k) U32(ld_v) U32(f32) F32(eps)
+
+/* The simple form of the attention itself, for sizes and precisions the tensor-core tiles do not take; out
+ * [rows][heads][ld_out]. */
+#define MF_GROUPED_ATTN_ARGS(U64, U32, F32) \
+  U64(q) U64(k_cache) U64(v_cache) U64(block_table) U64(out) U64(tok_pos) U32(heads) U32(kv_heads) U32(d) U32(e) U32(ld_q) \
+  U32(ld_k) U32(ld_v) U32(ld_out) U32(page) U32(bt_stride) U32(f32) F32(scale)
+
+/* out [rows][ld_out], head h at column h e = in [rows][heads][ld_in] (e columns) times sigmoid(g [rows][ld_g]). */
+#define MF_HEAD_GATE_ARGS(U64, U32, F32) \
+  U64(in) U64(g) U64(out) U32(heads) U32(e) U32(ld_in) U32(ld_g) U32(ld_out) U32(f32)
 
 #define MF_FIELD_U64(name) unsigned long long name;
 #define MF_FIELD_U32(name) uint32_t name;
@@ -176,9 +219,15 @@ MF_DECLARE(SumArgs, MF_SUM_ARGS, 64)
 MF_DECLARE(ConvArgs, MF_CONV_ARGS, 128)
 MF_DECLARE(ScanArgs, MF_SCAN_ARGS, 192)
 MF_DECLARE(MemoryArgs, MF_MEMORY_ARGS, 128)
-MF_DECLARE(HeadNormArgs, MF_HEAD_NORM_ARGS, 64)
+MF_DECLARE(HeadNormArgs, MF_HEAD_NORM_ARGS, 128)
 MF_DECLARE(LatentArgs, MF_LATENT_ARGS, 128)
 MF_DECLARE(LatentAttnArgs, MF_LATENT_ATTN_ARGS, 128)
 MF_DECLARE(LatentDirectArgs, MF_LATENT_DIRECT_ARGS, 128)
+MF_DECLARE(ResidualArgs, MF_RESIDUAL_ARGS, 192)
+MF_DECLARE(DecayArgs, MF_DECAY_ARGS, 128)
+MF_DECLARE(GatedMemoryArgs, MF_GATED_MEMORY_ARGS, 128)
+MF_DECLARE(QkvArgs, MF_QKV_ARGS, 128)
+MF_DECLARE(GroupedAttnArgs, MF_GROUPED_ATTN_ARGS, 128)
+MF_DECLARE(HeadGateArgs, MF_HEAD_GATE_ARGS, 64)
 
 }  // namespace mf

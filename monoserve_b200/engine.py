@@ -166,6 +166,8 @@ class Engine:
         self.fab, self.cfg, self.kv, self.table, self.pool = fab, cfg, kv, table, pool
         self.max_decode, self.token_budget = max_decode, token_budget
         self.max_len = max_len or table.bt_stride * kv.page
+        if getattr(cfg, "max_positions", None):   # a learned position per token: there are no more of them
+            self.max_len = min(self.max_len, cfg.max_positions)
         shared = dict(bt_stride=table.bt_stride, requests=table)
         lane_of = registry.lane_class(cfg, default=ModelLane)
         self.pre = lane_of(fab, PREFILL, cfg, weights, kv, max_tokens=token_budget, max_slots=table.slots,

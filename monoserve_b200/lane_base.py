@@ -17,6 +17,10 @@ GATED = (EPI_SILU_MUL, EPI_GELU_MUL)
 HEIGHTS = [16, 32, 64, 128, 256]
 
 
+def up(n, m):
+    return -(-n // m) * m
+
+
 def _block(name, **fields):
     return torch.frombuffer(bytearray(pack(name, **fields)), dtype=torch.uint8).cuda()
 

@@ -1,25 +1,32 @@
-"""Layer-list decoders (the Sinotar design) as fabric lane programs: the mixer of every layer is named by the
-configuration (selective scan, latent attention, matrix memory), the residual is a set of hyper-connected streams, and
-a span of layers may run several times in a row.
+"""Layer-list decoders as fabric lane programs: the configuration names the mixer of every layer.  What differs between
+designs otherwise is in DESIGNS: Sinotar (selective scan, latent attention, matrix memory; the residual a set of
+hyper-connected streams; a span of layers may run several times in a row) and Teganex (gated linear attention, and
+attention beside a gated delta rule: monoserve_b200/gated_mixers.py; a plain residual normed before and after each
+sublayer).
 
 `LayerListLane` builds the chain of one batch on the fabric's tiles, one run of a layer after the other:
 
-  streams (53: update of the streams by the sublayer before, the next sublayer's input, its norm)
+  streams (53: update of the streams by the sublayer before, the next sublayer's input, its norm), or
+  residual (66: the same for the plain residual)
     selective scan:    in GEMM (32) -> conv + silu (54) -> x GEMM (K ranges) -> slab sum (62) -> dt GEMM -> scan (55; one
                        token: 65) -> o GEMM
     matrix memory:     q k v g GEMM, gates GEMM beside it -> memory (57; one token: 56) -> head norm (58) -> o GEMM
     latent attention:  q + latent GEMM -> latent norm, rotation, cache append (59) -> per head W_uk^T q GEMM ->
                        attention over the cached latents (63 on the tensor cores, 60 in 32-bit; 61) -> per head W_uv
                        GEMM -> o GEMM; for a whole prompt: keys and values GEMM -> attention (64) -> o GEMM
-  streams -> gate / up GEMM with the gelu epilogue -> down GEMM
+    gated linear:      q k v g and decay GEMM -> decays (67) -> gated memory (68; one token: 69) -> head norm (58) -> o GEMM
+    parallel:          one GEMM for both sides; left: norms and append (70) -> paged attention (33 - 35, 44; 71 in 32-bit) ->
+                       head gate (72) -> o GEMM; right: conv (54), decays (67) and gate GEMM -> gated memory (68, 69) ->
+                       head norm (58) -> o GEMM
+  streams -> gate / up GEMM with the gated epilogue -> down GEMM
   ... -> final streams (gather) -> head GEMM (fp32) -> sample (43)
 
-Residual streams, norms, positions, gates, scores and recurrent state are 32-bit; GEMM operands are bf16.  With
+Residuals, norms, positions, gates, scores and recurrent state are 32-bit; GEMM operands are bf16.  With
 cfg.f32 set every activation is fp32 and every product runs in 32-bit arithmetic (tile 51): the exact form of the same
 programs, for checking.
 
-State: `LayerListCache` holds, per layer run, either pages of latents (addressed through the lane's block table) or
-slot-indexed recurrent state.  A request that starts at position 0 finds the state of its slot ignored (the tiles take
+State: `LayerListCache` holds, per layer run, pages of latents or of keys and values (addressed through the lane's block
+table) and slot-indexed recurrent state.  A request that starts at position 0 finds the state of its slot ignored (the tiles take
 it as zero), so slots and pages are handed on without clearing.
 """
 import types
@@ -30,10 +37,13 @@ import torch
 from monoserve_b200 import _C
 from monoserve_b200.checkpoint import checkpoint_files, safetensors_tensors
 from monoserve_b200.fabric import Program, Tile, tile_array
-from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_STORE, HEIGHTS, K_GEMM, K_SAMPLE, SPLIT_PARTS, SPLIT_ROWS,
-                                      LaneBase, _bm, _retarget)
+from monoserve_b200.fabric.args import pack
+from monoserve_b200.gated_mixers import GatedLinear, Parallel
+from monoserve_b200.lane_base import (EPI_F32, EPI_GELU_MUL, EPI_SILU_MUL, EPI_STORE, HEIGHTS, K_GEMM, K_SAMPLE, SPLIT_PARTS,
+                                      SPLIT_ROWS, LaneBase, _bm, _retarget, up)
 
 K_PRODUCT, K_GATED, K_STREAMS, K_CONV, K_SCAN, K_MEMORY_STEP, K_MEMORY, K_SCAN_STEP = 51, 52, 53, 54, 55, 56, 57, 65
+K_RESIDUAL = 66
 K_HEAD_NORM, K_LATENT_KV, K_LATENT_ATTN, K_LATENT_MERGE, K_SUM, K_LATENT_MMA, K_LATENT_DIRECT = 58, 59, 60, 61, 62, 63, 64
 MAX_STREAMS, MAX_TAPS, MAX_SCAN_STATE, MAX_MEMORY_DIM, MAX_LATENT_DIM = 8, 8, 128, 512, 1152
 SCAN_CHANNELS, MEMORY_COLUMNS, STEP_CHANNELS = 32, 32, 512   # of one tile
@@ -43,8 +53,13 @@ RING_BYTES, KEY_TILE = 216 * 1024, 128   # shared memory of a wide tile; keys pe
 DIRECT_ROWS = 32                         # a prompt of at least this many tokens maps its keys and values out of the latents
 
 
-def up(n, m):
-    return -(-n // m) * m
+# What a design fixes: its registry name, the mixers it has, what a norm weight is counted from, the feed-forward's
+# activation, and its residual: "streams", or "normed" on both sides of a sublayer.
+DESIGNS = {
+    "Sinotar": types.SimpleNamespace(name="sinotar", mixers=("mamba1", "mlstm", "latent_attention"), norm_from=1, act="gelu",
+                                     residual="streams"),
+    "Teganex": types.SimpleNamespace(name="teganex", mixers=("gla", "parallel"), norm_from=0, act="silu", residual="normed"),
+}
 
 
 # ---------------------------------------------------------------------------------------------- configuration
@@ -52,10 +67,11 @@ def read_config(c, dtype="bfloat16"):
     """The model shape from a parsed config.json with a list of layers."""
     if dtype not in ("bfloat16", "float32"):
         raise ValueError(f"dtype {dtype}")
+    design = DESIGNS[c.get("architecture", "Sinotar")]
     layers = []
     for i, e in enumerate(c["layers"]):
         kind, m, mlp = e["type"], dict(e["mixer"]), e.get("mlp")
-        if kind not in MIXERS:
+        if kind not in design.mixers:
             raise NotImplementedError(f"layer {i}: mixer {kind}")
         if mlp and mlp.get("kind", "dense") != "dense":
             raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']}")
@@ -66,12 +82,14 @@ def read_config(c, dtype="bfloat16"):
     if loop:
         a, b = loop["start"], loop["stop"]
         order = order[:a] + order[a:b] * loop["times"] + order[b:]
-    streams = c["streams"]
+    streams = c["streams"] if design.residual == "streams" else 1
     if not 1 <= streams <= MAX_STREAMS:
         raise NotImplementedError(f"{streams} residual streams (1 to {MAX_STREAMS})")
-    return types.SimpleNamespace(model_type="sinotar", hidden=c["width"], vocab=c["vocab"], eps=float(c["norm"]["eps"]),
-                                 streams=streams, layers=layers, order=order, num_layers=len(layers),
-                                 f32=dtype == "float32")
+    return types.SimpleNamespace(model_type=design.name, design=design, hidden=c["width"], vocab=c["vocab"],
+                                 eps=float(c["norm"]["eps"]), streams=streams, layers=layers, order=order,
+                                 num_layers=len(layers), f32=dtype == "float32",
+                                 embed_scale=float(c.get("embedding", {}).get("scale", 1.0)),
+                                 logit_scale=float(c.get("logit_scale", 1.0)), max_positions=c.get("max_positions"))
 
 
 def read_tensors(folder):
@@ -87,19 +105,24 @@ class Weights:
     def __init__(self, cfg, tensors):
         self.cfg = cfg
         t = tensors
+        design = cfg.design
         self.embed = t["embed"].to(torch.bfloat16).contiguous().cuda()
+        self.pos = t["pos"].to(torch.bfloat16).contiguous().cuda() if "pos" in t else None
         self.head = self.mat(t["head"])
-        self.final_norm = self.f32(1 + t["final.norm"].float())
+        # the logits' scale goes with the row in front of the head product
+        self.final_norm = self.f32((design.norm_from + t["final.norm"].float()) * cfg.logit_scale)
         self.ones = torch.ones(cfg.streams, device="cuda")
         self.layers = []
         for l, layer in enumerate(cfg.layers):
             g = lambda name: t[f"l{l}.{name}"]  # noqa: B023, E731
-            w = types.SimpleNamespace(norm1=self.f32(1 + g("norm1").float()))
-            w.hc1 = [self.f32(g(f"hc1.{n}").float()) for n in ("in", "out", "mix")]
+            norm = lambda name: self.f32(design.norm_from + g(name).float())  # noqa: B023, E731
+            # in front of the sublayer, and behind it: (hc_out, hc_mix) of the streams, or the norm of its output
+            after = (lambda i: [self.f32(g(f"hc{i}.{n}").float()) for n in ("in", "out", "mix")]) if design.residual == "streams" \
+                else (lambda i: [None, norm(f"norm{i}b")])  # noqa: B023
+            w = types.SimpleNamespace(norm1=norm("norm1"), hc1=after(1))
             MIXERS[layer.kind].place(self, w, layer.m, lambda name: g("mix." + name))
             if layer.ff:
-                w.norm2 = self.f32(1 + g("norm2").float())
-                w.hc2 = [self.f32(g(f"hc2.{n}").float()) for n in ("in", "out", "mix")]
+                w.norm2, w.hc2 = norm("norm2"), after(2)
                 w.gate_up = self.mat(torch.cat([g("mlp.gate"), g("mlp.up")]))
                 w.down = self.mat(g("mlp.down"))
             self.layers.append(w)
@@ -116,12 +139,13 @@ class Weights:
 
 
 class LayerListCache:
-    """Cache and state of every layer run, shared by the lanes: `page` tokens per page of latents (page 0 is the sink
-    unused block-table entries point at), `slots` requests' recurrent state."""
+    """Cache and state of every layer run, shared by the lanes: `page` tokens per page of latents, or of keys and values
+    (page 0 is the sink unused block-table entries point at), `slots` requests' recurrent state."""
 
     def __init__(self, cfg, n_pages, page_size=16, slots=8):
         self.n_pages, self.page, self.slots = n_pages, page_size, slots
-        self.runs = [MIXERS[cfg.layers[l].kind].state(cfg, cfg.layers[l].m, n_pages * page_size, slots) for l in cfg.order]
+        self.runs = [MIXERS[cfg.layers[l].kind].state(cfg, cfg.layers[l].m, n_pages * page_size, slots, page_size)
+                     for l in cfg.order]
 
 
 def latent_tile(m, page, tokens_per_request):
@@ -168,13 +192,20 @@ class SelectiveScan:
         w.A = W.f32(-torch.exp(g("A_log").float()))
 
     @staticmethod
-    def state(cfg, m, rows, slots):
+    def state(cfg, m, rows, slots, page):
         return dict(state=torch.zeros(slots, m.inner, m.state, device="cuda"),
                     tail=torch.zeros(slots, max(1, m.conv - 1), m.inner, device="cuda"))
 
     @staticmethod
-    def sizes(m):
+    def sizes(m, w):
         return dict(proj=2 * m.inner, act=m.inner, mix=m.inner, small=m.dt_rank + 2 * m.state, dt=m.inner, dt_in=m.dt_rank)
+
+    @staticmethod
+    def prepare(lane, layer, w, st):
+        m = layer.m
+        for t in (w.in_, w.x, w.dt, w.o):
+            lane.weight_map(t)
+        lane.act.maps(m.inner), lane.dt_in.maps(m.dt_rank), lane.mix.maps(m.inner)
 
     @staticmethod
     def build(lane, p, l, run, b, prev):
@@ -226,14 +257,19 @@ class MatrixMemory:
         w.gate_b, w.norm = W.f32(torch.cat([g("i.b"), g("f.b")])), W.f32(g("norm"))
 
     @staticmethod
-    def state(cfg, m, rows, slots):
+    def state(cfg, m, rows, slots, page):
         return dict(S=torch.zeros(slots, m.heads, m.vdim + 1, up(m.dim, 4), device="cuda"),
                     m=torch.zeros(slots, m.heads, up(m.vdim + 1, MEMORY_COLUMNS) // MEMORY_COLUMNS, device="cuda"))
 
     @staticmethod
-    def sizes(m):
+    def sizes(m, w):
         return dict(proj=2 * m.heads * (m.dim + m.vdim), mix=m.heads * m.vdim, small=2 * m.heads, raw=m.heads * up(m.vdim + 1, 4),
                     split=1)
+
+    @staticmethod
+    def prepare(lane, layer, w, st):
+        lane.weight_map(w.qkvg), lane.weight_map(w.gates), lane.weight_map(w.o)
+        lane.h.maps(3 * lane.split), lane.mix.maps(layer.m.heads * layer.m.vdim)
 
     @staticmethod
     def build(lane, p, l, run, b, prev):
@@ -249,11 +285,11 @@ class MatrixMemory:
         mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=raw.addr,
                         gate_parts=parts, gate_rows=lane.slab_rows(T), gate_bias=w.gate_b, state=st["S"], m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos,
                         ld_qkv=lane.proj.ld, ld_gates=ld, heads=H, d=d, e=e, f32=f32, q_scale=d ** -0.5, cap=m.gate_cap)
-        s_m = p.stage(_retarget(b.memory_tiles(H, e), a0=mem.data_ptr()), label=("memory", run))
+        s_m = p.stage(_retarget(b.memory_tiles(H, e + 1), a0=mem.data_ptr()), label=("memory", run))
         p.after(s, s_m)
         p.after(s_g, s_m)
         nrm = lane._dev("HeadNormArgs", o=lane.raw.addr, g=at + es * H * (2 * d + e), w=w.norm, out=lane.mix.addr, heads=H,
-                        e=e, ld_g=lane.proj.ld, ld_out=lane.mix.ld, f32=f32, eps=lane.cfg.eps)
+                        e=e, ld_g=lane.proj.ld, ld_out=lane.mix.ld, f32=f32, eps=lane.cfg.eps, divide=1, w_head=e)
         s_n = p.stage(lane._rows(K_HEAD_NORM, nrm, T * H, lane.items_per(T * H)), label=("head_norm", run))
         p.after(s_m, s_n)
         return lane.closing(p, s_n, lane.mix, w.o, T, H * e, ("memory_o", run))
@@ -278,15 +314,33 @@ class LatentAttention:
         w.uv = W.mat(g("uv").view(m.heads, m.vdim, m.kv_rank))                   # [head][value][latent]
 
     @staticmethod
-    def state(cfg, m, rows, slots):
+    def state(cfg, m, rows, slots, page):
         return dict(cache=torch.zeros(rows, up(m.kv_rank + m.rot_dim, 64), device="cuda",
                                       dtype=torch.float32 if cfg.f32 else torch.bfloat16))
 
     @staticmethod
-    def sizes(m):
+    def sizes(m, w):
         return dict(qc=m.heads * (m.dim + m.rot_dim) + m.kv_rank + m.rot_dim, mix=m.heads * m.vdim,
                     kvb=m.heads * (m.dim + m.vdim), c_rows=m.kv_rank + m.rot_dim, q_un=(m.heads, m.dim), q_all=(m.heads, m.kv_rank + m.rot_dim), o_lat=(m.heads, m.kv_rank),
                     ws=(m.heads, m.kv_rank))
+
+    @staticmethod
+    def prepare(lane, layer, w, st):
+        m = layer.m
+        for t in (w.qkv, w.uk, w.uv, w.ukv, w.o):
+            lane.weight_map(t)
+        lane.mix.maps(m.heads * m.vdim)
+        lane.head_maps(lane.q_un.addr, up(m.dim, 64), m.dim, m.heads)
+        lane.head_maps(lane.o_lat.addr, up(m.kv_rank, 64), m.kv_rank, m.heads)
+        lane.c_rows.maps(m.kv_rank)
+        if direct_buffers(m):
+            lane.direct_maps(m)
+        for n in range(1, 65):   # a program's tile shape follows its longest request
+            shape = latent_tile(m, lane.kv.page, n)
+            if shape:
+                lane.q_map(m, *shape[:2])
+        if latent_tile(m, lane.kv.page, 1):
+            lane.kv_map(m, st["cache"])
 
     @staticmethod
     def build(lane, p, l, run, b, prev):
@@ -358,7 +412,8 @@ class LatentAttention:
                                  ("latent_v", run))
 
 
-MIXERS = {"mamba1": SelectiveScan, "mlstm": MatrixMemory, "latent_attention": LatentAttention}
+MIXERS = {"mamba1": SelectiveScan, "mlstm": MatrixMemory, "latent_attention": LatentAttention, "gla": GatedLinear,
+          "parallel": Parallel}
 
 
 # ---------------------------------------------------------------------------------------------- the lane
@@ -369,10 +424,18 @@ class _Buf:
         self.ld = up(cols, 64)
         self.t = torch.zeros(rows, self.ld, dtype=dtype, device="cuda")
         self.addr, self.es = self.t.data_ptr(), self.t.element_size()
-        self.lane, self.rows, self._maps = lane, rows, {}
+        self.lane, self.rows, self._maps, self._views = lane, rows, {}, {}
 
     def data_ptr(self):
         return self.addr
+
+    def view(self, col):
+        """The buffer from column `col` on."""
+        if col not in self._views:
+            v = self._views[col] = object.__new__(_Buf)
+            v.ld, v.t, v.addr, v.es, v.lane, v.rows, v._maps, v._views = \
+                self.ld, None, self.addr + col * self.es, self.es, self.lane, self.rows, {}, {}
+        return self._views[col]
 
     def maps(self, k):
         """Maps of the first k columns (zero beyond them)."""
@@ -388,6 +451,7 @@ class _Batch:
     def __init__(self, lane, requests, pos0=None):
         self.lane, self.requests, self.pos0 = lane, requests, pos0
         self.T = sum(n for _, n, _ in requests)
+        self.first, self.plans = None, []   # the program's first stage; plan tiles to be given their dynamic region
         self._made = {}
 
     def split(self):
@@ -429,7 +493,7 @@ class _Batch:
             for row0, n, slot in self.requests:
                 r, c = np.meshgrid(np.arange(0, n, rows_per), np.arange(0, channels, ch_per), indexing="ij")
                 out.append(tile_array(K_CONV, i0=row0, i1=row0 + r,
-                                      i2=np.minimum(rows_per, n - r) | (np.minimum(ch_per, channels - c) << 16), i3=slot, a1=c))
+                                      i2=np.minimum(rows_per, n - r) | (np.minimum(ch_per, channels - c) << 16), i3=slot, a1=c, a2=n))
             return np.concatenate(out)
         return self._once(("conv", channels), make)
 
@@ -446,24 +510,24 @@ class _Batch:
             return np.concatenate(out)
         return self._once(("scan", channels), make)
 
-    def memory_tiles(self, heads, e):
-        """Portions: a tile per head and block of columns; single tokens: as many column blocks in a tile as leave every
-        worker one."""
+    def memory_tiles(self, heads, columns, kinds=(K_MEMORY, K_MEMORY_STEP), width=MEMORY_COLUMNS, step_width=MEMORY_COLUMNS):
+        """Portions: a tile per head and block of `width` columns; single tokens: as many blocks of step_width columns in a
+        tile as leave every worker one."""
         def make():
-            blocks = -(-(e + 1) // MEMORY_COLUMNS)
-            h, c = np.meshgrid(np.arange(heads), np.arange(blocks), indexing="ij")
-            out = [tile_array(K_MEMORY, i0=row0, i1=n, i2=h | (c << 16), i3=slot)
+            h, c = np.meshgrid(np.arange(heads), np.arange(-(-columns // width)), indexing="ij")
+            out = [tile_array(kinds[0], i0=row0, i1=n, i2=h | (c << 16), i3=slot, a1=width)
                    for row0, n, slot in sorted(self.requests, key=lambda q: -q[1]) if n > 1]
+            blocks = -(-columns // step_width)
             ones = [(row0, slot) for row0, n, slot in self.requests if n == 1]
             if ones:
                 row, slot = (np.array(v)[:, None, None] for v in zip(*ones))
                 per = min(128, -(-blocks // min(blocks, max(1, self.lane.fab.num_workers // (len(ones) * heads)))))
                 h, c = np.arange(heads)[None, :, None], np.arange(0, blocks, per)[None, None, :]
-                out.append(tile_array(K_MEMORY_STEP, i0=row, i1=np.minimum(per, blocks - c), i2=h | (c << 16), i3=slot))
+                out.append(tile_array(kinds[1], i0=row, i1=np.minimum(per, blocks - c), i2=h | (c << 16), i3=slot))
             return np.concatenate(out)
-        return self._once(("memory", heads, e), make)
+        return self._once(("memory", heads, columns, kinds, width, step_width), make)
 
-    def attn_tiles(self, heads, parts):
+    def attn_tiles(self, heads, parts, kind=K_LATENT_ATTN):
         """One tile per row, group of heads and part, the rows that see most keys first."""
         per = 4 if parts > 1 or self.T * -(-heads // 4) <= 4 * self.lane.fab.num_workers else heads
 
@@ -471,9 +535,9 @@ class _Batch:
             rows = np.concatenate([np.arange(row0 + n - 1, row0 - 1, -1) for row0, n, _ in self.requests])
             slots = np.concatenate([np.full(n, slot) for _, n, slot in self.requests])
             h = np.arange(0, heads, per)
-            return tile_array(K_LATENT_ATTN, i0=rows[:, None, None], i1=(h | (np.minimum(per, heads - h) << 16))[None, :, None],
+            return tile_array(kind, i0=rows[:, None, None], i1=(h | (np.minimum(per, heads - h) << 16))[None, :, None],
                               i2=np.arange(parts)[None, None, :], i3=parts, a1=slots[:, None, None])
-        return self._once(("attn", heads, parts), make)
+        return self._once(("attn", heads, parts, kind), make)
 
     def latent_tiles(self, heads, tokens, group, parts):
         """One tile per block of `tokens` rows of a request, group of heads and part, the blocks that see most keys first
@@ -504,23 +568,23 @@ class LayerListLane(LaneBase):
         act, f32 = torch.float32 if cfg.f32 else torch.bfloat16, torch.float32
         z = lambda *shape, dt=torch.float32: torch.zeros(*shape, dtype=dt, device="cuda")  # noqa: E731
         sizes = {}
-        for layer in cfg.layers:
-            for name, v in MIXERS[layer.kind].sizes(layer.m).items():
+        for layer, lw in zip(cfg.layers, weights.layers):
+            for name, v in MIXERS[layer.kind].sizes(layer.m, lw).items():
                 if isinstance(v, tuple):   # per head: the largest block of heads x padded columns
                     sizes[name] = max(sizes.get(name, 0), v[0] * up(v[1], 64))
                 else:
                     sizes[name] = max(sizes.get(name, 0), v)
-        self.xs = z(T, cfg.streams, H)
+        self.xs = z(T, cfg.streams, H)   # or the plain residual [T][H]
         # a row of h, and behind it what its bf16 rounding has left, for products that take the whole 32-bit row
         self.split = up(H, 64) if "split" in sizes and not cfg.f32 else 0
         self.h = _Buf(self, T, 3 * self.split or H, act)
         ff = max([layer.ff for layer in cfg.layers] + [0])
         self.hd = _Buf(self, T, ff, act) if ff else None
         self.gu = _Buf(self, T, 2 * ff, f32) if ff and cfg.f32 else None
-        for name, dt in (("proj", act), ("act", act), ("mix", act), ("dt_in", act), ("small", f32), ("dt", f32), ("qc", f32),
-                         ("raw", f32)) + (() if cfg.f32 else (("kvb", act), ("c_rows", act))):
+        for name, dt in (("proj", act), ("act", act), ("mix", act), ("dt_in", act), ("mix2", act), ("gate", act), ("small", f32),
+                         ("dt", f32), ("qc", f32), ("decay", f32), ("raw", f32)) + (() if cfg.f32 else (("kvb", act), ("c_rows", act))):
             setattr(self, name, _Buf(self, T, sizes[name], dt) if name in sizes else None)
-        for name in ("q_un", "q_all", "o_lat"):   # [head][T][columns]: addressed by the layer's own strides
+        for name in ("q_un", "q_all", "o_lat", "gq", "go"):   # [head][T][columns] or [T][head][columns]: addressed by the layer's own strides
             if name in sizes:
                 buf = types.SimpleNamespace(t=z(T * sizes[name], dt=act))
                 buf.addr = buf.t.data_ptr()
@@ -529,6 +593,9 @@ class LayerListLane(LaneBase):
         self.rows_slab = max(SPLIT_PARTS * SPLIT_ROWS, WIDE_PARTS * min(WIDE_ROWS, up(T, 64)), T)
         self.y = types.SimpleNamespace(t=z(self.rows_slab, H))
         self.y.addr = self.y.t.data_ptr()
+        if "y2" in sizes:   # the second of two mixers side by side
+            self.y2 = types.SimpleNamespace(t=z(self.rows_slab, H))
+            self.y2.addr = self.y2.t.data_ptr()
         if "small" in sizes:
             self.slabs = types.SimpleNamespace(t=z(self.rows_slab * sizes["small"]))
             self.slabs.addr = self.slabs.t.data_ptr()
@@ -539,16 +606,13 @@ class LayerListLane(LaneBase):
         self.residual = z(len(cfg.order), T, H) if keep_residual else None
         self._request_state(T, self.S, requests)
         self.max_pos = bt_stride * kv.page
-        self._cos_sin, self._wmaps, self._hmaps = {}, {}, {}
+        self._cos_sin, self._wmaps, self._hmaps, self.attn_blocks = {}, {}, {}, {}
         for layer in cfg.layers:
             if layer.kind == "latent_attention":
                 self.cos_sin(layer.m.rot["base"], layer.m.rot_dim)
         self._build_state((48 << 10) * (len(cfg.order) + 2))
         self.sample_args, self.step_args = self._sample_block(cfg.vocab), self._step_block()
         self._prepare()
-        for l, state in zip(cfg.order, kv.runs):
-            if cfg.layers[l].kind == "latent_attention" and not cfg.f32 and latent_tile(cfg.layers[l].m, kv.page, 1):
-                self.kv_map(cfg.layers[l].m, state["cache"])
 
     def _prepare(self):
         """Make every tensor map a program can name now: none may be made while the fabric is resident."""
@@ -560,25 +624,11 @@ class LayerListLane(LaneBase):
         self.h.maps(cfg.hidden)
         self.xlast.maps(cfg.hidden)
         for layer, lw in zip(cfg.layers, w.layers):
-            m = layer.m
             if layer.ff:
                 wm(lw.gate_up), wm(lw.down), self.hd.maps(layer.ff)
-            wm(lw.o)
-            if layer.kind == "mamba1":
-                wm(lw.in_), wm(lw.x), wm(lw.dt), self.act.maps(m.inner), self.dt_in.maps(m.dt_rank), self.mix.maps(m.inner)
-            elif layer.kind == "mlstm":
-                wm(lw.qkvg), wm(lw.gates), self.h.maps(3 * self.split), self.mix.maps(m.heads * m.vdim)
-            else:
-                wm(lw.qkv), wm(lw.uk), wm(lw.uv), self.mix.maps(m.heads * m.vdim)
-                self.head_maps(self.q_un.addr, up(m.dim, 64), m.dim, m.heads)
-                self.head_maps(self.o_lat.addr, up(m.kv_rank, 64), m.kv_rank, m.heads)
-                wm(lw.ukv), self.c_rows.maps(m.kv_rank)
-                if direct_buffers(m):
-                    self.direct_maps(m)
-                for n in range(1, 65):   # a program's tile shape follows its longest request
-                    shape = latent_tile(m, self.kv.page, n)
-                    if shape:
-                        self.q_map(m, *shape[:2])
+        for l, state in zip(cfg.order, self.kv.runs):
+            layer, lw = cfg.layers[l], w.layers[l]
+            MIXERS[layer.kind].prepare(self, layer, lw, state)
 
     def cos_sin(self, base, r):
         """fp32 [max_pos][r / 2][cos, sin] of the angles pos * base^(-2 i / r)."""
@@ -676,11 +726,12 @@ class LayerListLane(LaneBase):
         p.after(prev, s)
         return s
 
-    def closing(self, p, prev, x, w, rows, k, label):
-        """The product that ends a sublayer: y as fp32 slabs for the streams tile."""
+    def closing(self, p, prev, x, w, rows, k, label, out=None):
+        """The product that ends a sublayer: y (or `out`) as fp32 slabs for the streams or residual tile.  Returns (stage,
+        (slabs,)); a sublayer of two mixers has a pair of each."""
         parts = 1 if self.cfg.f32 else self.split_parts(rows, k)
-        s = self.product(p, prev, x, w, self.y, rows, self.cfg.hidden, k, label, parts=parts, ld_out=self.cfg.hidden)
-        return s, parts, self.slab_rows(rows) if parts > 1 else 0
+        s = self.product(p, prev, x, w, out or self.y, rows, self.cfg.hidden, k, label, parts=parts, ld_out=self.cfg.hidden)
+        return s, (parts,)
 
     def items_per(self, items):
         """Items (one warp each) per tile of an item-wise stage: a multiple of four, about two rounds of tiles."""
@@ -724,62 +775,78 @@ class LayerListLane(LaneBase):
         return self._hmaps[key]
 
     # ------------------------------------------------------------------ programs
-    def _streams(self, p, rows, prev, sub, before, label, split=False, gather=False, step=False):
-        """The streams stage in front of sublayer `sub` = (hc_in, norm): `before` = ((hc_out, hc_mix), parts, slab rows,
-        run whose residual this completes or None) of the sublayer behind it, or None at the embedding."""
+    def _between(self, p, rows, prev, sub, before, label, split=False, gather=False, step=False):
+        """The stage between two sublayers: the residual takes the output of the one behind it, and the one ahead of it,
+        `sub` = (hc_in, norm), gets its input.  `before` = (what of the layer's weights follows the sublayer, its slab
+        counts, its branches' norms or None, run whose residual this completes or None), or None at the embedding."""
         cfg = self.cfg
         hc_in, norm = sub
-        f = dict(xs=self.xs, hc_in=hc_in, w=norm, W=cfg.hidden, streams=cfg.streams, eps=cfg.eps)
+        streams = cfg.design.residual == "streams"
+        f = dict(w=norm, W=cfg.hidden, eps=cfg.eps)
+        f.update(dict(xs=self.xs, hc_in=hc_in, streams=cfg.streams) if streams else dict(x=self.xs))
         if before is None:
             f.update(embed=self.w.embed, **({"step": self.step_args} if step else {"tokens": self.tokens}))
+            if not streams:
+                f.update(embed_scale=cfg.embed_scale, tok_pos=self.tok_pos, max_pos=self.max_pos)
+                if self.w.pos is not None:
+                    f.update(pos=self.w.pos, max_pos=self.w.pos.shape[0])
         else:
-            (hc_out, hc_mix), parts, slab_rows, run = before
-            f.update(y=self.y.addr, hc_out=hc_out, hc_mix=hc_mix, y_parts=parts, y_rows=slab_rows)
+            after, parts, branches, run = before
+            y_rows = self.slab_rows(rows)
+            if streams:
+                f.update(y=self.y.addr, hc_out=after[0], hc_mix=after[1], y_parts=parts[0], y_rows=y_rows)
+            else:
+                f.update(y0=self.y.addr, y0_parts=parts[0], y_rows=y_rows, post_w=after[0])
+                if branches:
+                    f.update(y1=self.y2.addr, y1_parts=parts[1], w0=branches[0], w1=branches[1],
+                             branch_scale=Parallel.BRANCH_SCALE)
             if run is not None and self.residual is not None:
                 f.update(sum_out=self.residual[run])
         if gather:
             f.update(gather=self.gather, ld_out=self.xlast.ld, **{"out32" if cfg.f32 else "out16": self.xlast.addr})
+        elif cfg.f32:
+            f.update(h32=self.h.addr, ld_h32=self.h.ld)
         else:
-            if cfg.f32:
-                f.update(h32=self.h.addr, ld_h32=self.h.ld)
-            else:
-                f.update(h16=self.h.addr, ld_h16=self.h.ld, split=self.split if split else 0)
-        args = self._dev("StreamArgs", **f)
-        s = p.stage(self._rows(K_STREAMS, args, rows, self._per(rows)), label=label)
+            f.update(h16=self.h.addr, ld_h16=self.h.ld)
+            if split:
+                f.update(split=self.split)
+        args = self._dev("StreamArgs" if streams else "ResidualArgs", **f)
+        s = p.stage(self._rows(K_STREAMS if streams else K_RESIDUAL, args, rows, self._per(rows)), label=label)
         if prev is not None:
-            p.after(prev, s)
+            for stage in prev if isinstance(prev, list) else [prev]:
+                p.after(stage, s)
         return s
 
     def _chain(self, p, b, step):
-        """Every layer run; returns (first stage, final streams stage)."""
+        """Every layer run; returns (first stage, the final stage of the residual)."""
         cfg, T = self.cfg, b.T
         self.rows_now = T
-        first = prev = None
-        before = None
+        name = "streams" if cfg.design.residual == "streams" else "residual"
+        prev = before = None
         for run, l in enumerate(cfg.order):
             layer, w = cfg.layers[l], self.w.layers[l]
-            prev = self._streams(p, T, prev, (w.hc1[0], w.norm1), before, ("streams", run), split=layer.kind == "mlstm", step=step)
-            first = prev if first is None else first
-            prev, parts, slab = MIXERS[layer.kind].build(self, p, l, run, b, prev)
-            before = (w.hc1[1:], parts, slab, None if layer.ff else run)
+            prev = self._between(p, T, prev, (w.hc1[0], w.norm1), before, (name, run), split=layer.kind == "mlstm", step=step)
+            b.first = prev if b.first is None else b.first
+            prev, parts = MIXERS[layer.kind].build(self, p, l, run, b, prev)
+            before = (w.hc1[1:], parts, getattr(w, "branches", None), None if layer.ff else run)
             if layer.ff:
-                prev = self._streams(p, T, prev, (w.hc2[0], w.norm2), before, ("streams_ff", run))
+                prev = self._between(p, T, prev, (w.hc2[0], w.norm2), before, (name + "_ff", run))
                 if cfg.f32:
                     s = self.product(p, prev, self.h, w.gate_up, self.gu, T, 2 * layer.ff, cfg.hidden, ("ff_in", run))
                     g = self._dev("GatedArgs", out=self.hd.addr, ff=layer.ff, ld_in=self.gu.ld, ld_out=self.hd.ld,
-                                  **{"in": self.gu.addr})
+                                  silu=int(cfg.design.act == "silu"), **{"in": self.gu.addr})
                     s_g = p.stage(self._rows(K_GATED, g, T, self._per(T)), label=("ff_act", run))
                     p.after(s, s_g)
                     s = s_g
                 else:
                     s = self.product(p, prev, self.h, w.gate_up, self.hd, T, layer.ff, cfg.hidden, ("ff_in", run),
-                                     epi=EPI_GELU_MUL, up_offset=layer.ff)
-                prev, parts, slab = self.closing(p, s, self.hd, w.down, T, layer.ff, ("ff_out", run))
-                before = (w.hc2[1:], parts, slab, run)
-        last = self._streams(p, T, prev, (self.w.ones, self.w.final_norm), before, ("final", len(cfg.order)), gather=True)
-        return first, last
+                                     epi=EPI_SILU_MUL if cfg.design.act == "silu" else EPI_GELU_MUL, up_offset=layer.ff)
+                prev, parts = self.closing(p, s, self.hd, w.down, T, layer.ff, ("ff_out", run))
+                before = (w.hc2[1:], parts, None, run)
+        last = self._between(p, T, prev, (self.w.ones, self.w.final_norm), before, ("final", len(cfg.order)), gather=True)
+        return b.first, last
 
-    def _finish(self, p, prev, n_rows, sample_rows):
+    def _finish(self, p, b, prev, n_rows, sample_rows):
         if n_rows:
             s = self.product(p, prev, self.xlast, self.w.head, types.SimpleNamespace(t=self.logits, addr=self.logits.data_ptr(),
                                                                                      ld=self.cfg.vocab),
@@ -788,6 +855,11 @@ class LayerListLane(LaneBase):
             if tiles:
                 s_s = p.stage(tiles, label=("sample", -1))
                 p.after(s, s_s)
+        at = p.dynamic_first   # every static tile is counted: the plan tiles get their parts of the dynamic region
+        for blob, fields, most in b.plans:
+            p.reserve(most)
+            self.arena.patch(blob, pack("AttnPlanArgs", dyn_first=at, dyn_cap=most, **fields))
+            at += most
         self.rows_out = n_rows
         self.labels = p.labels()
         self.arena.flush()
@@ -803,7 +875,7 @@ class LayerListLane(LaneBase):
         p = Program()
         b = _Batch(self, [(row0, n, slot) for (row0, _, n, _), (slot, _, _) in zip(req_info, batch)], [q[2] for q in batch])
         first, last = self._chain(p, b, step=False)
-        self._finish(p, last, T if all_logits else sum(len(v) for v in places), sample_rows if want is None else [])
+        self._finish(p, b, last, T if all_logits else sum(len(v) for v in places), sample_rows if want is None else [])
         return p.upload(self.fab, first=first, iterations=iterations)
 
     def build_decode(self, slots, iterations=1, chunk_keys=0):
@@ -816,5 +888,5 @@ class LayerListLane(LaneBase):
         p = Program()
         b = _Batch(self, [(r, 1, slot) for r, slot in enumerate(slots)])
         first, last = self._chain(p, b, step=True)
-        self._finish(p, last, R, list(enumerate(slots)))
+        self._finish(p, b, last, R, list(enumerate(slots)))
         return p.upload(self.fab, first=first, iterations=iterations)

@@ -42,15 +42,16 @@ class _MoE:
 
 
 class _LayerList:
-    """Decoders whose configuration lists a mixer per layer: Sinotar (monoserve_b200/layer_list.py)."""
+    """Decoders whose configuration lists a mixer per layer: Sinotar, Teganex (monoserve_b200/layer_list.py)."""
 
     @staticmethod
     def matches(config):
-        return config.get("architecture") == "Sinotar"
+        from monoserve_b200.layer_list import DESIGNS
+        return config.get("architecture") in DESIGNS
 
     @staticmethod
     def owns(cfg):
-        return getattr(cfg, "model_type", None) == "sinotar"
+        return getattr(cfg, "model_type", None) in ("sinotar", "teganex")
 
     @staticmethod
     def load(folder, config, dtype):

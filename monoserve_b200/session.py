@@ -23,7 +23,7 @@ class Session:
         passes."""
         import torch
         n_pages = -(-max_tokens // page) + 2 * slots + 2
-        self.page, self.vocab = page, model.cfg.vocab
+        self.page, self.vocab, self.max_positions = page, model.cfg.vocab, getattr(model.cfg, "max_positions", None)
         workers = torch.cuda.get_device_properties(0).multi_processor_count - SPARE_SMS
         self.fab = Fabric(num_workers=workers, pool_bytes=256 << 20)
         self.fab.set_max_run(max_run_s)
@@ -77,6 +77,8 @@ class Session:
         if rid not in self.live:
             self.live[rid] = dict(slot=self.free.pop(), pages=[], length=0)
         r = self.live[rid]
+        if self.max_positions and r["length"] + len(tokens) > self.max_positions:
+            raise ValueError(f"request {rid}: {r['length']} + {len(tokens)} tokens, the model has {self.max_positions} positions")
         self._reserve(r, r["length"] + len(tokens))
         out = []
         for lo in range(0, len(tokens), self.pass_tokens):
