@@ -119,3 +119,7 @@ ONES = config([scan(inner=1, state=1, dt_rank=1, conv=2), latent(heads=1, dim=1,
                memory(heads=1, dim=1, vdim=2, cap=1.0)], width=16, vocab=16, streams=1, ff=1)
 ALONE = {"scan": config([SCAN], 96, 128, 3), "memory": config([MEMORY], 96, 128, 3), "latent": config([LATENT], 96, 128, 3),
          "ff": config([(scan(inner=8, state=1, dt_rank=1, conv=1), 80)], 96, 128, 4)}
+
+
+def copy_of(c):
+    return json.loads(json.dumps(c))
