@@ -757,13 +757,14 @@ def main():
     ap.add_argument("--sweep", action="store_true",
                     help="the batch x credits x form sweep of benchmark configuration 2 instead of the bench line")
     ap.add_argument("--layer-list", action="store_true",
-                    help="prefill and decode throughput of a layer-list decoder (Sinotar) beside the dense-layer decoder at equal "
+                    help="prefill and decode throughput of a layer-list decoder beside the dense-layer decoder at equal "
                          "size, with every stage against its roofline, instead of the bench line")
+    ap.add_argument("--design", default="Sinotar", choices=["Sinotar", "Teganex"], help="with --layer-list: the decoder's design")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.layer_list:
         from monoserve_b200.benchmarks import layer_list
-        layer_list.main(["--steps", str(min(args.steps, 50)), "--stages"])
+        layer_list.main(["--steps", str(min(args.steps, 50)), "--stages", "--design", args.design])
     elif args.sweep:
         run_sweep(args)
     elif args.ncu:

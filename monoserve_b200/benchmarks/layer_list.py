@@ -1,9 +1,10 @@
-"""Layer-list decoders (Sinotar) beside the closest model this library had: prefill and decode throughput at layer sizes
-of real models, random weights, one layer of each mixer with its feed-forward, against the dense-layer form of the
-GLM-style decoder (grouped-query attention and a gated feed-forward of the same width) at equal width, depth and
-feed-forward.
+"""Layer-list decoders beside the closest models of the library: prefill and decode throughput at layer sizes of real
+models, random weights, three layers with their feed-forward.  --design Sinotar (matrix memory, selective scan, latent
+attention; 4 residual streams) or Teganex (gated linear attention of two shapes around an attention / delta rule layer), and
+always `dense`: the dense-layer form of the GLM-style decoder (grouped-query attention and a gated feed-forward) at equal
+width, depth and feed-forward.  With Teganex the Sinotar layers are run as well: they have the like recurrence stages.
 
-    python -m monoserve_b200.benchmarks.layer_list [--sizes 2048,4096] [--steps 20] [--only new|dense] [--stages]
+    python -m monoserve_b200.benchmarks.layer_list [--design Sinotar] [--sizes 2048,4096] [--steps 20] [--only ...] [--stages]
 
 Timed by the fabric's iteration timer (device clock) over repeating programs on all SMs: `prefill` = 4 prompts of 1024
 tokens per iteration, `decode` = one token of 32 sequences with contexts around 4096 per iteration.  The weights of a
@@ -27,6 +28,54 @@ if os.path.exists(_path):
         PEAKS.update({k: v for k, v in json.load(_f).items() if k in PEAKS})
 
 PROMPTS, PROMPT_LEN, DECODE_ROWS, CONTEXT, PAGE, VOCAB = 4, 1024, 32, 4096, 16, 32768
+
+
+def teganex_config(W):
+    """A layer of many small memories, one with attention beside the delta rule, one of few large memories (the size of the
+    matrix memory's)."""
+    from monoserve_b200.layer_list import read_config
+    mixers = [("gla", dict(heads=W // 128, dim=64, vdim=128, tau=16.0)),
+              ("parallel", dict(left=dict(heads=W // 128, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5),
+                                right=dict(heads=W // 128, kv_heads=W // 256, dim=128, vdim=128, conv=4))),
+              ("gla", dict(heads=W // 512, dim=256, vdim=512, tau=16.0))]
+    return read_config(dict(architecture="Teganex", layers=[dict(type=k, mixer=m, mlp=dict(kind="dense", ff=3 * W)) for k, m in mixers],
+                            width=W, vocab=VOCAB, norm=dict(eps=1e-5), embedding=dict(scale=1.0), logit_scale=1.0,
+                            max_positions=CONTEXT * 2))
+
+
+def teganex_tensors(cfg):
+    """Random tensors, made on the device."""
+    W, t = cfg.hidden, {}
+    g = torch.Generator(device="cuda").manual_seed(0)
+    r = lambda *shape, scale=1.0: (torch.randn(*shape, generator=g, device="cuda") * scale).to(torch.bfloat16)  # noqa: E731
+    lin = lambda o, i: r(o, i, scale=i ** -0.5)  # noqa: E731
+    one = lambda n: 1 + r(n, scale=0.1)  # noqa: E731
+    t.update({"embed": r(cfg.vocab, W), "pos": r(cfg.max_positions, W, scale=0.1), "head": lin(cfg.vocab, W), "final.norm": one(W)})
+    for i, layer in enumerate(cfg.layers):
+        m, p, x = layer.m, f"l{i}.", f"l{i}.mix."
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            t[p + n] = one(W)
+        if layer.kind == "gla":
+            H, d, e = m.heads, m.dim, m.vdim
+            for n, o in (("q", H * d), ("k", H * d), ("v", H * e), ("g", H * e), ("a1", 16)):
+                t[x + n] = lin(o, W)
+            t[x + "a2"], t[x + "a2.b"], t[x + "norm"], t[x + "o"] = lin(H * d, 16), r(H * d) + 2, one(e), lin(W, H * e)
+        else:
+            a = m.left
+            for n, o in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim), ("g", a.heads)):
+                t[f"{x}left.{n}"] = lin(o, W)
+            t[x + "left.q.norm"], t[x + "left.k.norm"], t[x + "left.o"] = one(a.dim), one(a.dim), lin(W, a.heads * a.vdim)
+            a = m.right
+            for n, o in (("q", a.kv_heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.heads * a.vdim)):
+                t[f"{x}right.{n}"], t[f"{x}right.{n}.conv"] = lin(o, W), r(o, a.conv, scale=0.5)
+            for n, o in (("b", a.heads), ("a1", a.dim), ("g1", a.vdim)):
+                t[f"{x}right.{n}"] = lin(o, W)
+            t[x + "right.a2"], t[x + "right.g2"] = lin(a.heads * a.dim, a.dim), lin(a.heads * a.vdim, a.vdim)
+            t[x + "right.A_log"], t[x + "right.dt_bias"] = r(a.heads), r(a.heads * a.dim) - 3
+            t[x + "right.norm"], t[x + "right.o"] = one(a.vdim), lin(W, a.heads * a.vdim)
+            t[x + "left.out"], t[x + "right.out"] = one(W), one(W)
+        t[p + "mlp.gate"], t[p + "mlp.up"], t[p + "mlp.down"] = lin(layer.ff, W), lin(layer.ff, W), lin(W, layer.ff)
+    return t
 
 
 def new_config(W):
@@ -130,6 +179,33 @@ def new_roofline(cfg, T, R, pairs, keys):
     return st
 
 
+def teganex_roofline(cfg, T, R, pairs, keys):
+    """As new_roofline; stages of the two kinds of gla layers are told apart by their layer."""
+    W, f = cfg.hidden, cfg.layers[0].ff
+    row = lambda ys: seconds(T * W * (8.0 + 4 * ys + 2))  # noqa: E731
+    st = {"residual": row(1), "residual_ff": row(1), "final": seconds(T * W * 12.0), "residual_ff.1": row(2),
+          "ff_in": gemm(T, 2 * f, W, 1), "ff_out": gemm(T, W, f, 4), "head": gemm(R, cfg.vocab, W, 4), "sample": seconds(4.0 * R * cfg.vocab)}
+    # a memory: its inputs and outputs, its state read and written once, six operations per token and state element
+    memory = lambda H, G, d, e: seconds(T * (4.0 * G * d + 4 * H * d + 6 * H * e) + 8.0 * R * H * d * e, 6.0 * T * H * d * e)  # noqa: E731
+    for i, layer in enumerate(cfg.layers):
+        m = layer.m
+        if layer.kind == "gla":
+            H, d, e = m.heads, m.dim, m.vdim
+            st.update({f"gla_in.{i}": gemm(T, 2 * H * (d + e), W, 2), f"gla_decay.{i}": seconds(T * (4.0 * H * d + 32)),
+                       f"gla.{i}": memory(H, H, d, e), f"gla_norm.{i}": seconds(8.0 * T * H * e), f"gla_o.{i}": gemm(T, W, H * e, 4)})
+        else:
+            a, b = m.left, m.right
+            H, G, d, e = a.heads, a.kv_heads, a.dim, a.vdim
+            C = 2 * b.kv_heads * b.dim + b.heads * b.vdim
+            n = H * d + G * (d + e) + H + C + b.heads + b.dim + b.vdim
+            st.update(parallel_in=gemm(T, n, W, 2), qkv=seconds(4.0 * T * (H * d + G * (d + e))),
+                      attn=seconds(2.0 * keys * G * (d + e), 2.0 * pairs * H * (d + e)), head_gate=seconds(4.0 * T * H * e),
+                      attn_o=gemm(T, W, H * e, 4), delta_conv=seconds(4.0 * T * C), delta_decay=seconds(T * (4.0 * b.heads * b.dim + 2 * b.dim)),
+                      delta_gate=gemm(T, b.heads * b.vdim, b.vdim, 2), delta=memory(b.heads, b.kv_heads, b.dim, b.vdim),
+                      delta_norm=seconds(8.0 * T * b.heads * b.vdim), delta_o=gemm(T, W, b.heads * b.vdim, 4))
+    return st
+
+
 def dense_roofline(cfg, T, R, pairs, keys):
     W, f, hq, hkv = cfg.hidden, cfg.dense_intermediate, cfg.num_heads, cfg.num_kv_heads
     q = (hq + 2 * hkv) * 128
@@ -158,8 +234,9 @@ def timed(fab, lane, handle, tokens, steps, roofline, show):
     if error:
         raise RuntimeError(f"device error {error:#x}: {fab.wait_notes()}")
     us = {}
-    for name, _, _, t0, t1 in spans(records, lane.labels, 0):
-        us.setdefault(name, []).append((t1 - t0) / 1e3)
+    for name, layer, _, t0, t1 in spans(records, lane.labels, 0):
+        one = f"{name}.{layer}"   # stages that differ from layer to layer
+        us.setdefault(one if one in roofline or name.startswith("gla") else name, []).append((t1 - t0) / 1e3)
     stages = {}
     for name, v in us.items():
         mean = float(np.median(v))
@@ -184,26 +261,29 @@ def measure(kind, W, steps, show):
     from monoserve_b200.layer_list import LayerListCache, LayerListLane, Weights
     from monoserve_b200.model import KVCache, ModelLane
     rng = np.random.default_rng(0)
-    if kind == "new":
-        cfg = new_config(W)
-        weights = Weights(cfg, new_tensors(cfg))
+    listed = kind != "dense"
+    if listed:
+        make_config, make_tensors, roofline = {"Sinotar": (new_config, new_tensors, new_roofline),
+                                               "Teganex": (teganex_config, teganex_tensors, teganex_roofline)}[kind]
+        cfg = make_config(W)
+        weights = Weights(cfg, make_tensors(cfg))
     else:
-        cfg = dense_config(W)
+        cfg, roofline = dense_config(W), dense_roofline
         weights = dense_weights(cfg)
     ctx = rng.integers(CONTEXT // 2, CONTEXT * 3 // 2, size=DECODE_ROWS)
     grow = 4 * steps + 64
     dec_pages = [-(-(int(n) + grow) // PAGE) for n in ctx]
     pre_pages = -(-PROMPT_LEN // PAGE)
     n_pages = 1 + sum(dec_pages) + PROMPTS * pre_pages
-    kv = LayerListCache(cfg, n_pages, PAGE, DECODE_ROWS) if kind == "new" else KVCache(cfg, n_pages, PAGE)
-    if kind == "new":
+    kv = LayerListCache(cfg, n_pages, PAGE, DECODE_ROWS) if listed else KVCache(cfg, n_pages, PAGE)
+    if listed:
         for run in kv.runs:
             for t in run.values():
                 t.normal_(0, 0.5)
     else:
         for t in kv.k + kv.v:
             t.normal_(0, 1)
-    make = LayerListLane if kind == "new" else ModelLane
+    make = LayerListLane if listed else ModelLane
     out = {}
     fab = fabric()   # one per program: a stopped lane keeps the program it was running
     try:
@@ -217,7 +297,7 @@ def measure(kind, W, steps, show):
             at += pre_pages
             batch.append((s, rng.integers(0, cfg.vocab, size=PROMPT_LEN).tolist(), 0))
         pairs, keys = PROMPTS * PROMPT_LEN * (PROMPT_LEN + 1) / 2, T
-        roof = (new_roofline if kind == "new" else dense_roofline)(cfg, T, PROMPTS, pairs, keys)
+        roof = roofline(cfg, T, PROMPTS, pairs, keys)
         h = lane.build_prefill(batch, iterations=0)
         out["prefill"] = timed(fab, lane, h, T, steps, roof, show)
         fab.close()
@@ -229,7 +309,7 @@ def measure(kind, W, steps, show):
             at += n
             lane.set_request(s, seq_len=int(ctx[s]), last_token=int(rng.integers(0, cfg.vocab)))
         keys = float(ctx.sum())
-        roof = (new_roofline if kind == "new" else dense_roofline)(cfg, DECODE_ROWS, DECODE_ROWS, keys, keys)
+        roof = roofline(cfg, DECODE_ROWS, DECODE_ROWS, keys, keys)
         h = lane.build_decode(list(range(DECODE_ROWS)), iterations=0)
         out["decode"] = timed(fab, lane, h, DECODE_ROWS, steps, roof, show)
     finally:
@@ -242,16 +322,20 @@ def main(argv=None):
     ap = argparse.ArgumentParser()
     ap.add_argument("--sizes", default="2048,4096", help="model widths")
     ap.add_argument("--steps", type=int, default=20)
-    ap.add_argument("--only", choices=["new", "dense"])
+    ap.add_argument("--design", choices=["Sinotar", "Teganex"], default="Sinotar")
+    ap.add_argument("--only", choices=["Sinotar", "Teganex", "dense"])
     ap.add_argument("--stages", action="store_true")
     args = ap.parse_args(argv)
-    line = {"workload": "layer-list decoder (matrix memory, selective scan, latent attention; 4 residual streams) beside the "
+    what = {"Sinotar": "matrix memory, selective scan, latent attention; 4 residual streams",
+            "Teganex": "gated linear attention, attention beside a gated delta rule, gated linear attention of few large heads"}[args.design]
+    line = {"workload": f"layer-list decoder {args.design} ({what}) beside the "
                         f"dense-layer decoder, 3 layers each, ff 3 x width; prefill {PROMPTS} x {PROMPT_LEN}, decode {DECODE_ROWS} "
                         f"sequences at contexts {CONTEXT // 2}..{CONTEXT * 3 // 2}", "dtype": "bf16", "data": "synthetic",
             "l2": "the weights of a step exceed L2", "peaks": PEAKS, "sizes": {}}
+    kinds = ("Sinotar", "dense") if args.design == "Sinotar" else ("Teganex", "Sinotar", "dense")
     for W in [int(v) for v in args.sizes.split(",")]:
         line["sizes"][W] = {}
-        for kind in (args.only,) if args.only else ("new", "dense"):
+        for kind in (args.only,) if args.only else kinds:
             if args.stages:
                 print(f"== width {W}, {kind}", file=sys.stderr)
             line["sizes"][W][kind] = measure(kind, W, args.steps, args.stages)

@@ -76,6 +76,16 @@ __device__ __forceinline__ Pair fma_pair(Pair a, Pair b, Pair c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
   return r;
 }
+__device__ __forceinline__ Pair add_pair(Pair a, Pair b) {
+  Pair r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ Pair mul_pair(Pair a, Pair b) {
+  Pair r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
 __device__ __forceinline__ void ld_pairs(const float* p, Pair& a, Pair& b) {
   const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(p);
   a = q.x;
@@ -84,30 +94,30 @@ __device__ __forceinline__ void ld_pairs(const float* p, Pair& a, Pair& b) {
 
 // NV values per lane summed over groups of LB lanes: lane l of a group ends with values [l NV / LB, ..), max(1, NV / LB) of
 // them, at the front of v.
-template <int NV, int LB>
-__device__ __forceinline__ void group_sum(float (&v)[NV], int lane) {
-  int n = NV;
+template <int N, int BIT, int NV>
+__device__ __forceinline__ void group_sum_from(float (&v)[NV], int lane) {
+  if constexpr (BIT >= 1) {
+    if constexpr (N > 1) {
+      const bool hi = lane & BIT;
 #pragma unroll
-  for (int bit = LB / 2; bit >= 1; bit >>= 1) {
-    if (n > 1) {
-      n >>= 1;
-      const bool hi = lane & bit;
-#pragma unroll
-      for (int c = 0; c < n; ++c) {
-        const float give = hi ? v[c] : v[c + n], have = hi ? v[c + n] : v[c];
-        v[c] = have + __shfl_xor_sync(0xffffffffu, give, bit);
+      for (int c = 0; c < N / 2; ++c) {
+        const float give = hi ? v[c] : v[c + N / 2], have = hi ? v[c + N / 2] : v[c];
+        v[c] = have + __shfl_xor_sync(0xffffffffu, give, BIT);
       }
     } else {
-      v[0] += __shfl_xor_sync(0xffffffffu, v[0], bit);
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], BIT);
     }
+    group_sum_from<(N > 1 ? N / 2 : 1), BIT / 2>(v, lane);
   }
 }
+template <int NV, int LB>
+__device__ __forceinline__ void group_sum(float (&v)[NV], int lane) { group_sum_from<NV, LB / 2>(v, lane); }
 
 constexpr float kUnitFloor = 1e-6f;
 
 // ------------------------------------------------------------------ a request's rows
 // Kind 68, GatedMemoryArgs: rows [i0, i0 + i1) of one request; i2 = head | column block << 16, slot i3, a[1] columns of a
-// block (32 C).  A wide tile: inputs come kTokens rows at a time through double-buffered asynchronous copies into the ring.
+// block.  A wide tile: inputs come kTokens rows at a time through double-buffered asynchronous copies into the ring.
 //
 // Four tokens are one step.  With c_i the product of their decays up to token i, s_j that of the decays behind token j, and
 // d_ij that of the decays after j up to i (all per key channel), S the state in front of the four:
@@ -116,328 +126,328 @@ constexpr float kUnitFloor = 1e-6f;
 // so the state is read once and written once per step, and the dot products between keys and queries are numbers of the
 // step.  A pass over the chunk in front prepares c k, c q, s k and those numbers; no decay is ever divided by.  c_3 enters
 // as S + S (c_3 - 1), with c_3 - 1 composed from the decays' distances to one, so that rounding a factor just below one
-// does not add up over a long memory.
+// does not add up over a long memory.  Keys and queries stay as they come: their scales (unit norms, q_scale) go into the
+// numbers.
 //
-// A warp holds 8 C columns, 32 C in the tile: lane = 4 * (column group) + g, with rows 4 (g + 4 i) .. + 3 of its C columns
-// in registers for the whole portion.  Lane g ends with the read-out of token g of the step.
+// G lanes share C columns of the state, R rows each in groups of four, 4 (l + G i) .. + 3, in registers for the whole
+// portion: 128 C / G columns in a tile.  A column's sums end in 4 G / (4 C) lanes of its group, which solve for its u, and
+// hand them to the others through shared memory.
 constexpr int kStep = 4;
-constexpr int kCoefs = 36;   // of a step: [0] d_ij products with queries (rows of four), [16] key scales, [20] betas,
-                             // [24] products between keys (1,0) (2,0) (2,1) (3,0) (3,1) (3,2), [32] query scales
 
-template <int R, int C, bool DELTA>
+// i = 1: 0; i = 2: 1, 2; i = 3: 3, 4, 5 (j < i), and with the diagonal 0; 1, 2; 3, 4, 5; 6 .. 9
+__device__ __forceinline__ int below(int i, int j) { return i * (i - 1) / 2 + j; }
+__device__ __forceinline__ int upto(int i, int j) { return i * (i + 1) / 2 + j; }
+
+template <int G, int R, int C, bool DELTA, bool F32>
 __device__ __noinline__ void gated_rows(const TileDesc& t, int tid, uint8_t* ring) {
-  constexpr int DP = 4 * R;                                    // key channels, padded
-  constexpr int kTokens = R <= 32 ? 32 : R == 64 ? 16 : 8, kSteps = kTokens / kStep;
-  constexpr int CB = 32 * C, I4 = R / 4;
-  constexpr int LB = R < 32 ? R : 32, NV = DELTA ? 32 : 16;    // lanes that prepare a step, sums of a step
-  struct Shared {
-    float kh[DELTA ? kTokens : 1][DP], qh[kTokens][DP], kt[kTokens][DP], em[kSteps][DP];
-    float coef[kSteps][kCoefs], sums[kSteps][32], beta[32], v[kTokens][CB];
-    float decay[2][kTokens][DP];
+  using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
+  constexpr int DP = G * R;                                    // key channels, padded
+  constexpr int kTokens = DP <= 128 ? 32 : DP == 256 ? 16 : 8, kSteps = kTokens / kStep;
+  constexpr int kSide = 32 / G, CB = 4 * kSide * C, I4 = R / 4;
+  constexpr int LB = DP < 64 ? DP / 2 : 32, NV = DELTA ? 32 : 16;   // lanes that prepare a step, sums of a step
+  constexpr int NS = 4 * C > G ? 4 * C / G : 1;                // sums of a step that a lane ends with
+  constexpr int kPer16 = 16 / static_cast<int>(sizeof(T));
+  struct Raw {
+    T k[kTokens][DP], q[kTokens][DP], v[kTokens][CB];
+    float decay[kTokens][DP];
   };
-  static_assert(sizeof(Shared) + 2 * kTokens * (2 * DP + CB) * 4 <= 216 * 1024, "the operand ring");
-  static_assert(sizeof(Shared) % 16 == 0, "raw inputs start on 16 bytes");
+  struct Shared {
+    Raw in[2];
+    float kh[DELTA ? kTokens : 1][DP], qh[kTokens][DP], kt[kTokens][DP], em[kSteps][DP];
+    float mix[kSteps][16], keys[kSteps][8], scale[kSteps][8], sums[kSteps][32], beta[2][32];
+    float u[2][CB][4];
+    GatedMemoryArgs args;                                      // read again for each chunk rather than kept in registers
+  };
+  static_assert(sizeof(Shared) <= 216 * 1024, "the operand ring");
   __builtin_assume(__isShared(ring));
   Shared& sh = *reinterpret_cast<Shared*>(ring);
-  GatedMemoryArgs A;
-  load_block(A, t.a[0]);
+  GatedMemoryArgs& A = sh.args;
+  if (tid < static_cast<int>(sizeof(GatedMemoryArgs) / 16))
+    reinterpret_cast<uint4*>(&A)[tid] = __ldcg(reinterpret_cast<const uint4*>(t.a[0]) + tid);
+  exec_sync();
   const int row0 = static_cast<int>(t.i0), rows = static_cast<int>(t.i1), slot = static_cast<int>(t.i3);
   const int head = static_cast<int>(t.i2 & 0xffffu), col0 = static_cast<int>(t.i2 >> 16) * CB;
   const int H = static_cast<int>(A.heads), d = static_cast<int>(A.d), e = static_cast<int>(A.e), kv = head / static_cast<int>(A.group);
-  const int dp = (d + 3) & ~3, ds = (d + 7) & ~7, oe = (e + 3) & ~3, n_v = min(CB, e - col0);
-  const int warp = tid >> 5, lane = tid & 31, g = lane & 3;
-  const bool f32 = A.f32 != 0, unit = A.unit != 0;
-  const int es = f32 ? 4 : 2, per16 = 16 / es;
+  const int dp = (d + 3) & ~3, oe = (e + 3) & ~3, n_v = min(CB, e - col0);
+  const int warp = tid >> 5, lane = tid & 31, l = lane & (G - 1);
+  const bool unit = A.unit != 0;
+  const float q_scale = A.q_scale;
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row0] == 0;
-  // raw inputs: [2][k rows, q rows, v rows]
-  uint8_t* const raw = ring + sizeof(Shared);
-  const int raw_k = kTokens * ds * es, raw_bytes = 2 * raw_k + kTokens * CB * es;
-
-  const int c_lo = (warp * 8 + (lane >> 2)) * C;               // this lane's first column of the block
-  float* const state = reinterpret_cast<float*>(A.state) + (static_cast<size_t>(slot) * H + head) * e * dp;
+  const int c_lo = (warp * kSide + lane / G) * C;              // this lane's first column of the block
+  float* const state = reinterpret_cast<float*>(A.state) + (static_cast<size_t>(slot) * H + head) * e * dp + static_cast<size_t>(col0 + c_lo) * dp;
   Pair S[C][I4][2];
 #pragma unroll
   for (int c = 0; c < C; ++c)
 #pragma unroll
     for (int i = 0; i < I4; ++i) {
-      const int at = 4 * (g + 4 * i);
+      const int at = 4 * (l + G * i);
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!fresh && at < dp && col0 + c_lo + c < e) v = *reinterpret_cast<const float4*>(state + static_cast<size_t>(col0 + c_lo + c) * dp + at);
+      if (!fresh && at < dp && c_lo + c < n_v) v = *reinterpret_cast<const float4*>(state + static_cast<size_t>(c) * dp + at);
       S[c][i][0] = pair(v.x, v.y);
       S[c][i][1] = pair(v.z, v.w);
     }
 
   const size_t k_at = static_cast<size_t>(kv) * d, v_at = static_cast<size_t>(head) * e + col0;
-  const bool kq16 = (d % per16) == 0 && ((A.k | A.q) & 15) == 0;
-  const bool v16 = (e % per16) == 0 && (n_v % per16) == 0 && (A.v & 15) == 0;
-  const bool d16 = (d & 3) == 0;
-  if (d & 7) {   // the padding of keys, queries and decays stays zero
-    for (int i = tid; i < 2 * raw_bytes / 16; i += kExecThreads) reinterpret_cast<uint4*>(raw)[i] = make_uint4(0, 0, 0, 0);
-    for (int i = tid; i < 2 * kTokens * DP; i += kExecThreads) (&sh.decay[0][0][0])[i] = 0.f;
-    exec_sync();
-  }
+  const bool kq16 = (d % kPer16) == 0 && ((A.k | A.q) & 15) == 0, d16 = (d & 3) == 0;
+  const bool v16 = (e % kPer16) == 0 && (n_v % kPer16) == 0 && (A.v & 15) == 0;
+  if (d < DP)   // the padding of keys, queries and decays stays zero
+    for (int i = tid; i < static_cast<int>(sizeof(sh.in) / 16); i += kExecThreads) reinterpret_cast<uint4*>(sh.in)[i] = make_uint4(0, 0, 0, 0);
+  exec_sync();
   float beta_next = 0.f;
-  auto copy_elem = [&](uint8_t* dst, unsigned long long src, size_t at) {
-    if (f32) *reinterpret_cast<float*>(dst) = reinterpret_cast<const float*>(src)[at];
-    else *reinterpret_cast<__nv_bfloat16*>(dst) = reinterpret_cast<const __nv_bfloat16*>(src)[at];
+  // Rows of n elements, nt of them: 16-byte pieces (each thread keeps its place in a row), or single elements.  Rows past nt
+  // that belong to its last step become zero.
+  auto copy_rows = [&](auto* dst, const auto* src, size_t ld, auto width, int nt, int n, bool pieces) {
+    using E = std::remove_reference_t<decltype(*dst)>;
+    constexpr int N = decltype(width)::value, per = 16 / static_cast<int>(sizeof(E)), PP = N / per;
+    constexpr int kPass = kExecThreads / PP < kTokens ? kExecThreads / PP : kTokens;
+    const int tok0 = tid / PP, p = (tid % PP) * per, end = (nt + kStep - 1) & ~(kStep - 1);
+    if (pieces && tok0 < kPass && p < n) {
+      E* to = dst + tok0 * N + p;
+      const E* from = src + tok0 * ld + p;
+#pragma unroll
+      for (int tok = 0; tok < kTokens; tok += kPass) {
+        if (tok + tok0 < nt) cp16(to + tok * N, from + tok * ld);
+        else if (tok + tok0 < end) *reinterpret_cast<uint4*>(to + tok * N) = make_uint4(0, 0, 0, 0);
+      }
+    }
+    if (!pieces) {
+#pragma unroll 1
+      for (int tok = warp; tok < end; tok += kExecThreads / 32)
+        for (int i = lane; i < n; i += 32) dst[tok * N + i] = tok < nt ? src[tok * ld + i] : static_cast<E>(0.f);
+    }
   };
+  using DPc = std::integral_constant<int, DP>;
+  using CBc = std::integral_constant<int, CB>;
   auto stage = [&](int base, int b) {
     const int nt = min(kTokens, rows - base);
-    uint8_t *const rk = raw + b * raw_bytes, *const rq = rk + raw_k, *const rv = rq + raw_k;
-    for (int tok = warp; tok < nt; tok += kExecThreads / 32) {
-      const size_t row = static_cast<size_t>(row0 + base + tok), at = row * A.ld_qkv;
-      const float* dec = f32p(A.decay) + row * A.ld_decay + static_cast<size_t>(head) * d;
-      if (kq16) {
-        for (int p = lane; p < d / per16; p += 32) {
-          cp16(rk + (tok * ds + p * per16) * es, reinterpret_cast<const uint8_t*>(A.k) + (at + k_at + p * per16) * es);
-          cp16(rq + (tok * ds + p * per16) * es, reinterpret_cast<const uint8_t*>(A.q) + (at + k_at + p * per16) * es);
-        }
-      } else {
-        for (int p = lane; p < d; p += 32) {
-          copy_elem(rk + (tok * ds + p) * es, A.k, at + k_at + p);
-          copy_elem(rq + (tok * ds + p) * es, A.q, at + k_at + p);
-        }
-      }
-      if (d16) {
-        for (int p = lane; p < d / 4; p += 32) cp16(&sh.decay[b][tok][4 * p], dec + 4 * p);
-      } else {
-        for (int p = lane; p < d; p += 32) sh.decay[b][tok][p] = dec[p];
-      }
-      if (v16) {
-        if (lane < n_v / per16) cp16(rv + (tok * CB + lane * per16) * es, reinterpret_cast<const uint8_t*>(A.v) + (at + v_at + lane * per16) * es);
-      } else {
-        for (int p = lane; p < n_v; p += 32) copy_elem(rv + (tok * CB + p) * es, A.v, at + v_at + p);
-      }
-    }
+    Raw& in = sh.in[b];
+    const size_t row = static_cast<size_t>(row0 + base), at = row * A.ld_qkv, ld = A.ld_qkv;
+    copy_rows(&in.k[0][0], reinterpret_cast<const T*>(A.k) + at + k_at, ld, DPc(), nt, d, kq16);
+    copy_rows(&in.q[0][0], reinterpret_cast<const T*>(A.q) + at + k_at, ld, DPc(), nt, d, kq16);
+    copy_rows(&in.v[0][0], reinterpret_cast<const T*>(A.v) + at + v_at, ld, CBc(), nt, n_v, v16);
+    copy_rows(&in.decay[0][0], f32p(A.decay) + row * A.ld_decay + static_cast<size_t>(head) * d, static_cast<size_t>(A.ld_decay), DPc(), nt, d, d16);
     cp_commit();
-    if (DELTA && tid < nt) beta_next = act_ld(A.beta, static_cast<size_t>(row0 + base + tid) * A.ld_beta + head, f32);
+    if (DELTA && tid < nt) beta_next = act_ld(A.beta, (row + tid) * A.ld_beta + head, F32);
   };
-  auto load4 = [&](const uint8_t* p, float (&v)[4]) {
-    if (f32) {
-      ld_vec<4>(reinterpret_cast<const float*>(p), v);
-    } else {
-      const uint2 u = *reinterpret_cast<const uint2*>(p);
-      v[0] = __uint_as_float(u.x << 16);
-      v[1] = __uint_as_float(u.x & 0xffff0000u);
-      v[2] = __uint_as_float(u.y << 16);
-      v[3] = __uint_as_float(u.y & 0xffff0000u);
-    }
+  auto load2 = [&](const T* p) -> Pair {
+    if constexpr (F32) return *reinterpret_cast<const Pair*>(p);
+    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
+    return pair(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
   };
+  // the column and the tokens whose sums this lane ends with
+  const int first = l * 4 * C / G, my_col = c_lo + first / 4, my_tok = first & 3;
+  const bool owner = (l * 4 * C) % (4 * G) == 0;   // the first of the column's lanes
+  const int col_lane = lane - l + (first / 4) * G / C;
+  const size_t ld_out = static_cast<size_t>(H) * oe;
+  float* out = reinterpret_cast<float*>(A.out) + static_cast<size_t>(row0 + my_tok) * ld_out + static_cast<size_t>(head) * oe + col0 + my_col;
+
   stage(0, 0);
   for (int base = 0, b = 0; base < rows; base += kTokens, b ^= 1) {
     const int nt = min(kTokens, rows - base);
     cp_wait<0>();
-    if (DELTA && tid < kTokens) sh.beta[tid] = tid < nt ? sigmoid32(beta_next) : 0.f;
+    if (DELTA && tid < kTokens) sh.beta[b][tid] = tid < nt ? sigmoid32(beta_next) : 0.f;
     exec_sync();
     if (base + kTokens < rows) stage(base + kTokens, b ^ 1);
-    // ---- prepare the chunk's steps: LB lanes to a step, four rows of each at a time
-    const uint8_t *const rk = raw + b * raw_bytes, *const rq = rk + raw_k, *const rv = rq + raw_k;
+    // ---- prepare the chunk's steps: LB lanes to a step, two rows of each at a time
+    const Raw& in = sh.in[b];
     const int steps = (nt + kStep - 1) / kStep;
 #pragma unroll 1
     for (int s0 = warp * (32 / LB); s0 < steps; s0 += (kExecThreads / 32) * (32 / LB)) {
-      const int s = s0 + lane / LB, l = lane & (LB - 1);
-      float sum[NV];
+      const int s = s0 + lane / LB, pl = lane & (LB - 1);
+      Pair acc[24];   // products of queries and keys (10), of keys and keys (6), squares of keys, of queries
 #pragma unroll
-      for (int i = 0; i < NV; ++i) sum[i] = 0.f;
+      for (int i = 0; i < 24; ++i) acc[i] = 0ull;
       if (s < steps) {
 #pragma unroll 1
-        for (int r = 4 * l; r < DP; r += 4 * LB) {
-          float k[4][4], q[4][4], m[4][4];                     // [token][row]
+        for (int r = 2 * pl; r < DP; r += 2 * LB) {
+          Pair k[4], q[4], m[4];                               // by token
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            const int tok = s * kStep + i;
-            if (tok < nt && r < dp) {
-              load4(rk + (tok * ds + r) * es, k[i]);
-              load4(rq + (tok * ds + r) * es, q[i]);
-              ld_vec<4>(&sh.decay[b][tok][r], m[i]);
-            } else {
-#pragma unroll
-              for (int j = 0; j < 4; ++j) k[i][j] = q[i][j] = m[i][j] = 0.f;
-            }
+            k[i] = load2(&in.k[s * kStep + i][r]);
+            q[i] = load2(&in.q[s * kStep + i][r]);
+            m[i] = *reinterpret_cast<const Pair*>(&in.decay[s * kStep + i][r]);
           }
-          float kh[4][4], qh[4][4], kt[4][4], em[4];
+          auto put = [&](float* p, Pair v) { *reinterpret_cast<Pair*>(p + r) = v; };
+          const Pair one = pair(1.f, 1.f), a1 = add_pair(m[1], one), a2 = add_pair(m[2], one), a3 = add_pair(m[3], one);
+          Pair c = add_pair(m[0], one), x = m[0];
+          if constexpr (DELTA) put(sh.kh[s * kStep], mul_pair(c, k[0]));
+          put(sh.qh[s * kStep], mul_pair(c, q[0]));
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const float a1 = 1.f + m[1][j], a2 = 1.f + m[2][j], a3 = 1.f + m[3][j], a23 = a2 * a3;
-            float c = 1.f + m[0][j], x = m[0][j];
-            kh[0][j] = c * k[0][j];
-            qh[0][j] = c * q[0][j];
-#pragma unroll
-            for (int i = 1; i < 4; ++i) {
-              x += fmaf(x, m[i][j], m[i][j]);
-              c *= 1.f + m[i][j];
-              kh[i][j] = c * k[i][j];
-              qh[i][j] = c * q[i][j];
-            }
-            em[j] = x;
-            kt[3][j] = k[3][j];
-            kt[2][j] = a3 * k[2][j];
-            kt[1][j] = a23 * k[1][j];
-            kt[0][j] = a1 * a23 * k[0][j];
-            // keys as tokens 1, 2 and 3 find them
-            const float k10 = a1 * k[0][j], k20 = a2 * k10, k21 = a2 * k[1][j];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) sum[i * (i + 1) / 2 + i] = fmaf(q[i][j], k[i][j], sum[i * (i + 1) / 2 + i]);
-            sum[1] = fmaf(q[1][j], k10, sum[1]);
-            sum[3] = fmaf(q[2][j], k20, sum[3]);
-            sum[4] = fmaf(q[2][j], k21, sum[4]);
-            sum[6] = fmaf(q[3][j], kt[0][j], sum[6]);
-            sum[7] = fmaf(q[3][j], kt[1][j], sum[7]);
-            sum[8] = fmaf(q[3][j], kt[2][j], sum[8]);
-            if constexpr (DELTA) {
-              sum[10] = fmaf(k[1][j], k10, sum[10]);
-              sum[11] = fmaf(k[2][j], k20, sum[11]);
-              sum[12] = fmaf(k[2][j], k21, sum[12]);
-              sum[13] = fmaf(k[3][j], kt[0][j], sum[13]);
-              sum[14] = fmaf(k[3][j], kt[1][j], sum[14]);
-              sum[15] = fmaf(k[3][j], kt[2][j], sum[15]);
-#pragma unroll
-              for (int i = 0; i < 4; ++i) {
-                sum[16 + i] = fmaf(k[i][j], k[i][j], sum[16 + i]);
-                sum[20 + i] = fmaf(q[i][j], q[i][j], sum[20 + i]);
-              }
-            }
+          for (int i = 1; i < 4; ++i) {
+            x = add_pair(x, fma_pair(x, m[i], m[i]));
+            c = mul_pair(c, i == 1 ? a1 : i == 2 ? a2 : a3);
+            if constexpr (DELTA) put(sh.kh[s * kStep + i], mul_pair(c, k[i]));
+            put(sh.qh[s * kStep + i], mul_pair(c, q[i]));
           }
+          put(sh.em[s], x);
+          // keys as tokens 1, 2 and 3 find them; the last are also what the step leaves to the state
+          const Pair k10 = mul_pair(a1, k[0]), k20 = mul_pair(a2, k10), k21 = mul_pair(a2, k[1]);
+          const Pair kt[4] = {mul_pair(a3, k20), mul_pair(a3, k21), mul_pair(a3, k[2]), k[3]};
+          acc[0] = fma_pair(q[0], k[0], acc[0]);
+          acc[1] = fma_pair(q[1], k10, acc[1]);
+          acc[2] = fma_pair(q[1], k[1], acc[2]);
+          acc[3] = fma_pair(q[2], k20, acc[3]);
+          acc[4] = fma_pair(q[2], k21, acc[4]);
+          acc[5] = fma_pair(q[2], k[2], acc[5]);
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            if constexpr (DELTA) st_vec<4>(&sh.kh[s * kStep + i][r], kh[i]);
-            st_vec<4>(&sh.qh[s * kStep + i][r], qh[i]);
-            st_vec<4>(&sh.kt[s * kStep + i][r], kt[i]);
+            acc[6 + i] = fma_pair(q[3], kt[i], acc[6 + i]);
+            put(sh.kt[s * kStep + i], kt[i]);
           }
-          st_vec<4>(&sh.em[s][r], em);
+          if constexpr (DELTA) {
+            acc[10] = fma_pair(k[1], k10, acc[10]);
+            acc[11] = fma_pair(k[2], k20, acc[11]);
+            acc[12] = fma_pair(k[2], k21, acc[12]);
+#pragma unroll
+            for (int i = 0; i < 3; ++i) acc[13 + i] = fma_pair(k[3], kt[i], acc[13 + i]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              acc[16 + i] = fma_pair(k[i], k[i], acc[16 + i]);
+              acc[20 + i] = fma_pair(q[i], q[i], acc[20 + i]);
+            }
+          }
         }
+      }
+      float sum[NV];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const float2 f = unpair(i < 24 ? acc[i] : 0ull);
+        sum[i] = f.x + f.y;
       }
       group_sum<NV, LB>(sum, lane);
       if (s < steps) {
-        constexpr int kMine = NV > LB ? NV / LB : 1;
 #pragma unroll
-        for (int i = 0; i < kMine; ++i) sh.sums[s][l * NV / LB + i] = sum[i];
+        for (int i = 0; i < (NV > LB ? NV / LB : 1); ++i) sh.sums[s][pl * NV / LB + i] = sum[i];
+      }
+      __syncwarp();
+      if (s < steps && pl < 8) {   // scales of the four keys, of the four queries
+        float v = 1.f;
+        if constexpr (DELTA) v = unit ? 1.f / sqrtf(sh.sums[s][16 + pl] + kUnitFloor) : 1.f;
+        sh.scale[s][pl] = pl < 4 ? v : v * q_scale;
       }
       __syncwarp();
       if (s < steps) {
-        const float* z = sh.sums[s];
-        auto key_scale = [&](int i) { return DELTA && unit ? 1.f / sqrtf(z[16 + i] + kUnitFloor) : 1.f; };
-        auto query_scale = [&](int i) { return A.q_scale * (DELTA && unit ? 1.f / sqrtf(z[20 + i] + kUnitFloor) : 1.f); };
-        for (int x = l; x < kCoefs; x += LB) {
-          float v = 0.f;
-          if (x < 16) {
-            const int i = x >> 2, j = x & 3;
-            if (j <= i) v = query_scale(i) * key_scale(j) * z[i * (i + 1) / 2 + j];
-          } else if (x < 20) {
-            v = key_scale(x - 16);
-          } else if (x < 24) {
-            v = DELTA ? sh.beta[s * kStep + x - 20] : 0.f;
-          } else if (x < 30) {
-            const int i = x == 24 ? 1 : x < 27 ? 2 : 3, j = x - 24 - i * (i - 1) / 2;
-            if (DELTA) v = key_scale(i) * key_scale(j) * z[x - 14];
-          } else if (x >= 32) {
-            v = query_scale(x - 32);
-          }
-          sh.coef[s][x] = v;
+        const float *z = sh.sums[s], *zs = sh.scale[s];
+        for (int x = pl; x < 16 + (DELTA ? 6 : 0); x += LB) {
+          const int y = x - 16;
+          const int i = x < 16 ? x >> 2 : y < 1 ? 1 : y < 3 ? 2 : 3, j = x < 16 ? x & 3 : y - below(i, 0);
+          const float v = z[x < 16 ? min(upto(i, j), 9) : 10 + y] * zs[x < 16 ? 4 + i : i] * zs[j];
+          if (x < 16) sh.mix[s][x] = j <= i ? v : 0.f;
+          else sh.keys[s][y] = v;
         }
       }
       __syncwarp();
-    }
-    for (int i = tid; i < kTokens * CB; i += kExecThreads) {
-      const int tok = i / CB, c = i % CB;
-      float v = 0.f;
-      if (tok < nt && c < n_v) v = f32 ? reinterpret_cast<const float*>(rv)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(rv)[i]);
-      sh.v[tok][c] = v;
     }
     exec_sync();
     // ---- the steps
 #pragma unroll 1
     for (int s = 0; s < steps; ++s) {
-      Pair P[DELTA ? 4 : 1][C], O[4][C];
+      float p[4 * C], o[4 * C];                                // [column][token]
+      auto reads = [&](const float* rows4, float (&to)[4 * C]) {
+        Pair acc[4][C];
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+        for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int c = 0; c < C; ++c) {
-          O[i][c] = 0ull;
-          if constexpr (DELTA) P[i][c] = 0ull;
+          for (int c = 0; c < C; ++c) acc[i][c] = 0ull;
+        Pair x[2][4][2];   // loads run one group of rows ahead, and no further: more of them in flight would spill the state
+        auto load = [&](int i4) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) ld_pairs(rows4 + i * DP + 4 * (l + G * i4), x[i4 & 1][i][0], x[i4 & 1][i][1]);
+        };
+        load(0);
+#pragma unroll
+        for (int i4 = 0; i4 < I4; ++i4) {
+          asm volatile("" ::: "memory");
+          if (i4 + 1 < I4) load(i4 + 1);
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+              for (int c = 0; c < C; ++c) acc[i][c] = fma_pair(S[c][i4][j], x[i4 & 1][i][j], acc[i][c]);
         }
 #pragma unroll
-      for (int i4 = 0; i4 < I4; ++i4) {
-        const int at = 4 * (g + 4 * i4);
+        for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          Pair a, bb;
-          ld_pairs(&sh.qh[s * kStep + i][at], a, bb);
-#pragma unroll
-          for (int c = 0; c < C; ++c) O[i][c] = fma_pair(S[c][i4][1], bb, fma_pair(S[c][i4][0], a, O[i][c]));
-          if constexpr (DELTA) {
-            ld_pairs(&sh.kh[s * kStep + i][at], a, bb);
-#pragma unroll
-            for (int c = 0; c < C; ++c) P[i][c] = fma_pair(S[c][i4][1], bb, fma_pair(S[c][i4][0], a, P[i][c]));
+          for (int c = 0; c < C; ++c) {
+            const float2 f = unpair(acc[i][c]);
+            to[c * 4 + i] = f.x + f.y;
           }
-        }
+        group_sum<4 * C, G>(to, lane);
+      };
+      // (the order of the passes is kept, so that only one has its sums in registers)
+      if constexpr (DELTA) reads(sh.kh[s * kStep], p);
+      asm volatile("" ::: "memory");
+      reads(sh.qh[s * kStep], o);
+      asm volatile("" ::: "memory");
+      float u[4], zk[4];
+      if constexpr (DELTA) ld_vec<4>(sh.scale[s], zk);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const T v = in.v[s * kStep + i][my_col];
+        if constexpr (F32) u[i] = v;
+        else u[i] = __bfloat162float(v);
       }
-      const float* z = sh.coef[s];
-      float zk[4], mix[4];
-      ld_vec<4>(z + 16, zk);
-      ld_vec<4>(z + 4 * g, mix);
-      const float zq = z[32 + g];
+      if constexpr (DELTA) {
+        float pp[4], zb[4], kk[4], kk4[2];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {   // the column's other lanes hold its other tokens
+          if constexpr (NS == 4) pp[i] = p[i];
+          else pp[i] = __shfl_sync(0xffffffffu, p[i % NS], col_lane + i * G / (4 * C));
+        }
+        ld_vec<4>(sh.beta[b] + s * kStep, zb);
+        ld_vec<4>(sh.keys[s], kk);
+        kk4[0] = sh.keys[s][4];
+        kk4[1] = sh.keys[s][5];
+        u[0] = zb[0] * (u[0] - zk[0] * pp[0]);
+        u[1] = zb[1] * (u[1] - fmaf(kk[0], u[0], zk[1] * pp[1]));
+        u[2] = zb[2] * (u[2] - fmaf(kk[2], u[1], fmaf(kk[1], u[0], zk[2] * pp[2])));
+        u[3] = zb[3] * (u[3] - fmaf(kk4[1], u[2], fmaf(kk4[0], u[1], fmaf(kk[3], u[0], zk[3] * pp[3]))));
+      }
+      if constexpr (DELTA) {
+        if (owner) *reinterpret_cast<float4*>(sh.u[s & 1][my_col]) = make_float4(zk[0] * u[0], zk[1] * u[1], zk[2] * u[2], zk[3] * u[3]);
+      } else {
+        if (owner) *reinterpret_cast<float4*>(sh.u[s & 1][my_col]) = make_float4(u[0], u[1], u[2], u[3]);
+      }
+#pragma unroll
+      for (int n = 0; n < NS; ++n) {
+        float mix[4];
+        ld_vec<4>(sh.mix[s] + 4 * (my_tok + n), mix);
+        const float y = fmaf(mix[3], u[3], fmaf(mix[2], u[2], fmaf(mix[1], u[1], fmaf(mix[0], u[0], sh.scale[s][4 + my_tok + n] * o[n]))));
+        if (s * kStep + my_tok + n < nt && my_col < n_v) out[n * ld_out] = y;
+      }
+      out += kStep * ld_out;
+      __syncwarp();
       Pair U[4][C];
 #pragma unroll
       for (int c = 0; c < C; ++c) {
-        float u[4];
+        float x[4];
+        ld_vec<4>(sh.u[s & 1][c_lo + c], x);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) u[i] = sh.v[s * kStep + i][c_lo + c];
-        if constexpr (DELTA) {
-          float p[4], zb[4], kk[6];
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            const float2 f = unpair(P[i][c]);
-            p[i] = f.x + f.y;
-          }
-#pragma unroll
-          for (int bit = 1; bit <= 2; bit <<= 1)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) p[i] += __shfl_xor_sync(0xffffffffu, p[i], bit);
-          ld_vec<4>(z + 20, zb);
-#pragma unroll
-          for (int i = 0; i < 6; ++i) kk[i] = z[24 + i];
-          u[0] = zb[0] * (u[0] - zk[0] * p[0]);
-          u[1] = zb[1] * (u[1] - fmaf(kk[0], u[0], zk[1] * p[1]));
-          u[2] = zb[2] * (u[2] - fmaf(kk[2], u[1], fmaf(kk[1], u[0], zk[2] * p[2])));
-          u[3] = zb[3] * (u[3] - fmaf(kk[5], u[2], fmaf(kk[4], u[1], fmaf(kk[3], u[0], zk[3] * p[3]))));
-        }
-        float o[4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float2 f = unpair(O[i][c]);
-          o[i] = f.x + f.y;
-        }
-        group_sum<4, 4>(o, lane);
-        const float out = fmaf(mix[3], u[3], fmaf(mix[2], u[2], fmaf(mix[1], u[1], fmaf(mix[0], u[0], zq * o[0]))));
-        const int tok = s * kStep + g;
-        if (tok < nt && c_lo + c < n_v)
-          reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row0 + base + tok) * H + head) * oe + col0 + c_lo + c] = out;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float x = zk[i] * u[i];
-          U[i][c] = pair(x, x);
-        }
+        for (int i = 0; i < 4; ++i) U[i][c] = pair(x[i], x[i]);
       }
+      Pair x[2][5][2];
+      auto load = [&](int i4) {
+        const int at = 4 * (l + G * i4);
+        ld_pairs(&sh.em[s][at], x[i4 & 1][4][0], x[i4 & 1][4][1]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ld_pairs(&sh.kt[s * kStep + i][at], x[i4 & 1][i][0], x[i4 & 1][i][1]);
+      };
+      load(0);
 #pragma unroll
       for (int i4 = 0; i4 < I4; ++i4) {
-        const int at = 4 * (g + 4 * i4);
-        Pair a, bb;
-        ld_pairs(&sh.em[s][at], a, bb);
+        asm volatile("" ::: "memory");
+        if (i4 + 1 < I4) load(i4 + 1);
 #pragma unroll
-        for (int c = 0; c < C; ++c) {
-          S[c][i4][0] = fma_pair(S[c][i4][0], a, S[c][i4][0]);
-          S[c][i4][1] = fma_pair(S[c][i4][1], bb, S[c][i4][1]);
-        }
+        for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          ld_pairs(&sh.kt[s * kStep + i][at], a, bb);
+          for (int c = 0; c < C; ++c) S[c][i4][j] = fma_pair(S[c][i4][j], x[i4 & 1][4][j], S[c][i4][j]);
 #pragma unroll
-          for (int c = 0; c < C; ++c) {
-            S[c][i4][0] = fma_pair(a, U[i][c], S[c][i4][0]);
-            S[c][i4][1] = fma_pair(bb, U[i][c], S[c][i4][1]);
-          }
-        }
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int c = 0; c < C; ++c) S[c][i4][j] = fma_pair(x[i4 & 1][i][j], U[i][c], S[c][i4][j]);
       }
     }
   }
@@ -445,10 +455,10 @@ __device__ __noinline__ void gated_rows(const TileDesc& t, int tid, uint8_t* rin
   for (int c = 0; c < C; ++c)
 #pragma unroll
     for (int i = 0; i < I4; ++i) {
-      const int at = 4 * (g + 4 * i);
-      if (at < dp && col0 + c_lo + c < e) {
+      const int at = 4 * (l + G * i);
+      if (at < dp && c_lo + c < n_v) {
         const float2 a = unpair(S[c][i][0]), b = unpair(S[c][i][1]);
-        *reinterpret_cast<float4*>(state + static_cast<size_t>(col0 + c_lo + c) * dp + at) = make_float4(a.x, a.y, b.x, b.y);
+        *reinterpret_cast<float4*>(state + static_cast<size_t>(c) * dp + at) = make_float4(a.x, a.y, b.x, b.y);
       }
     }
 }
@@ -456,22 +466,29 @@ __device__ __noinline__ void gated_rows(const TileDesc& t, int tid, uint8_t* rin
 __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring) {
   const GatedMemoryArgs* p = reinterpret_cast<const GatedMemoryArgs*>(t.a[0]);
   const uint32_t d = __ldcg(&p->d);
-  const bool delta = __ldcg(&p->beta) != 0, two = t.a[1] == 64;
-  if (t.a[1] != 32 && !two) return false;
-#define MF_GATED(N, C)                                  \
-  if (d <= 4 * N && two == (C == 2)) {                  \
-    if (delta) gated_rows<N, C, true>(t, tid, ring);    \
-    else gated_rows<N, C, false>(t, tid, ring);         \
-    return true;                                        \
+  const bool delta = __ldcg(&p->beta) != 0;
+  const bool f32 = __ldcg(&p->f32) != 0;
+  // a[1]: the columns of a block, one of two widths; 32-bit activations have the narrower one only
+#define MF_GATED(N, G, C, F32)                                                          \
+  if (d <= N && t.a[1] == 128 * C / G && f32 == F32) {                                  \
+    if (delta) gated_rows<G, (N) / (G), C, true, F32>(t, tid, ring);                    \
+    else gated_rows<G, (N) / (G), C, false, F32>(t, tid, ring);                         \
+    return true;                                                                        \
   }
-  MF_GATED(8, 1)
-  MF_GATED(8, 2)
-  MF_GATED(16, 1)
-  MF_GATED(16, 2)
-  MF_GATED(32, 1)
-  MF_GATED(32, 2)
-  MF_GATED(64, 1)
-  MF_GATED(128, 1)
+  MF_GATED(32, 4, 2, false)
+  MF_GATED(32, 4, 1, false)
+  MF_GATED(32, 4, 1, true)
+  MF_GATED(64, 8, 4, false)
+  MF_GATED(64, 8, 2, false)
+  MF_GATED(64, 8, 2, true)
+  MF_GATED(128, 8, 4, false)
+  MF_GATED(128, 8, 2, false)
+  MF_GATED(128, 8, 2, true)
+  MF_GATED(256, 16, 4, false)
+  MF_GATED(256, 16, 2, false)
+  MF_GATED(256, 16, 2, true)
+  MF_GATED(512, 32, 4, false)
+  MF_GATED(512, 32, 4, true)
 #undef MF_GATED
   return false;
 }

@@ -63,13 +63,14 @@ def decay_stage(lane, p, prev, b, x, w, m, sign, label):
     return s
 
 
-def gated_columns(requests, heads, dim, columns, workers):
-    """Columns of a portion's tile, 32 or 64: a tile of twice the columns costs about one and a half times as much."""
-    if 2 * 32 > up(columns, 32) or dim > 128:
-        return 32
+def gated_columns(requests, heads, dim, columns, workers, f32=False):
+    """Columns of a portion's tile: the narrower or the wider form, which costs about one and a half times as much."""
+    narrow = 32 if dim <= 128 else 16
+    if f32 or dim > 256 or 2 * narrow > up(columns, narrow):
+        return narrow
     portions = sum(1 for _, n, _ in requests if n > 1) * heads
-    rounds = {c: -(-portions * -(-columns // c) // workers) for c in (32, 64)}
-    return 64 if 3 * rounds[64] <= 2 * rounds[32] else 32
+    rounds = {c: -(-portions * -(-columns // c) // workers) for c in (narrow, 2 * narrow)}
+    return 2 * narrow if 3 * rounds[2 * narrow] <= 2 * rounds[narrow] else narrow
 
 
 def step_columns(dim):
@@ -81,7 +82,7 @@ def memory_stage(lane, p, prev, b, m, group, q, k, v, ld, beta, ld_beta, state, 
     mem = lane._dev("GatedMemoryArgs", q=q, k=k, v=v, beta=beta, decay=lane.decay.addr, state=state, out=lane.raw.addr,
                     tok_pos=lane.tok_pos, ld_qkv=ld, ld_beta=ld_beta, ld_decay=lane.decay.ld, heads=m.heads, group=group, d=m.dim,
                     e=m.vdim, f32=int(lane.cfg.f32), unit=unit, q_scale=q_scale)
-    width = gated_columns(b.requests, m.heads, m.dim, m.vdim, lane.fab.num_workers)
+    width = gated_columns(b.requests, m.heads, m.dim, m.vdim, lane.fab.num_workers, lane.cfg.f32)
     tiles = b.memory_tiles(m.heads, m.vdim, kinds=(K_GATED, K_GATED_STEP), width=width, step_width=step_columns(m.dim))
     s = p.stage(_retarget(tiles, a0=mem.data_ptr()), label=label)
     for stage in prev:

@@ -77,7 +77,7 @@ def test_memory_tiles_cover_rows_heads_and_columns_once(heads, dim, e):
     from monoserve_b200.layer_list import _Batch
     b = _Batch(lane(), REQUESTS, POS0)
     width, step = gated_columns(REQUESTS, heads, dim, e, 140), step_columns(dim)
-    assert width in (32, 64) and (width == 32 or dim <= 128)
+    assert width in ((32, 64) if dim <= 128 else (16, 32) if dim <= 256 else (16,))
     seen = np.zeros((107, heads, e), int)
     t = fields(b.memory_tiles(heads, e, kinds=(K_GATED, K_GATED_STEP), width=width, step_width=step))
     slot_of = {row: slot for row0, n, slot in REQUESTS for row in range(row0, row0 + n)}
@@ -97,7 +97,8 @@ def test_wide_memory_tiles_are_used_where_they_save_a_round():
     from monoserve_b200.gated_mixers import gated_columns
     assert gated_columns([(0, 75, 0)], 24, 128, 192, 140) == 64     # 144 tiles of 32 columns are two rounds, 72 of 64 are one
     assert gated_columns([(0, 75, 0)], 24, 128, 128, 140) == 32     # 96 tiles are one round either way
-    assert gated_columns([(0, 75, 0)], 24, 192, 192, 140) == 32     # too many rows for twice the columns
+    assert gated_columns([(0, 75, 0)], 24, 192, 192, 140) == 32     # more rows, half the columns: 288 tiles or 144
+    assert gated_columns([(0, 75, 0)], 24, 300, 192, 140) == 16
     assert gated_columns([(0, 75, 0)], 400, 128, 32, 140) == 32     # a head has no more
 
 
