@@ -116,7 +116,7 @@ __device__ bool make_gemm_work(const TileDesc& t, GemmWork& w, uint32_t block = 
   w.block = -1;
   w.w_fp8 = A.w_fp8 != 0;   // e4m3 weights: the exec warps expand every stage to bf16 before its MMAs
   w.fetch = 0;
-  return w.k_tiles > 0 && A.epi <= kEpiGeluMul;
+  return w.k_tiles > 0 && A.epi <= kEpiDecay;
 }
 
 // Fetch tile (kind 49): i0 bytes from a[0] (host-resident weights) to a[1] (an HBM staging buffer).

@@ -87,11 +87,79 @@ __device__ __noinline__ void qkv_items(const TileDesc& t, int tid) {
   }
 }
 
+// The same for heads that are one 16-byte piece per lane at most: four rounds of items in flight.
+__device__ __noinline__ void qkv_narrow(const TileDesc& t, int tid) {
+  constexpr int U = 4;
+  QkvArgs A;
+  load_block(A, t.a[0]);
+  const int H = static_cast<int>(A.heads), G = static_cast<int>(A.kv_heads), per = H + 2 * G;
+  const int widest = static_cast<int>(max(max(A.ld_q, A.ld_k), A.ld_v));
+  int lanes = 1;   // of an item
+  while (lanes * 8 < widest) lanes <<= 1;
+  const int at_once = kExecThreads / lanes, mine = tid / lanes, c = (tid & (lanes - 1)) * 8;
+  const uint32_t end = t.i0 + t.i1;
+  for (uint32_t it0 = t.i0 + mine; it0 - mine < end; it0 += U * at_once) {
+    uint4 raw[U];
+    __nv_bfloat16* to[U];
+    const float* w[U];
+    int n[U];
+    float ss[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t it = min(it0 + u * at_once, end - 1), row = it / per;
+      const int k = static_cast<int>(it - row * per);
+      const bool is_q = k < H, is_v = k >= H + G;
+      const int head = is_q ? k : is_v ? k - H - G : k - H;
+      n[u] = static_cast<int>(is_v ? A.e : A.d);
+      w[u] = is_v ? nullptr : f32p(is_q ? A.q_norm : A.k_norm);
+      const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(is_q ? A.q : is_v ? A.v : A.k) + static_cast<size_t>(row) * A.ld_x + static_cast<size_t>(head) * n[u];
+      raw[u] = c < n[u] ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0, 0, 0, 0);
+      const int ld = static_cast<int>(is_q ? A.ld_q : is_v ? A.ld_v : A.ld_k);
+      const size_t place = is_q ? row : static_cast<size_t>(reinterpret_cast<const int*>(A.tok_slot)[row]);
+      to[u] = it0 + u * at_once < end && c < ld
+                  ? reinterpret_cast<__nv_bfloat16*>(is_q ? A.q_out : is_v ? A.v_cache : A.k_cache) + (place * (is_q ? H : G) + head) * ld + c
+                  : nullptr;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
+      ss[u] = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        ss[u] = fmaf(f.x, f.x, fmaf(f.y, f.y, ss[u]));
+      }
+    }
+    for (int o = lanes >> 1; o; o >>= 1)
+#pragma unroll
+      for (int u = 0; u < U; ++u) ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (!to[u]) continue;
+      if (w[u] && c < n[u]) {
+        const float inv = 1.f / sqrtf(ss[u] / static_cast<float>(n[u]) + A.eps);
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw[u]);
+        float wv[8];
+        ld_vec<4>(w[u] + c, *reinterpret_cast<float(*)[4]>(wv));
+        ld_vec<4>(w[u] + c + 4, *reinterpret_cast<float(*)[4]>(wv + 4));
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 f = __bfloat1622float2(h[i]);
+          h[i] = __floats2bfloat162_rn(f.x * inv * wv[2 * i], f.y * inv * wv[2 * i + 1]);
+        }
+      }
+      *reinterpret_cast<uint4*>(to[u]) = raw[u];
+    }
+  }
+}
+
 __device__ void tile_qkv(const TileDesc& t, int tid) {
   const QkvArgs* p = reinterpret_cast<const QkvArgs*>(t.a[0]);
   const uint32_t cols = __ldcg(&p->d) | __ldcg(&p->e) | __ldcg(&p->ld_q) | __ldcg(&p->ld_k) | __ldcg(&p->ld_v) | __ldcg(&p->ld_x);
   const unsigned long long at = __ldcg(&p->q) | __ldcg(&p->k) | __ldcg(&p->v);
-  if (!__ldcg(&p->f32) && (cols & 7) == 0 && (at & 15) == 0) qkv_items<8>(t, tid);
+  const bool pieces = !__ldcg(&p->f32) && (cols & 7) == 0 && (at & 15) == 0;
+  if (pieces && max(max(__ldcg(&p->ld_q), __ldcg(&p->ld_k)), __ldcg(&p->ld_v)) <= 256) qkv_narrow(t, tid);
+  else if (pieces) qkv_items<8>(t, tid);
   else qkv_items<1>(t, tid);
 }
 

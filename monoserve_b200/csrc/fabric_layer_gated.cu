@@ -9,54 +9,14 @@ namespace mf {
 namespace fab {
 
 // ------------------------------------------------------------------ decays
-// Kind 67, DecayArgs: rows [i0, i0 + i1), at most 32, channels [i2, i2 + i3), at most 128: a thread per channel.
-__device__ void tile_decay(const TileDesc& t, int tid, int* scratch) {
-  constexpr int KC = 32, kRows = 32;
-  static_assert(kRows * KC <= kLayerScratchInts, "decay scratch");
-  float* const sx = reinterpret_cast<float*>(scratch);   // [row][KC]
+// Kind 67, DecayArgs: rows [i0, i0 + i1).
+__device__ void tile_decay(const TileDesc& t, int tid) {
   DecayArgs A;
   load_block(A, t.a[0]);
-  const int rows = static_cast<int>(t.i1), R = static_cast<int>(A.r);
-  const bool ok = tid < static_cast<int>(t.i3);
-  const int ch = static_cast<int>(t.i2) + (ok ? tid : 0);
-  const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(A.w) + static_cast<size_t>(ch) * A.ld_w;
-  float acc[kRows];
-#pragma unroll
-  for (int r = 0; r < kRows; ++r) acc[r] = 0.f;
-  for (int k0 = 0; k0 < R; k0 += KC) {
-    for (int i = tid; i < kRows * KC; i += kExecThreads) {
-      const int r = i / KC, k = k0 + i % KC;
-      sx[i] = r < rows && k < R ? act_ld(A.x, static_cast<size_t>(t.i0 + r) * A.ld_x + k, A.f32 != 0) : 0.f;
-    }
-    exec_sync();
-    // rows of w are padded with zeros to whole 64-column steps
-#pragma unroll 1
-    for (int k = 0; k < KC && k0 + k < R; k += 8) {
-      const uint4 raw = *reinterpret_cast<const uint4*>(w + k0 + k);
-      const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-      float wv[8];
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float2 f = __bfloat1622float2(h[i]);
-        wv[2 * i] = f.x;
-        wv[2 * i + 1] = f.y;
-      }
-#pragma unroll
-      for (int r = 0; r < kRows; ++r) {
-        if (r >= rows) break;
-        const float4 a = *reinterpret_cast<const float4*>(sx + r * KC + k), b = *reinterpret_cast<const float4*>(sx + r * KC + k + 4);
-        acc[r] += fmaf(a.x, wv[0], fmaf(a.y, wv[1], fmaf(a.z, wv[2], a.w * wv[3]))) +
-                  fmaf(b.x, wv[4], fmaf(b.y, wv[5], fmaf(b.z, wv[6], b.w * wv[7])));
-      }
-    }
-    exec_sync();
+  for (uint32_t r = t.i0; r < t.i0 + t.i1; ++r) {
+    float* z = reinterpret_cast<float*>(A.z) + static_cast<size_t>(r) * A.ld;
+    for (uint32_t c = tid; c < A.n; c += kExecThreads) z[c] = expm1f(-f32p(A.coef)[c] * softplus32(z[c] + f32p(A.bias)[c]));
   }
-  if (!ok) return;
-  const float bias = f32p(A.bias)[ch], coef = f32p(A.coef)[ch / static_cast<int>(A.d)];
-  float* out = reinterpret_cast<float*>(A.out) + static_cast<size_t>(t.i0) * A.ld_out + ch;
-#pragma unroll
-  for (int r = 0; r < kRows; ++r)
-    if (r < rows) out[static_cast<size_t>(r) * A.ld_out] = expm1f(-coef * softplus32(A.sign * (acc[r] + bias)));
 }
 
 // ------------------------------------------------------------------ packed fp32 pairs (each half rounded like the scalar)
@@ -494,110 +454,153 @@ __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring) {
 }
 
 // ------------------------------------------------------------------ one token
-// Kind 69, GatedMemoryArgs: row i0, i2 = head | first column block << 16, i1 column blocks, slot i3.  G lanes share a
-// column (ND four-row groups of it each); a column block is 32 (32 / G) columns.  The state streams through registers, the
-// next block's loads issued before this one's arithmetic; the read-out comes from the state in front of the token's write,
-// S^T q + (k q) u, so one round of sums per column serves both products.
-template <int G, int ND, bool DELTA>
+// Kind 69, GatedMemoryArgs: row i0, slot i3, i1 column blocks from block i2 on, counted through the heads (blocks of a head:
+// its columns over kBlock, rounded up).  G lanes share a column (ND four-row groups of it each), NC columns a lane.  The
+// state streams through registers, the next block's loads issued before this one's arithmetic; the read-out comes from the
+// state in front of the token's write, S^T q + (k q) u, so one round of sums per column serves both products.
+template <int G, int ND, int NC, bool DELTA, bool F32>
 __device__ __noinline__ void gated_step(const TileDesc& t, int tid) {
-  constexpr int kSide = 32 / G, kBlock = 32 * kSide;           // columns side by side in a warp; of a block
+  using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
+  constexpr int kSide = 32 / G, kBlock = 4 * NC * kSide;       // columns side by side in a warp; of a block
+  struct Block {
+    float4 S[NC][ND];
+    float k[ND][4], q[ND][4], m[ND][4], v, beta;
+  };
   GatedMemoryArgs A;
   load_block(A, t.a[0]);
-  const int row = static_cast<int>(t.i0), slot = static_cast<int>(t.i3), n_blocks = static_cast<int>(t.i1);
-  const int head = static_cast<int>(t.i2 & 0xffffu), block0 = static_cast<int>(t.i2 >> 16);
-  const int H = static_cast<int>(A.heads), d = static_cast<int>(A.d), e = static_cast<int>(A.e), kv = head / static_cast<int>(A.group);
+  const int row = static_cast<int>(t.i0), slot = static_cast<int>(t.i3), first = static_cast<int>(t.i2), last = first + static_cast<int>(t.i1);
+  const int H = static_cast<int>(A.heads), d = static_cast<int>(A.d), e = static_cast<int>(A.e), group = static_cast<int>(A.group);
   const int dp = (d + 3) & ~3, oe = (e + 3) & ~3, warp = tid >> 5, lane = tid & 31, l = lane & (G - 1), side = lane / G;
-  const bool f32 = A.f32 != 0, unit = A.unit != 0;
-  const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row] == 0;
-  const size_t at_row = static_cast<size_t>(row) * A.ld_qkv;
-  float* const state = reinterpret_cast<float*>(A.state) + (static_cast<size_t>(slot) * H + head) * e * dp;
-  // column c of this lane's eight is c_lo + c * kSide; after the sums the lane owns column c_lo + own * kSide
-  const int own = l * 8 / G;
-  const bool writes = G == 8 || (l & (G / 8 - 1)) == 0;
-  float4 st[2][8][ND];
-  float v1[2];
-  auto fetch = [&](int b, float4 (&S)[8][ND], float& v) {
-    const int c_lo = b * kBlock + warp * 8 * kSide + side;
+  const int blocks = (e + kBlock - 1) / kBlock;
+  const bool unit = A.unit != 0;
+  const T* const k_row = reinterpret_cast<const T*>(A.k) + static_cast<size_t>(row) * A.ld_qkv;
+  const T* const q_row = reinterpret_cast<const T*>(A.q) + static_cast<size_t>(row) * A.ld_qkv;
+  const T* const v_row = reinterpret_cast<const T*>(A.v) + static_cast<size_t>(row) * A.ld_qkv;
+  const float* const m_row = f32p(A.decay) + static_cast<size_t>(row) * A.ld_decay;
+  const bool vec = (d & 3) == 0 && ((A.k | A.q) & (4 * sizeof(T) - 1)) == 0;
+  float* const state = reinterpret_cast<float*>(A.state) + static_cast<size_t>(slot) * H * e * dp;
+  // column c of this lane's NC is c_lo + c * kSide; after the sums the lane owns column c_lo + own * kSide
+  const int own = l * NC / G;
+  const bool writes = (l * NC) % G == 0;
+  auto value = [](T v) -> float {
+    if constexpr (F32) return v;
+    else return __bfloat162float(v);
+  };
+  auto load4 = [&](const T* p, float (&v)[4]) {
+    if constexpr (F32) {
+      ld_vec<4>(p, v);
+    } else {
+      const uint2 u = *reinterpret_cast<const uint2*>(p);
+      v[0] = __uint_as_float(u.x << 16);
+      v[1] = __uint_as_float(u.x & 0xffff0000u);
+      v[2] = __uint_as_float(u.y << 16);
+      v[3] = __uint_as_float(u.y & 0xffff0000u);
+    }
+  };
+  auto fetch = [&](int b, Block& B) {
+    const int head = b / blocks, c_lo = (b - head * blocks) * kBlock + warp * NC * kSide + side, kv = head / group;
+    const float* S = state + static_cast<size_t>(head) * e * dp;
 #pragma unroll
-    for (int c = 0; c < 8; ++c)
+    for (int c = 0; c < NC; ++c)
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
         const int at = 4 * (l + G * i), col = c_lo + c * kSide;
-        S[c][i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (!fresh && at < dp && col < e) S[c][i] = __ldcs(reinterpret_cast<const float4*>(state + static_cast<size_t>(col) * dp + at));
+        B.S[c][i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (at < dp && col < e) B.S[c][i] = __ldcs(reinterpret_cast<const float4*>(S + static_cast<size_t>(col) * dp + at));
       }
-    const int col = c_lo + own * kSide;
-    v = col < e ? act_ld(A.v, at_row + static_cast<size_t>(head) * e + col, f32) : 0.f;
-  };
-  fetch(block0, st[0], v1[0]);
-  float k[ND][4], q[ND][4], m[ND][4];
-  float dots[4] = {0.f, 0.f, 0.f, 0.f};                        // k k, q q, k q
 #pragma unroll
-  for (int i = 0; i < ND; ++i)
+    for (int i = 0; i < ND; ++i) {
+      const int at = 4 * (l + G * i);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int at = 4 * (l + G * i) + j;
-      k[i][j] = at < d ? act_ld(A.k, at_row + static_cast<size_t>(kv) * d + at, f32) : 0.f;
-      q[i][j] = at < d ? act_ld(A.q, at_row + static_cast<size_t>(kv) * d + at, f32) : 0.f;
-      m[i][j] = at < d ? f32p(A.decay)[static_cast<size_t>(row) * A.ld_decay + static_cast<size_t>(head) * d + at] : 0.f;
-      dots[0] = fmaf(k[i][j], k[i][j], dots[0]);
-      dots[1] = fmaf(q[i][j], q[i][j], dots[1]);
-      dots[2] = fmaf(k[i][j], q[i][j], dots[2]);
+      for (int j = 0; j < 4; ++j) B.k[i][j] = B.q[i][j] = B.m[i][j] = 0.f;
+      if (vec) {
+        if (at < d) {
+          load4(k_row + kv * d + at, B.k[i]);
+          load4(q_row + kv * d + at, B.q[i]);
+          ld_vec<4>(m_row + head * d + at, B.m[i]);
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (at + j < d) {
+            B.k[i][j] = value(k_row[kv * d + at + j]);
+            B.q[i][j] = value(q_row[kv * d + at + j]);
+            B.m[i][j] = m_row[head * d + at + j];
+          }
+      }
     }
+    const int col = c_lo + own * kSide;
+    B.v = col < e ? value(v_row[static_cast<size_t>(head) * e + col]) : 0.f;
+    if constexpr (DELTA) B.beta = value(reinterpret_cast<const T*>(A.beta)[static_cast<size_t>(row) * A.ld_beta + head]);
+  };
+  Block blk[2];
+  fetch(first, blk[0]);
+  const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row] == 0;
+  auto run = [&](int b, Block& B) {
+    const int head = b / blocks, c_lo = (b - head * blocks) * kBlock + warp * NC * kSide + side;
+    float* const S0 = state + static_cast<size_t>(head) * e * dp;
+    float dots[3] = {0.f, 0.f, 0.f};                           // k k, q q, k q
 #pragma unroll
-  for (int bit = G / 2; bit >= 1; bit >>= 1)
+    for (int i = 0; i < ND; ++i)
 #pragma unroll
-    for (int i = 0; i < 3; ++i) dots[i] += __shfl_xor_sync(0xffffffffu, dots[i], bit);
-  const float zk = unit ? 1.f / sqrtf(dots[0] + kUnitFloor) : 1.f;
-  const float zq = A.q_scale * (unit ? 1.f / sqrtf(dots[1] + kUnitFloor) : 1.f), kq = dots[2] * zk * zq;
-  const float beta = DELTA ? sigmoid32(act_ld(A.beta, static_cast<size_t>(row) * A.ld_beta + head, f32)) : 0.f;
-  auto run = [&](int b, float4 (&S)[8][ND], float v) {
-    const int c_lo = b * kBlock + warp * 8 * kSide + side;
-    float o[8], p[8];
+      for (int j = 0; j < 4; ++j) {
+        dots[0] = fmaf(B.k[i][j], B.k[i][j], dots[0]);
+        dots[1] = fmaf(B.q[i][j], B.q[i][j], dots[1]);
+        dots[2] = fmaf(B.k[i][j], B.q[i][j], dots[2]);
+      }
 #pragma unroll
-    for (int c = 0; c < 8; ++c) {
+    for (int bit = G / 2; bit >= 1; bit >>= 1)
+#pragma unroll
+      for (int i = 0; i < 3; ++i) dots[i] += __shfl_xor_sync(0xffffffffu, dots[i], bit);
+    const float zk = unit ? 1.f / sqrtf(dots[0] + kUnitFloor) : 1.f;
+    const float zq = A.q_scale * (unit ? 1.f / sqrtf(dots[1] + kUnitFloor) : 1.f), kq = dots[2] * zk * zq;
+    float o[NC], p[NC];
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
       o[c] = p[c] = 0.f;
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
-        float4& s = S[c][i];
-        s.x = fmaf(s.x, m[i][0], s.x);
-        s.y = fmaf(s.y, m[i][1], s.y);
-        s.z = fmaf(s.z, m[i][2], s.z);
-        s.w = fmaf(s.w, m[i][3], s.w);
-        o[c] = fmaf(s.x, q[i][0], fmaf(s.y, q[i][1], fmaf(s.z, q[i][2], fmaf(s.w, q[i][3], o[c]))));
-        if constexpr (DELTA) p[c] = fmaf(s.x, k[i][0], fmaf(s.y, k[i][1], fmaf(s.z, k[i][2], fmaf(s.w, k[i][3], p[c]))));
+        float4& s = B.S[c][i];
+        if (fresh) s = make_float4(0.f, 0.f, 0.f, 0.f);
+        s.x = fmaf(s.x, B.m[i][0], s.x);
+        s.y = fmaf(s.y, B.m[i][1], s.y);
+        s.z = fmaf(s.z, B.m[i][2], s.z);
+        s.w = fmaf(s.w, B.m[i][3], s.w);
+        o[c] = fmaf(s.x, B.q[i][0], fmaf(s.y, B.q[i][1], fmaf(s.z, B.q[i][2], fmaf(s.w, B.q[i][3], o[c]))));
+        if constexpr (DELTA) p[c] = fmaf(s.x, B.k[i][0], fmaf(s.y, B.k[i][1], fmaf(s.z, B.k[i][2], fmaf(s.w, B.k[i][3], p[c]))));
       }
     }
-    group_sum<8, G>(o, lane);
-    float u = v;
+    group_sum<NC, G>(o, lane);
+    float u = B.v;
     if constexpr (DELTA) {
-      group_sum<8, G>(p, lane);
-      u = beta * (v - zk * p[0]);
+      group_sum<NC, G>(p, lane);
+      u = sigmoid32(B.beta) * (B.v - zk * p[0]);
     }
     const int mine = c_lo + own * kSide;
     if (writes && mine < e) reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row) * H + head) * oe + mine] = fmaf(kq, u, zq * o[0]);
 #pragma unroll
-    for (int c = 0; c < 8; ++c) {
-      const float x = zk * __shfl_sync(0xffffffffu, u, side * G + c * G / 8);
+    for (int c = 0; c < NC; ++c) {
+      const float x = zk * __shfl_sync(0xffffffffu, u, side * G + c * G / NC);
       const int col = c_lo + c * kSide;
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
-        float4 s = S[c][i];
-        s.x = fmaf(k[i][0], x, s.x);
-        s.y = fmaf(k[i][1], x, s.y);
-        s.z = fmaf(k[i][2], x, s.z);
-        s.w = fmaf(k[i][3], x, s.w);
+        float4 s = B.S[c][i];
+        s.x = fmaf(B.k[i][0], x, s.x);
+        s.y = fmaf(B.k[i][1], x, s.y);
+        s.z = fmaf(B.k[i][2], x, s.z);
+        s.w = fmaf(B.k[i][3], x, s.w);
         const int at = 4 * (l + G * i);
-        if (at < dp && col < e) __stcs(reinterpret_cast<float4*>(state + static_cast<size_t>(col) * dp + at), s);
+        if (at < dp && col < e) __stcs(reinterpret_cast<float4*>(S0 + static_cast<size_t>(col) * dp + at), s);
       }
     }
   };
-  for (int b = block0; b < block0 + n_blocks; b += 2) {
-    if (b + 1 < block0 + n_blocks) fetch(b + 1, st[1], v1[1]);
-    run(b, st[0], v1[0]);
-    if (b + 1 < block0 + n_blocks) {
-      if (b + 2 < block0 + n_blocks) fetch(b + 2, st[0], v1[0]);
-      run(b + 1, st[1], v1[1]);
+#pragma unroll 1
+  for (int b = first; b < last; b += 2) {
+    if (b + 1 < last) fetch(b + 1, blk[1]);
+    run(b, blk[0]);
+    if (b + 1 < last) {
+      if (b + 2 < last) fetch(b + 2, blk[0]);
+      run(b + 1, blk[1]);
     }
   }
 }
@@ -605,18 +608,20 @@ __device__ __noinline__ void gated_step(const TileDesc& t, int tid) {
 __device__ bool tile_gated_step(const TileDesc& t, int tid) {
   const GatedMemoryArgs* p = reinterpret_cast<const GatedMemoryArgs*>(t.a[0]);
   const uint32_t d = __ldcg(&p->d);
-  const bool delta = __ldcg(&p->beta) != 0;
-#define MF_STEP(N, G, ND)                           \
-  if (d <= N) {                                     \
-    if (delta) gated_step<G, ND, true>(t, tid);     \
-    else gated_step<G, ND, false>(t, tid);          \
-    return true;                                    \
+  const bool delta = __ldcg(&p->beta) != 0, f32 = __ldcg(&p->f32) != 0;
+#define MF_STEP(N, G, ND, NC)                                 \
+  if (d <= N) {                                               \
+    if (delta && f32) gated_step<G, ND, NC, true, true>(t, tid);   \
+    else if (delta) gated_step<G, ND, NC, true, false>(t, tid);    \
+    else if (f32) gated_step<G, ND, NC, false, true>(t, tid);      \
+    else gated_step<G, ND, NC, false, false>(t, tid);              \
+    return true;                                              \
   }
-  MF_STEP(32, 8, 1)
-  MF_STEP(64, 16, 1)
-  MF_STEP(128, 32, 1)
-  MF_STEP(256, 32, 2)
-  MF_STEP(512, 32, 4)
+  MF_STEP(32, 8, 1, 8)
+  MF_STEP(64, 16, 1, 16)
+  MF_STEP(128, 32, 1, 16)
+  MF_STEP(256, 32, 2, 8)
+  MF_STEP(512, 32, 4, 4)
 #undef MF_STEP
   return false;
 }

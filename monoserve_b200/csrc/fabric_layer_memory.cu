@@ -461,9 +461,66 @@ __device__ __noinline__ void head_norm_items(const TileDesc& t, int tid) {
   }
 }
 
+// Heads of at most 128 columns, bf16: four items of a warp in flight.
+__device__ __noinline__ void head_norm_narrow(const TileDesc& t, int tid) {
+  constexpr int U = 4;
+  HeadNormArgs A;
+  load_block(A, t.a[0]);
+  const int warp = tid >> 5, lane = tid & 31, e = static_cast<int>(A.e), oe = (e + (A.divide ? 4 : 3)) & ~3, c = lane * 4;
+  const bool in = c < e;
+  const uint32_t end = t.i0 + t.i1;
+  for (uint32_t it0 = t.i0 + warp * U; it0 < end; it0 += U * (kExecThreads / 32)) {
+    float v[U][4], w[U][4], den[U], ss[U];
+    uint2 g[U];
+    size_t to[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t it = min(it0 + u, end - 1), row = it / A.heads, head = it - row * A.heads;
+      const float* o = f32p(A.o) + static_cast<size_t>(it) * oe;
+      to[u] = static_cast<size_t>(row) * A.ld_out + head * e + c;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[u][j] = 0.f;
+      if (in) {
+        ld_vec<4>(o + c, v[u]);
+        ld_vec<4>(f32p(A.w) + head * A.w_head + c, w[u]);
+        g[u] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(A.g) + static_cast<size_t>(row) * A.ld_g + head * e + c);
+      }
+      den[u] = A.divide ? o[e] : 1.f;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const float inv_den = 1.f / den[u];
+      ss[u] = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        v[u][j] *= inv_den;
+        ss[u] = fmaf(v[u][j], v[u][j], ss[u]);
+      }
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1)
+#pragma unroll
+      for (int u = 0; u < U; ++u) ss[u] += __shfl_xor_sync(0xffffffffu, ss[u], o);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (!in || it0 + u >= end) continue;
+      const float inv = 1.f / sqrtf(ss[u] / static_cast<float>(e) + A.eps);
+      const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g[u].x));
+      const float2 gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g[u].y));
+      const float gate[4] = {ga.x, ga.y, gb.x, gb.y};
+      float x[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[j] = v[u][j] * inv * w[u][j] * __fdividef(A.silu ? gate[j] : 1.f, 1.f + __expf(-gate[j]));
+      const __nv_bfloat162 q[2] = {__floats2bfloat162_rn(x[0], x[1]), __floats2bfloat162_rn(x[2], x[3])};
+      *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(A.out) + to[u]) = *reinterpret_cast<const uint2*>(q);
+    }
+  }
+}
+
 __device__ void tile_head_norm(const TileDesc& t, int tid) {
   const HeadNormArgs* p = reinterpret_cast<const HeadNormArgs*>(t.a[0]);
-  if ((__ldcg(&p->e) & 3) == 0 && (__ldcg(&p->g) & 7) == 0) head_norm_items<4>(t, tid);
+  if (!__ldcg(&p->f32) && __ldcg(&p->e) <= 128 && (__ldcg(&p->e) & 3) == 0 && (__ldcg(&p->g) & 7) == 0) head_norm_narrow(t, tid);
+  else if ((__ldcg(&p->e) & 3) == 0 && (__ldcg(&p->g) & 7) == 0) head_norm_items<4>(t, tid);
   else head_norm_items<1>(t, tid);
 }
 

@@ -307,7 +307,7 @@ __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx) 
     case kTileLatentMerge: tile_latent_merge(t, tid); return true;
     case kTileSumSlabs: tile_sum_slabs(t, tid); return true;
     case kTileResidual: tile_residual(t, tid, scratch); return true;
-    case kTileDecay: tile_decay(t, tid, scratch); return true;
+    case kTileDecay: tile_decay(t, tid); return true;
     case kTileGatedMemory: return tile_gated_memory(t, tid, ctx.ring);
     case kTileGatedStep: return tile_gated_step(t, tid);
     case kTileQkv: tile_qkv(t, tid); return true;

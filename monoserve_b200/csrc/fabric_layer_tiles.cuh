@@ -60,7 +60,7 @@ __device__ bool tile_latent_mma(const TileDesc& t, int tid, const LayerCtx& ctx)
 __device__ bool tile_latent_direct(const TileDesc& t, int tid, const LayerCtx& ctx);
 __device__ void tile_latent_merge(const TileDesc& t, int tid);
 __device__ void tile_residual(const TileDesc& t, int tid, int* scratch);
-__device__ void tile_decay(const TileDesc& t, int tid, int* scratch);
+__device__ void tile_decay(const TileDesc& t, int tid);
 __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring);
 __device__ bool tile_gated_step(const TileDesc& t, int tid);
 __device__ void tile_qkv(const TileDesc& t, int tid);

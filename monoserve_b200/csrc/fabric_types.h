@@ -63,7 +63,7 @@ enum TileKind : uint16_t {
   kTileLatentDirect = 64,   // the same for a whole prompt, with keys and values mapped out of the latents
   kTileScanStep = 65,       // selective scan, one token
   kTileResidual = 66,       // normed sublayer output into the plain residual, next sublayer's input and its norm
-  kTileDecay = 67,          // decays of a gated memory from their low-rank projection
+  kTileDecay = 67,          // decays of a gated memory from their projection, 32-bit form
   kTileGatedMemory = 68,    // gated linear attention / gated delta rule over a request's rows
   kTileGatedStep = 69,      // the same, one token
   kTileQkv = 70,            // query / key norms and K / V append of grouped-query attention

@@ -46,6 +46,7 @@ constexpr int kEpiStoreF32 = 3;    // out32[m][n] = acc (+ bias[n])
 constexpr int kEpiAtomicF32 = 4;   // out32[m][n] += acc : K-split partial sums
 constexpr int kEpiRowsF32 = 5;     // out32[m][n] = acc : per-pair rows for the deterministic combine (not in the reference)
 constexpr int kEpiGeluMul = 6;     // as kEpiSiluMul with the tanh form of gelu on the gate (not in the reference)
+constexpr int kEpiDecay = 7;       // out32[m][n] = expm1(-coef[n] softplus(acc + bias[n])), coef in pair_weight (not in the reference)
 // A tile of 64 gate and 64 up rows whose epilogue multiplies act(gate) by up.
 __host__ __device__ __forceinline__ bool epi_gated(int epi) { return epi == kEpiSiluMul || epi == kEpiGeluMul; }
 
@@ -391,6 +392,16 @@ __device__ __forceinline__ float gelu_mul(float g, float u) {
   return __fdividef(g, 1.f + __expf(-t2)) * u;
 }
 
+// expm1(-coef softplus(z)), coef >= 0, to a few units of 2^-24: the distance to one of a decay e^(-coef softplus(z)).  Power
+// series where the sums 1 + t and e^x - 1 would cancel.
+__device__ __forceinline__ float decay_less_one(float z, float coef) {
+  const float t = __expf(-fabsf(z));
+  const float log1p_t = t < 0.02f ? t * fmaf(t, fmaf(t, fmaf(t, -0.25f, 1.f / 3.f), -0.5f), 1.f) : __logf(1.f + t);
+  const float x = -coef * (fmaxf(z, 0.f) + log1p_t);
+  const float series = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+  return x > -0.25f ? series : __expf(x) - 1.f;
+}
+
 // Epilogue of one tile from accumulator buffer `buf` (the four epilogue warps
 // call): everything except handing the buffer back to the MMA warp.
 template <bool kFetch = true>
@@ -489,6 +500,14 @@ __device__ __forceinline__ bool gemm_epilogue_body(const GemmWork& w, GemmBarrie
 #pragma unroll
         for (int j = 0; j < 32; ++j)
           if (c0 + j < w.rows) atomicAdd(out + static_cast<size_t>(j) * w.ld_out, __uint_as_float(r[j]) * sc + bias);
+      }
+    } else if (w.epi == kEpiDecay) {
+      float* out = reinterpret_cast<float*>(w.out) + static_cast<size_t>(w.b_row0 + c0) * w.ld_out + f;
+      if (f_ok) {
+        const float coef = w.pair_weight[f];
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+          if (c0 + j < w.rows) out[static_cast<size_t>(j) * w.ld_out] = decay_less_one(__uint_as_float(r[j]) * sc + bias, coef);
       }
     } else {
       // fp32 rows that are read once, later (per-pair expert outputs, logits): streaming stores

@@ -158,10 +158,9 @@ namespace mf {
   U64(pos) U64(tokens) U64(tok_pos) U64(step) U64(sum_out) U32(W) U32(ld_h16) U32(ld_h32) U32(ld_out) U32(y0_parts) \
   U32(y1_parts) U32(y_rows) U32(max_pos) F32(eps) F32(embed_scale) F32(branch_scale)
 
-/* out fp32 [rows][ld_out] = expm1(-coef[channel / d] * softplus(sign * (x w^T + bias))) for n channels: one minus the
- * decay of a gated memory, negated.  x: r activations per row, w bf16 [n][ld_w]. */
-#define MF_DECAY_ARGS(U64, U32, F32) \
-  U64(x) U64(w) U64(bias) U64(coef) U64(out) U32(ld_x) U32(ld_w) U32(ld_out) U32(r) U32(n) U32(d) U32(f32) F32(sign)
+/* z fp32 [rows][ld] in place: expm1(-coef[channel] * softplus(z + bias[channel])) for n channels, the distance to one of a
+ * gated memory's decays; bias, coef fp32 [n].  (bf16 models have it as the projection's epilogue.) */
+#define MF_DECAY_ARGS(U64, U32, F32) U64(z) U64(bias) U64(coef) U32(ld) U32(n)
 
 /* Gated memory: per head S <- diag(1 + decay) S + k u^T, o = S^T q, state fp32 [slot][head][e][d padded to 4].
  * beta = 0: u = v; else the delta rule u = sigmoid(beta) (v - S^T k) on the decayed S.  unit: keys and queries are
@@ -224,7 +223,7 @@ MF_DECLARE(LatentArgs, MF_LATENT_ARGS, 128)
 MF_DECLARE(LatentAttnArgs, MF_LATENT_ATTN_ARGS, 128)
 MF_DECLARE(LatentDirectArgs, MF_LATENT_DIRECT_ARGS, 128)
 MF_DECLARE(ResidualArgs, MF_RESIDUAL_ARGS, 192)
-MF_DECLARE(DecayArgs, MF_DECAY_ARGS, 128)
+MF_DECLARE(DecayArgs, MF_DECAY_ARGS, 64)
 MF_DECLARE(GatedMemoryArgs, MF_GATED_MEMORY_ARGS, 128)
 MF_DECLARE(QkvArgs, MF_QKV_ARGS, 128)
 MF_DECLARE(GroupedAttnArgs, MF_GROUPED_ATTN_ARGS, 128)

@@ -13,14 +13,13 @@ import torch
 from monoserve_b200 import _C
 from monoserve_b200.attention import fabric_maps, fabric_tiles, plan_items
 from monoserve_b200.fabric import tile_array
-from monoserve_b200.lane_base import _block, _retarget, up
+from monoserve_b200.lane_base import EPI_DECAY, _block, _retarget, up
 
 K_CONV, K_HEAD_NORM = 54, 58
 K_DECAY, K_GATED, K_GATED_STEP, K_QKV, K_GROUPED_ATTN, K_HEAD_GATE = 67, 68, 69, 70, 71, 72
 K_ATTN_PREFILL, K_ATTN_PLAN = 33, 44
 MAX_GATED_DIM, MAX_CONV_TAPS, MAX_HEAD_COLUMNS = 512, 8, 512
 PAD_HEAD, MAX_PLAN_ROWS, MAX_CHUNKS = 128, 256, 8   # of the paged attention tiles: head width, decode rows, key ranges of a row
-DECAY_ROWS, DECAY_CHANNELS = 32, 128                # of one tile
 QKV_ITEMS = 64
 
 
@@ -47,20 +46,24 @@ def gated_state(m, slots):
     return torch.zeros(slots, m.heads, m.vdim, up(m.dim, 4), device="cuda")
 
 
-def decay_stage(lane, p, prev, b, x, w, m, sign, label):
-    """expm1 of the log decays of every head and key channel from their low-rank activations x [rows][w.rank]."""
+def decay_stage(lane, p, prev, b, x, w, m, label):
+    """expm1 of the log decays of every head and key channel, -coef softplus(x a2^T + bias), from their low-rank activations
+    x [rows][w.rank]: the epilogue of the product, or in 32-bit a tile behind it."""
     n = m.heads * m.dim
-    args = lane._dev("DecayArgs", x=x.addr, w=w.a2, bias=w.a_bias, coef=w.coef, out=lane.decay.addr, ld_x=x.ld, ld_w=w.a2.shape[1],
-                     ld_out=lane.decay.ld, r=w.rank, n=n, d=m.dim, f32=int(lane.cfg.f32), sign=sign)
+    if not lane.cfg.f32:
+        return lane.product(p, prev, x, w.a2, lane.decay, b.T, n, w.rank, label, epi=EPI_DECAY, bias=w.a_bias, coef=w.coef)
+    s = lane.product(p, prev, x, w.a2, lane.decay, b.T, n, w.rank, label)
+    args = lane._dev("DecayArgs", z=lane.decay.addr, bias=w.a_bias, coef=w.coef, ld=lane.decay.ld, n=n)
+    s_d = p.stage(lane._rows(K_DECAY, args, b.T, lane._per(b.T)), label=label)
+    p.after(s, s_d)
+    return s_d
 
-    def make():
-        rows = np.concatenate([np.arange(row0, row0 + k, DECAY_ROWS) for row0, k in b.spans()])
-        count = np.concatenate([np.minimum(DECAY_ROWS, k - np.arange(0, k, DECAY_ROWS)) for _, k in b.spans()])
-        c = np.arange(0, n, DECAY_CHANNELS)[None]
-        return tile_array(K_DECAY, i0=rows[:, None], i1=count[:, None], i2=c, i3=np.minimum(DECAY_CHANNELS, n - c))
-    s = p.stage(_retarget(b._once(("decay", n), make), a0=args.data_ptr()), label=label)
-    p.after(prev, s)
-    return s
+
+def place_decay(W, a2, bias, coef, dim):
+    """a2 [heads * dim, rank] and bias as the decay stage takes them (the bias in fp32 for its tile, else the checkpoint's
+    bf16 as a GEMM's), the heads' coefficients once per channel."""
+    return types.SimpleNamespace(a2=W.mat(a2), a_bias=W.f32(bias) if W.cfg.f32 else bias.to(torch.bfloat16).contiguous().cuda(),
+                                 coef=coef.float().repeat_interleave(dim).contiguous().cuda(), rank=a2.shape[1])
 
 
 def gated_columns(requests, heads, dim, columns, workers, f32=False):
@@ -74,16 +77,34 @@ def gated_columns(requests, heads, dim, columns, workers, f32=False):
 
 
 def step_columns(dim):
-    """Columns of one block of the one-token tile: 8, 16 or 32 lanes hold a column of up to 32, 64 or more rows."""
-    return 32 * (4 if dim <= 32 else 2 if dim <= 64 else 1)
+    """Columns of one block of the one-token tile: its four warps hold 128 columns of up to 64 rows, 64 of up to 128, ..."""
+    return next(c for rows, c in ((64, 128), (128, 64), (256, 32), (512, 16)) if dim <= rows)
+
+
+def gated_tiles(b, heads, dim, e, workers, f32):
+    """Portions: a tile per head and block of columns, the longest first; single tokens: each row's column blocks, counted
+    through its heads, in as many tiles as leave no worker two."""
+    def make():
+        width = gated_columns(b.requests, heads, dim, e, workers, f32)
+        h, c = np.meshgrid(np.arange(heads), np.arange(-(-e // width)), indexing="ij")
+        out = [tile_array(K_GATED, i0=row0, i1=n, i2=h | (c << 16), i3=slot, a1=width)
+               for row0, n, slot in sorted(b.requests, key=lambda q: -q[1]) if n > 1]
+        ones = [(row0, slot) for row0, n, slot in b.requests if n == 1]
+        if ones:
+            row, slot = (np.array(v)[:, None] for v in zip(*ones))
+            blocks = heads * -(-e // step_columns(dim))
+            per = -(-blocks // min(blocks, max(1, workers // len(ones))))
+            first = np.arange(0, blocks, per)[None]
+            out.append(tile_array(K_GATED_STEP, i0=row, i1=np.minimum(per, blocks - first), i2=first, i3=slot))
+        return np.concatenate(out)
+    return b._once(("gated", heads, dim, e), make)
 
 
 def memory_stage(lane, p, prev, b, m, group, q, k, v, ld, beta, ld_beta, state, unit, q_scale, label):
     mem = lane._dev("GatedMemoryArgs", q=q, k=k, v=v, beta=beta, decay=lane.decay.addr, state=state, out=lane.raw.addr,
                     tok_pos=lane.tok_pos, ld_qkv=ld, ld_beta=ld_beta, ld_decay=lane.decay.ld, heads=m.heads, group=group, d=m.dim,
                     e=m.vdim, f32=int(lane.cfg.f32), unit=unit, q_scale=q_scale)
-    width = gated_columns(b.requests, m.heads, m.dim, m.vdim, lane.fab.num_workers, lane.cfg.f32)
-    tiles = b.memory_tiles(m.heads, m.vdim, kinds=(K_GATED, K_GATED_STEP), width=width, step_width=step_columns(m.dim))
+    tiles = gated_tiles(b, m.heads, m.dim, m.vdim, lane.fab.num_workers, lane.cfg.f32)
     s = p.stage(_retarget(tiles, a0=mem.data_ptr()), label=label)
     for stage in prev:
         p.after(stage, s)
@@ -111,8 +132,8 @@ class GatedLinear:
     def place(W, w, m, g):
         w.stack = Stack([(n, g(n)) for n in ("q", "k", "v", "g", "a1")])
         w.in_, w.o, w.norm = W.mat(w.stack.rows), W.mat(g("o")), W.f32(g("norm"))
-        w.a2, w.a_bias, w.rank = W.mat(g("a2")), W.f32(g("a2.b")), g("a1").shape[0]
-        w.coef = torch.full((m.heads,), 1.0 / m.tau, device="cuda")
+        # log of sigmoid(z)^(1 / tau) = -softplus(-z) / tau
+        w.decay = place_decay(W, -g("a2"), -g("a2.b"), torch.full((m.heads,), 1.0 / m.tau), m.dim)
 
     @staticmethod
     def state(cfg, m, rows, slots, page):
@@ -124,15 +145,15 @@ class GatedLinear:
 
     @staticmethod
     def prepare(lane, layer, w, run_state):
-        lane.weight_map(w.in_), lane.mix.maps(layer.m.heads * layer.m.vdim)
+        lane.weight_map(w.in_), lane.weight_map(w.o), lane.weight_map(w.decay.a2)
+        lane.mix.maps(layer.m.heads * layer.m.vdim), lane.proj.view(w.stack.at["a1"]).maps(w.decay.rank)
 
     @staticmethod
     def build(lane, p, l, run, b, prev):
         m, w, T = lane.cfg.layers[l].m, lane.w.layers[l], b.T
         s = lane.product(p, prev, lane.h, w.in_, lane.proj, T, w.stack.n, lane.cfg.hidden, ("gla_in", run), out16=True)
         at = {name: lane.proj.view(col) for name, col in w.stack.at.items()}
-        # log of sigmoid(z)^(1 / tau) = -softplus(-z) / tau
-        s_a = decay_stage(lane, p, s, b, at["a1"], w, m, -1.0, ("gla_decay", run))
+        s_a = decay_stage(lane, p, s, b, at["a1"], w.decay, m, ("gla_decay", run))
         s_m = memory_stage(lane, p, [s_a], b, m, 1, at["q"].addr, at["k"].addr, at["v"].addr, lane.proj.ld, 0, 0,
                            lane.kv.runs[run]["S"], 0, m.dim ** -0.5, ("gla", run))
         s_n = head_norm_stage(lane, p, [s_m], T, m, at["g"], w.norm, 1, ("gla_norm", run))
@@ -292,8 +313,8 @@ class GatedDelta:
         g_ = lambda n: g("right." + n)  # noqa: E731
         return types.SimpleNamespace(
             o=W.mat(g_("o")), norm=W.f32(g_("norm")), out=W.f32(g_("out")), conv=W.f32(torch.cat([g_(f"{n}.conv") for n in "qkv"])),
-            a2=W.mat(g_("a2")), a_bias=W.f32(g_("dt_bias")), coef=W.f32(torch.exp(g_("A_log").float())), rank=g_("a1").shape[0],
-            g2=W.mat(g_("g2")), gate_rank=g_("g1").shape[0])
+            decay=place_decay(W, g_("a2"), g_("dt_bias"), torch.exp(g_("A_log").float()), m.dim), g2=W.mat(g_("g2")),
+            gate_rank=g_("g1").shape[0])
 
     @staticmethod
     def state(m, slots):
@@ -306,8 +327,10 @@ class GatedDelta:
 
     @staticmethod
     def prepare(lane, m, w, at):
-        lane.weight_map(w.g2), lane.weight_map(w.o)
+        for t in (w.g2, w.o, w.decay.a2):
+            lane.weight_map(t)
         lane.mix.maps(m.heads * m.vdim), lane.proj.view(at["right.g1"]).maps(w.gate_rank)
+        lane.proj.view(at["right.a1"]).maps(w.decay.rank)
 
     @staticmethod
     def build(lane, p, m, w, st, at, run, b, prev):
@@ -316,7 +339,7 @@ class GatedDelta:
                          ld_x=lane.proj.ld, ld_out=lane.act.ld, channels=GatedDelta.channels(m), taps=m.conv, f32=f32, advance=1)
         s_c = p.stage(_retarget(b.conv_tiles(GatedDelta.channels(m)), a0=conv.data_ptr()), label=("delta_conv", run))
         p.after(prev, s_c)
-        s_a = decay_stage(lane, p, prev, b, at["right.a1"], w, m, 1.0, ("delta_decay", run))
+        s_a = decay_stage(lane, p, prev, b, at["right.a1"], w.decay, m, ("delta_decay", run))
         s_g = lane.product(p, prev, at["right.g1"], w.g2, lane.gate, T, m.heads * m.vdim, w.gate_rank, ("delta_gate", run), out16=True)
         s_m = memory_stage(lane, p, [s_c, s_a], b, m, m.heads // m.kv_heads, lane.act.addr, lane.act.view(kd).addr,
                            lane.act.view(2 * kd).addr, lane.act.ld, at["right.b"].addr, lane.proj.ld, st["S"], 1, m.dim ** -0.5,

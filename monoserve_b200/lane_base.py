@@ -12,7 +12,7 @@ from monoserve_b200.fabric.args import pack
 
 K_GEMM, K_SAMPLE = 32, 43
 SPLIT_ROWS, SPLIT_PARTS = 64, 8   # a dense GEMM of at most SPLIT_ROWS rows may run as up to SPLIT_PARTS K ranges
-EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_ROWS_F32, EPI_GELU_MUL = 0, 1, 3, 5, 6
+EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_ROWS_F32, EPI_GELU_MUL, EPI_DECAY = 0, 1, 3, 5, 6, 7
 GATED = (EPI_SILU_MUL, EPI_GELU_MUL)
 HEIGHTS = [16, 32, 64, 128, 256]
 
@@ -247,16 +247,17 @@ class LaneBase:
         return p.stage(tiles, mark=mark, label=label)
 
     def _gemm(self, p, wmap, amaps, rows, n_out, k, out, ld_out, epi, label, residual=None, ld_res=0, mark=None,
-              mat=None, bias=None, up_offset=0, bm=None):
+              mat=None, bias=None, up_offset=0, bm=None, coef=None):
         """A dense GEMM stage: out[rows][n_out] = act[rows][k] x weight[n_out (x2 for SiLU-mul)][k]^T.
         mat: the weight's Mat (e4m3 weights carry their scales into the tiles); bm: the row-block height, when not the
-        largest."""
+        largest; coef: fp32 per output of the decay epilogue."""
         bm = bm or _bm(rows)
         fp8 = mat is not None and mat.fp8
         args = self.arena.put(_C.gemm_args(
             out=out.data_ptr(), ld_out=ld_out, k_tiles=-(-k // 64), epi=epi, bm=bm, n_limit=n_out,
             residual=residual.data_ptr() if residual is not None else 0, ld_res=ld_res,
-            bias=bias.data_ptr() if bias is not None else 0, up_offset=up_offset, w_fp8=int(fp8)))
+            bias=bias.data_ptr() if bias is not None else 0, up_offset=up_offset, w_fp8=int(fp8),
+            pair_weight=coef.data_ptr() if coef is not None else 0))
         xm = amaps[HEIGHTS.index(bm)]
         step = 64 if epi in GATED else 128
         key = ("gemm", rows, bm, n_out, step)

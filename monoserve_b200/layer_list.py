@@ -14,9 +14,9 @@ sublayer).
     latent attention:  q + latent GEMM -> latent norm, rotation, cache append (59) -> per head W_uk^T q GEMM ->
                        attention over the cached latents (63 on the tensor cores, 60 in 32-bit; 61) -> per head W_uv
                        GEMM -> o GEMM; for a whole prompt: keys and values GEMM -> attention (64) -> o GEMM
-    gated linear:      q k v g and decay GEMM -> decays (67) -> gated memory (68; one token: 69) -> head norm (58) -> o GEMM
+    gated linear:      q k v g and low-rank decay GEMM -> decay GEMM with the decay epilogue -> gated memory (68; one token: 69) -> head norm (58) -> o GEMM
     parallel:          one GEMM for both sides; left: norms and append (70) -> paged attention (33 - 35, 44; 71 in 32-bit) ->
-                       head gate (72) -> o GEMM; right: conv (54), decays (67) and gate GEMM -> gated memory (68, 69) ->
+                       head gate (72) -> o GEMM; right: conv (54), decay and gate GEMMs -> gated memory (68, 69) ->
                        head norm (58) -> o GEMM
   streams -> gate / up GEMM with the gated epilogue -> down GEMM
   ... -> final streams (gather) -> head GEMM (fp32) -> sample (43)
@@ -285,7 +285,7 @@ class MatrixMemory:
         mem = lane._dev("MemoryArgs", q=at, k=at + es * H * d, v=at + es * 2 * H * d, gates=raw.addr,
                         gate_parts=parts, gate_rows=lane.slab_rows(T), gate_bias=w.gate_b, state=st["S"], m=st["m"], out=lane.raw.addr, tok_pos=lane.tok_pos,
                         ld_qkv=lane.proj.ld, ld_gates=ld, heads=H, d=d, e=e, f32=f32, q_scale=d ** -0.5, cap=m.gate_cap)
-        s_m = p.stage(_retarget(b.memory_tiles(H, e + 1), a0=mem.data_ptr()), label=("memory", run))
+        s_m = p.stage(_retarget(b.memory_tiles(H, e), a0=mem.data_ptr()), label=("memory", run))
         p.after(s, s_m)
         p.after(s_g, s_m)
         nrm = lane._dev("HeadNormArgs", o=lane.raw.addr, g=at + es * H * (2 * d + e), w=w.norm, out=lane.mix.addr, heads=H,
@@ -510,22 +510,22 @@ class _Batch:
             return np.concatenate(out)
         return self._once(("scan", channels), make)
 
-    def memory_tiles(self, heads, columns, kinds=(K_MEMORY, K_MEMORY_STEP), width=MEMORY_COLUMNS, step_width=MEMORY_COLUMNS):
-        """Portions: a tile per head and block of `width` columns; single tokens: as many blocks of step_width columns in a
-        tile as leave every worker one."""
+    def memory_tiles(self, heads, e):
+        """Portions: a tile per head and block of columns; single tokens: as many column blocks in a tile as leave every
+        worker one."""
         def make():
-            h, c = np.meshgrid(np.arange(heads), np.arange(-(-columns // width)), indexing="ij")
-            out = [tile_array(kinds[0], i0=row0, i1=n, i2=h | (c << 16), i3=slot, a1=width)
+            blocks = -(-(e + 1) // MEMORY_COLUMNS)
+            h, c = np.meshgrid(np.arange(heads), np.arange(blocks), indexing="ij")
+            out = [tile_array(K_MEMORY, i0=row0, i1=n, i2=h | (c << 16), i3=slot)
                    for row0, n, slot in sorted(self.requests, key=lambda q: -q[1]) if n > 1]
-            blocks = -(-columns // step_width)
             ones = [(row0, slot) for row0, n, slot in self.requests if n == 1]
             if ones:
                 row, slot = (np.array(v)[:, None, None] for v in zip(*ones))
                 per = min(128, -(-blocks // min(blocks, max(1, self.lane.fab.num_workers // (len(ones) * heads)))))
                 h, c = np.arange(heads)[None, :, None], np.arange(0, blocks, per)[None, None, :]
-                out.append(tile_array(kinds[1], i0=row, i1=np.minimum(per, blocks - c), i2=h | (c << 16), i3=slot))
+                out.append(tile_array(K_MEMORY_STEP, i0=row, i1=np.minimum(per, blocks - c), i2=h | (c << 16), i3=slot))
             return np.concatenate(out)
-        return self._once(("memory", heads, columns, kinds, width, step_width), make)
+        return self._once(("memory", heads, e), make)
 
     def attn_tiles(self, heads, parts, kind=K_LATENT_ATTN):
         """One tile per row, group of heads and part, the rows that see most keys first."""
@@ -660,7 +660,8 @@ class LayerListLane(LaneBase):
     def slab_rows(self, rows):
         return SPLIT_ROWS if rows <= SPLIT_ROWS else min(WIDE_ROWS, up(self.T, 64)) if rows <= WIDE_ROWS else self.T
 
-    def product(self, p, prev, x, w, out, rows, n, k, label, out16=False, parts=1, ld_out=None, epi=None, up_offset=0):
+    def product(self, p, prev, x, w, out, rows, n, k, label, out16=False, parts=1, ld_out=None, epi=None, up_offset=0,
+                bias=None, coef=None):
         """A stage out[rows][n] = x[rows][k] w[n][k]^T after `prev`.  out16: the output is of the activations' type,
         else fp32; parts > 1: that many fp32 slabs."""
         ld = ld_out or out.ld
@@ -673,7 +674,7 @@ class LayerListLane(LaneBase):
         else:
             s = self._gemm(p, self.weight_map(w), x.maps(k), rows, n, k, out.t, ld,
                            epi if epi is not None else (EPI_STORE if out16 else EPI_F32), label, up_offset=up_offset,
-                           bm=self.row_block(rows, n))
+                           bm=self.row_block(rows, n), bias=bias, coef=coef)
         for stage in prev if isinstance(prev, list) else [prev]:
             p.after(stage, s)
         return s

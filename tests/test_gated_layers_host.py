@@ -73,24 +73,30 @@ def test_stacked_projections_start_on_eight_columns():
 
 @pytest.mark.parametrize("heads,dim,e", [(3, 40, 24), (24, 128, 192), (40, 24, 130), (1, 512, 33), (2, 64, 64), (1, 1, 1), (48, 52, 128)])
 def test_memory_tiles_cover_rows_heads_and_columns_once(heads, dim, e):
-    from monoserve_b200.gated_mixers import K_GATED, K_GATED_STEP, gated_columns, step_columns
+    from monoserve_b200.gated_mixers import K_GATED, K_GATED_STEP, gated_columns, gated_tiles, step_columns
     from monoserve_b200.layer_list import _Batch
-    b = _Batch(lane(), REQUESTS, POS0)
-    width, step = gated_columns(REQUESTS, heads, dim, e, 140), step_columns(dim)
-    assert width in ((32, 64) if dim <= 128 else (16, 32) if dim <= 256 else (16,))
-    seen = np.zeros((107, heads, e), int)
-    t = fields(b.memory_tiles(heads, e, kinds=(K_GATED, K_GATED_STEP), width=width, step_width=step))
     slot_of = {row: slot for row0, n, slot in REQUESTS for row in range(row0, row0 + n)}
-    for k, row, a, what, slot, cols in zip(t["kind"], t["i0"], t["i1"], t["i2"], t["i3"], t["a1"]):
-        head, block = what & 0xFFFF, what >> 16
-        assert slot_of[row] == slot
-        if k == K_GATED:
-            assert cols == width and slot_of[row + a - 1] == slot
-            seen[row:row + a, head, block * width:(block + 1) * width] += 1
-        else:
-            assert k == K_GATED_STEP
-            seen[row, head, block * step:(block + a) * step] += 1
-    assert (seen == 1).all()
+    for f32, workers in ((False, 140), (True, 3)):
+        b = _Batch(lane(), REQUESTS, POS0)
+        width, step = gated_columns(REQUESTS, heads, dim, e, workers, f32), step_columns(dim)
+        assert width in ((32, 64) if dim <= 128 else (16, 32) if dim <= 256 else (16,)) and not (f32 and width == 64)
+        seen = np.zeros((107, heads, e), int)
+        t = fields(gated_tiles(b, heads, dim, e, workers, f32))
+        of_row = {}
+        for k, row, a, what, slot, cols in zip(t["kind"], t["i0"], t["i1"], t["i2"], t["i3"], t["a1"]):
+            assert slot_of[row] == slot
+            if k == K_GATED:
+                head, block = what & 0xFFFF, what >> 16
+                assert cols == width and slot_of[row + a - 1] == slot
+                seen[row:row + a, head, block * width:(block + 1) * width] += 1
+            else:
+                assert k == K_GATED_STEP
+                of_row[row] = of_row.get(row, 0) + 1
+                blocks = -(-e // step)
+                for v in range(what, what + a):
+                    seen[row, v // blocks, v % blocks * step:(v % blocks + 1) * step] += 1
+        assert (seen == 1).all()
+        assert all(n <= max(1, workers // 2) for n in of_row.values()) and len(of_row) == 2
 
 
 def test_wide_memory_tiles_are_used_where_they_save_a_round():

@@ -111,7 +111,7 @@ def test_tile_lists_cover_rows_channels_columns_and_heads_once():
     for heads, e in ((3, 40), (2, 31), (8, 512), (1, 32)):
         blocks = e // 32 + 1
         seen = np.zeros((107, heads, blocks), int)
-        t = fields(b.memory_tiles(heads, e + 1))
+        t = fields(b.memory_tiles(heads, e))
         for k, row, a, what, slot in zip(t["kind"], t["i0"], t["i1"], t["i2"], t["i3"]):
             head, block = what & 0xFFFF, what >> 16
             rows, count = (a, 1) if k == K_MEMORY else (1, a)
