@@ -3,6 +3,7 @@
 //   S <- diag(a) S;  u = v, or beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // and the decays themselves.  All of it is 32-bit arithmetic on the tensors' values.
 #include "fabric_layer_tiles.cuh"
+#include "ptx.cuh"
 #include "wide_tile.cuh"
 
 namespace mf {
@@ -455,16 +456,20 @@ __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring) {
 
 // ------------------------------------------------------------------ one token
 // Kind 69, GatedMemoryArgs: row i0, slot i3, i1 column blocks from block i2 on, counted through the heads (blocks of a head:
-// its columns over kBlock, rounded up).  G lanes share a column (ND four-row groups of it each), NC columns a lane.  The
-// state streams through registers, the next block's loads issued before this one's arithmetic; the read-out comes from the
-// state in front of the token's write, S^T q + (k q) u, so one round of sums per column serves both products.
+// its columns over kBlock, rounded up).  G lanes share a column (ND four-row groups of it each), NC columns a lane.  A wide
+// tile: a warp's columns of a block are one piece of memory, which comes and goes by bulk copies through kDepth stages of
+// its own in the ring.  The read-out comes from the state in front of the token's write, S^T q + (k q) u, so one round of
+// sums per column serves both products.
 template <int G, int ND, int NC, bool DELTA, bool F32>
-__device__ __noinline__ void gated_step(const TileDesc& t, int tid) {
+__device__ __noinline__ bool gated_step(const TileDesc& t, int tid, const LayerCtx& ctx) {
   using T = typename std::conditional<F32, float, __nv_bfloat16>::type;
-  constexpr int kSide = 32 / G, kBlock = 4 * NC * kSide;       // columns side by side in a warp; of a block
-  struct Block {
-    float4 S[NC][ND];
-    float k[ND][4], q[ND][4], m[ND][4], v, beta;
+  constexpr int kSide = 32 / G, kWarp = NC * kSide, kBlock = 4 * kWarp;   // columns side by side in a warp; of a warp; of a block
+  constexpr int kDepth = 6, kStageBytes = kWarp * G * ND * 16;
+  static_assert(4 * kDepth * kStageBytes <= 216 * 1024 && kStageBytes % 128 == 0, "the operand ring");
+  __builtin_assume(__isShared(ctx.ring));
+  __builtin_assume(__isShared(ctx.scratch));
+  struct Head {
+    float k[ND][4], q[ND][4], m[ND][4], beta;
   };
   GatedMemoryArgs A;
   load_block(A, t.a[0]);
@@ -497,125 +502,180 @@ __device__ __noinline__ void gated_step(const TileDesc& t, int tid) {
       v[3] = __uint_as_float(u.y & 0xffff0000u);
     }
   };
-  auto fetch = [&](int b, Block& B) {
-    const int head = b / blocks, c_lo = (b - head * blocks) * kBlock + warp * NC * kSide + side, kv = head / group;
-    const float* S = state + static_cast<size_t>(head) * e * dp;
-#pragma unroll
-    for (int c = 0; c < NC; ++c)
-#pragma unroll
-      for (int i = 0; i < ND; ++i) {
-        const int at = 4 * (l + G * i), col = c_lo + c * kSide;
-        B.S[c][i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (at < dp && col < e) B.S[c][i] = __ldcs(reinterpret_cast<const float4*>(S + static_cast<size_t>(col) * dp + at));
-      }
+  uint8_t* const stages = ctx.ring + warp * kDepth * kStageBytes;
+  uint64_t* const bar = reinterpret_cast<uint64_t*>(ctx.scratch) + warp * kDepth;
+  struct Place {
+    int head, col, n;   // first column of this warp in the block, and how many it has
+  };
+  auto place = [&](int b) {
+    Place x;
+    x.head = b / blocks;
+    x.col = (b - x.head * blocks) * kBlock + warp * kWarp;
+    x.n = max(0, min(kWarp, e - x.col));
+    return x;
+  };
+  auto state_at = [&](const Place& x) { return state + (static_cast<size_t>(x.head) * e + x.col) * dp; };
+  auto fetch = [&](int i) {   // lane 0
+    const Place x = place(first + i);
+    if (x.n == 0) return;
+    const uint32_t bytes = static_cast<uint32_t>(x.n * dp) * 4;
+    mbar_arrive_expect_tx(bar + i % kDepth, bytes);
+    bulk_in(stages + i % kDepth * kStageBytes, state_at(x), bytes, bar + i % kDepth);
+  };
+  auto fetch_v = [&](int b) {   // of the column this lane owns
+    const Place x = place(min(b, last - 1));
+    const int c = own * kSide + side;
+    return c < x.n ? value(v_row[static_cast<size_t>(x.head) * e + x.col + c]) : 0.f;
+  };
+  auto fetch_head = [&](int head, Head& X) {
+    const int kv = head / group;
 #pragma unroll
     for (int i = 0; i < ND; ++i) {
       const int at = 4 * (l + G * i);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) B.k[i][j] = B.q[i][j] = B.m[i][j] = 0.f;
+      for (int j = 0; j < 4; ++j) X.k[i][j] = X.q[i][j] = X.m[i][j] = 0.f;
       if (vec) {
         if (at < d) {
-          load4(k_row + kv * d + at, B.k[i]);
-          load4(q_row + kv * d + at, B.q[i]);
-          ld_vec<4>(m_row + head * d + at, B.m[i]);
+          load4(k_row + kv * d + at, X.k[i]);
+          load4(q_row + kv * d + at, X.q[i]);
+          ld_vec<4>(m_row + head * d + at, X.m[i]);
         }
       } else {
 #pragma unroll
         for (int j = 0; j < 4; ++j)
           if (at + j < d) {
-            B.k[i][j] = value(k_row[kv * d + at + j]);
-            B.q[i][j] = value(q_row[kv * d + at + j]);
-            B.m[i][j] = m_row[head * d + at + j];
+            X.k[i][j] = value(k_row[kv * d + at + j]);
+            X.q[i][j] = value(q_row[kv * d + at + j]);
+            X.m[i][j] = m_row[head * d + at + j];
           }
       }
     }
-    const int col = c_lo + own * kSide;
-    B.v = col < e ? value(v_row[static_cast<size_t>(head) * e + col]) : 0.f;
-    if constexpr (DELTA) B.beta = value(reinterpret_cast<const T*>(A.beta)[static_cast<size_t>(row) * A.ld_beta + head]);
+    if constexpr (DELTA) X.beta = value(reinterpret_cast<const T*>(A.beta)[static_cast<size_t>(row) * A.ld_beta + head]);
   };
-  Block blk[2];
-  fetch(first, blk[0]);
+  fence_proxy_async_all();   // the state may have been written, and the ring used, by plain loads and stores
+  if (lane < kDepth) mbar_init(bar + lane, 1);
+  fence_barrier_init();
+  exec_sync();
+  const int n_blocks = last - first;
+  if (lane == 0)
+    for (int i = 0; i < min(n_blocks, kDepth - 1); ++i) fetch(i);
+  Head next, X;
+  fetch_head(first / blocks, next);
+  float v0 = fetch_v(first), v1 = fetch_v(first + 1);
   const bool fresh = reinterpret_cast<const int*>(A.tok_pos)[row] == 0;
-  auto run = [&](int b, Block& B) {
-    const int head = b / blocks, c_lo = (b - head * blocks) * kBlock + warp * NC * kSide + side;
-    float* const S0 = state + static_cast<size_t>(head) * e * dp;
-    float dots[3] = {0.f, 0.f, 0.f};                           // k k, q q, k q
+  int at_head = -1;
+  float zk = 1.f, zq = 0.f, kq = 0.f, beta = 0.f;
+  uint32_t phases = 0;   // a bit per stage: loads are counted only where the warp has columns
+  bool ok = true;
+#pragma unroll 1
+  for (int it = 0; it < n_blocks; ++it) {
+    const int s = it % kDepth;
+    const Place at_block = place(first + it);
+    const int head = at_block.head, n_cols = at_block.n;
+    const float v = v0;
+    v0 = v1;
+    v1 = fetch_v(first + it + 2);
+    if (head != at_head) {   // the next head's row, and the one after it on its way
+      at_head = head;
+      X = next;
+      if (head < (last - 1) / blocks) fetch_head(head + 1, next);
+      float dots[3] = {0.f, 0.f, 0.f};                         // k k, q q, k q
 #pragma unroll
-    for (int i = 0; i < ND; ++i)
+      for (int i = 0; i < ND; ++i)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        dots[0] = fmaf(B.k[i][j], B.k[i][j], dots[0]);
-        dots[1] = fmaf(B.q[i][j], B.q[i][j], dots[1]);
-        dots[2] = fmaf(B.k[i][j], B.q[i][j], dots[2]);
+        for (int j = 0; j < 4; ++j) {
+          dots[0] = fmaf(X.k[i][j], X.k[i][j], dots[0]);
+          dots[1] = fmaf(X.q[i][j], X.q[i][j], dots[1]);
+          dots[2] = fmaf(X.k[i][j], X.q[i][j], dots[2]);
+        }
+#pragma unroll
+      for (int bit = G / 2; bit >= 1; bit >>= 1)
+#pragma unroll
+        for (int i = 0; i < 3; ++i) dots[i] += __shfl_xor_sync(0xffffffffu, dots[i], bit);
+      zk = unit ? 1.f / sqrtf(dots[0] + kUnitFloor) : 1.f;
+      zq = A.q_scale * (unit ? 1.f / sqrtf(dots[1] + kUnitFloor) : 1.f);
+      kq = dots[2] * zk * zq;
+      if constexpr (DELTA) beta = sigmoid32(X.beta);
+    }
+    if (n_cols > 0) {
+      ok = __all_sync(0xffffffffu, mbar_wait_bounded(bar + s, (phases >> s) & 1u, ctx.abort_flag, kWideWaitNs));
+      if (!ok) {   // the loads behind this one end, or run out of their time, before the ring is left
+        for (int j = it; j < min(n_blocks, it + kDepth - 1); ++j)
+          for (int tries = 0; place(first + j).n > 0 && tries < 1 << 16 && !mbar_try_wait(bar + j % kDepth, (phases >> j % kDepth) & 1u); ++tries) {}
+        break;
       }
-#pragma unroll
-    for (int bit = G / 2; bit >= 1; bit >>= 1)
-#pragma unroll
-      for (int i = 0; i < 3; ++i) dots[i] += __shfl_xor_sync(0xffffffffu, dots[i], bit);
-    const float zk = unit ? 1.f / sqrtf(dots[0] + kUnitFloor) : 1.f;
-    const float zq = A.q_scale * (unit ? 1.f / sqrtf(dots[1] + kUnitFloor) : 1.f), kq = dots[2] * zk * zq;
+      phases ^= 1u << s;
+    }
+    float* const S = reinterpret_cast<float*>(stages + s * kStageBytes) + side * dp;   // column c of this lane: c * kSide * dp on
+    float4 reg[NC][ND];
     float o[NC], p[NC];
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       o[c] = p[c] = 0.f;
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
-        float4& s = B.S[c][i];
-        if (fresh) s = make_float4(0.f, 0.f, 0.f, 0.f);
-        s.x = fmaf(s.x, B.m[i][0], s.x);
-        s.y = fmaf(s.y, B.m[i][1], s.y);
-        s.z = fmaf(s.z, B.m[i][2], s.z);
-        s.w = fmaf(s.w, B.m[i][3], s.w);
-        o[c] = fmaf(s.x, B.q[i][0], fmaf(s.y, B.q[i][1], fmaf(s.z, B.q[i][2], fmaf(s.w, B.q[i][3], o[c]))));
-        if constexpr (DELTA) p[c] = fmaf(s.x, B.k[i][0], fmaf(s.y, B.k[i][1], fmaf(s.z, B.k[i][2], fmaf(s.w, B.k[i][3], p[c]))));
+        const int at = 4 * (l + G * i);
+        float4& r = reg[c][i];
+        r = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (!fresh && at < dp && c * kSide + side < n_cols) r = *reinterpret_cast<const float4*>(S + c * kSide * dp + at);
+        r.x = fmaf(r.x, X.m[i][0], r.x);
+        r.y = fmaf(r.y, X.m[i][1], r.y);
+        r.z = fmaf(r.z, X.m[i][2], r.z);
+        r.w = fmaf(r.w, X.m[i][3], r.w);
+        o[c] = fmaf(r.x, X.q[i][0], fmaf(r.y, X.q[i][1], fmaf(r.z, X.q[i][2], fmaf(r.w, X.q[i][3], o[c]))));
+        if constexpr (DELTA) p[c] = fmaf(r.x, X.k[i][0], fmaf(r.y, X.k[i][1], fmaf(r.z, X.k[i][2], fmaf(r.w, X.k[i][3], p[c]))));
       }
     }
     group_sum<NC, G>(o, lane);
-    float u = B.v;
+    float u = v;
     if constexpr (DELTA) {
       group_sum<NC, G>(p, lane);
-      u = sigmoid32(B.beta) * (B.v - zk * p[0]);
+      u = beta * (v - zk * p[0]);
     }
-    const int mine = c_lo + own * kSide;
-    if (writes && mine < e) reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row) * H + head) * oe + mine] = fmaf(kq, u, zq * o[0]);
+    if (writes && own * kSide + side < n_cols)
+      reinterpret_cast<float*>(A.out)[(static_cast<size_t>(row) * H + head) * oe + at_block.col + own * kSide + side] = fmaf(kq, u, zq * o[0]);
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
       const float x = zk * __shfl_sync(0xffffffffu, u, side * G + c * G / NC);
-      const int col = c_lo + c * kSide;
 #pragma unroll
       for (int i = 0; i < ND; ++i) {
-        float4 s = B.S[c][i];
-        s.x = fmaf(B.k[i][0], x, s.x);
-        s.y = fmaf(B.k[i][1], x, s.y);
-        s.z = fmaf(B.k[i][2], x, s.z);
-        s.w = fmaf(B.k[i][3], x, s.w);
+        float4 r = reg[c][i];
+        r.x = fmaf(X.k[i][0], x, r.x);
+        r.y = fmaf(X.k[i][1], x, r.y);
+        r.z = fmaf(X.k[i][2], x, r.z);
+        r.w = fmaf(X.k[i][3], x, r.w);
         const int at = 4 * (l + G * i);
-        if (at < dp && col < e) __stcs(reinterpret_cast<float4*>(S0 + static_cast<size_t>(col) * dp + at), s);
+        if (at < dp && c * kSide + side < n_cols) *reinterpret_cast<float4*>(S + c * kSide * dp + at) = r;
       }
     }
-  };
-#pragma unroll 1
-  for (int b = first; b < last; b += 2) {
-    if (b + 1 < last) fetch(b + 1, blk[1]);
-    run(b, blk[0]);
-    if (b + 1 < last) {
-      if (b + 2 < last) fetch(b + 2, blk[0]);
-      run(b + 1, blk[1]);
+    fence_proxy_async_smem();
+    __syncwarp();
+    if (lane == 0) {
+      if (n_cols > 0) bulk_store(state_at(at_block), stages + s * kStageBytes, static_cast<uint32_t>(n_cols * dp) * 4);
+      bulk_commit();
+      if (it + kDepth - 1 < n_blocks) {   // into the stage of the block before, once its store has read it
+        bulk_wait_read<1>();
+        fetch(it + kDepth - 1);
+      }
     }
+    __syncwarp();
   }
+  if (lane == 0) bulk_wait_all();
+  ok = exec_and(ok);
+  if (lane < kDepth) mbar_inval(bar + lane);
+  return ok;
 }
 
-__device__ bool tile_gated_step(const TileDesc& t, int tid) {
+__device__ bool tile_gated_step(const TileDesc& t, int tid, const LayerCtx& ctx) {
   const GatedMemoryArgs* p = reinterpret_cast<const GatedMemoryArgs*>(t.a[0]);
   const uint32_t d = __ldcg(&p->d);
   const bool delta = __ldcg(&p->beta) != 0, f32 = __ldcg(&p->f32) != 0;
-#define MF_STEP(N, G, ND, NC)                                 \
-  if (d <= N) {                                               \
-    if (delta && f32) gated_step<G, ND, NC, true, true>(t, tid);   \
-    else if (delta) gated_step<G, ND, NC, true, false>(t, tid);    \
-    else if (f32) gated_step<G, ND, NC, false, true>(t, tid);      \
-    else gated_step<G, ND, NC, false, false>(t, tid);              \
-    return true;                                              \
+#define MF_STEP(N, G, ND, NC)                                             \
+  if (d <= N) {                                                           \
+    if (delta && f32) return gated_step<G, ND, NC, true, true>(t, tid, ctx);   \
+    if (delta) return gated_step<G, ND, NC, true, false>(t, tid, ctx);         \
+    if (f32) return gated_step<G, ND, NC, false, true>(t, tid, ctx);           \
+    return gated_step<G, ND, NC, false, false>(t, tid, ctx);                   \
   }
   MF_STEP(32, 8, 1, 8)
   MF_STEP(64, 16, 1, 16)

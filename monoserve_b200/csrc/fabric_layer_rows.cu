@@ -309,7 +309,7 @@ __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx) 
     case kTileResidual: tile_residual(t, tid, scratch); return true;
     case kTileDecay: tile_decay(t, tid); return true;
     case kTileGatedMemory: return tile_gated_memory(t, tid, ctx.ring);
-    case kTileGatedStep: return tile_gated_step(t, tid);
+    case kTileGatedStep: return tile_gated_step(t, tid, ctx);
     case kTileQkv: tile_qkv(t, tid); return true;
     case kTileGroupedAttn: return tile_grouped_attn(t, tid);
     case kTileHeadGate: tile_head_gate(t, tid); return true;

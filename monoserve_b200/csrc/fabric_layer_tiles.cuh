@@ -41,7 +41,7 @@ struct LayerCtx {
 __device__ bool run_layer_tile(const TileDesc& t, int tid, const LayerCtx& ctx);
 // Wide tiles: their exec warps use the operand ring as scratch memory, and TMEM.
 __device__ __forceinline__ bool tile_is_wide(uint32_t kind) {
-  return kind == kTileMemory || kind == kTileScan || kind == kTileGatedMemory || kind == kTileLatentMma || kind == kTileLatentDirect;
+  return kind == kTileMemory || kind == kTileScan || kind == kTileGatedMemory || kind == kTileGatedStep || kind == kTileLatentMma || kind == kTileLatentDirect;
 }
 
 __device__ void tile_streams(const TileDesc& t, int tid, int* scratch);
@@ -62,7 +62,7 @@ __device__ void tile_latent_merge(const TileDesc& t, int tid);
 __device__ void tile_residual(const TileDesc& t, int tid, int* scratch);
 __device__ void tile_decay(const TileDesc& t, int tid);
 __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring);
-__device__ bool tile_gated_step(const TileDesc& t, int tid);
+__device__ bool tile_gated_step(const TileDesc& t, int tid, const LayerCtx& ctx);
 __device__ void tile_qkv(const TileDesc& t, int tid);
 __device__ bool tile_grouped_attn(const TileDesc& t, int tid);
 __device__ void tile_head_gate(const TileDesc& t, int tid);
