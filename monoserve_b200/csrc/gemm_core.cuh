@@ -392,14 +392,15 @@ __device__ __forceinline__ float gelu_mul(float g, float u) {
   return __fdividef(g, 1.f + __expf(-t2)) * u;
 }
 
-// expm1(-coef softplus(z)), coef >= 0, to a few units of 2^-24: the distance to one of a decay e^(-coef softplus(z)).  Power
-// series where the sums 1 + t and e^x - 1 would cancel.
+// expm1(-coef softplus(z)), coef >= 0: the distance to one of a decay e^(-coef softplus(z)).  Power series where the sums
+// 1 + t and e^x - 1 would cancel; no branches.
 __device__ __forceinline__ float decay_less_one(float z, float coef) {
   const float t = __expf(-fabsf(z));
-  const float log1p_t = t < 0.02f ? t * fmaf(t, fmaf(t, fmaf(t, -0.25f, 1.f / 3.f), -0.5f), 1.f) : __logf(1.f + t);
-  const float x = -coef * (fmaxf(z, 0.f) + log1p_t);
-  const float series = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
-  return x > -0.25f ? series : __expf(x) - 1.f;
+  const float log_small = t * fmaf(t, fmaf(t, fmaf(t, -0.25f, 1.f / 3.f), -0.5f), 1.f), log_large = __logf(1.f + t);
+  const float x = -coef * (fmaxf(z, 0.f) + (t < 0.02f ? log_small : log_large));
+  const float small = x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+  const float large = __expf(x) - 1.f;
+  return x > -0.25f ? small : large;
 }
 
 // Epilogue of one tile from accumulator buffer `buf` (the four epilogue warps
@@ -506,8 +507,10 @@ __device__ __forceinline__ bool gemm_epilogue_body(const GemmWork& w, GemmBarrie
       if (f_ok) {
         const float coef = w.pair_weight[f];
 #pragma unroll
+        for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(decay_less_one(__uint_as_float(r[j]) * sc + bias, coef));
+#pragma unroll
         for (int j = 0; j < 32; ++j)
-          if (c0 + j < w.rows) out[static_cast<size_t>(j) * w.ld_out] = decay_less_one(__uint_as_float(r[j]) * sc + bias, coef);
+          if (c0 + j < w.rows) out[static_cast<size_t>(j) * w.ld_out] = __uint_as_float(r[j]);
       }
     } else {
       // fp32 rows that are read once, later (per-pair expert outputs, logits): streaming stores
