@@ -5,12 +5,15 @@ always `dense`: the dense-layer form of the GLM-style decoder (grouped-query att
 width, depth and feed-forward.  With Teganex the Sinotar layers are run as well: they have the like recurrence stages.
 
     python -m monoserve_b200.benchmarks.layer_list [--design Sinotar] [--sizes 2048,4096] [--steps 20] [--only ...] [--stages]
+                                                  [--serial]
 
 Timed by the fabric's iteration timer (device clock) over repeating programs on all SMs: `prefill` = 4 prompts of 1024
 tokens per iteration, `decode` = one token of 32 sequences with contexts around 4096 per iteration.  The weights of a
 step (more than 250 MB) exceed L2.  Every stage's mean span comes with its roofline time: the larger of its algorithmic
 bytes over the measured copy bandwidth and its products' FLOPs over the measured bf16 GEMM rate (MEASURED_PEAKS.json),
-and `frac` = roofline time / span.  One JSON line; --stages prints the tables to stderr.
+and `frac` = roofline time / span.  One JSON line; --stages prints the tables to stderr.  Stages that do not depend on one
+another share the SMs, and their spans include one another's work; --serial chains the stages of the layer-list decoders, for
+the spans of each alone.
 """
 import argparse
 import json
@@ -250,6 +253,22 @@ def timed(fab, lane, handle, tokens, steps, roofline, show):
     return dict(ms=round(float(np.median(ms)), 4), tokens_per_s=round(tokens / float(np.median(ms)) * 1e3, 1), stages=stages)
 
 
+def serial_program():
+    from monoserve_b200.fabric import Program
+
+    class Serial(Program):
+        """Every stage waits for the one added before it."""
+        last = None
+
+        def stage(self, *args, **kwargs):
+            s = super().stage(*args, **kwargs)
+            if self.last is not None:
+                self.after(self.last, s)
+            self.last = s
+            return s
+    return Serial
+
+
 def fabric():
     from monoserve_b200.fabric import Fabric
     fab = Fabric(pool_bytes=512 << 20)
@@ -257,7 +276,7 @@ def fabric():
     return fab
 
 
-def measure(kind, W, steps, show):
+def measure(kind, W, steps, show, serial=False):
     from monoserve_b200.layer_list import LayerListCache, LayerListLane, Weights
     from monoserve_b200.model import KVCache, ModelLane
     rng = np.random.default_rng(0)
@@ -284,6 +303,7 @@ def measure(kind, W, steps, show):
         for t in kv.k + kv.v:
             t.normal_(0, 1)
     make = LayerListLane if listed else ModelLane
+    programs = dict(program=serial_program()) if serial and listed else {}
     out = {}
     fab = fabric()   # one per program: a stopped lane keeps the program it was running
     try:
@@ -291,6 +311,7 @@ def measure(kind, W, steps, show):
         stride = max(dec_pages)
         perm = rng.permutation(n_pages - 1) + 1
         lane = make(fab, 0, cfg, weights, kv, max_tokens=T, max_slots=DECODE_ROWS, bt_stride=stride, logit_rows=DECODE_ROWS)
+        vars(lane).update(programs)
         at, batch = 0, []
         for s in range(PROMPTS):
             lane.set_pages(s, perm[at:at + pre_pages].tolist())
@@ -304,6 +325,7 @@ def measure(kind, W, steps, show):
         del lane
         fab = fabric()
         lane = make(fab, 0, cfg, weights, kv, max_tokens=DECODE_ROWS, max_slots=DECODE_ROWS, bt_stride=stride, logit_rows=DECODE_ROWS)
+        vars(lane).update(programs)
         for s, n in enumerate(dec_pages):
             lane.set_pages(s, perm[at:at + n].tolist())
             at += n
@@ -325,6 +347,7 @@ def main(argv=None):
     ap.add_argument("--design", choices=["Sinotar", "Teganex"], default="Sinotar")
     ap.add_argument("--only", choices=["Sinotar", "Teganex", "dense"])
     ap.add_argument("--stages", action="store_true")
+    ap.add_argument("--serial", action="store_true")
     args = ap.parse_args(argv)
     what = {"Sinotar": "matrix memory, selective scan, latent attention; 4 residual streams",
             "Teganex": "gated linear attention, attention beside a gated delta rule, gated linear attention of few large heads"}[args.design]
@@ -338,7 +361,7 @@ def main(argv=None):
         for kind in (args.only,) if args.only else kinds:
             if args.stages:
                 print(f"== width {W}, {kind}", file=sys.stderr)
-            line["sizes"][W][kind] = measure(kind, W, args.steps, args.stages)
+            line["sizes"][W][kind] = measure(kind, W, args.steps, args.stages, args.serial)
             torch.cuda.empty_cache()
     print(json.dumps(line), flush=True)
 

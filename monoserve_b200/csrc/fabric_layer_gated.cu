@@ -429,7 +429,7 @@ __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring) {
   const uint32_t d = __ldcg(&p->d);
   const bool delta = __ldcg(&p->beta) != 0;
   const bool f32 = __ldcg(&p->f32) != 0;
-  // a[1]: the columns of a block, one of two widths; 32-bit activations have the narrower one only
+  // a[1]: the columns of a block; 32-bit activations have the narrowest form only
 #define MF_GATED(N, G, C, F32)                                                          \
   if (d <= N && t.a[1] == 128 * C / G && f32 == F32) {                                  \
     if (delta) gated_rows<G, (N) / (G), C, true, F32>(t, tid, ring);                    \
@@ -445,6 +445,7 @@ __device__ bool tile_gated_memory(const TileDesc& t, int tid, uint8_t* ring) {
   MF_GATED(128, 8, 4, false)
   MF_GATED(128, 8, 2, false)
   MF_GATED(128, 8, 2, true)
+  MF_GATED(256, 8, 4, false)
   MF_GATED(256, 16, 4, false)
   MF_GATED(256, 16, 2, false)
   MF_GATED(256, 16, 2, true)

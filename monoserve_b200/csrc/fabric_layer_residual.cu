@@ -5,7 +5,9 @@ namespace mf {
 namespace fab {
 
 // Kind 66, ResidualArgs: rows [i0, i0 + i1), the four exec warps on one row.
-// Sums of two values over the exec threads; `slot` alternates, so that one barrier is enough.
+
+// Sums of two values over the exec threads.  Successive reductions of a row use scratch of their own, so that one barrier
+// each is enough.
 __device__ __forceinline__ void block_sum2(float& a, float& b, float* red, int tid) {
   a = warp_sum(a);
   b = warp_sum(b);

@@ -15,7 +15,7 @@ from monoserve_b200.attention import fabric_maps, fabric_tiles, plan_items
 from monoserve_b200.fabric import tile_array
 from monoserve_b200.lane_base import EPI_DECAY, _block, _retarget, up
 
-K_CONV, K_HEAD_NORM = 54, 58
+K_HEAD_NORM = 58
 K_DECAY, K_GATED, K_GATED_STEP, K_QKV, K_GROUPED_ATTN, K_HEAD_GATE = 67, 68, 69, 70, 71, 72
 K_ATTN_PREFILL, K_ATTN_PLAN = 33, 44
 MAX_GATED_DIM, MAX_CONV_TAPS, MAX_HEAD_COLUMNS = 512, 8, 512
@@ -67,13 +67,12 @@ def place_decay(W, a2, bias, coef, dim):
 
 
 def gated_columns(requests, heads, dim, columns, workers, f32=False):
-    """Columns of a portion's tile: the narrower or the wider form, which costs about one and a half times as much."""
-    narrow = 32 if dim <= 128 else 16
-    if f32 or dim > 256 or 2 * narrow > up(columns, narrow):
-        return narrow
+    """Columns of a portion's tile: the width whose rounds of tiles over the workers cost least, a tile of twice the columns
+    costing about a third more."""
+    widths = (32, 64) if dim <= 128 else (16, 32, 64) if dim <= 256 else (16,)
     portions = sum(1 for _, n, _ in requests if n > 1) * heads
-    rounds = {c: -(-portions * -(-columns // c) // workers) for c in (narrow, 2 * narrow)}
-    return 2 * narrow if 3 * rounds[2 * narrow] <= 2 * rounds[narrow] else narrow
+    fit = [w for w in widths[:1 if f32 else None] if w == widths[0] or w <= up(columns, widths[0])]
+    return min(fit, key=lambda w: -(-portions * -(-columns // w) // workers) * (4 / 3) ** widths.index(w))
 
 
 def step_columns(dim):

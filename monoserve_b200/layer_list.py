@@ -557,6 +557,8 @@ class _Batch:
 class LayerListLane(LaneBase):
     """One lane of the fabric running a layer-list decoder; the interface of ModelLane."""
 
+    program = Program   # what programs are built with
+
     def __init__(self, fab, lane_id, cfg, weights, kv, max_tokens, max_slots, bt_stride, logit_rows=None, requests=None,
                  keep_residual=False):
         """keep_residual: every program also stores the sum of the streams after each layer run (`residual`)."""
@@ -873,7 +875,7 @@ class LayerListLane(LaneBase):
         self._reset_build()
         places = want if want is not None else [[len(toks) - 1] for _, toks, _ in batch]
         T, req_info, sample_rows = self._batch_rows(batch, places, all_logits)
-        p = Program()
+        p = self.program()
         b = _Batch(self, [(row0, n, slot) for (row0, _, n, _), (slot, _, _) in zip(req_info, batch)], [q[2] for q in batch])
         first, last = self._chain(p, b, step=False)
         self._finish(p, b, last, T if all_logits else sum(len(v) for v in places), sample_rows if want is None else [])
@@ -886,7 +888,7 @@ class LayerListLane(LaneBase):
         self._reset_build()
         self._put(self.row_req, slots)
         self._put(self.gather, np.arange(R))
-        p = Program()
+        p = self.program()
         b = _Batch(self, [(r, 1, slot) for r, slot in enumerate(slots)])
         first, last = self._chain(p, b, step=True)
         self._finish(p, b, last, R, list(enumerate(slots)))

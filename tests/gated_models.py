@@ -12,7 +12,7 @@ def parallel(left, right):
                             right=dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), right)))
 
 
-def config(layers, width, vocab, ff=None, eps=1e-5, embed=3.0, logits=2.0, positions=512):
+def config(layers, width, vocab, ff=None, eps=2e-5, embed=2.5, logits=1.5, positions=512):
     """layers: mixers, or (mixer, ff) pairs; ff: the feed-forward width of layers that name none (None: no feed-forward)."""
     out = []
     for entry in layers:
@@ -108,10 +108,12 @@ MODELS = {
                    (parallel((5, 5, 7, 50, 0.5), (3, 3, 67, 5, 7)), 53)], 90, 203, ff=41, eps=3e-4, embed=0.7, logits=1.3),
     # many heads: tiles of 64 columns; 128 key channels; one key head for all query heads
     "heads": config([gla(24, 128, 192), parallel((16, 1, 128, 128, 0.09), (20, 5, 128, 256, 4)), (gla(40, 24, 130), None),
-                     (gla(48, 52, 128), None)], 256, 160, ff=128),
+                     (gla(48, 52, 128), None), (gla(10, 136, 258), None)], 256, 160, ff=128),
     # wider than the paged attention tiles and than one register block of the memories
     "big": config([gla(2, 200, 72), parallel((4, 2, 144, 160, 0.1), (2, 1, 300, 40, 5)), (gla(1, 512, 33), None)], 320, 333, ff=200),
-    "long_rows": config([gla(1, 16, 16)], 4100, 64),
+    # rows of the residual beyond one and beyond both of its register blocks
+    "wide_rows": config([gla(1, 16, 16), parallel((2, 1, 16, 16, 0.2), (1, 1, 16, 16, 2))], 2564, 64),
+    "long_rows": config([gla(1, 16, 16), (parallel((2, 1, 16, 16, 0.2), (1, 1, 16, 16, 2)), 64)], 4100, 64),
     "ones": config([gla(1, 1, 1, 1.0), parallel((1, 1, 1, 1, 1.0), (1, 1, 1, 1, 1))], 16, 16, ff=1),
 }
 SERVED = config([GLA, BOTH, gla(2, 64, 96, 8.0)], 112, 160, ff=64)

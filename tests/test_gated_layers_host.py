@@ -79,7 +79,7 @@ def test_memory_tiles_cover_rows_heads_and_columns_once(heads, dim, e):
     for f32, workers in ((False, 140), (True, 3)):
         b = _Batch(lane(), REQUESTS, POS0)
         width, step = gated_columns(REQUESTS, heads, dim, e, workers, f32), step_columns(dim)
-        assert width in ((32, 64) if dim <= 128 else (16, 32) if dim <= 256 else (16,)) and not (f32 and width == 64)
+        assert width in ((32, 64) if dim <= 128 else (16, 32, 64) if dim <= 256 else (16,)) and not (f32 and width == 64)
         seen = np.zeros((107, heads, e), int)
         t = fields(gated_tiles(b, heads, dim, e, workers, f32))
         of_row = {}
@@ -103,7 +103,8 @@ def test_wide_memory_tiles_are_used_where_they_save_a_round():
     from monoserve_b200.gated_mixers import gated_columns
     assert gated_columns([(0, 75, 0)], 24, 128, 192, 140) == 64     # 144 tiles of 32 columns are two rounds, 72 of 64 are one
     assert gated_columns([(0, 75, 0)], 24, 128, 128, 140) == 32     # 96 tiles are one round either way
-    assert gated_columns([(0, 75, 0)], 24, 192, 192, 140) == 32     # more rows, half the columns: 288 tiles or 144
+    assert gated_columns([(0, 75, 0)], 24, 192, 192, 140) == 64     # more rows: three rounds of 16 columns, two of 32, one of 64
+    assert gated_columns([(0, 75, 0)], 2, 192, 192, 140) == 16      # one round of any
     assert gated_columns([(0, 75, 0)], 24, 300, 192, 140) == 16
     assert gated_columns([(0, 75, 0)], 400, 128, 32, 140) == 32     # a head has no more
 
